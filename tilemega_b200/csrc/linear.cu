@@ -30,8 +30,13 @@ struct LinearParams {
   int t, n, out_stride, outputs;
   int chunks, chunks_per_split;
   Glu glu;
+  ExpertSlots slots;
   unsigned* status;
 };
+
+// Which products read gathered rows, and which run per expert.
+__host__ __device__ constexpr bool Gathers(int epilogue) { return epilogue == kLinearExpertUp; }
+__host__ __device__ constexpr bool PerExpert(int epilogue) { return epilogue == kLinearExpertUp || epilogue == kLinearExpertDown; }
 
 template <int BN> struct LinearShape {
   static constexpr int kStages = BN == 256 ? 4 : BN == 128 ? 3 : BN == 64 ? 4 : 5;   // about 100 KB (two CTAs per SM), 192 KB for the widest
@@ -43,7 +48,9 @@ template <int BN> struct LinearShape {
   static_assert(!kStaged || kStages * kStageBytes >= kRowsM * BN * 4, "the fp32 tile must fit the stages");
 };
 
+// gelu(g) = g (1 + tanh(z)) / 2 = g / (1 + exp(-2 z)), z = sqrt(2 / pi) (g + 0.044715 g^3)
 __device__ __forceinline__ float glu_value(float g, float u, const Glu& p) {
+  if (p.gelu) return g / (1.f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g))) * u;
   g = fminf(g, p.limit);
   u = fminf(fmaxf(u, -p.limit), p.limit);
   return g / (1.f + __expf(-p.alpha * g)) * (u + p.shift);
@@ -69,10 +76,17 @@ template <int EPI> __device__ __forceinline__ void emit(const LinearParams& g, i
   if (EPI == kLinearStore) static_cast<__nv_bfloat16*>(g.out)[size_t(t) * g.out_stride + n] = __float2bfloat16_rn(v);
   if (EPI == kLinearAdd) static_cast<float*>(g.out)[size_t(t) * g.out_stride + n] += v;
   if (EPI == kLinearFloat) static_cast<float*>(g.out)[size_t(t) * g.out_stride + n] = v;
+  if (EPI == kLinearExpertUp) {
+    const float r = fmaxf(v * g.slots.score[t], 0.f);
+    static_cast<__nv_bfloat16*>(g.out)[size_t(t) * g.out_stride + n] = __float2bfloat16_rn(r * r);
+  }
+  if (EPI == kLinearExpertDown) static_cast<__nv_bfloat16*>(g.out)[size_t(g.slots.list[t]) * g.out_stride + n] = __float2bfloat16_rn(v);
 }
 
 // blockIdx = (token tile, weight tile, K split): CTAs that run together share weight tiles, so a prompt's weights are read
-// once while its activations stay in L2. The CTAs of one (weight, token) tile form a cluster along z.
+// once while its activations stay in L2. The CTAs of one (weight, token) tile form a cluster along z. Per expert, token
+// tiles are those of the slot table (the grid holds as many as there could be), tokens are slots, and weight tiles start at
+// the expert's rows; rows beyond the tile's slots belong to other experts and are dropped.
 template <int BN, int EPI>
 __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap tmap,
                                                                const LinearParams g) {
@@ -85,7 +99,20 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
   uint64_t* accum = empty + S;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(accum + 1);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n0 = blockIdx.y * kRowsM, t0 = blockIdx.x * BN;
+  const int n0 = blockIdx.y * kRowsM;
+  int t0 = blockIdx.x * BN, t_end = g.t, weight_row = n0;
+  if constexpr (PerExpert(EPI)) {
+    // ExpertUp follows the kernel that writes the table; for ExpertDown it is there before the wait
+    if (Gathers(EPI)) dependency_wait();
+    if (int(blockIdx.x) >= *g.slots.tile_count) {
+      if (!Gathers(EPI)) dependency_wait();
+      return;
+    }
+    const ExpertTile tile = g.slots.tiles[blockIdx.x];
+    t0 = tile.first;
+    t_end = tile.first + min(tile.count, BN);
+    weight_row = tile.expert * g.n + n0;
+  }
   const int splits = gridDim.z;
   const int c0 = blockIdx.z * g.chunks_per_split;
   const int chunks = max(0, min(g.chunks_per_split, g.chunks - c0));
@@ -109,11 +136,39 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
   if (threadIdx.x == 0)
     for (int c = 0; c < early; ++c) {   // weights do not depend on the kernel before this one
       mbar_expect_tx(&full[c], Shape::kStageBytes);
-      tma_load_2d(tiles + c * Shape::kStageBytes, &wmap, (c0 + c) * kStepK, n0, &full[c]);
+      tma_load_2d(tiles + c * Shape::kStageBytes, &wmap, (c0 + c) * kStepK, weight_row, &full[c]);
     }
-  dependency_wait();
+  if (!Gathers(EPI)) dependency_wait();
 
-  if (warp == 0) {
+  if (Gathers(EPI) && warp == 0) {
+    // every lane fetches four rows of the tile (BN = 256: eight)
+    constexpr int Q = BN == 256 ? 2 : 1;
+    int rows[Q][4];
+#pragma unroll
+    for (int i = 0; i < 4 * Q; ++i) {
+      const int slot = min(t0 + (i / 4) * 128 + lane * 4 + i % 4, t_end - 1);
+      rows[i / 4][i % 4] = g.slots.list[slot] / g.slots.top;
+    }
+    int issued = 0;
+    bool ok = true;
+    for (int c = 0; c < chunks; ++c) {
+      const int s = c % S;
+      if (c >= S) ok = __all_sync(0xffffffffu, wait_bounded(&empty[s], uint32_t((c / S) - 1) & 1u, g.status, 1));
+      if (!ok) break;
+      unsigned char* w = tiles + s * Shape::kStageBytes;
+      if (lane == 0 && c >= early) {
+        mbar_expect_tx(&full[s], Shape::kStageBytes);
+        tma_load_2d(w, &wmap, (c0 + c) * kStepK, weight_row, &full[s]);
+      }
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < Q; ++i)
+        if (lane < BN / 4) tma_gather_rows(w + kWeightBytes + (i * 32 + lane) * 4 * kStepK * 2, &tmap, (c0 + c) * kStepK, rows[i], &full[s]);
+      issued = c + 1;
+    }
+    if (!ok)
+      for (int c = issued > S ? issued - S : 0; c < issued; ++c) wait_bounded(&full[c % S], uint32_t(c / S) & 1u, g.status, 2);
+  } else if (warp == 0) {
     if (lane == 0) {
       int issued = 0;
       bool ok = true;
@@ -124,7 +179,7 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
         unsigned char* w = tiles + s * Shape::kStageBytes;
         if (c >= early) {
           mbar_expect_tx(&full[s], Shape::kStageBytes);
-          tma_load_2d(w, &wmap, (c0 + c) * kStepK, n0, &full[s]);
+          tma_load_2d(w, &wmap, (c0 + c) * kStepK, weight_row, &full[s]);
         }
         tma_load_2d(w + kWeightBytes, &tmap, (c0 + c) * kStepK, t0, &full[s]);
         issued = c + 1;
@@ -177,7 +232,7 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
     if (worker >= 0 && ok) {
       const uint32_t rank = splits > 1 ? cluster_rank() : 0;
       const int per = (BN + splits - 1) / splits, first = int(rank) * per;
-      const int cols = min(min(per, BN - first), g.t - t0 - first);   // this CTA's tokens of the tile
+      const int cols = min(min(per, BN - first), t_end - t0 - first);   // this CTA's tokens of the tile
       const uint32_t base = smem_u32(tile);
       auto total = [&](int c, int row) {
         if (splits == 1) return tile[c * kRowsM + row];
@@ -211,10 +266,10 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
     const int n = n0 + 32 * quarter + lane;
     const float bias = g.bias && n < g.n ? g.bias[n] : 0.f;
     for (int c = column_half * (BN / 2); c < (column_half + 1) * (BN / 2); c += 32) {
-      if (t0 + c >= g.t) break;
+      if (t0 + c >= t_end) break;
       float v[32];
       tmem_load_32(tmem + (uint32_t(32 * quarter) << 16) + uint32_t(c), v);
-      const int cols = min(32, g.t - t0 - c);
+      const int cols = min(32, t_end - t0 - c);
       if constexpr (EPI == kLinearGlu) {
         const bool upper = lane >= kGluUnit;          // lanes 0..15 hold gate rows, 16..31 the matching up rows
         const int out = (n0 + 32 * quarter) / 2 + (lane & (kGluUnit - 1));
@@ -258,16 +313,25 @@ constexpr int kTile32 = 64, kStep32 = 16;
 template <int EPI>
 __global__ void __launch_bounds__(256) linear_f32(const float* activations, const float* weight, const LinearParams g, int k_stride) {
   __shared__ float as[kStep32][kTile32 + 4], ws[kStep32][kTile32 + 4];
-  const int n0 = blockIdx.x * kTile32, t0 = blockIdx.y * kTile32;
+  const int n0 = blockIdx.x * kTile32;
+  int t0 = blockIdx.y * kTile32, t_end = g.t;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   dependency_wait();
   allow_dependents();
+  if constexpr (PerExpert(EPI)) {
+    if (int(blockIdx.y) >= *g.slots.tile_count) return;
+    const ExpertTile tile = g.slots.tiles[blockIdx.y];
+    t0 = tile.first;
+    t_end = tile.first + min(tile.count, kTile32);
+    weight += size_t(tile.expert) * g.n * k_stride;
+  }
+  auto row_of = [&](int t) { return Gathers(EPI) ? g.slots.list[t] / g.slots.top : t; };
   float acc[4][4] = {};
   for (int k0 = 0; k0 < k_stride; k0 += kStep32) {
 #pragma unroll
     for (int i = threadIdx.x; i < kTile32 * kStep32; i += 256) {
       const int r = i / kStep32, k = i % kStep32;
-      as[k][r] = t0 + r < g.t && k0 + k < k_stride ? activations[size_t(t0 + r) * k_stride + k0 + k] : 0.f;
+      as[k][r] = t0 + r < t_end && k0 + k < k_stride ? activations[size_t(row_of(t0 + r)) * k_stride + k0 + k] : 0.f;
       ws[k][r] = n0 + r < g.n && k0 + k < k_stride ? weight[size_t(n0 + r) * k_stride + k0 + k] : 0.f;
     }
     __syncthreads();
@@ -284,10 +348,11 @@ __global__ void __launch_bounds__(256) linear_f32(const float* activations, cons
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
-      if (t >= g.t || n >= g.n) continue;
+      if (t >= t_end || n >= g.n) continue;
       const float v = acc[i][j] + (g.bias ? g.bias[n] : 0.f);
-      float* out = static_cast<float*>(g.out) + size_t(t) * g.out_stride + n;
-      *out = EPI == kLinearAdd ? *out + v : v;
+      float* out = static_cast<float*>(g.out) + size_t(EPI == kLinearExpertDown ? g.slots.list[t] : t) * g.out_stride + n;
+      const float positive = fmaxf(EPI == kLinearExpertUp ? v * g.slots.score[t] : 0.f, 0.f);
+      *out = EPI == kLinearAdd ? *out + v : EPI == kLinearExpertUp ? positive * positive : v;
     }
 }
 
@@ -298,25 +363,35 @@ __global__ void __launch_bounds__(256) glu_rows(const T* in, T* out, int t, int 
   const int j = blockIdx.x * 256 + threadIdx.x, row = blockIdx.y;
   if (j >= outputs || row >= t) return;
   const T* pair = in + size_t(row) * in_stride + (j / kGluUnit) * 2 * kGluUnit + j % kGluUnit;
+  if (glu.gelu) {
+    const float z = to_f(pair[0]);
+    out[size_t(row) * out_stride + j] = from_f<T>(z / (1.f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))) * to_f(pair[kGluUnit]));
+    return;
+  }
   const float g = fminf(to_f(pair[0]), glu.limit), u = fminf(fmaxf(to_f(pair[kGluUnit]), -glu.limit), glu.limit);
   out[size_t(row) * out_stride + j] = from_f<T>(g / (1.f + expf(-glu.alpha * g)) * (u + glu.shift));
 }
 
 template <int BN> cudaError_t RaiseLimit() {
   const int smem = LinearShape<BN>::kSmem;
-  for (auto kernel : {linear_tiles<BN, kLinearStore>, linear_tiles<BN, kLinearAdd>, linear_tiles<BN, kLinearGlu>, linear_tiles<BN, kLinearFloat>}) {
+  for (auto kernel : {linear_tiles<BN, kLinearStore>, linear_tiles<BN, kLinearAdd>, linear_tiles<BN, kLinearGlu>, linear_tiles<BN, kLinearFloat>,
+                      linear_tiles<BN, kLinearExpertUp>, linear_tiles<BN, kLinearExpertDown>}) {
     const cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (err != cudaSuccess) return err;
   }
   return cudaSuccess;
 }
 
+// Most tiles the slots of a step can fall into: full ones, and one more for every expert in use.
+int MostTiles(const ExpertSlots& s) { return s.slots / s.tile_rows + std::min(s.experts, s.slots); }
+
 template <int BN>
 cudaError_t LaunchTiles(const Queue& q, const LinearArgs& a, const LinearParams& p, int map, int splits) {
   auto kernel = a.epilogue == kLinearAdd ? linear_tiles<BN, kLinearAdd> : a.epilogue == kLinearGlu ? linear_tiles<BN, kLinearGlu>
-                : a.epilogue == kLinearFloat ? linear_tiles<BN, kLinearFloat> : linear_tiles<BN, kLinearStore>;
+                : a.epilogue == kLinearFloat ? linear_tiles<BN, kLinearFloat> : a.epilogue == kLinearExpertUp ? linear_tiles<BN, kLinearExpertUp>
+                : a.epilogue == kLinearExpertDown ? linear_tiles<BN, kLinearExpertDown> : linear_tiles<BN, kLinearStore>;
   cudaLaunchConfig_t config{};
-  config.gridDim = dim3(unsigned((a.t + BN - 1) / BN), unsigned((a.n + kRowsM - 1) / kRowsM), unsigned(splits));
+  config.gridDim = dim3(unsigned(PerExpert(a.epilogue) ? MostTiles(a.slots) : (a.t + BN - 1) / BN), unsigned((a.n + kRowsM - 1) / kRowsM), unsigned(splits));
   config.blockDim = dim3(kLinearThreads);
   config.dynamicSmemBytes = LinearShape<BN>::kSmem;
   config.stream = q.stream;
@@ -334,7 +409,7 @@ cudaError_t LaunchTiles(const Queue& q, const LinearArgs& a, const LinearParams&
   }
   config.attrs = attributes;
   config.numAttrs = unsigned(count);
-  return cudaLaunchKernelEx(&config, kernel, a.maps->weight, a.maps->rows[map], p);
+  return cudaLaunchKernelEx(&config, kernel, a.maps->weight, Gathers(a.epilogue) ? a.maps->row : a.maps->rows[map], p);
 }
 
 // Tile width (index into 16, 32, 64, 128, 256 tokens) and K splits: the widest tile that gives most SMs a CTA, else
@@ -353,7 +428,25 @@ void ChooseLinear(int t, int n, int chunks, int sms, int* index, int* splits) {
   while (*splits < kMaxCluster && grid * *splits <= sms && chunks / (*splits * 2) >= (grid * *splits * 10 < sms * 8 ? 4 : 16)) *splits *= 2;
 }
 
+// The same per expert: the tile width is that of the slot table; K splits until the tiles to be expected cover the SMs.
+void ChooseExpertLinear(const ExpertSlots& s, int n, int chunks, int sms, int* index, int* splits) {
+  *index = 0;
+  while ((16 << *index) < s.tile_rows) ++*index;
+  *splits = 1;
+  if (*index == 4) return;
+  const int grid = MostTiles(s) * ((n + kRowsM - 1) / kRowsM);
+  while (*splits < kMaxCluster && grid * *splits <= sms && chunks / (*splits * 2) >= 4) *splits *= 2;
+}
+
 }  // namespace
+
+int ExpertTileRows(const Queue& q, int slots, int experts) {
+  if (q.f32) return kTile32;
+  const int share = (slots + experts - 1) / experts;   // slots of an expert on average; most have no more than 4/3 of it
+  int rows = 16;
+  while (rows < 256 && rows * 3 < share * 4) rows *= 2;
+  return rows;
+}
 
 int PrepareLinear() {
   cudaError_t err = RaiseLimit<16>();
@@ -368,11 +461,13 @@ bool EncodeLinear(LinearMaps* maps, const void* weight, uint64_t n, const void* 
   if (!EncodeMatrix(&maps->weight, false, weight, n, k_stride, kRowsM)) return false;
   for (int i = 0; i < 5; ++i)
     if (!EncodeMatrix(&maps->rows[i], false, activations, rows, k_stride, 16u << i)) return false;
-  return true;
+  return EncodeMatrix(&maps->row, false, activations, rows, k_stride, 1);
 }
 
 int Linear(const Queue& q, const LinearArgs& a) {
   if (a.t <= 0) return 0;
+  const bool experts = PerExpert(a.epilogue);
+  if (experts && (a.slots.slots <= 0 || a.slots.tile_rows < 16 || !a.slots.tiles)) return int(cudaErrorInvalidValue);
   LinearParams p{};
   p.bias = a.bias;
   p.out = a.out;
@@ -381,17 +476,21 @@ int Linear(const Queue& q, const LinearArgs& a) {
   p.out_stride = a.out_stride;
   p.outputs = a.outputs;
   p.glu = a.glu;
+  p.slots = a.slots;
   p.status = q.status;
   if (q.f32) {
     if (a.epilogue == kLinearGlu) return int(cudaErrorInvalidValue);   // two operations in fp32: the product, then GluRows
-    auto kernel = a.epilogue == kLinearAdd ? linear_f32<kLinearAdd> : linear_f32<kLinearStore>;
-    const dim3 grid(unsigned((a.n + kTile32 - 1) / kTile32), unsigned((a.t + kTile32 - 1) / kTile32));
+    auto kernel = a.epilogue == kLinearAdd ? linear_f32<kLinearAdd> : a.epilogue == kLinearExpertUp ? linear_f32<kLinearExpertUp>
+                  : a.epilogue == kLinearExpertDown ? linear_f32<kLinearExpertDown> : linear_f32<kLinearStore>;
+    if (experts && a.slots.tile_rows != kTile32) return int(cudaErrorInvalidValue);
+    const dim3 grid(unsigned((a.n + kTile32 - 1) / kTile32), unsigned(experts ? MostTiles(a.slots) : (a.t + kTile32 - 1) / kTile32));
     return int(Launch(kernel, grid, dim3(256), 0, q.stream, q.chained, static_cast<const float*>(a.activations),
                       static_cast<const float*>(a.weight), p, a.k_stride));
   }
   p.chunks = (a.k_stride + kStepK - 1) / kStepK;
   int index = 0, splits = 1;
-  ChooseLinear(a.t, a.n, p.chunks, q.sm_count, &index, &splits);
+  if (experts) ChooseExpertLinear(a.slots, a.n, p.chunks, q.sm_count, &index, &splits);
+  else ChooseLinear(a.t, a.n, p.chunks, q.sm_count, &index, &splits);
   p.chunks_per_split = (p.chunks + splits - 1) / splits;
   switch (index) {
     case 0: return int(LaunchTiles<16>(q, a, p, 0, splits));

@@ -17,38 +17,49 @@ namespace tmb {
 namespace {
 
 // ---- rotary + append ------------------------------------------------------------------------------------------------
+struct AppendParams {
+  int stride, heads, kv_heads, dim, vdim, pool_dim, v_pool_dim;
+  bool value_is_key;
+  const float *q_norm, *k_norm;
+  float eps;
+  Rotary rot;
+};
+
 template <typename T>
-__global__ void __launch_bounds__(128) rotate_append(StepRows r, T* proj, int stride, T* k_pool, T* v_pool, int heads, int kv_heads, int dim,
-                                                     int pool_dim, bool value_is_key, Rotary rot, bool portions_only) {
+__global__ void __launch_bounds__(128) rotate_append(StepRows r, T* proj, T* k_pool, T* v_pool, AppendParams p, bool portions_only) {
+  __shared__ float2 part[4];
   dependency_wait();
   allow_dependents();
   const int row = blockIdx.x;
   if (portions_only && r.entry[r.row_entry[row]].rows == 1) return;
-  const int half = rot.dims / 2, units = dim - half;   // a unit: one rotated pair, or one entry behind the rotated ones
-  const float2* angle = rot.table + size_t(min(r.row_position[row], rot.capacity - 1)) * half;
+  const int half = p.rot.dims / 2, units = p.dim - half;   // a unit: one rotated pair, or one entry behind the rotated ones
+  const float2* angle = p.rot.table + size_t(min(r.row_position[row], p.rot.capacity - 1)) * half;
   const int kv = r.row_kv[row];
-  T* line = proj + size_t(row) * stride;
-  for (int i = threadIdx.x; i < (heads + kv_heads) * units; i += 128) {
-    const int head = i / units, u = i % units, group = head - heads;
-    T* at = line + size_t(head) * dim;
-    const size_t pool = group < 0 ? 0 : pool_offset(kv, group, kv_heads, pool_dim);
-    const T* value = value_is_key ? at : line + size_t(heads + kv_heads + group) * dim;
+  T* line = proj + size_t(row) * p.stride;
+  const T* keys = line + size_t(p.heads) * p.dim;
+  float2 inv = make_float2(1.f, 1.f);
+  if (p.q_norm) {
+    const int q_count = p.heads * p.dim, k_count = p.kv_heads * p.dim;
+    inv = inverse_rms<128>(make_float2(square_sum(line, q_count, 128), square_sum(keys, k_count, 128)), q_count, k_count, p.eps, part);
+  }
+  const T* values = p.value_is_key ? keys : keys + size_t(p.kv_heads) * p.dim;
+  for (int i = threadIdx.x; i < p.kv_heads * p.vdim; i += 128)
+    v_pool[pool_offset(kv, i / p.vdim, p.kv_heads, p.v_pool_dim) + i % p.vdim] = values[i];
+  for (int i = threadIdx.x; i < (p.heads + p.kv_heads) * units; i += 128) {
+    const int head = i / units, u = i % units, group = head - p.heads;
+    if (u >= half && group < 0 && !p.q_norm) continue;      // (an entry of q that stays as it is)
+    T* at = line + size_t(head) * p.dim;
+    T* to = group < 0 ? at : k_pool + pool_offset(kv, group, p.kv_heads, p.pool_dim);
+    const float scale = group < 0 ? inv.x : inv.y;
+    const float* weight = group < 0 ? p.q_norm : p.k_norm;
+    auto value = [&](int d) { return weight ? to_f(at[d]) * scale * weight[(group < 0 ? head : group) * p.dim + d] : to_f(at[d]); };
     if (u < half) {
-      const T a = at[u], b = at[u + half];
+      const float a = value(u), b = value(u + half);
       const float2 cs = angle[u];
-      const T x = from_f<T>(to_f(a) * cs.x - to_f(b) * cs.y), y = from_f<T>(to_f(b) * cs.x + to_f(a) * cs.y);
-      if (group < 0) {
-        at[u] = x;
-        at[u + half] = y;
-      } else {
-        k_pool[pool + u] = x;
-        k_pool[pool + u + half] = y;
-        v_pool[pool + u] = value[u];
-        v_pool[pool + u + half] = value[u + half];
-      }
-    } else if (group >= 0) {
-      k_pool[pool + u + half] = at[u + half];
-      v_pool[pool + u + half] = value[u + half];
+      to[u] = from_f<T>(a * cs.x - b * cs.y);
+      to[u + half] = from_f<T>(b * cs.x + a * cs.y);
+    } else {
+      to[u + half] = from_f<T>(value(u + half));
     }
   }
 }
@@ -58,8 +69,8 @@ constexpr int kPlainWarps = 4;
 
 template <typename T>
 __global__ void __launch_bounds__(32 * kPlainWarps) attend_rows(StepRows r, const T* proj, int stride, const T* k_pool, const T* v_pool, T* out,
-                                                                int out_stride, int heads, int kv_heads, int dim, int pool_dim, int window,
-                                                                int keep, float scale) {
+                                                                int out_stride, int heads, int kv_heads, int dim, int vdim, int pool_dim,
+                                                                int v_pool_dim, int window, int keep, float scale, float sink, int gate_at) {
   __shared__ float qs[kPlainWarps][kMaxHeadDim];
   dependency_wait();
   allow_dependents();
@@ -73,14 +84,16 @@ __global__ void __launch_bounds__(32 * kPlainWarps) attend_rows(StepRows r, cons
   for (int d = lane; d < dim; d += 32) qs[warp][d] = to_f(proj[size_t(row) * stride + size_t(head) * dim + d]);
   __syncwarp();
   constexpr int N = kMaxHeadDim / 32;
-  float acc[N] = {}, top = -INFINITY, sum = 0.f;
+  float acc[N] = {}, top = sink, sum = sink == -INFINITY ? 0.f : 1.f;   // (the null key, if there is one)
   auto walk = [&](int from, int to) {
     for (int base = from; base < to; base += 32) {
       const int j = base + lane;
-      long long at = 0;
+      long long v_at = 0;
       float score = -INFINITY;
       if (j < to) {
-        at = (long long)(pool_offset(key_row(table, j, r), group, kv_heads, pool_dim));
+        const int key = key_row(table, j, r);
+        const size_t at = pool_offset(key, group, kv_heads, pool_dim);
+        v_at = (long long)(pool_offset(key, group, kv_heads, v_pool_dim));
         float dot = 0.f;
         for (int d = 0; d < dim; ++d) dot = fmaf(qs[warp][d], to_f(k_pool[at + d]), dot);
         score = dot * scale;
@@ -94,10 +107,10 @@ __global__ void __launch_bounds__(32 * kPlainWarps) attend_rows(StepRows r, cons
       const int count = min(32, to - base);
       for (int jj = 0; jj < count; ++jj) {
         const float weight = __shfl_sync(0xffffffffu, p, jj);
-        const T* v = v_pool + __shfl_sync(0xffffffffu, at, jj);
+        const T* v = v_pool + __shfl_sync(0xffffffffu, v_at, jj);
 #pragma unroll
         for (int i = 0; i < N; ++i)
-          if (lane + 32 * i < dim) acc[i] = fmaf(weight, to_f(v[lane + 32 * i]), acc[i]);
+          if (lane + 32 * i < vdim) acc[i] = fmaf(weight, to_f(v[lane + 32 * i]), acc[i]);
       }
     }
   };
@@ -105,8 +118,12 @@ __global__ void __launch_bounds__(32 * kPlainWarps) attend_rows(StepRows r, cons
   walk(0, min(keep, low));
   walk(low, position + 1);
 #pragma unroll
-  for (int i = 0; i < N; ++i)
-    if (lane + 32 * i < dim) out[size_t(row) * out_stride + size_t(head) * dim + lane + 32 * i] = from_f<T>(acc[i] / sum);
+  for (int i = 0; i < N; ++i) {
+    const int c = lane + 32 * i;
+    if (c >= vdim) continue;
+    const float gate = gate_at < 0 ? 1.f : sigmoid(to_f(proj[size_t(row) * stride + gate_at + size_t(head) * vdim + c]));
+    out[size_t(row) * out_stride + size_t(head) * vdim + c] = from_f<T>(acc[i] / sum * gate);
+  }
 }
 
 // ---- retention by its recurrence ----------------------------------------------------------------------------------------
@@ -303,15 +320,16 @@ __global__ void __launch_bounds__(128) retention_gate(const float* raw, const T*
 }
 
 template <typename T> int RotateAppendAs(const Queue& q, const StepRows& r, const AttentionArgs& a) {
-  return int(Launch(rotate_append<T>, dim3(unsigned(r.rows)), dim3(128), 0, q.stream, q.chained, r, static_cast<T*>(a.proj), a.proj_stride,
-                    static_cast<T*>(a.k_pool), static_cast<T*>(a.v_pool), a.heads, a.kv_heads, a.dim, a.pool_dim, a.value_is_key, a.rotary, !q.f32));
+  const AppendParams p{a.proj_stride, a.heads, a.kv_heads, a.dim, a.vdim, a.pool_dim, a.v_pool_dim, a.value_is_key, a.q_norm, a.k_norm, a.eps, a.rotary};
+  return int(Launch(rotate_append<T>, dim3(unsigned(r.rows)), dim3(128), 0, q.stream, q.chained, r, static_cast<T*>(a.proj),
+                    static_cast<T*>(a.k_pool), static_cast<T*>(a.v_pool), p, !q.f32));
 }
 
 template <typename T> int AttendAs(const Queue& q, const StepRows& r, const AttentionArgs& a) {
   const dim3 grid(unsigned((a.heads + kPlainWarps - 1) / kPlainWarps), unsigned(r.rows));
   return int(Launch(attend_rows<T>, grid, dim3(32 * kPlainWarps), 0, q.stream, q.chained, r, static_cast<const T*>(a.proj), a.proj_stride,
                     static_cast<const T*>(a.k_pool), static_cast<const T*>(a.v_pool), static_cast<T*>(a.out), a.out_stride, a.heads,
-                    a.kv_heads, a.dim, a.pool_dim, a.window, a.keep, a.scale));
+                    a.kv_heads, a.dim, a.vdim, a.pool_dim, a.v_pool_dim, a.window, a.keep, a.scale, a.sink, a.gate_at));
 }
 
 template <typename T> int RetainAs(const Queue& q, const StepRows& r, const RetentionArgs& a, bool singles_only) {

@@ -1,7 +1,8 @@
-// Addressing and rotary helpers shared by the mixer kernels of a ragged step.
+// Addressing, norm and rotary helpers shared by the mixer kernels of a ragged step.
 #pragma once
 #include "element.cuh"
 #include "ops.h"
+#include "ptx.cuh"
 
 namespace tmb {
 
@@ -24,5 +25,52 @@ template <typename T> __device__ __forceinline__ float rotated(const T* head, in
   const float2 cs = angle[i];
   return d < half ? u * cs.x - v * cs.y : v * cs.x + u * cs.y;
 }
+
+// The same for a head whose entries are first scaled: entry d by inv * weight[d] (weight null: not at all).
+template <typename T>
+__device__ __forceinline__ float normed_rotated(const T* head, const float* weight, float inv, int d, int half, const float2* angle) {
+  if (!weight) return rotated(head, d, half, angle);
+  if (d >= 2 * half) return to_f(head[d]) * inv * weight[d];
+  const int i = d < half ? d : d - half;
+  const float u = to_f(head[i]) * inv * weight[i], v = to_f(head[i + half]) * inv * weight[i + half];
+  const float2 cs = angle[i];
+  return d < half ? u * cs.x - v * cs.y : v * cs.x + u * cs.y;
+}
+
+// A thread's share of the squares of `count` consecutive elements, spread over `threads` threads.
+template <typename T> __device__ __forceinline__ float square_sum(const T* at, int count, int threads) {
+  float sq = 0.f;
+  if (sizeof(T) == 2 && (reinterpret_cast<uintptr_t>(at) & 15) == 0 && count % 8 == 0) {
+    for (int i = threadIdx.x; i < count / 8; i += threads) {
+      float v[8];
+      unpack8(reinterpret_cast<const uint4*>(at)[i], v);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) sq = fmaf(v[j], v[j], sq);
+    }
+  } else {
+    for (int i = threadIdx.x; i < count; i += threads) {
+      const float v = to_f(at[i]);
+      sq = fmaf(v, v, sq);
+    }
+  }
+  return sq;
+}
+// 1 / rms of two vectors from every thread's shares of their squares; `part` holds one entry per warp.
+template <int THREADS>
+__device__ __forceinline__ float2 inverse_rms(float2 squares, int count_a, int count_b, float eps, float2* part) {
+  squares.x = warp_sum(squares.x);
+  squares.y = warp_sum(squares.y);
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = squares;
+  __syncthreads();
+  float2 sum = make_float2(0.f, 0.f);
+#pragma unroll
+  for (int w = 0; w < THREADS / 32; ++w) {
+    sum.x += part[w].x;
+    sum.y += part[w].y;
+  }
+  return make_float2(1.f / sqrtf(sum.x / float(count_a) + eps), 1.f / sqrtf(sum.y / float(count_b) + eps));
+}
+
+__device__ __forceinline__ float sigmoid(float v) { return 1.f / (1.f + expf(-v)); }
 
 }  // namespace tmb

@@ -63,9 +63,10 @@ struct AttendParams {
   bf16* out;
   float* part;
   unsigned* count;
-  int proj_stride, out_stride, heads, kv_heads, dim, pool_dim, window, keep, splits;
+  const float *q_norm, *k_norm;
+  int proj_stride, out_stride, heads, kv_heads, dim, vdim, pool_dim, v_pool_dim, window, keep, splits, gate_at;
   int subs, sub_heads;      // query heads of one key head are served in `subs` units of up to `sub_heads`
-  float scale_log2;
+  float scale_log2, sink_log2, eps;
   bool value_is_key;
   Rotary rotary;
 };
@@ -81,8 +82,9 @@ template <int DT, int WM> struct AttendShape {
 // Rows of a tile are (token, query head of the unit) pairs, token-major. WM = 8: a prompt portion, 128 rows, each warp 16
 // of them against all keys of a block; q is rotated and the portion's keys are in the pools already (RotateAppend).
 // WM = 1: one decoded token, 16 rows, each of the four warps a quarter of a block's keys; the CTA rotates q itself, and
-// the one that holds the newest position rotates and appends its key and value. blockIdx = (token tile | split, unit,
-// entry).
+// the one that holds the newest position rotates and appends its key and value (both norm them first, if the model does,
+// which takes the squares of the whole projected row). DT: 16-column tiles of the wider of keys and values. blockIdx =
+// (token tile | split, unit, entry).
 template <int DT, int WM>
 __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM > 1 ? 2 : 3) attend_tiles(StepRows r, AttendParams p) {
   using Shape = AttendShape<DT, WM>;
@@ -92,6 +94,7 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
   bf16* ks = qs + Shape::kRows * P;
   bf16* vs = ks + 2 * Shape::kTile;
   __shared__ unsigned last;
+  __shared__ float2 square_part[NT / 32];
   __shared__ int key_at[2][kKeys];   // pool rows of a block's keys (-1: none)
   // Every kernel of a step lets the next one start only behind its own dependency wait, so what kernels before the last
   // one wrote is there already: the step's tables, and the keys of earlier steps. A decoded token's first block of keys
@@ -133,10 +136,10 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
 #pragma unroll 4
     for (int i = threadIdx.x; i < kKeys * C; i += NT) {
       const int key = i / C, c = (i % C) * 8, row = key_at[stage][key];
-      const bool live = row >= 0 && c < p.pool_dim;
-      const size_t at = live ? pool_offset(row, group, p.kv_heads, p.pool_dim) + c : 0;
-      copy16(ks + stage * Shape::kTile + key * P + c, p.k_pool + at, live);
-      copy16(vs + stage * Shape::kTile + key * P + c, p.v_pool + at, live);
+      const bool live = row >= 0;
+      const size_t line = live ? size_t(row / kRaggedBlock * p.kv_heads + group) * kRaggedBlock + row % kRaggedBlock : 0;
+      if (c < p.pool_dim) copy16(ks + stage * Shape::kTile + key * P + c, p.k_pool + line * p.pool_dim + c, live);
+      if (c < p.v_pool_dim) copy16(vs + stage * Shape::kTile + key * P + c, p.v_pool + line * p.v_pool_dim + c, live);
     }
     copy_commit();
   };
@@ -150,9 +153,16 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
   const int half = p.rotary.dims / 2;
   const float2* angle = p.rotary.table + size_t(min(p1, p.rotary.capacity - 1)) * half;   // WM == 1: the token's
   const bool wide = (p.dim & 7) == 0;
+  float2 inv = make_float2(1.f, 1.f);
+  if (WM == 1 && p.q_norm) {
+    const bf16* line = p.proj + size_t(e.first_row) * p.proj_stride;
+    const int q_count = p.heads * p.dim, k_count = p.kv_heads * p.dim;
+    inv = inverse_rms<NT>(make_float2(square_sum(line, q_count, NT), square_sum(line + q_count, k_count, NT)), q_count, k_count, p.eps, square_part);
+  }
   for (int i = threadIdx.x; i < Shape::kRows * (P / 8); i += NT) {
     const int m = i / (P / 8), c = (i % (P / 8)) * 8, t = m / gq;
     const bf16* head = p.proj + size_t(e.first_row + t0 + t) * p.proj_stride + size_t(head0 + m % gq) * p.dim;
+    const float* weight = p.q_norm ? p.q_norm + (head0 + m % gq) * p.dim : nullptr;
     uint4 word = make_uint4(0, 0, 0, 0);
     if (t < tokens && c < p.dim) {
       if (wide && WM > 1) {
@@ -161,7 +171,7 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
         bf16 e8[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j)
-          e8[j] = c + j >= p.dim ? __float2bfloat16_rn(0.f) : WM > 1 ? head[c + j] : __float2bfloat16_rn(rotated(head, c + j, half, angle));
+          e8[j] = c + j >= p.dim ? __float2bfloat16_rn(0.f) : WM > 1 ? head[c + j] : __float2bfloat16_rn(normed_rotated(head, weight, inv.x, c + j, half, angle));
         word = *reinterpret_cast<uint4*>(e8);
       }
     }
@@ -189,16 +199,20 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
     if (WM == 1 && b + 1 == blocks) {   // the newest position: over whatever the copy found in its pool row
       const bf16* k = p.proj + size_t(e.first_row) * p.proj_stride + size_t(p.heads + group) * p.dim;
       const bf16* v = p.value_is_key ? k : k + size_t(p.kv_heads) * p.dim;
-      const size_t pool = pool_offset(key_row(table, p1, r), group, p.kv_heads, p.pool_dim);
-      const int key = p1 - block_base(b);
+      v += size_t(group) * (p.vdim - p.dim);
+      const float* weight = p.k_norm ? p.k_norm + group * p.dim : nullptr;
+      const int row = key_row(table, p1, r), key = p1 - block_base(b);
+      bf16* k_to = p.k_pool + pool_offset(row, group, p.kv_heads, p.pool_dim);
+      bf16* v_to = p.v_pool + pool_offset(row, group, p.kv_heads, p.v_pool_dim);
       for (int d = threadIdx.x; d < p.dim; d += NT) {
-        const bf16 kd = __float2bfloat16_rn(rotated(k, d, half, angle)), vd = v[d];
+        const bf16 kd = __float2bfloat16_rn(normed_rotated(k, weight, inv.y, d, half, angle));
         ks[stage * Shape::kTile + key * P + d] = kd;
+        if (first_head == 0) k_to[d] = kd;
+      }
+      for (int d = threadIdx.x; d < p.vdim; d += NT) {
+        const bf16 vd = v[d];
         vs[stage * Shape::kTile + key * P + d] = vd;
-        if (first_head == 0) {
-          p.k_pool[pool + d] = kd;
-          p.v_pool[pool + d] = vd;
-        }
+        if (first_head == 0) v_to[d] = vd;
       }
       __syncthreads();
     }
@@ -209,6 +223,7 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
     for (int t = 0; t < KN / 8; ++t) s[t][0] = s[t][1] = s[t][2] = s[t][3] = 0.f;
 #pragma unroll
     for (int kk = 0; kk < DT; ++kk) {
+      if (kk * 16 >= p.pool_dim) break;
       uint32_t a[4];
       load_a(a, qs, P, row0, kk * 16, lane);
 #pragma unroll
@@ -275,6 +290,7 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
       }
 #pragma unroll
       for (int d = 0; d < DT; ++d) {
+        if (d * 16 >= p.v_pool_dim) break;
         uint32_t bb[4];
         load_b_transposed(bb, vt, P, kk * 16, d * 16, lane);
         mma16816(o[2 * d], hi, bb[0], bb[1]);
@@ -291,14 +307,27 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
     sum_b += __shfl_xor_sync(0xffffffffu, sum_b, x);
   }
   if constexpr (WM > 1) {
-    const float inv_a = 1.f / sum_a, inv_b = 1.f / sum_b;
+    // (a null key that stands above every key takes the maximum's place: the values then count by the distance)
+    auto share = [&](float top, float sum) {
+      if (p.sink_log2 == -INFINITY) return 1.f / sum;
+      const float high = fmaxf(top, p.sink_log2), f = ex2(top - high);
+      return f / fmaf(sum, f, ex2(p.sink_log2 - high));
+    };
+    const float inv_a = share(top_a, sum_a), inv_b = share(top_b, sum_b);
     auto write = [&](int m, float inv, int i, int at) {
-      const int t = m / gq;
-      if (t >= tokens) return;
-      bf16* dst = p.out + size_t(e.first_row + t0 + t) * p.out_stride + size_t(head0 + m % gq) * p.dim;
-      const int c = i * 8 + 2 * (lane & 3);
-      if (c < p.dim) dst[c] = __float2bfloat16_rn(o[i][at] * inv);
-      if (c + 1 < p.dim) dst[c + 1] = __float2bfloat16_rn(o[i][at + 1] * inv);
+      const int t = m / gq, c = i * 8 + 2 * (lane & 3);
+      if (t >= tokens || c >= p.vdim) return;
+      const size_t row = size_t(e.first_row + t0 + t), column = size_t(head0 + m % gq) * p.vdim + c;
+      bf16* dst = p.out + row * p.out_stride + column;
+      float y0 = o[i][at] * inv, y1 = o[i][at + 1] * inv;
+      const bool pair = c + 1 < p.vdim;
+      if (p.gate_at >= 0) {
+        const bf16* gate = p.proj + row * p.proj_stride + p.gate_at + column;
+        y0 *= sigmoid(__bfloat162float(gate[0]));
+        if (pair) y1 *= sigmoid(__bfloat162float(gate[1]));
+      }
+      dst[0] = __float2bfloat16_rn(y0);
+      if (pair) dst[1] = __float2bfloat16_rn(y1);
     };
 #pragma unroll
     for (int i = 0; i < 2 * DT; ++i) {
@@ -325,11 +354,14 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
       *reinterpret_cast<float2*>(os + (warp * 16 + rb) * D + c) = make_float2(o[i][2], o[i][3]);
     }
     __syncthreads();
-    const int record = p.dim + 2;
+    const bf16* gates = p.proj + size_t(e.first_row) * p.proj_stride + p.gate_at + size_t(head0) * p.vdim;   // [head of the unit][column]
+    bf16* dst = p.out + size_t(e.first_row) * p.out_stride + size_t(head0) * p.vdim;
+    auto gated = [&](float v, int i) { return __float2bfloat16_rn(p.gate_at < 0 ? v : v * sigmoid(__bfloat162float(gates[i]))); };
+    const int record = p.vdim + 2;
     float* parts = p.part + (size_t(blockIdx.z) * p.heads + head0) * p.splits * record;   // [head of the unit][split][record]
-    for (int i = threadIdx.x; i < gq * p.dim; i += NT) {
-      const int h = i / p.dim, c = i % p.dim;
-      float high = -INFINITY, sum = 0.f, value = 0.f;
+    for (int i = threadIdx.x; i < gq * p.vdim; i += NT) {
+      const int h = i / p.vdim, c = i % p.vdim;
+      float high = p.splits == 1 ? p.sink_log2 : -INFINITY, sum = 0.f, value = 0.f;
 #pragma unroll
       for (int w = 0; w < 4; ++w) high = fmaxf(high, ms[w * 16 + h]);
       const float ref = high == -INFINITY ? 0.f : high;
@@ -340,7 +372,7 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
         value = fmaf(os[(w * 16 + h) * D + c], f, value);
       }
       if (p.splits == 1) {
-        p.out[size_t(e.first_row) * p.out_stride + size_t(head0 + h) * p.dim + c] = __float2bfloat16_rn(value / sum);
+        dst[i] = gated(value / (sum + ex2(p.sink_log2 - ref)), i);
       } else {
         float* mine = parts + (size_t(h) * p.splits + split) * record;
         mine[2 + c] = value;
@@ -367,8 +399,9 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
       if (int(threadIdx.x) < gq) {
         float* f = factor + threadIdx.x * p.splits;
         const float* l = f + gq * p.splits;
-        float high = -INFINITY, sum = 0.f;
+        float high = p.sink_log2;
         for (int s = 0; s < p.splits; ++s) high = fmaxf(high, f[s]);
+        float sum = ex2(p.sink_log2 - high);
         for (int s = 0; s < p.splits; ++s) {         // in split order
           f[s] = ex2(f[s] - high);
           sum = fmaf(l[s], f[s], sum);
@@ -376,15 +409,15 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
         for (int s = 0; s < p.splits; ++s) f[s] /= sum;
       }
       __syncthreads();
-      const int outputs = gq * p.dim;
+      const int outputs = gq * p.vdim;
       for (int i0 = threadIdx.x; i0 < outputs; i0 += 4 * NT) {
         float value[4] = {};
         const float* at[4];
         const float* f[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          const int i = min(i0 + j * NT, outputs - 1), h = i / p.dim;
-          at[j] = parts + size_t(h) * p.splits * record + 2 + i % p.dim;
+          const int i = min(i0 + j * NT, outputs - 1), h = i / p.vdim;
+          at[j] = parts + size_t(h) * p.splits * record + 2 + i % p.vdim;
           f[j] = factor + h * p.splits;
         }
 #pragma unroll 8
@@ -394,7 +427,7 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int i = i0 + j * NT;
-          if (i < outputs) p.out[size_t(e.first_row) * p.out_stride + size_t(head0 + i / p.dim) * p.dim + i % p.dim] = __float2bfloat16_rn(value[j]);
+          if (i < outputs) dst[i] = gated(value[j], i);
         }
       }
     }
@@ -703,7 +736,7 @@ template <int DT> int AttendWith(const Queue& q, const StepRows& r, const Attent
         one.splits = s;
       }
     }
-    if (size_t(r.entries) * a.heads * one.splits * (a.dim + 2) > a.part_floats || r.entries * units > a.count_words) one.splits = 1;
+    if (size_t(r.entries) * a.heads * one.splits * (a.vdim + 2) > a.part_floats || r.entries * units > a.count_words) one.splits = 1;
     const int status = LaunchAttend<DT, 1>(q, r, one, one.splits);
     if (status != 0) return status;
   }
@@ -749,7 +782,13 @@ int AttendTiles(const Queue& q, const StepRows& r, const AttentionArgs& a) {
   p.heads = a.heads;
   p.kv_heads = a.kv_heads;
   p.dim = a.dim;
+  p.vdim = a.vdim;
   p.pool_dim = a.pool_dim;
+  p.v_pool_dim = a.v_pool_dim;
+  p.q_norm = a.q_norm;
+  p.k_norm = a.k_norm;
+  p.eps = a.eps;
+  p.gate_at = a.gate_at;
   p.window = a.window;
   p.keep = a.keep;
   const int gq = a.heads / a.kv_heads;
@@ -757,7 +796,8 @@ int AttendTiles(const Queue& q, const StepRows& r, const AttentionArgs& a) {
   p.sub_heads = (gq + p.subs - 1) / p.subs;
   p.subs = (gq + p.sub_heads - 1) / p.sub_heads;
   p.scale_log2 = a.scale * 1.4426950408889634f;
-  const int tiles = (a.dim + 15) / 16;
+  p.sink_log2 = a.sink * 1.4426950408889634f;
+  const int tiles = (std::max(a.dim, a.vdim) + 15) / 16;
   return tiles <= 2 ? AttendWith<2>(q, r, a, p) : tiles <= 4 ? AttendWith<4>(q, r, a, p) : tiles <= 6 ? AttendWith<6>(q, r, a, p)
          : tiles <= 8 ? AttendWith<8>(q, r, a, p) : tiles <= 12 ? AttendWith<12>(q, r, a, p) : AttendWith<16>(q, r, a, p);
 }

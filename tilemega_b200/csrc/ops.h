@@ -37,8 +37,8 @@ struct StepRows {
   int* row_kv = nullptr;                    // [rows] pool row: block * 16 + position mod 16
 };
 
-// x[row] = embed[token]; the row tables.
-int StartStep(const Queue& q, const StepRows& r, const int* tokens, const void* embed, float* x, int width, int vocab);
+// x[row] = embed[token] (and as an element in `copy`, rows of copy_stride, unless null); the row tables.
+int StartStep(const Queue& q, const StepRows& r, const int* tokens, const void* embed, float* x, void* copy, int copy_stride, int width, int vocab);
 
 // out[i] = x[r] / sqrt(mean(x[r]^2) + eps) * weight, r = select ? select[i] : i. With `again`, x[r] += embed[token[r]]
 // first (and is written back). Rows of `out` are out_stride elements apart.
@@ -54,25 +54,57 @@ struct NormArgs {
 };
 int RmsNorm(const Queue& q, const NormArgs& a);
 
+// A sublayer's output normed and added: x[i] += y / sqrt(mean(y^2) + eps) * weight, and out[i] = x[i] as elements. y is
+// branch[i] (fp32 [rows][width]), or with `parts` > 0 the sum of the elements parts_of[i * parts + 0 .. parts - 1].
+struct AddNormArgs {
+  float* x;
+  const float* branch;
+  const void* parts_of;
+  int parts;
+  const float* weight;
+  void* out;
+  int rows, width, out_stride;
+  float eps;
+};
+int AddNorm(const Queue& q, const AddNormArgs& a);
+
 // Rotary table [capacity][dims / 2] of (cos, sin), or dims = 0: none.
 struct Rotary {
   const float2* table = nullptr;
   int dims = 0, capacity = 0;
 };
 
-// y = min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + shift)
+// y = min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u, -limit, limit) + shift), or with `gelu` y = gelu(g) u, the
+// tanh form
 struct Glu {
   float limit = 0.f, alpha = 1.f, shift = 0.f;
+  bool gelu = false;
 };
 
-enum LinearEpilogue { kLinearStore = 0, kLinearAdd = 1, kLinearGlu = 2, kLinearFloat = 3 };
+enum LinearEpilogue { kLinearStore = 0, kLinearAdd = 1, kLinearGlu = 2, kLinearFloat = 3, kLinearExpertUp = 4, kLinearExpertDown = 5 };
+
+// The assignments of a step's rows to experts, sorted by expert (written by Route). Assignment a is the a % top-th choice
+// of row a / top; slot s, in sorted order, runs assignment list[s] on the expert of its tile.
+struct ExpertTile {
+  int expert, first, count, unused;   // slots [first, first + count)
+};
+struct ExpertSlots {
+  const ExpertTile* tiles = nullptr;
+  const int* tile_count = nullptr;
+  const int* list = nullptr;          // [slots]
+  const float* score = nullptr;       // [slots]
+  int experts = 0, top = 1, slots = 0, tile_rows = 0;
+};
 
 // D[t][n] = sum_k activations[t][k] weight[n][k] (+ bias[n]), then by epilogue: store as an element; x[t][n] += D; the
 // gated unit of interleaved gate/up rows, stored as an element (column n of the output is pair n); store as fp32.
 // Activation and weight rows are k_stride elements long (a multiple of 8, zero weights behind k).
+// Per expert (weight rows expert * n ..., slots in place of t): ExpertUp reads activation row list[s] / top for slot s
+// and stores relu(score[s] D)^2 in row s; ExpertDown reads row s and stores D in row list[s]; both as elements.
 struct LinearMaps {
   CUtensorMap weight;        // bf16 only: 128-row boxes
   CUtensorMap rows[5];       // boxes of 16, 32, 64, 128, 256 activation rows
+  CUtensorMap row;           // boxes of one activation row (gathered rows)
 };
 struct LinearArgs {
   const void* activations;
@@ -84,7 +116,9 @@ struct LinearArgs {
   int outputs;               // kLinearGlu: columns stored (pairs beyond it are padding)
   int epilogue;
   Glu glu;
+  ExpertSlots slots;         // expert epilogues
 };
+int ExpertTileRows(const Queue& q, int slots, int experts);   // slots per tile that suits this many
 int PrepareLinear();         // raises the kernels' shared-memory limits (once per device)
 bool EncodeLinear(LinearMaps* maps, const void* weight, uint64_t n, const void* activations, uint64_t rows, uint64_t k_stride);
 int Linear(const Queue& q, const LinearArgs& a);
@@ -92,17 +126,42 @@ int Linear(const Queue& q, const LinearArgs& a);
 // The gated unit by itself: in [t][2 * padded] interleaved pairs, out [t][outputs].
 int GluRows(const Queue& q, const void* in, void* out, int t, int in_stride, int out_stride, int outputs, const Glu& glu);
 
+// Mixture of experts: the `top` largest of z = router h per row (the smaller index on a tie), scores sigmoid(z), and the
+// assignments sorted by expert in tiles of slots->tile_rows. RouteFused: does Route compute z itself? (If not, the
+// caller has put it into `logits`.)
+struct RouteArgs {
+  const void* h;             // elements, rows of k_stride
+  const void* router;        // [experts][k_stride]
+  int k_stride, rows, experts, top, tile_rows;
+  float* logits;             // [rows][experts]
+  int* choice;               // [rows * top]
+  float* score;              // [rows * top]
+  int* list;                 // [rows * top], sorted
+  float* slot_score;         // [rows * top], sorted
+  ExpertTile* tiles;
+  int* tile_count;
+  unsigned* count;           // arrival counter, zero between launches
+};
+bool RouteFused(int rows);
+int Route(const Queue& q, const RouteArgs& a);
+
 // Attention with grouped heads, a sliding window of `window` positions and the first `keep` positions always seen.
-// proj rows hold q | k (| v): q heads x dim, k kv_heads x dim; the values are v, or k before rotation (value_is_key).
+// proj rows hold q | k (| v) (| g): q heads x dim, k kv_heads x dim, v kv_heads x vdim, g heads x vdim; the values are v,
+// or k before rotation (value_is_key). q_norm / k_norm: RMS norm over all heads together before the rotation. A null key
+// of score `sink` (-infinity: none) without a value joins the softmax. gate_at >= 0: outputs times sigmoid(g).
 struct AttentionArgs {
   void* proj;
   int proj_stride;
   void* k_pool;              // [num_blocks][kv_heads][16][pool_dim]
-  void* v_pool;
-  void* out;                 // [rows][out_stride], heads x dim
+  void* v_pool;              // [num_blocks][kv_heads][16][v_pool_dim]
+  void* out;                 // [rows][out_stride], heads x vdim
   int out_stride;
-  int heads, kv_heads, dim, pool_dim;
+  int heads, kv_heads, dim, vdim, pool_dim, v_pool_dim;
   bool value_is_key;
+  const float* q_norm;       // [heads * dim], or null
+  const float* k_norm;       // [kv_heads * dim]
+  float eps, sink;
+  int gate_at;               // first gate column of a projected row, or -1
   int window, keep;
   float scale;
   Rotary rotary;
@@ -111,7 +170,7 @@ struct AttentionArgs {
   unsigned* count;           // arrival counters, zero between launches
   int count_words;
 };
-// Rotates q in place and appends rotated k and v to the pools. (bf16: rows of portions only; a decoded token's attention
+// Norms and rotates q in place and appends such k, and v, to the pools. (bf16: rows of portions only; a decoded token's attention
 // does it itself.)
 int RotateAppend(const Queue& q, const StepRows& r, const AttentionArgs& a);
 int Attend(const Queue& q, const StepRows& r, const AttentionArgs& a);

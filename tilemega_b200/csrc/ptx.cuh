@@ -213,6 +213,15 @@ __device__ __forceinline__ void tma_load_3d(void* dst, const void* tensor_map, i
       : "memory");
 }
 
+// Four rows y[0..3] of a 2-D map whose box is one row high, `x` as above: four consecutive box rows in shared memory.
+__device__ __forceinline__ void tma_gather_rows(void* dst, const void* tensor_map, int x, const int (&y)[4], uint64_t* bar) {
+  asm volatile(
+      "cp.async.bulk.tensor.2d.shared::cta.global.tile::gather4.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4, %5, %6}], [%7];" ::"r"(
+          smem_u32(dst)),
+      "l"(tensor_map), "r"(x), "r"(y[0]), "r"(y[1]), "r"(y[2]), "r"(y[3]), "r"(smem_u32(bar))
+      : "memory");
+}
+
 // Tensor memory columns for this CTA (a power of two >= 32); the base address lands in
 // shared memory. Executed by one whole warp, which also frees the columns.
 __device__ __forceinline__ void tmem_alloc(uint32_t* base_in_smem, uint32_t columns) {

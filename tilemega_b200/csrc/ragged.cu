@@ -25,6 +25,15 @@ struct RaggedPlan {
   void* mixed = nullptr;       // [max_rows][widest mixer output]
   void* mlp = nullptr;         // [max_rows][widest feed-forward]
   void* pairs = nullptr;       // fp32 plans: gate/up rows before the gated unit
+  float* branch = nullptr;     // fp32 outputs of sublayers that are normed before they are added
+  // mixtures of experts: logits, choices and scores per row, the assignments sorted by expert, their hidden rows and outputs
+  float* logits = nullptr;
+  int *choice = nullptr, *list = nullptr, *tile_count = nullptr;
+  float *score = nullptr, *slot_score = nullptr;
+  ExpertTile* tiles = nullptr;
+  unsigned* route_count = nullptr;
+  void* expert_hidden = nullptr;   // [max_rows * most experts of a token][widest expert]
+  void* expert_out = nullptr;      // [max_rows * most experts of a token][width]
   float* raw = nullptr;        // retention outputs before their norm
   void* split = nullptr;       // bf16 plans: rotated retention queries and keys of portions
   float* part = nullptr;       // attention partials
@@ -33,7 +42,7 @@ struct RaggedPlan {
   int count_words = 0;
   std::vector<float*> decay;   // per layer
   struct Maps {
-    LinearMaps in, out, gate_up, down;
+    LinearMaps in, out, gate_up, down, router;   // (gate_up, down: of the gated unit or of the experts)
   };
   std::vector<Maps> maps;      // per layer (bf16 plans)
   LinearMaps head;
@@ -72,7 +81,8 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     const int status_ = (call);      \
     if (status_ != 0) return status_; \
   } while (0)
-  TMB_TRY(StartStep(q, r, tokens, buffer(s.embed), x, W, s.vocab));
+  const bool norm_output = s.layers[0].norm_output;   // sublayers then read the stream itself: `normed` holds it as elements
+  TMB_TRY(StartStep(q, r, tokens, buffer(s.embed), x, norm_output ? plan->normed : nullptr, W8, W, s.vocab));
   auto norm = [&](int weight, bool again) {
     NormArgs a{};
     a.x = x;
@@ -102,13 +112,32 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     a.epilogue = epilogue;
     return a;
   };
+  // a sublayer's last product (rows of `in` times `weight`): added to the stream, or normed and added
+  auto add_output = [&](const void* in, int weight, int bias, const LinearMaps* maps, int k) {
+    if (!norm_output) return Linear(q, linear(in, weight, bias, maps, W, k, x, W, kLinearAdd));
+    return Linear(q, linear(in, weight, bias, maps, W, k, plan->branch, W, kLinearFloat));
+  };
+  auto add_norm = [&](int weight, int parts) {
+    AddNormArgs a{};
+    a.x = x;
+    a.branch = plan->branch;
+    a.parts_of = plan->expert_out;
+    a.parts = parts;
+    a.weight = floats(weight);
+    a.out = plan->normed;
+    a.rows = r.rows;
+    a.width = W;
+    a.out_stride = W8;
+    a.eps = float(s.eps);
+    return AddNorm(q, a);
+  };
   for (size_t i = 0; i < s.runs.size(); ++i) {
     const RaggedRun& run = s.runs[i];
     const RaggedLayer& layer = s.layers[size_t(run.layer)];
     const RaggedMixer& m = layer.mixer;
     const RaggedPlan::Maps* maps = s.f32 ? nullptr : &plan->maps[size_t(run.layer)];
     const int stride = (m.proj_rows() + 7) / 8 * 8, mixed_stride = padded_columns(m.out_columns());
-    TMB_TRY(norm(layer.norm1, run.add_embedding));
+    if (!norm_output) TMB_TRY(norm(layer.norm1, run.add_embedding));
     TMB_TRY(Linear(q, linear(plan->normed, layer.in_weight, layer.in_bias, maps ? &maps->in : nullptr, m.proj_rows(), W, plan->proj, stride, kLinearStore)));
     Rotary rotary;
     if (m.rotary >= 0) {
@@ -144,7 +173,14 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.heads = m.heads;
       a.kv_heads = m.kv_heads;
       a.dim = m.dim;
+      a.vdim = m.vdim;
       a.pool_dim = m.pool_dim();
+      a.v_pool_dim = m.v_pool_dim();
+      a.q_norm = floats(layer.q_norm);
+      a.k_norm = floats(layer.k_norm);
+      a.eps = float(s.eps);
+      a.sink = m.sink ? float(m.sink_score) : -INFINITY;
+      a.gate_at = m.gate_at();
       a.value_is_key = m.value_is_key;
       a.window = m.window;
       a.keep = m.keep;
@@ -157,21 +193,61 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       TMB_TRY(RotateAppend(q, r, a));
       TMB_TRY(Attend(q, r, a));
     }
-    TMB_TRY(Linear(q, linear(plan->mixed, layer.out_weight, layer.out_bias, maps ? &maps->out : nullptr, W, m.out_columns(), x, W, kLinearAdd)));
-    if (layer.mlp.present) {
-      const Glu glu{float(layer.mlp.limit), float(layer.mlp.alpha), float(layer.mlp.shift)};
-      const int packed = layer.mlp.packed_rows(), mlp_stride = padded_columns(layer.mlp.ff);
-      TMB_TRY(norm(layer.norm2, false));
+    TMB_TRY(add_output(plan->mixed, layer.out_weight, layer.out_bias, maps ? &maps->out : nullptr, m.out_columns()));
+    if (norm_output) TMB_TRY(add_norm(layer.norm1, 0));
+    const RaggedMlp& mlp = layer.mlp;
+    if (mlp.kind == RaggedMlp::kGlu) {
+      const Glu glu{float(mlp.limit), float(mlp.alpha), float(mlp.shift), mlp.gelu};
+      const int packed = mlp.packed_rows(), mlp_stride = padded_columns(mlp.ff);
+      if (!norm_output) TMB_TRY(norm(layer.norm2, false));
       if (s.f32) {
         TMB_TRY(Linear(q, linear(plan->normed, layer.gate_up, -1, nullptr, packed, W, plan->pairs, packed, kLinearStore)));
-        TMB_TRY(GluRows(q, plan->pairs, plan->mlp, r.rows, packed, mlp_stride, layer.mlp.ff, glu));
+        TMB_TRY(GluRows(q, plan->pairs, plan->mlp, r.rows, packed, mlp_stride, mlp.ff, glu));
       } else {
         LinearArgs a = linear(plan->normed, layer.gate_up, -1, &maps->gate_up, packed, W, plan->mlp, mlp_stride, kLinearGlu);
-        a.outputs = layer.mlp.ff;
+        a.outputs = mlp.ff;
         a.glu = glu;
         TMB_TRY(Linear(q, a));
       }
-      TMB_TRY(Linear(q, linear(plan->mlp, layer.down, -1, maps ? &maps->down : nullptr, W, layer.mlp.ff, x, W, kLinearAdd)));
+      TMB_TRY(add_output(plan->mlp, layer.down, -1, maps ? &maps->down : nullptr, mlp.ff));
+      if (norm_output) TMB_TRY(add_norm(layer.norm2, 0));
+    } else if (mlp.kind == RaggedMlp::kExperts) {
+      ExpertSlots slots;
+      slots.tiles = plan->tiles;
+      slots.tile_count = plan->tile_count;
+      slots.list = plan->list;
+      slots.score = plan->slot_score;
+      slots.experts = mlp.experts;
+      slots.top = mlp.top;
+      slots.slots = r.rows * mlp.top;
+      slots.tile_rows = ExpertTileRows(q, slots.slots, slots.experts);
+      RouteArgs a{};
+      a.h = plan->normed;
+      a.router = buffer(layer.router);
+      a.k_stride = W8;
+      a.rows = r.rows;
+      a.experts = mlp.experts;
+      a.top = mlp.top;
+      a.tile_rows = slots.tile_rows;
+      a.logits = plan->logits;
+      a.choice = plan->choice;
+      a.score = plan->score;
+      a.list = plan->list;
+      a.slot_score = plan->slot_score;
+      a.tiles = plan->tiles;
+      a.tile_count = plan->tile_count;
+      a.count = plan->route_count;
+      if (!RouteFused(r.rows))
+        TMB_TRY(Linear(q, linear(plan->normed, layer.router, -1, maps ? &maps->router : nullptr, mlp.experts, W, plan->logits, mlp.experts, kLinearFloat)));
+      TMB_TRY(Route(q, a));
+      const int stride = padded_columns(mlp.ff);
+      LinearArgs up = linear(plan->normed, layer.expert_up, -1, maps ? &maps->gate_up : nullptr, mlp.ff, W, plan->expert_hidden, stride, kLinearExpertUp);
+      up.slots = slots;
+      TMB_TRY(Linear(q, up));
+      LinearArgs down = linear(plan->expert_hidden, layer.expert_down, -1, maps ? &maps->down : nullptr, W, mlp.ff, plan->expert_out, W, kLinearExpertDown);
+      down.slots = slots;
+      TMB_TRY(Linear(q, down));
+      TMB_TRY(add_norm(layer.norm2, mlp.top));
     }
     if (s.write_residuals) {
       const cudaError_t err = cudaMemcpyAsync(floats(s.residuals) + i * size_t(s.max_rows) * W, x, size_t(rows) * W * sizeof(float),
@@ -216,29 +292,40 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
   };
   const size_t element = spec.f32 ? 4 : 2;
   size_t proj = 0, mixed = 0, mlp = 0, pairs = 0, raw = 0, split = 0, heads = 1, partial = 0;
+  size_t top = 0, experts = 0, expert_columns = 0;
   for (const RaggedLayer& layer : spec.layers) {
     const RaggedMixer& m = layer.mixer;
     proj = std::max(proj, size_t(m.proj_rows() + 7) / 8 * 8);
     mixed = std::max(mixed, size_t(padded_columns(m.out_columns())));
-    if (layer.mlp.present) {
+    if (layer.mlp.kind == RaggedMlp::kGlu) {
       mlp = std::max(mlp, size_t(padded_columns(layer.mlp.ff)));
       pairs = std::max(pairs, size_t(layer.mlp.packed_rows()));
+    } else if (layer.mlp.kind == RaggedMlp::kExperts) {
+      top = std::max(top, size_t(layer.mlp.top));
+      experts = std::max(experts, size_t(layer.mlp.experts));
+      expert_columns = std::max(expert_columns, size_t(padded_columns(layer.mlp.ff)));
     }
     if (m.kind == RaggedMixer::kRetention) {
       raw = std::max(raw, size_t(m.out_columns()));
       split = std::max(split, size_t(m.heads) * 4 * m.pool_dim());
     } else {
       heads = std::max(heads, size_t(m.heads));
-      partial = std::max(partial, size_t(m.heads) * (m.dim + 2));
+      partial = std::max(partial, size_t(m.heads) * (m.vdim + 2));
     }
   }
-  const size_t rows = size_t(spec.max_rows), W8 = size_t(padded_columns(spec.width));
+  const size_t rows = size_t(spec.max_rows), W8 = size_t(padded_columns(spec.width)), slots = rows * top;
   plan->count_words = int(heads) * spec.slots;
   // a decode step cuts a long window into parts: at most eight CTAs per SM's worth of parts in all, one per head at least
   plan->part_floats = partial * (size_t(spec.slots) + 8 * size_t(sm_count));
   if (!Own(plan, &plan->normed, rows * W8 * element) || !Own(plan, &plan->picked, size_t(spec.max_wanted) * W8 * element) ||
       !Own(plan, &plan->proj, rows * proj * element) || !Own(plan, &plan->mixed, rows * mixed * element) ||
       !Own(plan, &plan->mlp, rows * mlp * element) || !Own(plan, &plan->pairs, spec.f32 ? rows * pairs * element : 0) ||
+      !Own(plan, &plan->branch, spec.layers[0].norm_output ? rows * size_t(spec.width) * sizeof(float) : 0) ||
+      !Own(plan, &plan->logits, rows * experts * sizeof(float)) || !Own(plan, &plan->choice, slots * sizeof(int)) ||
+      !Own(plan, &plan->list, slots * sizeof(int)) || !Own(plan, &plan->tile_count, sizeof(int)) ||
+      !Own(plan, &plan->score, slots * sizeof(float)) || !Own(plan, &plan->slot_score, slots * sizeof(float)) ||
+      !Own(plan, &plan->tiles, (slots / 16 + experts) * sizeof(ExpertTile)) || !Own(plan, &plan->route_count, sizeof(unsigned)) ||
+      !Own(plan, &plan->expert_hidden, slots * expert_columns * element) || !Own(plan, &plan->expert_out, slots * size_t(spec.width) * element) ||
       !Own(plan, &plan->raw, rows * raw * sizeof(float)) || !Own(plan, &plan->split, spec.f32 ? 0 : rows * split * 2) ||
       !Own(plan, &plan->part, plan->part_floats * sizeof(float)) ||
       !Own(plan, &plan->count, size_t(plan->count_words) * sizeof(unsigned)) || !Own(plan, &plan->queue.status, 64) ||
@@ -275,9 +362,15 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
       RaggedPlan::Maps& maps = plan->maps[i];
       bool ok = EncodeLinear(&maps.in, at(layer.in_weight), uint64_t(m.proj_rows()), plan->normed, rows, W8) &&
                 EncodeLinear(&maps.out, at(layer.out_weight), uint64_t(spec.width), plan->mixed, rows, uint64_t(padded_columns(m.out_columns())));
-      if (layer.mlp.present)
-        ok = ok && EncodeLinear(&maps.gate_up, at(layer.gate_up), uint64_t(layer.mlp.packed_rows()), plan->normed, rows, W8) &&
-             EncodeLinear(&maps.down, at(layer.down), uint64_t(spec.width), plan->mlp, rows, uint64_t(padded_columns(layer.mlp.ff)));
+      const RaggedMlp& mlp = layer.mlp;
+      if (mlp.kind == RaggedMlp::kExperts)
+        ok = ok && EncodeLinear(&maps.router, at(layer.router), uint64_t(mlp.experts), plan->normed, rows, W8) &&
+             EncodeLinear(&maps.gate_up, at(layer.expert_up), uint64_t(mlp.experts) * mlp.ff, plan->normed, rows, W8) &&
+             EncodeLinear(&maps.down, at(layer.expert_down), uint64_t(mlp.experts) * spec.width, plan->expert_hidden, slots,
+                          uint64_t(padded_columns(mlp.ff)));
+      if (mlp.kind == RaggedMlp::kGlu)
+        ok = ok && EncodeLinear(&maps.gate_up, at(layer.gate_up), uint64_t(mlp.packed_rows()), plan->normed, rows, W8) &&
+             EncodeLinear(&maps.down, at(layer.down), uint64_t(spec.width), plan->mlp, rows, uint64_t(padded_columns(mlp.ff)));
       if (!ok) return fail("cuTensorMapEncodeTiled rejected a layer's buffers");
     }
     if (!EncodeLinear(&plan->head, at(spec.head), uint64_t(spec.vocab), plan->picked, uint64_t(spec.max_wanted), W8))

@@ -33,6 +33,14 @@ std::string Name(const Json& object, const char* key) {
 
 std::string AliasRecipe(const std::string& name) { return "{\"kind\":\"alias\",\"source\":" + Json::Quote(name) + "}"; }
 
+std::string QuotedList(const Json& names, const char* key, int count) {
+  Require(names.has(key) && names.at(key).kind == Json::kArray && int(names.at(key).items.size()) == count,
+          std::string("a layer needs one tensor per expert for '") + key + "'");
+  std::string out = "[";
+  for (const Json& name : names.at(key).items) out += (out.size() > 1 ? "," : "") + Json::Quote(name.text);
+  return out + "]";
+}
+
 // Matrices stacked by rows, each row zero-padded to `columns`.
 std::string StackRecipe(const std::string& sources, int columns) {
   return "{\"kind\":\"pad_columns\",\"columns\":" + std::to_string(columns) + ",\"source\":{\"kind\":\"stack_rows\",\"sources\":" + sources + "}}";
@@ -109,14 +117,17 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     if (mixer.has("rotary") && mixer.at("rotary").kind == Json::kObject) {
       const Json& rot = mixer.at("rotary");
       const double base = rot.num("base", 0);
+      const double factor = rot.num("factor", 1);
       m.rot_dims = int(rot.integer("dims", 0));
+      Require(factor > 0, "the rotary scaling factor must be positive");
       Require(base > 0 && m.rot_dims >= 0 && m.rot_dims % 2 == 0 && m.rot_dims <= m.dim, "rotary dims must be even and at most the head size");
       if (m.rot_dims) {
         for (size_t r = 0; r < s.rotaries.size(); ++r)
-          if (s.rotaries[r].base == base && s.rotaries[r].dims == m.rot_dims) m.rotary = int(r);
+          if (s.rotaries[r].base == base && s.rotaries[r].dims == m.rot_dims && s.rotaries[r].factor == factor) m.rotary = int(r);
         if (m.rotary < 0) {
           RotaryTable table;
           table.base = base;
+          table.factor = factor;
           table.dims = m.rot_dims;
           m.rotary = int(s.rotaries.size());
           table.buffer = add("rotary." + std::to_string(m.rotary), 1, 1, uint64_t(s.capacity) * m.rot_dims, 0, "");
@@ -134,18 +145,33 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
       sources = Quoted(names, {"q", "k", "v", "g"});
     } else {
       m.value_is_key = mixer.str("values", "projected") == "keys";
-      Require(m.vdim == m.dim, "attention value heads are as wide as its key heads");
+      Require(m.vdim <= kMaxHeadDim, "head sizes must lie in [1, 256]");
+      Require(!m.value_is_key || m.vdim == m.dim, "values that are keys are as wide as keys");
+      m.qk_norm = mixer.flag("qk_norm", false);
+      m.gate = mixer.flag("gate", false);
+      m.sink = mixer.has("sink") && mixer.at("sink").kind == Json::kNumber;
+      m.sink_score = mixer.num("sink", 0);
       const Json none;
       const Json& mask = mixer.has("mask") && mixer.at("mask").kind == Json::kObject ? mixer.at("mask") : none;
       m.window = int(std::min<long long>(mask.integer("size", s.capacity), s.capacity));   // no window: everything before
       m.keep = int(std::min<long long>(mask.integer("keep_first", 0), s.capacity));
       m.scale = mixer.num("scale", 0);
       Require(m.window >= 1 && m.keep >= 0, "a window holds at least one position");
-      sources = m.value_is_key ? Quoted(names, {"q", "k"}) : Quoted(names, {"q", "k", "v"});
+      sources = m.value_is_key ? (m.gate ? Quoted(names, {"q", "k", "g"}) : Quoted(names, {"q", "k"}))
+                               : (m.gate ? Quoted(names, {"q", "k", "v", "g"}) : Quoted(names, {"q", "k", "v"}));
+      Require(!bias || !m.gate, "gated attention has no projection biases");
     }
+    const std::string place = in.str("norm_at", "input");
+    Require(place == "input" || place == "output", "a layer's norms act on its sublayers' input or output (norm_at)");
+    layer.norm_output = place == "output";
+    Require(i == 0 || layer.norm_output == s.layers[0].norm_output, "every layer of a model has its norms in the same place");
     layer.norm1 = add(p + "norm1", 1, 1, W, 0, AliasRecipe(Name(in, "norm1")));
     layer.in_weight = matrix(p + "in.weight", StackRecipe(sources, padded_columns(s.width)), m.proj_rows(), s.width);
     layer.out_weight = matrix(p + "out.weight", StackRecipe(Quoted(names, {"o"}), padded_columns(m.out_columns())), s.width, m.out_columns());
+    if (m.qk_norm) {
+      layer.q_norm = add(p + "q.norm", 1, 1, uint64_t(m.heads) * m.dim, 0, AliasRecipe(Name(names, "q.norm")));
+      layer.k_norm = add(p + "k.norm", 1, 1, uint64_t(m.kv_heads) * m.dim, 0, AliasRecipe(Name(names, "k.norm")));
+    }
     if (bias) {
       const std::string biases = m.value_is_key ? Quoted(names, {"q.b", "k.b"}) : Quoted(names, {"q.b", "k.b", "v.b"});
       layer.in_bias = add(p + "in.bias", 1, 1, uint64_t(m.proj_rows()), 0, "{\"kind\":\"concat\",\"sources\":" + biases + "}");
@@ -154,20 +180,39 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     if (in.has("mlp") && in.at("mlp").kind == Json::kObject) {
       const Json& mlp = in.at("mlp");
       const Json& parts = mlp.at("tensors");
-      Require(mlp.str("kind", "") == "glu", "unknown kind of feed-forward");
-      layer.mlp.present = true;
+      const std::string unit = mlp.str("kind", "");
+      Require(unit == "glu" || unit == "experts", "unknown kind of feed-forward");
+      layer.mlp.kind = unit == "glu" ? RaggedMlp::kGlu : RaggedMlp::kExperts;
       layer.mlp.ff = int(mlp.integer("ff", 0));
-      layer.mlp.limit = mlp.num("limit", 3.0e38);
-      layer.mlp.alpha = mlp.num("alpha", 1.0);
-      layer.mlp.shift = mlp.num("shift", 0.0);
       Require(layer.mlp.ff > 0, "the feed-forward width must be positive");
       layer.norm2 = add(p + "norm2", 1, 1, W, 0, AliasRecipe(Name(in, "norm2")));
-      layer.gate_up = matrix(p + "gate_up.weight",
-                             "{\"kind\":\"pad_columns\",\"columns\":" + std::to_string(padded_columns(s.width)) +
-                                 ",\"source\":{\"kind\":\"gate_up_interleave\",\"pad\":true,\"u\":" + std::to_string(kGluUnit) +
-                                 ",\"sources\":" + Quoted(parts, {"gate", "up"}) + "}}",
-                             layer.mlp.packed_rows(), s.width);
-      layer.down = matrix(p + "down.weight", StackRecipe(Quoted(parts, {"down"}), padded_columns(layer.mlp.ff)), s.width, layer.mlp.ff);
+      const std::string activation = mlp.str("activation", "silu");
+      if (layer.mlp.kind == RaggedMlp::kGlu) {
+        Require(activation == "silu" || activation == "gelu_tanh", "unknown activation of a gated unit");
+        layer.mlp.gelu = activation == "gelu_tanh";
+        layer.mlp.limit = mlp.num("limit", 3.0e38);
+        layer.mlp.alpha = mlp.num("alpha", 1.0);
+        layer.mlp.shift = mlp.num("shift", 0.0);
+        layer.gate_up = matrix(p + "gate_up.weight",
+                               "{\"kind\":\"pad_columns\",\"columns\":" + std::to_string(padded_columns(s.width)) +
+                                   ",\"source\":{\"kind\":\"gate_up_interleave\",\"pad\":true,\"u\":" + std::to_string(kGluUnit) +
+                                   ",\"sources\":" + Quoted(parts, {"gate", "up"}) + "}}",
+                               layer.mlp.packed_rows(), s.width);
+        layer.down = matrix(p + "down.weight", StackRecipe(Quoted(parts, {"down"}), padded_columns(layer.mlp.ff)), s.width, layer.mlp.ff);
+      } else {
+        RaggedMlp& e = layer.mlp;
+        e.experts = int(mlp.integer("experts", 0));
+        e.top = int(mlp.integer("top", 0));
+        Require(e.experts >= 1 && e.experts <= kMaxExperts, "a layer has 1..1024 experts");
+        Require(e.top >= 1 && e.top <= e.experts && e.top <= kMaxTop, "a token uses 1..32 of a layer's experts (top)");
+        Require(uint64_t(s.max_rows) * e.top <= (1u << 20), "max_rows times the experts of a token is at most 2^20");
+        Require(activation == "relu2" && mlp.str("scores", "") == "sigmoid" && mlp.str("weighted", "") == "input",
+                "experts use the square of relu, sigmoid scores and weights on their inputs");
+        Require(layer.norm_output, "expert layers need their norms on the sublayers' outputs");
+        layer.router = matrix(p + "router.weight", StackRecipe(Quoted(parts, {"router"}), padded_columns(s.width)), e.experts, s.width);
+        layer.expert_up = matrix(p + "experts.up", StackRecipe(QuotedList(parts, "up", e.experts), padded_columns(s.width)), e.experts * e.ff, s.width);
+        layer.expert_down = matrix(p + "experts.down", StackRecipe(QuotedList(parts, "down", e.experts), padded_columns(e.ff)), e.experts * s.width, e.ff);
+      }
     }
     s.layers.push_back(layer);
   }
@@ -181,12 +226,14 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     if (m.kind == RaggedMixer::kRetention) {
       run.state = add("retention." + at, 1, 1, 0, uint64_t(m.heads) * m.dim * m.vdim, "");
     } else {
-      const uint64_t pool = uint64_t(s.num_blocks) * m.kv_heads * kRaggedBlock * m.pool_dim();
-      run.k_pool = add("kv_pool.k." + at, 1, element, pool, 0, "");
-      run.v_pool = add("kv_pool.v." + at, 1, element, pool, 0, "");
+      const uint64_t rows = uint64_t(s.num_blocks) * m.kv_heads * kRaggedBlock;
+      run.k_pool = add("kv_pool.k." + at, 1, element, rows * m.pool_dim(), 0, "");
+      run.v_pool = add("kv_pool.v." + at, 1, element, rows * m.v_pool_dim(), 0, "");
     }
-    const RaggedGlu& mlp = s.layers[size_t(run.layer)].mlp;
-    s.weight_bytes += element_bytes * W * uint64_t(m.proj_rows() + m.out_columns() + (mlp.present ? 3 * mlp.ff : 0));
+    const RaggedMlp& mlp = s.layers[size_t(run.layer)].mlp;
+    Require(!run.add_embedding || !s.layers[size_t(run.layer)].norm_output, "layers with norms on their outputs are not looped");
+    const int mlp_rows = mlp.kind == RaggedMlp::kGlu ? 3 * mlp.ff : mlp.kind == RaggedMlp::kExperts ? 2 * mlp.top * mlp.ff + mlp.experts : 0;
+    s.weight_bytes += element_bytes * W * uint64_t(m.proj_rows() + m.out_columns() + mlp_rows);
     s.runs.push_back(run);
   }
   Require(!s.runs.empty(), "the model runs no layer");

@@ -1,6 +1,6 @@
 // Description of a ragged-step plan: a decoder given as a list of layers, each with its own kind of token mixer and
 // its own sizes, run in a given order (a layer may run several times). Read from the "model" object of the sidecar,
-// which serving/registry.py derives from a model's config.json.
+// which registry.py derives from a model's config.json.
 #pragma once
 #include <stdint.h>
 
@@ -19,31 +19,44 @@ struct RaggedMixer {
   int rot_dims = 0, rotary = -1;          // rotary: index into RaggedSpec::rotaries (-1: no rotation)
   // attention
   bool value_is_key = false;
+  bool qk_norm = false;                   // RMS norm over all query heads together, and over all key heads, before the rotation
+  bool gate = false;                      // the heads' outputs are multiplied by sigmoid of a projection of their own
+  bool sink = false;                      // a null key of score sink_score without a value joins every softmax
+  double sink_score = 0;
   int window = 0, keep = 0;
   double scale = 1.0;
   // retention
   std::vector<float> decay;
 
-  int proj_rows() const {                 // rows of the stacked input projection: q | k (| v), or q | k | v | g
+  int proj_rows() const {                 // rows of the stacked input projection: q | k (| v) (| g), or q | k | v | g
     if (kind == kRetention) return 2 * heads * dim + 2 * heads * vdim;
-    return heads * dim + kv_heads * dim * (value_is_key ? 1 : 2);
+    return (heads + kv_heads) * dim + (value_is_key ? 0 : kv_heads * vdim) + (gate ? heads * vdim : 0);
   }
+  int gate_at() const { return gate ? proj_rows() - heads * vdim : -1; }   // attention: first gate column of a projected row
   int out_columns() const { return heads * vdim; }
   int pool_dim() const { return (dim + 15) / 16 * 16; }
+  int v_pool_dim() const { return (vdim + 15) / 16 * 16; }
 };
 
-struct RaggedGlu {
-  bool present = false;
+struct RaggedMlp {
+  enum Kind { kNone, kGlu, kExperts };
+  Kind kind = kNone;
   int ff = 0;
+  // gated unit
+  bool gelu = false;                      // tanh form of GELU on the gate, else the clipped SiLU
   double limit = 0, alpha = 1, shift = 0;
   int packed_rows() const { return (ff + 15) / 16 * 32; }
+  // mixture of experts
+  int experts = 0, top = 0;
 };
 
 struct RaggedLayer {
   RaggedMixer mixer;
-  RaggedGlu mlp;
+  RaggedMlp mlp;
+  bool norm_output = false;               // the norms act on the sublayers' outputs; the sublayers read the stream itself
   // indices into the plan's buffer table
-  int norm1 = -1, in_weight = -1, in_bias = -1, out_weight = -1, out_bias = -1, norm2 = -1, gate_up = -1, down = -1, decay = -1;
+  int norm1 = -1, in_weight = -1, in_bias = -1, out_weight = -1, out_bias = -1, norm2 = -1, gate_up = -1, down = -1, decay = -1,
+      q_norm = -1, k_norm = -1, router = -1, expert_up = -1, expert_down = -1;
 };
 
 struct RaggedRun {
@@ -53,7 +66,7 @@ struct RaggedRun {
 };
 
 struct RotaryTable {
-  double base = 0;
+  double base = 0, factor = 1;
   int dims = 0, buffer = -1;
 };
 
@@ -70,7 +83,7 @@ struct RaggedSpec {
 
   // Fills the description and appends the plan's buffer table. Throws std::invalid_argument on anything unsupported.
   static RaggedSpec FromJson(const Json& plan, std::vector<BufferSpec>* buffers);
-  uint64_t weight_bytes = 0;              // matrices one step reads (every layer run, and the head)
+  uint64_t weight_bytes = 0;              // matrices a step of one token reads (every layer run, and the head)
 };
 
 inline int padded_columns(int k) { return (k + 7) / 8 * 8; }   // 16-byte rows for bf16

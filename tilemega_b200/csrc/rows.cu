@@ -1,5 +1,5 @@
-// Row operations of a ragged step: embedding and row tables, RMS norm over the fp32 residual stream, greedy sampling,
-// and the hand-over of sampled tokens to the next step.
+// Row operations of a ragged step: embedding and row tables, RMS norm over the fp32 residual stream and of what is added
+// to it, greedy sampling, and the hand-over of sampled tokens to the next step.
 #include <cuda_bf16.h>
 
 #include "element.cuh"
@@ -12,7 +12,8 @@ namespace {
 
 // One CTA per row. The row's entry is found by bisection over the entries' first rows (ascending, no gaps).
 template <typename T>
-__global__ void __launch_bounds__(256) start_step(StepRows r, const int* tokens, const T* embed, float* x, int width, int vocab) {
+__global__ void __launch_bounds__(256) start_step(StepRows r, const int* tokens, const T* embed, float* x, T* copy,
+                                                  int copy_stride, int width, int vocab) {
   const int row = blockIdx.x;
   dependency_wait();
   allow_dependents();
@@ -33,7 +34,11 @@ __global__ void __launch_bounds__(256) start_step(StepRows r, const int* tokens,
   }
   const int token = min(max(tokens[row], 0), vocab - 1);
 #pragma unroll 8
-  for (int i = threadIdx.x; i < width; i += 256) x[size_t(row) * width + i] = to_f(embed[size_t(token) * width + i]);
+  for (int i = threadIdx.x; i < width; i += 256) {
+    const T value = embed[size_t(token) * width + i];
+    x[size_t(row) * width + i] = to_f(value);
+    if (copy) copy[size_t(row) * copy_stride + i] = value;
+  }
 }
 
 template <typename T>
@@ -123,6 +128,100 @@ __global__ void __launch_bounds__(512) rms_norm_quads(NormArgs a) {
   }
 }
 
+// A sublayer's output normed and added to the stream, see AddNormArgs. QUADS: widths that are multiples of 4 up to 8192
+// (the row in registers); otherwise a thread forms the output's columns twice.
+template <typename T>
+__device__ __forceinline__ float branch_value(const AddNormArgs& a, int row, int c) {
+  if (a.parts == 0) return a.branch[size_t(row) * a.width + c];
+  const T* at = static_cast<const T*>(a.parts_of) + size_t(row) * a.parts * a.width + c;
+  float v = 0.f;
+  for (int k = 0; k < a.parts; ++k) v += to_f(at[size_t(k) * a.width]);
+  return v;
+}
+template <typename T> __device__ __forceinline__ float4 four(const T* at);
+template <> __device__ __forceinline__ float4 four<float>(const float* at) { return *reinterpret_cast<const float4*>(at); }
+template <> __device__ __forceinline__ float4 four<__nv_bfloat16>(const __nv_bfloat16* at) {
+  const uint2 w = *reinterpret_cast<const uint2*>(at);
+  return make_float4(bf_lo(w.x), bf_hi(w.x), bf_lo(w.y), bf_hi(w.y));
+}
+
+template <typename T, bool QUADS>
+__global__ void __launch_bounds__(512) add_norm(AddNormArgs a) {
+  __shared__ float part[16];
+  const int row = blockIdx.x, quads = a.width / 4;
+  float4 weight[kQuads], y[kQuads], x[kQuads];
+  if (QUADS) {
+#pragma unroll
+    for (int n = 0; n < kQuads; ++n) {
+      const int c = threadIdx.x + 512 * n;
+      if (c >= quads) continue;
+      weight[n] = reinterpret_cast<const float4*>(a.weight)[c];
+    }
+  }
+  dependency_wait();
+  allow_dependents();
+  float* line = a.x + size_t(row) * a.width;
+  float sq = 0.f;
+  if (QUADS) {
+#pragma unroll
+    for (int n = 0; n < kQuads; ++n) {
+      const int c = threadIdx.x + 512 * n;
+      y[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c >= quads) continue;
+      x[n] = reinterpret_cast<const float4*>(line)[c];
+      if (a.parts == 0) {
+        y[n] = reinterpret_cast<const float4*>(a.branch + size_t(row) * a.width)[c];
+      } else {
+        const T* at = static_cast<const T*>(a.parts_of) + size_t(row) * a.parts * a.width + 4 * c;
+#pragma unroll 8
+        for (int k = 0; k < a.parts; ++k) {
+          const float4 v = four<T>(at + size_t(k) * a.width);
+          y[n].x += v.x;
+          y[n].y += v.y;
+          y[n].z += v.z;
+          y[n].w += v.w;
+        }
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < kQuads; ++n) sq += y[n].x * y[n].x + y[n].y * y[n].y + y[n].z * y[n].z + y[n].w * y[n].w;
+  } else {
+    for (int c = threadIdx.x; c < a.width; c += 512) {
+      const float v = branch_value<T>(a, row, c);
+      sq = fmaf(v, v, sq);
+    }
+  }
+  sq = warp_sum(sq);
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = sq;
+  __syncthreads();
+  sq = 0.f;
+#pragma unroll
+  for (int w = 0; w < 16; ++w) sq += part[w];
+  const float inv = 1.f / sqrtf(sq / float(a.width) + a.eps);
+  T* out = static_cast<T*>(a.out) + size_t(row) * a.out_stride;
+  if (QUADS) {
+#pragma unroll
+    for (int n = 0; n < kQuads; ++n) {
+      const int c = threadIdx.x + 512 * n;
+      if (c >= quads) continue;
+      x[n].x += y[n].x * inv * weight[n].x;
+      x[n].y += y[n].y * inv * weight[n].y;
+      x[n].z += y[n].z * inv * weight[n].z;
+      x[n].w += y[n].w * inv * weight[n].w;
+      reinterpret_cast<float4*>(line)[c] = x[n];
+      alignas(16) T e[4] = {from_f<T>(x[n].x), from_f<T>(x[n].y), from_f<T>(x[n].z), from_f<T>(x[n].w)};
+      if (sizeof(T) == 2) reinterpret_cast<uint2*>(out)[c] = *reinterpret_cast<const uint2*>(e);
+      else reinterpret_cast<uint4*>(out)[c] = *reinterpret_cast<const uint4*>(e);
+    }
+  } else {
+    for (int c = threadIdx.x; c < a.width; c += 512) {
+      const float v = line[c] + branch_value<T>(a, row, c) * inv * a.weight[c];
+      line[c] = v;
+      out[c] = from_f<T>(v);
+    }
+  }
+}
+
 __global__ void __launch_bounds__(1024) arg_max(const float* logits, int vocab, int* next) {
   __shared__ float best_v[32];
   __shared__ int best_i[32];
@@ -186,10 +285,13 @@ __global__ void feed(Entry* entries, int count, const int* next, int* tokens, in
 
 }  // namespace
 
-int StartStep(const Queue& q, const StepRows& r, const int* tokens, const void* embed, float* x, int width, int vocab) {
+int StartStep(const Queue& q, const StepRows& r, const int* tokens, const void* embed, float* x, void* copy, int copy_stride, int width, int vocab) {
   const dim3 grid(unsigned(r.rows));
-  if (q.f32) return int(Launch(start_step<float>, grid, dim3(256), 0, q.stream, false, r, tokens, static_cast<const float*>(embed), x, width, vocab));
-  return int(Launch(start_step<__nv_bfloat16>, grid, dim3(256), 0, q.stream, false, r, tokens, static_cast<const __nv_bfloat16*>(embed), x, width, vocab));
+  if (q.f32)
+    return int(Launch(start_step<float>, grid, dim3(256), 0, q.stream, false, r, tokens, static_cast<const float*>(embed), x, static_cast<float*>(copy),
+                      copy_stride, width, vocab));
+  return int(Launch(start_step<__nv_bfloat16>, grid, dim3(256), 0, q.stream, false, r, tokens, static_cast<const __nv_bfloat16*>(embed), x,
+                    static_cast<__nv_bfloat16*>(copy), copy_stride, width, vocab));
 }
 
 int RmsNorm(const Queue& q, const NormArgs& a) {
@@ -200,6 +302,14 @@ int RmsNorm(const Queue& q, const NormArgs& a) {
   }
   auto kernel = q.f32 ? rms_norm<float> : rms_norm<__nv_bfloat16>;
   return int(Launch(kernel, dim3(unsigned(a.rows)), dim3(256), 0, q.stream, q.chained, a));
+}
+
+int AddNorm(const Queue& q, const AddNormArgs& a) {
+  if (a.rows <= 0) return 0;
+  const bool quads = a.width % 4 == 0 && a.width <= 512 * 4 * kQuads;
+  auto kernel = q.f32 ? (quads ? add_norm<float, true> : add_norm<float, false>)
+                      : (quads ? add_norm<__nv_bfloat16, true> : add_norm<__nv_bfloat16, false>);
+  return int(Launch(kernel, dim3(unsigned(a.rows)), dim3(512), 0, q.stream, q.chained, a));
 }
 
 int ArgMax(const Queue& q, const float* logits, int rows, int vocab, int* next) {

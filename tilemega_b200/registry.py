@@ -68,11 +68,48 @@ def bamudra_program(config: dict) -> dict:
             "head": "head", "layers": layers, "runs": looped_runs(len(layers), config.get("loop"))}
 
 
+def _nadilorn_mixer(kind: str, mixer: dict, prefix: str) -> dict:
+    if kind != "attention":
+        raise ValueError(f"unknown layer type {kind!r}")
+    rot = mixer.get("rot")
+    rotary = rot and {"base": rot["base"], "dims": rot["dims"], "factor": (rot.get("scaling") or {}).get("factor", 1.0)}
+    # queries and keys are normed before their rotation, the softmax has a null key of score 0, the heads' outputs a gate
+    return {"kind": kind, "heads": mixer["heads"], "kv_heads": mixer["kv_heads"], "dim": mixer["dim"], "vdim": mixer["vdim"],
+            "rotary": rotary, "mask": mixer.get("mask"), "scale": mixer["scale"], "values": "projected", "qk_norm": True, "sink": 0.0,
+            "gate": True, "tensors": _names(prefix, "q", "k", "v", "g", "o", "q.norm", "k.norm")}
+
+
+def _nadilorn_mlp(mlp: dict | None, prefix: str) -> dict | None:
+    if mlp is None:
+        return None
+    if mlp["kind"] == "dense":
+        return {"kind": "glu", "ff": mlp["ff"], "activation": "gelu_tanh", "tensors": _names(prefix, "gate", "up", "down")}
+    if mlp["kind"] != "moe":
+        raise ValueError(f"unknown feed-forward {mlp['kind']!r}")
+    count = int(mlp["router"]["experts"])
+    # a token's scores weigh the rows its experts read, as they are
+    return {"kind": "experts", "ff": mlp["expert"]["ff"], "experts": count, "top": mlp["router"]["top"], "activation": "relu2",
+            "scores": "sigmoid", "weighted": "input",
+            "tensors": {"router": prefix + "router"} | {part: [f"{prefix}e{expert}.{part}" for expert in range(count)] for part in ("up", "down")}}
+
+
+def nadilorn_program(config: dict) -> dict:
+    layers = []
+    for index, layer in enumerate(config["layers"]):
+        prefix = f"l{index}."
+        mlp = _nadilorn_mlp(layer.get("mlp"), prefix + "mlp.")
+        layers.append({"norm_at": "output", "norm1": prefix + "norm1", "mixer": _nadilorn_mixer(layer["type"], layer["mixer"], prefix + "mix."),
+                       "norm2": prefix + "norm2" if mlp else None, "mlp": mlp})
+    return {"width": config["width"], "vocab": config["vocab"], "eps": config["norm"]["eps"], "embed": "embed", "final_norm": "final.norm",
+            "head": "head", "layers": layers, "runs": looped_runs(len(layers), None)}
+
+
 FAMILIES = {
     "LlamaForCausalLM": Family("llama", ("decode", "prefill")),
     "Qwen3MoeForCausalLM": Family("qwen3-moe", ("decode",)),
     "BertModel": Family("bert", ("forward",)),
     "Bamudra": Family("bamudra", ("ragged",), bamudra_program),
+    "Nadilorn": Family("nadilorn", ("ragged",), nadilorn_program),
 }
 
 
@@ -110,13 +147,20 @@ def tensor_shapes(config: dict) -> dict[str, tuple[int, ...]]:
         sizes = {"q": q, "k": k, "v": mixer.get("kv_heads", mixer["heads"]) * mixer["vdim"], "g": out}
         shapes[layer["norm1"]] = (width,)
         for part, name in names.items():
-            if part.endswith(".b"):
+            if part.endswith(".norm"):
+                shapes[name] = (sizes[part[:-5]],)
+            elif part.endswith(".b"):
                 shapes[name] = (width if part == "o.b" else sizes[part[:-2]],)
             else:
                 shapes[name] = (width, out) if part == "o" else (sizes[part], width)
         if layer["mlp"]:
             ff, parts = layer["mlp"]["ff"], layer["mlp"]["tensors"]
-            shapes |= {layer["norm2"]: (width,), parts["gate"]: (ff, width), parts["up"]: (ff, width), parts["down"]: (width, ff)}
+            shapes[layer["norm2"]] = (width,)
+            if layer["mlp"]["kind"] == "experts":
+                shapes[parts["router"]] = (layer["mlp"]["experts"], width)
+                shapes |= {name: (ff, width) for name in parts["up"]} | {name: (width, ff) for name in parts["down"]}
+            else:
+                shapes |= {parts["gate"]: (ff, width), parts["up"]: (ff, width), parts["down"]: (width, ff)}
     shapes[program["final_norm"]] = (width,)
     shapes[program["head"]] = (program["vocab"], width)
     return shapes

@@ -79,10 +79,10 @@ def rotary_tables(config: dict, capacity: int, device: torch.device | str) -> tu
             table.sin().to(torch.bfloat16).to(device).contiguous())
 
 
-def rotary_pairs(base: float, dims: int, capacity: int) -> torch.Tensor:
-    """fp32 [capacity][dims/2][2]: cosine and sine of position * base^(-2i/dims) for the pairs of a rotate-half
+def rotary_pairs(base: float, dims: int, capacity: int, factor: float = 1.0) -> torch.Tensor:
+    """fp32 [capacity][dims/2][2]: cosine and sine of position * base^(-2i/dims) / factor for the pairs of a rotate-half
     rotation, the angles taken in float64."""
-    frequency = base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    frequency = base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims) / factor
     angles = torch.arange(capacity, dtype=torch.float64)[:, None] * frequency[None, :]
     return torch.stack((angles.cos(), angles.sin()), dim=-1).float()
 
@@ -200,15 +200,16 @@ def allocate_ragged_state(ragged: PlanLibrary, device: str | torch.device = "cud
     tables = []
     for layer in model["layers"]:
         rot = layer["mixer"].get("rotary")
-        if rot and rot["dims"] and (rot["base"], rot["dims"]) not in tables:
-            tables.append((rot["base"], rot["dims"]))
+        if rot and rot["dims"] and (rot["base"], rot["dims"], rot.get("factor", 1.0)) not in tables:
+            tables.append((rot["base"], rot["dims"], rot.get("factor", 1.0)))
     result = {}
     for buffer in ragged.buffers:
         if buffer.role != 1 or buffer.pack_json:
             continue
         count = buffer.elements_constant + slots * buffer.elements_per_batch
         if buffer.name.startswith("rotary."):
-            tensor = rotary_pairs(*tables[int(buffer.name.split(".")[1])], capacity).to(device).reshape(-1).contiguous()
+            base, dims, factor = tables[int(buffer.name.split(".")[1])]
+            tensor = rotary_pairs(base, dims, capacity, factor).to(device).reshape(-1).contiguous()
         else:
             tensor = torch.zeros(count, dtype={0: torch.bfloat16, 1: torch.float32, 2: torch.int32}[buffer.dtype], device=device)
         if tensor.numel() != count:
