@@ -69,7 +69,9 @@ def measured_peak_gbs() -> tuple[float, str]:
 MODELS = {"llama-3.1-8b": synthetic.LLAMA_3_1_8B, "llama-3.2-1b": synthetic.LLAMA_3_2_1B,
           "llama-3.1-70b": synthetic.LLAMA_3_1_70B, "qwen3-30b-a3b": synthetic.QWEN3_30B_A3B,
           "bert-base": synthetic.BERT_BASE,   # the encoder forward workload (run_forward)
-          "bamudra-8b": synthetic.BAMUDRA_8B, "bamudra-1b": synthetic.BAMUDRA_1B}   # ragged-step plans (run_ragged)
+          "bamudra-8b": synthetic.BAMUDRA_8B, "bamudra-1b": synthetic.BAMUDRA_1B,   # ragged-step plans (run_ragged)
+          "nadilorn-8b": synthetic.NADILORN_8B, "nadilorn-1b": synthetic.NADILORN_1B, "nadilorn-30b-a3b": synthetic.NADILORN_30B_A3B}
+LAYERED = ("bamudra", "nadilorn")   # decoders given as a list of layers
 
 
 def workload(args) -> dict:
@@ -497,8 +499,8 @@ def run_forward(args) -> None:
 
 
 def run_ragged(args) -> None:
-    """Secondary workload: a Bamudra-shaped decoder (`--model bamudra-8b | bamudra-1b`) through a ragged-step plan (phase 3
-    of the plan ABI). Decode: `--batch` sequences at `--context` positions, one step = one decoded token of each, the
+    """Secondary workload: a decoder given as a list of layers (`--model bamudra-8b | bamudra-1b | nadilorn-8b | nadilorn-1b |
+    nadilorn-30b-a3b`) through a ragged-step plan (phase 3 of the plan ABI). Decode: `--batch` sequences at `--context` positions, one step = one decoded token of each, the
     sampled tokens fed back on the device. `--prefill T`: a prompt of T tokens in portions of `--portion` rows, one step =
     one portion. One JSON line in the shape of the decode line; same weights, widths and vocabulary as the Llama-shaped
     model of the same name, so the two lines stand side by side."""
@@ -534,19 +536,25 @@ def run_ragged(args) -> None:
     runs = executor.library.manifest["model"]["runs"]
     state_bytes = sum(2 * 4 * m["heads"] * m["dim"] * m["vdim"] for m in (config["layers"][run["layer"]]["mixer"] for run in runs) if "decay" in m)
 
+    attention = [mixer for mixer in (config["layers"][run["layer"]]["mixer"] for run in runs) if "mask" in mixer]
+
+    def seen(mixer: dict, position: int) -> int:
+        size, keep = mixer["mask"]["size"], mixer["mask"].get("keep_first", 0)
+        return min(position + 1, size) + min(keep, max(0, position + 1 - size))
+
     def cached(position: int) -> int:
         """Bytes of keys and values one token at this position reads, all attention layers."""
-        total = 0
-        for run in runs:
-            mixer = config["layers"][run["layer"]]["mixer"]
-            if "mask" in mixer:
-                size, keep = mixer["mask"]["size"], mixer["mask"]["keep_first"]
-                seen = min(position + 1, size) + min(keep, max(0, position + 1 - size))
-                total += seen * 2 * 2 * mixer["kv_heads"] * mixer["dim"]
-        return total
+        return sum(seen(mixer, position) * 2 * mixer["kv_heads"] * (mixer["dim"] + mixer["vdim"]) for mixer in attention)
+
+    def attention_flops(position: int) -> int:
+        return sum(seen(mixer, position) * 2 * mixer["heads"] * (mixer["dim"] + mixer["vdim"]) for mixer in attention)
 
     weight_bytes = executor.plan.step_bytes(0)
-    weight_elements = weight_bytes // 2
+    weight_elements = weight_bytes // 2                          # of one token: its own experts
+    mixtures = [layer["mlp"] for layer in config["layers"] if layer["mlp"] and layer["mlp"]["kind"] == "moe"]
+    for mlp in mixtures:                                         # experts a batch reads, if its tokens spread evenly
+        experts, top = mlp["router"]["experts"], mlp["router"]["top"]
+        weight_bytes += round(2 * 2 * width * mlp["expert"]["ff"] * (experts * (1.0 - (1.0 - top / experts) ** batch) - top))
     peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
     if args.prefill:
         prompt = synthetic.seeded_tokens(1, context, vocab, seed=3)[0].tolist()
@@ -578,7 +586,7 @@ def run_ragged(args) -> None:
         head_elements = vocab * width
         flops = 2.0 * (context * (weight_elements - head_elements) + head_elements)
         for position in range(context):
-            flops += cached(position) / 4 * 4 * (config["layers"][1]["mixer"]["heads"] / config["layers"][1]["mixer"]["kv_heads"]) / 2
+            flops += attention_flops(position)
         flops += context * 4.0 * state_bytes / 8
         peak = float(peaks.get("bf16_tflops", 1590.0))
         steps_run = -(-context // portion)
@@ -840,7 +848,7 @@ def main() -> None:
                         help="--model bert-base: element type of the forward plan (f16: the benchmark configuration; bf16: what the reference's export runs)")
     parser.add_argument("--prefill", type=int, default=0,
                         help="secondary workload: chunked prefill of one prompt of this many tokens (one GPU)")
-    parser.add_argument("--portion", type=int, default=2048, help="--model bamudra-*: rows per step of a prefilled prompt")
+    parser.add_argument("--portion", type=int, default=2048, help="--model bamudra-* / nadilorn-*: rows per step of a prefilled prompt")
     parser.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     parser.add_argument("--trace", action="store_true",
                         help="after the timed runs, stamp one more step and print the per-stage table (rank 0)")
@@ -848,7 +856,7 @@ def main() -> None:
                         help="several GPUs: independent copies of the one-GPU workload instead of one sharded model")
     parser.add_argument("--tp", action="store_true", help="accepted for compatibility: several GPUs shard one model by default")
     args = parser.parse_args()
-    if args.impl == "reference" and (args.model or "").startswith("bamudra"):
+    if args.impl == "reference" and (args.model or "").startswith(LAYERED):
         print(json.dumps({"impl": "reference", "unavailable": "the reference has no model of this design"}), flush=True)
     elif args.impl == "reference" and args.model == "bert-base":
         run_forward_reference(args)
@@ -856,7 +864,7 @@ def main() -> None:
         run_reference(args)
     elif args.model == "bert-base":
         run_forward(args)
-    elif (args.model or "").startswith("bamudra"):
+    elif (args.model or "").startswith(LAYERED):
         run_ragged(args)
     elif args.prefill:
         run_prefill(args)

@@ -217,6 +217,24 @@ BAMUDRA_8B = bamudra_config(4096, 32, 8, 128, 14336, 32, 128256, 2048, 4)
 BAMUDRA_1B = bamudra_config(2048, 32, 8, 64, 8192, 16, 128256, 1024, 4)
 
 
+# Nadilorn-shaped decoders with the layer sizes of the models above: windowed attention in every layer; the first two with
+# gated units throughout, the third with a gated unit in the first layer and mixtures of experts behind it (an expert has
+# two matrices where Qwen3's has three, so its width is half as large again).
+def nadilorn_config(width: int, heads: int, kv_heads: int, dim: int, ff: int, layers: int, vocab: int, window: int,
+                    experts: int = 0, top: int = 0, expert_ff: int = 0) -> dict:
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window},
+             "rot": {"base": 500000.0, "dims": dim // 2, "scaling": {"factor": 4.0}}}
+    dense = {"kind": "dense", "ff": ff}
+    mixture = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": expert_ff}} if experts else dense
+    order = [{"type": "attention", "mixer": mixer, "mlp": mixture if index else dense} for index in range(layers)]
+    return {"architecture": "Nadilorn", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "layers": order}
+
+
+NADILORN_8B = nadilorn_config(4096, 32, 8, 128, 14336, 32, 128256, 2048)
+NADILORN_1B = nadilorn_config(2048, 32, 8, 64, 8192, 16, 128256, 1024)
+NADILORN_30B_A3B = nadilorn_config(2048, 32, 4, 128, 6144, 48, 151936, 2048, 128, 8, 1152)
+
+
 class LazyShapedCheckpoint:
     """Like LazySeededCheckpoint for any table of tensor shapes (registry.tensor_shapes): matrices N(0, std), norm
     weights 1, biases N(0, std), each tensor from its own generator when it is asked for."""
