@@ -31,48 +31,83 @@ template <> __device__ __forceinline__ float dot16<float>(const uint4& a, const 
   return fmaf(__uint_as_float(a.w), __uint_as_float(b.w), sum);
 }
 
-// The warp's row: its `top` largest logits in falling order, the smaller index first where two are equal. Every turn
-// takes the largest of those behind the one before it in that order.
-__device__ __forceinline__ void choose(const RouteArgs& a, int row, int lane) {
+// Floats as unsigned integers of the same order.
+__device__ __forceinline__ unsigned ordered(float v) {
+  const unsigned u = __float_as_uint(v);
+  return u & 0x80000000u ? ~u : u | 0x80000000u;
+}
+
+// The warp's row: its `top` largest logits in falling order, the smaller index first where two are equal. HELD: up to
+// 32 * kMine experts, a lane keeps its own in registers and strikes out what was taken; otherwise every turn takes the
+// largest of those behind the one before it in that order.
+constexpr int kMine = 8;
+template <bool HELD> __device__ __forceinline__ void choose(const RouteArgs& a, int row, int lane) {
   const float* z = a.logits + size_t(row) * a.experts;
-  float before = INFINITY;
+  unsigned key[kMine];
+  if (HELD)
+#pragma unroll
+    for (int i = 0; i < kMine; ++i) key[i] = lane + 32 * i < a.experts ? max(ordered(__ldcg(z + lane + 32 * i)), 1u) : 0u;   // 0: taken, or none
+  unsigned before = 0xffffffffu;
   int before_at = -1;
   for (int k = 0; k < a.top; ++k) {
-    float best = -INFINITY;
+    unsigned best = 0u;
     int at = 0x7fffffff;
-    for (int e = lane; e < a.experts; e += 32) {
-      const float v = __ldcg(z + e);
-      if (v > before || (v == before && e <= before_at)) continue;
-      if (v > best || at == 0x7fffffff) {
-        best = v;
-        at = e;
-      }
-    }
+    if (HELD) {
 #pragma unroll
-    for (int o = 16; o; o >>= 1) {
-      const float v = __shfl_xor_sync(0xffffffffu, best, o);
-      const int i = __shfl_xor_sync(0xffffffffu, at, o);
-      if (v > best || (v == best && i < at)) {
-        best = v;
-        at = i;
+      for (int i = 0; i < kMine; ++i)
+        if (key[i] > best) {
+          best = key[i];
+          at = lane + 32 * i;
+        }
+    } else {
+      for (int e = lane; e < a.experts; e += 32) {
+        const unsigned v = max(ordered(__ldcg(z + e)), 1u);
+        if (v > before || (v == before && e <= before_at)) continue;
+        if (v > best) {
+          best = v;
+          at = e;
+        }
       }
     }
-    at = min(at, a.experts - 1);      // (logits that are not numbers: any expert, but a valid one)
-    if (lane == 0) {
-      a.choice[row * a.top + k] = at;
-      a.score[row * a.top + k] = 1.f / (1.f + expf(-best));
+    const unsigned high = __reduce_max_sync(0xffffffffu, best);
+    at = __reduce_min_sync(0xffffffffu, best == high ? at : 0x7fffffff);
+    if (HELD) {
+#pragma unroll
+      for (int i = 0; i < kMine; ++i)
+        if (at == lane + 32 * i) key[i] = 0u;
     }
-    before = best;
+    before = high;
     before_at = at;
+    if (lane == 0) {
+      at = min(at, a.experts - 1);
+      a.choice[row * a.top + k] = at;
+      a.score[row * a.top + k] = 1.f / (1.f + expf(-__ldcg(z + at)));
+    }
   }
+}
+__device__ __forceinline__ void choose(const RouteArgs& a, int row, int lane) {
+  if (a.experts <= 32 * kMine) choose<true>(a, row, lane);
+  else choose<false>(a, row, lane);
 }
 
 // The step's assignments sorted by expert, by one CTA. `first` holds every expert's first slot, then its next free one.
 __device__ __forceinline__ void sort_assignments(const RouteArgs& a, int* counts, int* first) {
+  constexpr int U = 8;                  // assignments a thread has in flight
   const int n = a.rows * a.top, threads = blockDim.x, lane = threadIdx.x & 31;
+  int choice[U];
+  auto load = [&](int base) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) choice[u] = base + u * threads < n ? __ldcg(a.choice + base + u * threads) : -1;
+  };
+  load(threadIdx.x);
   for (int e = threadIdx.x; e < a.experts; e += threads) counts[e] = 0;
   __syncthreads();
-  for (int i = threadIdx.x; i < n; i += threads) atomicAdd(&counts[__ldcg(a.choice + i)], 1);
+  for (int base = threadIdx.x; base < n; base += U * threads) {
+    if (base >= U * threads) load(base);
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (choice[u] >= 0) atomicAdd(&counts[choice[u]], 1);
+  }
   __syncthreads();
   if (threadIdx.x < 32) {
     int slots = 0, tiles = 0;
@@ -98,15 +133,35 @@ __device__ __forceinline__ void sort_assignments(const RouteArgs& a, int* counts
   }
   __syncthreads();
   // (the order of an expert's slots is whatever the counters make it: every slot is computed by itself)
-  for (int i = threadIdx.x; i < n; i += threads) {
-    const int slot = atomicAdd(&first[__ldcg(a.choice + i)], 1);
-    a.list[slot] = i;
-    a.slot_score[slot] = __ldcg(a.score + i);
+  for (int base = threadIdx.x; base < n; base += U * threads) {
+    if (n > U * threads) load(base);
+    float score[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) score[u] = choice[u] >= 0 ? __ldcg(a.score + base + u * threads) : 0.f;
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (choice[u] < 0) continue;
+      const int slot = atomicAdd(&first[choice[u]], 1);
+      a.list[slot] = base + u * threads;
+      a.slot_score[slot] = score[u];
+    }
   }
 }
 
-// FUSED: a warp takes one expert and runs its router row over all rows; the last CTA chooses and sorts. Otherwise the
-// logits are there and a warp takes one row; the last CTA sorts.
+// True for the CTA that arrives last of `of`; the counter is left at zero. Every thread takes part.
+__device__ __forceinline__ bool arrives_last(unsigned* counter, unsigned of, unsigned* flag) {
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    *flag = atom_acq_rel_add(counter, 1u) == of - 1 ? 1u : 0u;
+    if (*flag) *counter = 0;
+  }
+  __syncthreads();
+  return *flag != 0;
+}
+
+// FUSED: blockIdx = (eight experts, eight rows); a warp runs its expert's router row over the rows, the last CTA of the
+// rows chooses, a warp a row, and the last of all sorts. Otherwise the logits are there, a warp chooses for one row, and
+// the last CTA sorts.
 template <typename T, bool FUSED>
 __global__ void __launch_bounds__(FUSED ? 256 : 1024) route(RouteArgs a) {
   __shared__ int counts[kMaxExperts], first[kMaxExperts];
@@ -114,7 +169,7 @@ __global__ void __launch_bounds__(FUSED ? 256 : 1024) route(RouteArgs a) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   if constexpr (FUSED) {
     constexpr int N = 16 / sizeof(T);
-    const int e = blockIdx.x * warps + warp, pieces = a.k_stride / N;
+    const int e = blockIdx.x * 8 + warp, pieces = a.k_stride / N, row0 = blockIdx.y * 8, rows = min(8, a.rows - row0);
     const uint4* w = reinterpret_cast<const uint4*>(static_cast<const T*>(a.router) + size_t(min(e, a.experts - 1)) * a.k_stride);
     uint4 held[kHeld];
 #pragma unroll
@@ -122,36 +177,44 @@ __global__ void __launch_bounds__(FUSED ? 256 : 1024) route(RouteArgs a) {
     dependency_wait();
     allow_dependents();
     if (e < a.experts)
-      for (int row = 0; row < a.rows; ++row) {
+      for (int row = row0; row < row0 + rows; ++row) {
         const uint4* h = reinterpret_cast<const uint4*>(static_cast<const T*>(a.h) + size_t(row) * a.k_stride);
+        uint4 x[kHeld];
+#pragma unroll
+        for (int i = 0; i < kHeld; ++i) x[i] = lane + 32 * i < pieces ? h[lane + 32 * i] : make_uint4(0, 0, 0, 0);
         float sum = 0.f;
 #pragma unroll
-        for (int i = 0; i < kHeld; ++i)
-          if (lane + 32 * i < pieces) sum += dot16<T>(h[lane + 32 * i], held[i]);
+        for (int i = 0; i < kHeld; ++i) sum += dot16<T>(x[i], held[i]);
         for (int i = lane + 32 * kHeld; i < pieces; i += 32) sum += dot16<T>(h[i], w[i]);
         sum = warp_sum(sum);
         if (lane == 0) a.logits[size_t(row) * a.experts + e] = sum;
       }
+    if (!arrives_last(a.count + 1 + blockIdx.y, gridDim.x, &last)) return;
+    if (warp < rows) choose(a, row0 + warp, lane);
+    if (gridDim.y == 1) __syncthreads();
+    else if (!arrives_last(a.count, gridDim.y, &last)) return;
   } else {
     dependency_wait();
     allow_dependents();
     const int row = blockIdx.x * warps + warp;
     if (row < a.rows) choose(a, row, lane);
-  }
-  __syncthreads();
-  if (threadIdx.x == 0) last = atom_acq_rel_add(a.count, 1u) == gridDim.x - 1 ? 1u : 0u;
-  __syncthreads();
-  if (!last) return;
-  if (threadIdx.x == 0) *a.count = 0;   // for the next launch
-  if constexpr (FUSED) {
-    for (int row = warp; row < a.rows; row += warps) choose(a, row, lane);
-    __syncthreads();
+    if (!arrives_last(a.count, gridDim.x, &last)) return;
   }
   sort_assignments(a, counts, first);
 }
 
+// out[slot] = h[list[slot] / top], 16 bytes a thread.
+__global__ void __launch_bounds__(256) gather_rows(const uint4* h, const int* list, int top, uint4* out, int pieces) {
+  dependency_wait();
+  allow_dependents();
+  const size_t slot = blockIdx.x;
+  const uint4* from = h + size_t(list[slot] / top) * pieces;
+  for (int i = threadIdx.x; i < pieces; i += 256) out[slot * pieces + i] = from[i];
+}
+
 template <typename T> int RouteAs(const Queue& q, const RouteArgs& a) {
-  if (RouteFused(a.rows)) return int(Launch(route<T, true>, dim3(unsigned((a.experts + 7) / 8)), dim3(256), 0, q.stream, q.chained, a));
+  if (RouteFused(a.rows))
+    return int(Launch(route<T, true>, dim3(unsigned((a.experts + 7) / 8), unsigned((a.rows + 7) / 8)), dim3(256), 0, q.stream, q.chained, a));
   return int(Launch(route<T, false>, dim3(unsigned((a.rows + 31) / 32)), dim3(1024), 0, q.stream, q.chained, a));
 }
 
@@ -163,6 +226,12 @@ int Route(const Queue& q, const RouteArgs& a) {
   if (a.rows <= 0) return 0;
   if (a.experts > kMaxExperts || a.top > a.experts || a.tile_rows < 1 || a.k_stride % 8) return int(cudaErrorInvalidValue);
   return q.f32 ? RouteAs<float>(q, a) : RouteAs<__nv_bfloat16>(q, a);
+}
+
+int GatherRows(const Queue& q, const void* h, int k_stride, const ExpertSlots& slots, void* out) {
+  if (q.f32 || slots.slots <= 0) return q.f32 ? int(cudaErrorInvalidValue) : 0;
+  return int(Launch(gather_rows, dim3(unsigned(slots.slots)), dim3(256), 0, q.stream, q.chained, static_cast<const uint4*>(h), slots.list, slots.top,
+                    static_cast<uint4*>(out), k_stride / 8));
 }
 
 }  // namespace tmb

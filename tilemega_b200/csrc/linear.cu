@@ -35,7 +35,7 @@ struct LinearParams {
 };
 
 // Which products read gathered rows, and which run per expert.
-__host__ __device__ constexpr bool Gathers(int epilogue) { return epilogue == kLinearExpertUp; }
+__host__ __device__ constexpr bool Gathers(int epilogue, int tokens) { return epilogue == kLinearExpertUp && tokens <= kGatherRows; }
 __host__ __device__ constexpr bool PerExpert(int epilogue) { return epilogue == kLinearExpertUp || epilogue == kLinearExpertDown; }
 
 template <int BN> struct LinearShape {
@@ -84,9 +84,10 @@ template <int EPI> __device__ __forceinline__ void emit(const LinearParams& g, i
 }
 
 // blockIdx = (token tile, weight tile, K split): CTAs that run together share weight tiles, so a prompt's weights are read
-// once while its activations stay in L2. The CTAs of one (weight, token) tile form a cluster along z. Per expert, token
+// once while its activations stay in L2. The CTAs of one (weight, token) tile form a cluster along z. Per expert the
+// first two axes change places (an expert's weights are read by few tiles, its tokens by all of its weight tiles), token
 // tiles are those of the slot table (the grid holds as many as there could be), tokens are slots, and weight tiles start at
-// the expert's rows; rows beyond the tile's slots belong to other experts and are dropped.
+// the expert's rows; what a tile computes beyond its slots or its expert's rows is dropped.
 template <int BN, int EPI>
 __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap tmap,
                                                                const LinearParams g) {
@@ -99,20 +100,27 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
   uint64_t* accum = empty + S;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(accum + 1);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n0 = blockIdx.y * kRowsM;
-  int t0 = blockIdx.x * BN, t_end = g.t, weight_row = n0;
+  const int n0 = (PerExpert(EPI) ? blockIdx.x : blockIdx.y) * kRowsM, token_tile = PerExpert(EPI) ? blockIdx.y : blockIdx.x;
+  int t0 = token_tile * BN, t_end = g.t, weight_row = n0;
+  // per expert only the tokens there are cost anything: wide tiles load them 32 rows at a time
+  constexpr bool kGather = Gathers(EPI, BN);
+  constexpr int kBoxes = PerExpert(EPI) && BN > 32 ? BN / 32 : 1;
+  int columns = BN, boxes = kBoxes;
   if constexpr (PerExpert(EPI)) {
-    // ExpertUp follows the kernel that writes the table; for ExpertDown it is there before the wait
-    if (Gathers(EPI)) dependency_wait();
-    if (int(blockIdx.x) >= *g.slots.tile_count) {
-      if (!Gathers(EPI)) dependency_wait();
+    // a product that gathers follows the kernel that writes the table; for the others it is there before the wait
+    if (kGather) dependency_wait();
+    const ExpertTile tile = g.slots.tiles[token_tile];
+    if (token_tile >= *g.slots.tile_count) {
+      if (!kGather) dependency_wait();
       return;
     }
-    const ExpertTile tile = g.slots.tiles[blockIdx.x];
     t0 = tile.first;
     t_end = tile.first + min(tile.count, BN);
     weight_row = tile.expert * g.n + n0;
+    columns = (t_end - t0 + 15) / 16 * 16;
+    if (kBoxes > 1) boxes = (t_end - t0 + 31) / 32;
   }
+  const uint32_t stage_bytes = uint32_t(kWeightBytes + boxes * (Shape::kTokenBytes / kBoxes));
   const int splits = gridDim.z;
   const int c0 = blockIdx.z * g.chunks_per_split;
   const int chunks = max(0, min(g.chunks_per_split, g.chunks - c0));
@@ -135,20 +143,15 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
   const int early = chunks < S ? chunks : S;
   if (threadIdx.x == 0)
     for (int c = 0; c < early; ++c) {   // weights do not depend on the kernel before this one
-      mbar_expect_tx(&full[c], Shape::kStageBytes);
+      mbar_expect_tx(&full[c], stage_bytes);
       tma_load_2d(tiles + c * Shape::kStageBytes, &wmap, (c0 + c) * kStepK, weight_row, &full[c]);
     }
-  if (!Gathers(EPI)) dependency_wait();
+  if (!kGather) dependency_wait();
 
-  if (Gathers(EPI) && warp == 0) {
-    // every lane fetches four rows of the tile (BN = 256: eight)
-    constexpr int Q = BN == 256 ? 2 : 1;
-    int rows[Q][4];
+  if (kGather && warp == 0) {
+    int rows[4];                                        // every lane of the first BN / 4 fetches four rows of the tile
 #pragma unroll
-    for (int i = 0; i < 4 * Q; ++i) {
-      const int slot = min(t0 + (i / 4) * 128 + lane * 4 + i % 4, t_end - 1);
-      rows[i / 4][i % 4] = g.slots.list[slot] / g.slots.top;
-    }
+    for (int i = 0; i < 4; ++i) rows[i] = g.slots.list[min(t0 + lane * 4 + i, t_end - 1)] / g.slots.top;
     int issued = 0;
     bool ok = true;
     for (int c = 0; c < chunks; ++c) {
@@ -157,13 +160,11 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
       if (!ok) break;
       unsigned char* w = tiles + s * Shape::kStageBytes;
       if (lane == 0 && c >= early) {
-        mbar_expect_tx(&full[s], Shape::kStageBytes);
+        mbar_expect_tx(&full[s], stage_bytes);
         tma_load_2d(w, &wmap, (c0 + c) * kStepK, weight_row, &full[s]);
       }
       __syncwarp();
-#pragma unroll
-      for (int i = 0; i < Q; ++i)
-        if (lane < BN / 4) tma_gather_rows(w + kWeightBytes + (i * 32 + lane) * 4 * kStepK * 2, &tmap, (c0 + c) * kStepK, rows[i], &full[s]);
+      if (lane < BN / 4) tma_gather_rows(w + kWeightBytes + lane * 4 * kStepK * 2, &tmap, (c0 + c) * kStepK, rows, &full[s]);
       issued = c + 1;
     }
     if (!ok)
@@ -178,10 +179,12 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
         if (!ok) break;
         unsigned char* w = tiles + s * Shape::kStageBytes;
         if (c >= early) {
-          mbar_expect_tx(&full[s], Shape::kStageBytes);
+          mbar_expect_tx(&full[s], stage_bytes);
           tma_load_2d(w, &wmap, (c0 + c) * kStepK, weight_row, &full[s]);
         }
-        tma_load_2d(w + kWeightBytes, &tmap, (c0 + c) * kStepK, t0, &full[s]);
+        if constexpr (kBoxes == 1) tma_load_2d(w + kWeightBytes, &tmap, (c0 + c) * kStepK, t0, &full[s]);
+        else
+          for (int i = 0; i < boxes; ++i) tma_load_2d(w + kWeightBytes + i * 32 * kStepK * 2, &tmap, (c0 + c) * kStepK, t0 + 32 * i, &full[s]);
         issued = c + 1;
       }
       if (!ok)   // leaving early: let the copies already issued land first
@@ -189,7 +192,7 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
     }
   } else if (warp == 1) {
     if (lane == 0) {
-      const uint32_t idesc = umma_idesc_bf16(kRowsM, BN);
+      const uint32_t idesc = umma_idesc_bf16(kRowsM, columns);
       for (int c = 0; c < chunks; ++c) {
         const int s = c % S;
         if (!wait_bounded(&full[s], uint32_t(c / S) & 1u, g.status, 3)) break;
@@ -218,6 +221,7 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
       constexpr int L = W == 8 ? 16 : W;              // columns per tensor-memory load
 #pragma unroll
       for (int c = column_half * (BN / 2); c < (column_half + 1) * (BN / 2); c += W) {
+        if (PerExpert(EPI) && c >= columns) break;
         float v[L];
         const uint32_t at = tmem + (uint32_t(32 * quarter) << 16) + uint32_t(W == 8 ? 0 : c);
         if constexpr (L == 32) tmem_load_32(at, v);
@@ -325,7 +329,7 @@ __global__ void __launch_bounds__(256) linear_f32(const float* activations, cons
     t_end = tile.first + min(tile.count, kTile32);
     weight += size_t(tile.expert) * g.n * k_stride;
   }
-  auto row_of = [&](int t) { return Gathers(EPI) ? g.slots.list[t] / g.slots.top : t; };
+  auto row_of = [&](int t) { return EPI == kLinearExpertUp ? g.slots.list[t] / g.slots.top : t; };
   float acc[4][4] = {};
   for (int k0 = 0; k0 < k_stride; k0 += kStep32) {
 #pragma unroll
@@ -391,7 +395,9 @@ cudaError_t LaunchTiles(const Queue& q, const LinearArgs& a, const LinearParams&
                 : a.epilogue == kLinearFloat ? linear_tiles<BN, kLinearFloat> : a.epilogue == kLinearExpertUp ? linear_tiles<BN, kLinearExpertUp>
                 : a.epilogue == kLinearExpertDown ? linear_tiles<BN, kLinearExpertDown> : linear_tiles<BN, kLinearStore>;
   cudaLaunchConfig_t config{};
-  config.gridDim = dim3(unsigned(PerExpert(a.epilogue) ? MostTiles(a.slots) : (a.t + BN - 1) / BN), unsigned((a.n + kRowsM - 1) / kRowsM), unsigned(splits));
+  const unsigned weight_tiles = unsigned((a.n + kRowsM - 1) / kRowsM);
+  config.gridDim = PerExpert(a.epilogue) ? dim3(weight_tiles, unsigned(MostTiles(a.slots)), unsigned(splits))
+                                         : dim3(unsigned((a.t + BN - 1) / BN), weight_tiles, unsigned(splits));
   config.blockDim = dim3(kLinearThreads);
   config.dynamicSmemBytes = LinearShape<BN>::kSmem;
   config.stream = q.stream;
@@ -409,7 +415,7 @@ cudaError_t LaunchTiles(const Queue& q, const LinearArgs& a, const LinearParams&
   }
   config.attrs = attributes;
   config.numAttrs = unsigned(count);
-  return cudaLaunchKernelEx(&config, kernel, a.maps->weight, Gathers(a.epilogue) ? a.maps->row : a.maps->rows[map], p);
+  return cudaLaunchKernelEx(&config, kernel, a.maps->weight, Gathers(a.epilogue, BN) ? a.maps->row : a.maps->rows[PerExpert(a.epilogue) ? std::min(map, 1) : map], p);
 }
 
 // Tile width (index into 16, 32, 64, 128, 256 tokens) and K splits: the widest tile that gives most SMs a CTA, else
@@ -444,7 +450,7 @@ int ExpertTileRows(const Queue& q, int slots, int experts) {
   if (q.f32) return kTile32;
   const int share = (slots + experts - 1) / experts;   // slots of an expert on average; most have no more than 4/3 of it
   int rows = 16;
-  while (rows < 256 && rows * 3 < share * 4) rows *= 2;
+  while (rows < 128 && rows * 3 < share * 4) rows *= 2;
   return rows;
 }
 
@@ -461,6 +467,10 @@ bool EncodeLinear(LinearMaps* maps, const void* weight, uint64_t n, const void* 
   if (!EncodeMatrix(&maps->weight, false, weight, n, k_stride, kRowsM)) return false;
   for (int i = 0; i < 5; ++i)
     if (!EncodeMatrix(&maps->rows[i], false, activations, rows, k_stride, 16u << i)) return false;
+  return true;
+}
+
+bool EncodeGathered(LinearMaps* maps, const void* activations, uint64_t rows, uint64_t k_stride) {
   return EncodeMatrix(&maps->row, false, activations, rows, k_stride, 1);
 }
 

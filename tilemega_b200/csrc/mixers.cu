@@ -64,6 +64,70 @@ __global__ void __launch_bounds__(128) rotate_append(StepRows r, T* proj, T* k_p
   }
 }
 
+// The same for bf16 rows whose head sizes and half rotations are multiples of 8: eight pairs, or eight entries behind the
+// rotated ones, a turn. Portions only.
+__global__ void __launch_bounds__(256) rotate_append_wide(StepRows r, __nv_bfloat16* proj, __nv_bfloat16* k_pool, __nv_bfloat16* v_pool, AppendParams p) {
+  __shared__ float2 part[8];
+  dependency_wait();
+  allow_dependents();
+  const int row = blockIdx.x;
+  if (r.entry[r.row_entry[row]].rows == 1) return;
+  const int half = p.rot.dims / 2, turned = half / 8, units = p.dim / 8 - turned;
+  const float2* angle = p.rot.table + size_t(min(r.row_position[row], p.rot.capacity - 1)) * half;
+  const int kv = r.row_kv[row];
+  __nv_bfloat16* line = proj + size_t(row) * p.stride;
+  const __nv_bfloat16* keys = line + size_t(p.heads) * p.dim;
+  const __nv_bfloat16* values = p.value_is_key ? keys : keys + size_t(p.kv_heads) * p.dim;
+  const int v_units = p.vdim / 8;
+  for (int i = threadIdx.x; i < p.kv_heads * v_units; i += 256)
+    *reinterpret_cast<uint4*>(v_pool + pool_offset(kv, i / v_units, p.kv_heads, p.v_pool_dim) + i % v_units * 8) = reinterpret_cast<const uint4*>(values)[i];
+  float2 inv = make_float2(1.f, 1.f);
+  if (p.q_norm) {
+    const int q_count = p.heads * p.dim, k_count = p.kv_heads * p.dim;
+    inv = inverse_rms<256>(make_float2(square_sum(line, q_count, 256), square_sum(keys, k_count, 256)), q_count, k_count, p.eps, part);
+  }
+  for (int i = threadIdx.x; i < (p.heads + p.kv_heads) * units; i += 256) {
+    const int head = i / units, u = i % units, group = head - p.heads;
+    if (u >= turned && group < 0 && !p.q_norm) continue;
+    const int d = u < turned ? 8 * u : 8 * u + half;
+    __nv_bfloat16* at = line + size_t(head) * p.dim + d;
+    __nv_bfloat16* to = group < 0 ? at : k_pool + pool_offset(kv, group, p.kv_heads, p.pool_dim) + d;
+    const float* weight = group < 0 ? p.q_norm : p.k_norm;
+    const float scale = group < 0 ? inv.x : inv.y;
+    auto load = [&](int offset, float (&v)[8]) {
+      unpack8(*reinterpret_cast<const uint4*>(at + offset), v);
+      if (!weight) return;
+      const float4* w = reinterpret_cast<const float4*>(weight + (group < 0 ? head : group) * p.dim + d + offset);
+      const float4 lo = w[0], hi = w[1];
+      const float by[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] *= scale * by[j];
+    };
+    auto store = [&](int offset, const float (&v)[8]) {
+      *reinterpret_cast<uint4*>(to + offset) =
+          make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+    };
+    float a[8];
+    load(0, a);
+    if (u < turned) {
+      float b[8];
+      load(half, b);
+      const float4* turn = reinterpret_cast<const float4*>(angle + d);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float4 cs = turn[j];
+        const float x0 = a[2 * j], y0 = b[2 * j], x1 = a[2 * j + 1], y1 = b[2 * j + 1];
+        a[2 * j] = x0 * cs.x - y0 * cs.y;
+        b[2 * j] = y0 * cs.x + x0 * cs.y;
+        a[2 * j + 1] = x1 * cs.z - y1 * cs.w;
+        b[2 * j + 1] = y1 * cs.z + x1 * cs.w;
+      }
+      store(half, b);
+    }
+    store(0, a);
+  }
+}
+
 // ---- attention, one warp per (row, query head) -------------------------------------------------------------------------
 constexpr int kPlainWarps = 4;
 
@@ -321,6 +385,11 @@ __global__ void __launch_bounds__(128) retention_gate(const float* raw, const T*
 
 template <typename T> int RotateAppendAs(const Queue& q, const StepRows& r, const AttentionArgs& a) {
   const AppendParams p{a.proj_stride, a.heads, a.kv_heads, a.dim, a.vdim, a.pool_dim, a.v_pool_dim, a.value_is_key, a.q_norm, a.k_norm, a.eps, a.rotary};
+  if constexpr (sizeof(T) == 2) {
+    if (a.dim % 8 == 0 && a.vdim % 8 == 0 && a.rotary.dims % 16 == 0 && a.proj_stride % 8 == 0)
+      return int(Launch(rotate_append_wide, dim3(unsigned(r.rows)), dim3(256), 0, q.stream, q.chained, r, static_cast<T*>(a.proj),
+                        static_cast<T*>(a.k_pool), static_cast<T*>(a.v_pool), p));
+  }
   return int(Launch(rotate_append<T>, dim3(unsigned(r.rows)), dim3(128), 0, q.stream, q.chained, r, static_cast<T*>(a.proj),
                     static_cast<T*>(a.k_pool), static_cast<T*>(a.v_pool), p, !q.f32));
 }

@@ -67,7 +67,7 @@ struct AttendParams {
   int proj_stride, out_stride, heads, kv_heads, dim, vdim, pool_dim, v_pool_dim, window, keep, splits, gate_at;
   int subs, sub_heads;      // query heads of one key head are served in `subs` units of up to `sub_heads`
   float scale_log2, sink_log2, eps;
-  bool value_is_key;
+  bool value_is_key, even;
   Rotary rotary;
 };
 
@@ -83,9 +83,9 @@ template <int DT, int WM> struct AttendShape {
 // of them against all keys of a block; q is rotated and the portion's keys are in the pools already (RotateAppend).
 // WM = 1: one decoded token, 16 rows, each of the four warps a quarter of a block's keys; the CTA rotates q itself, and
 // the one that holds the newest position rotates and appends its key and value (both norm them first, if the model does,
-// which takes the squares of the whole projected row). DT: 16-column tiles of the wider of keys and values. blockIdx =
-// (token tile | split, unit, entry).
-template <int DT, int WM>
+// which takes the squares of the whole projected row). DT: 16-column tiles of the wider of keys and values; FULL: both
+// fill them. blockIdx = (token tile | split, unit, entry).
+template <int DT, int WM, bool FULL>
 __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM > 1 ? 2 : 3) attend_tiles(StepRows r, AttendParams p) {
   using Shape = AttendShape<DT, WM>;
   constexpr int WN = WM == 1 ? 4 : 1, KN = kKeys / WN, P = Shape::kPitch, NT = Shape::kThreads;
@@ -138,8 +138,8 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
       const int key = i / C, c = (i % C) * 8, row = key_at[stage][key];
       const bool live = row >= 0;
       const size_t line = live ? size_t(row / kRaggedBlock * p.kv_heads + group) * kRaggedBlock + row % kRaggedBlock : 0;
-      if (c < p.pool_dim) copy16(ks + stage * Shape::kTile + key * P + c, p.k_pool + line * p.pool_dim + c, live);
-      if (c < p.v_pool_dim) copy16(vs + stage * Shape::kTile + key * P + c, p.v_pool + line * p.v_pool_dim + c, live);
+      if (FULL || c < p.pool_dim) copy16(ks + stage * Shape::kTile + key * P + c, p.k_pool + line * p.pool_dim + c, live);
+      if (FULL || c < p.v_pool_dim) copy16(vs + stage * Shape::kTile + key * P + c, p.v_pool + line * p.v_pool_dim + c, live);
     }
     copy_commit();
   };
@@ -152,30 +152,51 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
 
   const int half = p.rotary.dims / 2;
   const float2* angle = p.rotary.table + size_t(min(p1, p.rotary.capacity - 1)) * half;   // WM == 1: the token's
-  const bool wide = (p.dim & 7) == 0;
   float2 inv = make_float2(1.f, 1.f);
-  if (WM == 1 && p.q_norm) {
+  if constexpr (WM == 1) {
     const bf16* line = p.proj + size_t(e.first_row) * p.proj_stride;
-    const int q_count = p.heads * p.dim, k_count = p.kv_heads * p.dim;
-    inv = inverse_rms<NT>(make_float2(square_sum(line, q_count, NT), square_sum(line + q_count, k_count, NT)), q_count, k_count, p.eps, square_part);
-  }
-  for (int i = threadIdx.x; i < Shape::kRows * (P / 8); i += NT) {
-    const int m = i / (P / 8), c = (i % (P / 8)) * 8, t = m / gq;
-    const bf16* head = p.proj + size_t(e.first_row + t0 + t) * p.proj_stride + size_t(head0 + m % gq) * p.dim;
-    const float* weight = p.q_norm ? p.q_norm + (head0 + m % gq) * p.dim : nullptr;
-    uint4 word = make_uint4(0, 0, 0, 0);
-    if (t < tokens && c < p.dim) {
-      if (wide && WM > 1) {
-        word = *reinterpret_cast<const uint4*>(head + c);
-      } else {
-        bf16 e8[8];
-#pragma unroll
-        for (int j = 0; j < 8; ++j)
-          e8[j] = c + j >= p.dim ? __float2bfloat16_rn(0.f) : WM > 1 ? head[c + j] : __float2bfloat16_rn(normed_rotated(head, weight, inv.x, c + j, half, angle));
-        word = *reinterpret_cast<uint4*>(e8);
-      }
+    for (int i = threadIdx.x; i < Shape::kRows * (P / 8); i += NT) *reinterpret_cast<uint4*>(qs + 8 * i) = make_uint4(0, 0, 0, 0);
+    if (p.q_norm) {
+      const int q_count = p.heads * p.dim, k_count = p.kv_heads * p.dim;
+      inv = inverse_rms<NT>(make_float2(square_sum(line, q_count, NT), square_sum(line + q_count, k_count, NT)), q_count, k_count, p.eps, square_part);
+    } else {
+      __syncthreads();
     }
-    *reinterpret_cast<uint4*>(qs + m * P + c) = word;
+    const int units = p.dim - half;                      // a unit: one rotated pair, or one entry behind the rotated ones
+#pragma unroll 4
+    for (int i = threadIdx.x; i < gq * units; i += NT) {
+      const int m = i / units, u = i % units, d = u < half ? u : u + half, head = head0 + m;
+      const bf16* q = line + size_t(head) * p.dim;
+      const float* weight = p.q_norm ? p.q_norm + size_t(head) * p.dim : nullptr;
+      float a = __bfloat162float(q[d]);
+      if (weight) a *= inv.x * weight[d];
+      if (u < half) {
+        float b = __bfloat162float(q[d + half]);
+        if (weight) b *= inv.x * weight[d + half];
+        const float2 cs = angle[u];
+        qs[m * P + d + half] = __float2bfloat16_rn(b * cs.x + a * cs.y);
+        a = a * cs.x - b * cs.y;
+      }
+      qs[m * P + d] = __float2bfloat16_rn(a);
+    }
+  } else {
+    const bool wide = (p.dim & 7) == 0;
+    for (int i = threadIdx.x; i < Shape::kRows * (P / 8); i += NT) {
+      const int m = i / (P / 8), c = (i % (P / 8)) * 8, t = m / gq;
+      const bf16* head = p.proj + size_t(e.first_row + t0 + t) * p.proj_stride + size_t(head0 + m % gq) * p.dim;
+      uint4 word = make_uint4(0, 0, 0, 0);
+      if (t < tokens && c < p.dim) {
+        if (wide) {
+          word = *reinterpret_cast<const uint4*>(head + c);
+        } else {
+          bf16 e8[8];
+#pragma unroll
+          for (int j = 0; j < 8; ++j) e8[j] = c + j >= p.dim ? __float2bfloat16_rn(0.f) : head[c + j];
+          word = *reinterpret_cast<uint4*>(e8);
+        }
+      }
+      *reinterpret_cast<uint4*>(qs + m * P + c) = word;
+    }
   }
 
   const int row0 = WM == 1 ? 0 : warp * 16, key0 = WM == 1 ? warp * KN : 0;
@@ -223,7 +244,7 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
     for (int t = 0; t < KN / 8; ++t) s[t][0] = s[t][1] = s[t][2] = s[t][3] = 0.f;
 #pragma unroll
     for (int kk = 0; kk < DT; ++kk) {
-      if (kk * 16 >= p.pool_dim) break;
+      if (!FULL && kk * 16 >= p.pool_dim) break;
       uint32_t a[4];
       load_a(a, qs, P, row0, kk * 16, lane);
 #pragma unroll
@@ -290,7 +311,7 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
       }
 #pragma unroll
       for (int d = 0; d < DT; ++d) {
-        if (d * 16 >= p.v_pool_dim) break;
+        if (!FULL && d * 16 >= p.v_pool_dim) break;
         uint32_t bb[4];
         load_b_transposed(bb, vt, P, kk * 16, d * 16, lane);
         mma16816(o[2 * d], hi, bb[0], bb[1]);
@@ -321,6 +342,15 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
       bf16* dst = p.out + row * p.out_stride + column;
       float y0 = o[i][at] * inv, y1 = o[i][at + 1] * inv;
       const bool pair = c + 1 < p.vdim;
+      if (p.even) {                                      // both columns, and words of two at the addresses
+        if (p.gate_at >= 0) {
+          const uint32_t gate = *reinterpret_cast<const uint32_t*>(p.proj + row * p.proj_stride + p.gate_at + column);
+          y0 = __fdividef(y0, 1.f + ex2(-1.4426950408889634f * bf_lo(gate)));
+          y1 = __fdividef(y1, 1.f + ex2(-1.4426950408889634f * bf_hi(gate)));
+        }
+        *reinterpret_cast<uint32_t*>(dst) = pack(y0, y1);
+        return;
+      }
       if (p.gate_at >= 0) {
         const bf16* gate = p.proj + row * p.proj_stride + p.gate_at + column;
         y0 *= sigmoid(__bfloat162float(gate[0]));
@@ -715,7 +745,8 @@ __global__ void __launch_bounds__(128) retain_chunks(StepRows r, const bf16* pro
 
 template <int DT, int WM> int LaunchAttend(const Queue& q, const StepRows& r, const AttendParams& p, int x) {
   const int units = p.kv_heads * p.subs;
-  return int(Launch(attend_tiles<DT, WM>, dim3(unsigned(x), unsigned(units), unsigned(r.entries)), dim3(AttendShape<DT, WM>::kThreads), AttendShape<DT, WM>::kSmem, q.stream,
+  auto kernel = p.pool_dim == 16 * DT && p.v_pool_dim == 16 * DT ? attend_tiles<DT, WM, true> : attend_tiles<DT, WM, false>;
+  return int(Launch(kernel, dim3(unsigned(x), unsigned(units), unsigned(r.entries)), dim3(AttendShape<DT, WM>::kThreads), AttendShape<DT, WM>::kSmem, q.stream,
                     q.chained, r, p));
 }
 
@@ -759,9 +790,11 @@ template <int DT> int RetainWith(const Queue& q, const StepRows& r, const Retent
 }
 
 template <int DT> cudaError_t Raise() {
-  cudaError_t err = cudaFuncSetAttribute(attend_tiles<DT, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, AttendShape<DT, 1>::kSmem);
-  if (err == cudaSuccess) err = cudaFuncSetAttribute(attend_tiles<DT, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, AttendShape<DT, 8>::kSmem);
-  if (err == cudaSuccess) err = cudaFuncSetAttribute(retain_chunks<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, RetainShape<DT>::kSmem);
+  cudaError_t err = cudaFuncSetAttribute(retain_chunks<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, RetainShape<DT>::kSmem);
+  for (auto kernel : {attend_tiles<DT, 1, false>, attend_tiles<DT, 1, true>})
+    if (err == cudaSuccess) err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, AttendShape<DT, 1>::kSmem);
+  for (auto kernel : {attend_tiles<DT, 8, false>, attend_tiles<DT, 8, true>})
+    if (err == cudaSuccess) err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, AttendShape<DT, 8>::kSmem);
   return err;
 }
 
@@ -789,6 +822,7 @@ int AttendTiles(const Queue& q, const StepRows& r, const AttentionArgs& a) {
   p.k_norm = a.k_norm;
   p.eps = a.eps;
   p.gate_at = a.gate_at;
+  p.even = a.vdim % 2 == 0 && a.out_stride % 2 == 0 && a.proj_stride % 2 == 0 && (a.gate_at < 0 || a.gate_at % 2 == 0);
   p.window = a.window;
   p.keep = a.keep;
   const int gq = a.heads / a.kv_heads;

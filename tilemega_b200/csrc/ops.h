@@ -100,7 +100,9 @@ struct ExpertSlots {
 // gated unit of interleaved gate/up rows, stored as an element (column n of the output is pair n); store as fp32.
 // Activation and weight rows are k_stride elements long (a multiple of 8, zero weights behind k).
 // Per expert (weight rows expert * n ..., slots in place of t): ExpertUp reads activation row list[s] / top for slot s
-// and stores relu(score[s] D)^2 in row s; ExpertDown reads row s and stores D in row list[s]; both as elements.
+// (from `activations`; bf16 tiles of more than kGatherRows slots read row s of rows gathered before, see GatherRows) and
+// stores relu(score[s] D)^2 in row s; ExpertDown reads row s and stores D in row list[s]; both as elements.
+constexpr int kGatherRows = 32;
 struct LinearMaps {
   CUtensorMap weight;        // bf16 only: 128-row boxes
   CUtensorMap rows[5];       // boxes of 16, 32, 64, 128, 256 activation rows
@@ -121,6 +123,7 @@ struct LinearArgs {
 int ExpertTileRows(const Queue& q, int slots, int experts);   // slots per tile that suits this many
 int PrepareLinear();         // raises the kernels' shared-memory limits (once per device)
 bool EncodeLinear(LinearMaps* maps, const void* weight, uint64_t n, const void* activations, uint64_t rows, uint64_t k_stride);
+bool EncodeGathered(LinearMaps* maps, const void* activations, uint64_t rows, uint64_t k_stride);   // maps->row only
 int Linear(const Queue& q, const LinearArgs& a);
 
 // The gated unit by itself: in [t][2 * padded] interleaved pairs, out [t][outputs].
@@ -140,10 +143,13 @@ struct RouteArgs {
   float* slot_score;         // [rows * top], sorted
   ExpertTile* tiles;
   int* tile_count;
-  unsigned* count;           // arrival counter, zero between launches
+  unsigned* count;           // kRouteCounters arrival counters, zero between launches
 };
+constexpr int kRouteCounters = 9;
 bool RouteFused(int rows);
 int Route(const Queue& q, const RouteArgs& a);
+// out[slot] = h[list[slot] / top] (bf16 rows of k_stride).
+int GatherRows(const Queue& q, const void* h, int k_stride, const ExpertSlots& slots, void* out);
 
 // Attention with grouped heads, a sliding window of `window` positions and the first `keep` positions always seen.
 // proj rows hold q | k (| v) (| g): q heads x dim, k kv_heads x dim, v kv_heads x vdim, g heads x vdim; the values are v,

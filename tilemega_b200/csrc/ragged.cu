@@ -32,6 +32,7 @@ struct RaggedPlan {
   float *score = nullptr, *slot_score = nullptr;
   ExpertTile* tiles = nullptr;
   unsigned* route_count = nullptr;
+  void* gathered = nullptr;        // bf16 plans: [max_rows * most experts of a token][padded width]
   void* expert_hidden = nullptr;   // [max_rows * most experts of a token][widest expert]
   void* expert_out = nullptr;      // [max_rows * most experts of a token][width]
   float* raw = nullptr;        // retention outputs before their norm
@@ -240,6 +241,7 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       if (!RouteFused(r.rows))
         TMB_TRY(Linear(q, linear(plan->normed, layer.router, -1, maps ? &maps->router : nullptr, mlp.experts, W, plan->logits, mlp.experts, kLinearFloat)));
       TMB_TRY(Route(q, a));
+      if (!s.f32 && slots.tile_rows > kGatherRows) TMB_TRY(GatherRows(q, plan->normed, W8, slots, plan->gathered));
       const int stride = padded_columns(mlp.ff);
       LinearArgs up = linear(plan->normed, layer.expert_up, -1, maps ? &maps->gate_up : nullptr, mlp.ff, W, plan->expert_hidden, stride, kLinearExpertUp);
       up.slots = slots;
@@ -324,7 +326,8 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
       !Own(plan, &plan->logits, rows * experts * sizeof(float)) || !Own(plan, &plan->choice, slots * sizeof(int)) ||
       !Own(plan, &plan->list, slots * sizeof(int)) || !Own(plan, &plan->tile_count, sizeof(int)) ||
       !Own(plan, &plan->score, slots * sizeof(float)) || !Own(plan, &plan->slot_score, slots * sizeof(float)) ||
-      !Own(plan, &plan->tiles, (slots / 16 + experts) * sizeof(ExpertTile)) || !Own(plan, &plan->route_count, sizeof(unsigned)) ||
+      !Own(plan, &plan->tiles, (slots / 16 + experts) * sizeof(ExpertTile)) || !Own(plan, &plan->route_count, kRouteCounters * sizeof(unsigned)) ||
+      !Own(plan, &plan->gathered, spec.f32 ? 0 : slots * W8 * element) ||
       !Own(plan, &plan->expert_hidden, slots * expert_columns * element) || !Own(plan, &plan->expert_out, slots * size_t(spec.width) * element) ||
       !Own(plan, &plan->raw, rows * raw * sizeof(float)) || !Own(plan, &plan->split, spec.f32 ? 0 : rows * split * 2) ||
       !Own(plan, &plan->part, plan->part_floats * sizeof(float)) ||
@@ -365,7 +368,8 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
       const RaggedMlp& mlp = layer.mlp;
       if (mlp.kind == RaggedMlp::kExperts)
         ok = ok && EncodeLinear(&maps.router, at(layer.router), uint64_t(mlp.experts), plan->normed, rows, W8) &&
-             EncodeLinear(&maps.gate_up, at(layer.expert_up), uint64_t(mlp.experts) * mlp.ff, plan->normed, rows, W8) &&
+             EncodeLinear(&maps.gate_up, at(layer.expert_up), uint64_t(mlp.experts) * mlp.ff, plan->gathered, slots, W8) &&
+             EncodeGathered(&maps.gate_up, plan->normed, rows, W8) &&
              EncodeLinear(&maps.down, at(layer.expert_down), uint64_t(mlp.experts) * spec.width, plan->expert_hidden, slots,
                           uint64_t(padded_columns(mlp.ff)));
       if (mlp.kind == RaggedMlp::kGlu)
