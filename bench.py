@@ -500,8 +500,8 @@ def run_forward(args) -> None:
 
 def run_ragged(args) -> None:
     """Secondary workload: a decoder given as a list of layers (`--model bamudra-8b | bamudra-1b | nadilorn-8b | nadilorn-1b |
-    nadilorn-30b-a3b`) through a ragged-step plan (phase 3 of the plan ABI). Decode: `--batch` sequences at `--context` positions, one step = one decoded token of each, the
-    sampled tokens fed back on the device. `--prefill T`: a prompt of T tokens in portions of `--portion` rows, one step =
+    nadilorn-30b-a3b`) through a ragged-step plan (phase 3 of the plan ABI). Decode: `--batch` sequences at `--context`
+    positions, one step = one decoded token of each, the sampled tokens fed back on the device. `--prefill T`: a prompt of T tokens in portions of `--portion` rows, one step =
     one portion. One JSON line in the shape of the decode line; same weights, widths and vocabulary as the Llama-shaped
     model of the same name, so the two lines stand side by side."""
     if int(os.environ.get("RANK", "0")) != 0:
