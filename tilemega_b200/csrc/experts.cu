@@ -42,7 +42,7 @@ __device__ __forceinline__ unsigned ordered(float v) {
 // largest of those behind the one before it in that order.
 constexpr int kMine = 8;
 template <bool HELD> __device__ __forceinline__ void choose(const RouteArgs& a, int row, int lane) {
-  const float* z = a.logits + size_t(row) * a.experts;
+  const float* z = a.logits + size_t(row) * (a.experts + a.extra);
   unsigned key[kMine];
   if (HELD)
 #pragma unroll
@@ -85,9 +85,110 @@ template <bool HELD> __device__ __forceinline__ void choose(const RouteArgs& a, 
     }
   }
 }
-__device__ __forceinline__ void choose(const RouteArgs& a, int row, int lane) {
-  if (a.experts <= 32 * kMine) choose<true>(a, row, lane);
-  else choose<false>(a, row, lane);
+// The same where scores are not the logits' order: ranked by score + correction, from the best groups only. `line` holds the
+// row's ranks (shared memory where HELD, else a.ranks).
+template <bool HELD> __device__ __forceinline__ void choose_ranked(const RouteArgs& a, int row, int lane, float* line) {
+  const float* z = a.logits + size_t(row) * (a.experts + a.extra);
+  float high = -INFINITY, sum = 0.f;
+  if (a.softmax) {
+    for (int e = lane; e < a.experts; e += 32) high = fmaxf(high, __ldcg(z + e));
+    high = warp_max(high);
+    for (int e = lane; e < a.experts; e += 32) sum += expf(__ldcg(z + e) - high);
+    sum = warp_sum(sum);
+  }
+  auto score = [&](int e) { return a.softmax ? expf(__ldcg(z + e) - high) / sum : 1.f / (1.f + expf(-__ldcg(z + e))); };
+  for (int e = lane; e < a.experts; e += 32) line[e] = score(e) + (a.correction ? a.correction[e] : 0.f);
+  __syncwarp();
+  // the largest key behind (before, before_at) in falling order, the smaller index first where two are equal
+  auto next = [&](unsigned best, int at, unsigned& before, int& before_at) {
+    before = __reduce_max_sync(0xffffffffu, best);
+    before_at = __reduce_min_sync(0xffffffffu, best == before ? at : 0x7fffffff);
+  };
+  if (a.keep_groups < a.groups) {
+    const int size = a.experts / a.groups;
+    auto largest = [&](int g) {
+      unsigned v = 1u;
+      for (int e = g * size; e < (g + 1) * size; ++e) v = max(v, ordered(line[e]));
+      return v;
+    };
+    unsigned before = 0xffffffffu;
+    int before_at = -1;
+    for (int k = 0; k < a.keep_groups; ++k) {
+      unsigned best = 0u;
+      int at = 0x7fffffff;
+      for (int g = lane; g < a.groups; g += 32) {
+        const unsigned v = largest(g);
+        if (v > before || (v == before && g <= before_at)) continue;
+        if (v > best) {
+          best = v;
+          at = g;
+        }
+      }
+      next(best, at, before, before_at);
+    }
+    __syncwarp();
+    for (int g = lane; g < a.groups; g += 32) {
+      const unsigned v = largest(g);
+      if (v > before || (v == before && g <= before_at)) continue;
+      for (int e = g * size; e < (g + 1) * size; ++e) line[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  unsigned key[kMine];
+  if (HELD)
+#pragma unroll
+    for (int i = 0; i < kMine; ++i) key[i] = lane + 32 * i < a.experts ? max(ordered(line[lane + 32 * i]), 1u) : 0u;
+  unsigned before = 0xffffffffu;
+  int before_at = -1, mine_at = 0;
+  float total = 0.f, mine = 0.f;
+  for (int k = 0; k < a.top; ++k) {
+    unsigned best = 0u;
+    int at = 0x7fffffff;
+    if (HELD) {
+#pragma unroll
+      for (int i = 0; i < kMine; ++i)
+        if (key[i] > best) {
+          best = key[i];
+          at = lane + 32 * i;
+        }
+    } else {
+      for (int e = lane; e < a.experts; e += 32) {
+        const unsigned v = max(ordered(line[e]), 1u);
+        if (v > before || (v == before && e <= before_at)) continue;
+        if (v > best) {
+          best = v;
+          at = e;
+        }
+      }
+    }
+    next(best, at, before, before_at);
+    if (HELD) {
+#pragma unroll
+      for (int i = 0; i < kMine; ++i)
+        if (before_at == lane + 32 * i) key[i] = 0u;
+    }
+    const int expert = min(before_at, a.experts - 1);
+    const float s = score(expert);
+    total += s;
+    if (lane == k) {
+      mine = s;
+      mine_at = expert;
+    }
+  }
+  if (lane < a.top) {
+    a.choice[row * a.top + lane] = mine_at;
+    a.score[row * a.top + lane] = a.weights ? mine / (total + 1e-20f) : mine;
+  }
+}
+__device__ __forceinline__ void choose(const RouteArgs& a, int row, int lane, float* line) {
+  const bool held = a.experts <= 32 * kMine;
+  if (a.ranks) {
+    if (held) choose_ranked<true>(a, row, lane, line);
+    else choose_ranked<false>(a, row, lane, a.ranks + size_t(row) * a.experts);
+  } else {
+    if (held) choose<true>(a, row, lane);
+    else choose<false>(a, row, lane);
+  }
 }
 
 // The step's assignments sorted by expert, by one CTA. `first` holds every expert's first slot, then its next free one.
@@ -166,17 +267,18 @@ template <typename T, bool FUSED>
 __global__ void __launch_bounds__(FUSED ? 256 : 1024) route(RouteArgs a) {
   __shared__ int counts[kMaxExperts], first[kMaxExperts];
   __shared__ unsigned last;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  __shared__ float ranks[FUSED ? 8 : 32][32 * kMine];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5, logits = a.experts + a.extra;
   if constexpr (FUSED) {
     constexpr int N = 16 / sizeof(T);
     const int e = blockIdx.x * 8 + warp, pieces = a.k_stride / N, row0 = blockIdx.y * 8, rows = min(8, a.rows - row0);
-    const uint4* w = reinterpret_cast<const uint4*>(static_cast<const T*>(a.router) + size_t(min(e, a.experts - 1)) * a.k_stride);
+    const uint4* w = reinterpret_cast<const uint4*>(static_cast<const T*>(a.router) + size_t(min(e, logits - 1)) * a.k_stride);
     uint4 held[kHeld];
 #pragma unroll
     for (int i = 0; i < kHeld; ++i) held[i] = lane + 32 * i < pieces ? w[lane + 32 * i] : make_uint4(0, 0, 0, 0);
     dependency_wait();
     allow_dependents();
-    if (e < a.experts)
+    if (e < logits)
       for (int row = row0; row < row0 + rows; ++row) {
         const uint4* h = reinterpret_cast<const uint4*>(static_cast<const T*>(a.h) + size_t(row) * a.k_stride);
         uint4 x[kHeld];
@@ -187,17 +289,17 @@ __global__ void __launch_bounds__(FUSED ? 256 : 1024) route(RouteArgs a) {
         for (int i = 0; i < kHeld; ++i) sum += dot16<T>(x[i], held[i]);
         for (int i = lane + 32 * kHeld; i < pieces; i += 32) sum += dot16<T>(h[i], w[i]);
         sum = warp_sum(sum);
-        if (lane == 0) a.logits[size_t(row) * a.experts + e] = sum;
+        if (lane == 0) a.logits[size_t(row) * logits + e] = sum;
       }
     if (!arrives_last(a.count + 1 + blockIdx.y, gridDim.x, &last)) return;
-    if (warp < rows) choose(a, row0 + warp, lane);
+    if (warp < rows) choose(a, row0 + warp, lane, ranks[warp]);
     if (gridDim.y == 1) __syncthreads();
     else if (!arrives_last(a.count, gridDim.y, &last)) return;
   } else {
     dependency_wait();
     allow_dependents();
     const int row = blockIdx.x * warps + warp;
-    if (row < a.rows) choose(a, row, lane);
+    if (row < a.rows) choose(a, row, lane, ranks[warp]);
     if (!arrives_last(a.count, gridDim.x, &last)) return;
   }
   sort_assignments(a, counts, first);
@@ -214,7 +316,7 @@ __global__ void __launch_bounds__(256) gather_rows(const uint4* h, const int* li
 
 template <typename T> int RouteAs(const Queue& q, const RouteArgs& a) {
   if (RouteFused(a.rows))
-    return int(Launch(route<T, true>, dim3(unsigned((a.experts + 7) / 8), unsigned((a.rows + 7) / 8)), dim3(256), 0, q.stream, q.chained, a));
+    return int(Launch(route<T, true>, dim3(unsigned((a.experts + a.extra + 7) / 8), unsigned((a.rows + 7) / 8)), dim3(256), 0, q.stream, q.chained, a));
   return int(Launch(route<T, false>, dim3(unsigned((a.rows + 31) / 32)), dim3(1024), 0, q.stream, q.chained, a));
 }
 
@@ -224,7 +326,8 @@ bool RouteFused(int rows) { return rows <= kFusedRows; }
 
 int Route(const Queue& q, const RouteArgs& a) {
   if (a.rows <= 0) return 0;
-  if (a.experts > kMaxExperts || a.top > a.experts || a.tile_rows < 1 || a.k_stride % 8) return int(cudaErrorInvalidValue);
+  if (a.experts > kMaxExperts || a.top > a.experts || a.tile_rows < 1 || a.k_stride % 8 || (!a.ranks && (a.softmax || a.correction || a.keep_groups < a.groups)) || a.top > kMaxTop)
+    return int(cudaErrorInvalidValue);
   return q.f32 ? RouteAs<float>(q, a) : RouteAs<__nv_bfloat16>(q, a);
 }
 

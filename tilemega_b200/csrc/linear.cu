@@ -28,6 +28,7 @@ struct LinearParams {
   const float* bias;
   void* out;
   int t, n, out_stride, outputs;
+  int head_in, head_out;
   int chunks, chunks_per_split;
   Glu glu;
   ExpertSlots slots;
@@ -35,8 +36,14 @@ struct LinearParams {
 };
 
 // Which products read gathered rows, and which run per expert.
-__host__ __device__ constexpr bool Gathers(int epilogue, int tokens) { return epilogue == kLinearExpertUp && tokens <= kGatherRows; }
-__host__ __device__ constexpr bool PerExpert(int epilogue) { return epilogue == kLinearExpertUp || epilogue == kLinearExpertDown; }
+__host__ __device__ constexpr bool Gathers(int epilogue, int tokens) {
+  return (epilogue == kLinearExpertUp || epilogue == kLinearExpertGlu) && tokens <= kGatherRows;
+}
+__host__ __device__ constexpr bool PerExpert(int epilogue) {
+  return epilogue == kLinearExpertUp || epilogue == kLinearExpertDown || epilogue == kLinearExpertGlu || epilogue == kLinearExpertStore;
+}
+// Gated units: products of interleaved gate and up rows.
+__host__ __device__ constexpr bool IsGlu(int epilogue) { return epilogue == kLinearGlu || epilogue == kLinearExpertGlu; }
 
 template <int BN> struct LinearShape {
   static constexpr int kStages = BN == 256 ? 4 : BN == 128 ? 3 : BN == 64 ? 4 : 5;   // about 100 KB (two CTAs per SM), 192 KB for the widest
@@ -73,7 +80,7 @@ __device__ __forceinline__ float ld_peer(uint32_t local, uint32_t rank) {
 }
 
 template <int EPI> __device__ __forceinline__ void emit(const LinearParams& g, int t, int n, float v) {
-  if (EPI == kLinearStore) static_cast<__nv_bfloat16*>(g.out)[size_t(t) * g.out_stride + n] = __float2bfloat16_rn(v);
+  if (EPI == kLinearStore || EPI == kLinearHeads) static_cast<__nv_bfloat16*>(g.out)[size_t(t) * g.out_stride + n] = __float2bfloat16_rn(v);
   if (EPI == kLinearAdd) static_cast<float*>(g.out)[size_t(t) * g.out_stride + n] += v;
   if (EPI == kLinearFloat) static_cast<float*>(g.out)[size_t(t) * g.out_stride + n] = v;
   if (EPI == kLinearExpertUp) {
@@ -87,7 +94,9 @@ template <int EPI> __device__ __forceinline__ void emit(const LinearParams& g, i
 // once while its activations stay in L2. The CTAs of one (weight, token) tile form a cluster along z. Per expert the
 // first two axes change places (an expert's weights are read by few tiles, its tokens by all of its weight tiles), token
 // tiles are those of the slot table (the grid holds as many as there could be), tokens are slots, and weight tiles start at
-// the expert's rows; what a tile computes beyond its slots or its expert's rows is dropped.
+// the expert's rows; what a tile computes beyond its slots or its expert's rows is dropped. Products by heads count the weight
+// tiles of one head after the other; columns behind a head's in its chunks of activations meet zeros, the map's fill
+// behind a weight row.
 template <int BN, int EPI>
 __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap tmap,
                                                                const LinearParams g) {
@@ -100,8 +109,16 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
   uint64_t* accum = empty + S;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(accum + 1);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n0 = (PerExpert(EPI) ? blockIdx.x : blockIdx.y) * kRowsM, token_tile = PerExpert(EPI) ? blockIdx.y : blockIdx.x;
-  int t0 = token_tile * BN, t_end = g.t, weight_row = n0;
+  int n0 = (PerExpert(EPI) ? blockIdx.x : blockIdx.y) * kRowsM;
+  const int token_tile = PerExpert(EPI) ? blockIdx.y : blockIdx.x;
+  int t0 = token_tile * BN, t_end = g.t, weight_row = n0, k_at = 0, out_at = 0;
+  if constexpr (EPI == kLinearHeads) {
+    const int tiles = (g.n + kRowsM - 1) / kRowsM, head = blockIdx.y / tiles;
+    n0 = (blockIdx.y % tiles) * kRowsM;
+    weight_row = head * g.n + n0;
+    k_at = head * g.head_in;
+    out_at = head * g.head_out;
+  }
   // per expert only the tokens there are cost anything: wide tiles load them 32 rows at a time
   constexpr bool kGather = Gathers(EPI, BN);
   constexpr int kBoxes = PerExpert(EPI) && BN > 32 ? BN / 32 : 1;
@@ -182,7 +199,7 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
           mbar_expect_tx(&full[s], stage_bytes);
           tma_load_2d(w, &wmap, (c0 + c) * kStepK, weight_row, &full[s]);
         }
-        if constexpr (kBoxes == 1) tma_load_2d(w + kWeightBytes, &tmap, (c0 + c) * kStepK, t0, &full[s]);
+        if constexpr (kBoxes == 1) tma_load_2d(w + kWeightBytes, &tmap, k_at + (c0 + c) * kStepK, t0, &full[s]);
         else
           for (int i = 0; i < boxes; ++i) tma_load_2d(w + kWeightBytes + i * 32 * kStepK * 2, &tmap, (c0 + c) * kStepK, t0 + 32 * i, &full[s]);
         issued = c + 1;
@@ -249,7 +266,7 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
           if (p < splits) sum += part[p];               // in split order
         return sum;
       };
-      if constexpr (EPI == kLinearGlu) {
+      if constexpr (IsGlu(EPI)) {
         for (int i = worker; i < cols * (kRowsM / 2); i += 256) {
           const int c = first + i / (kRowsM / 2), pair = i % (kRowsM / 2);
           const int row = (pair / kGluUnit) * 2 * kGluUnit + pair % kGluUnit, out = n0 / 2 + pair;
@@ -261,7 +278,7 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
         const int row = worker & (kRowsM - 1), n = n0 + row;
         if (n < g.n) {
           const float bias = g.bias ? g.bias[n] : 0.f;
-          for (int c = first + (worker >> 7); c < first + cols; c += 2) emit<EPI>(g, t0 + c, n, total(c, row) + bias);
+          for (int c = first + (worker >> 7); c < first + cols; c += 2) emit<EPI>(g, t0 + c, out_at + n, total(c, row) + bias);
         }
       }
     }
@@ -274,7 +291,7 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
       float v[32];
       tmem_load_32(tmem + (uint32_t(32 * quarter) << 16) + uint32_t(c), v);
       const int cols = min(32, t_end - t0 - c);
-      if constexpr (EPI == kLinearGlu) {
+      if constexpr (IsGlu(EPI)) {
         const bool upper = lane >= kGluUnit;          // lanes 0..15 hold gate rows, 16..31 the matching up rows
         const int out = (n0 + 32 * quarter) / 2 + (lane & (kGluUnit - 1));
 #pragma unroll
@@ -298,7 +315,7 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            if (i < cols) emit<EPI>(g, t0 + c + i, n, v[i] + bias);
+            if (i < cols) emit<EPI>(g, t0 + c + i, out_at + n, v[i] + bias);
         }
       }
     }
@@ -315,7 +332,7 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
 constexpr int kTile32 = 64, kStep32 = 16;
 
 template <int EPI>
-__global__ void __launch_bounds__(256) linear_f32(const float* activations, const float* weight, const LinearParams g, int k_stride) {
+__global__ void __launch_bounds__(256) linear_f32(const float* activations, const float* weight, const LinearParams g, int k_stride, int in_stride) {
   __shared__ float as[kStep32][kTile32 + 4], ws[kStep32][kTile32 + 4];
   const int n0 = blockIdx.x * kTile32;
   int t0 = blockIdx.y * kTile32, t_end = g.t;
@@ -329,13 +346,16 @@ __global__ void __launch_bounds__(256) linear_f32(const float* activations, cons
     t_end = tile.first + min(tile.count, kTile32);
     weight += size_t(tile.expert) * g.n * k_stride;
   }
-  auto row_of = [&](int t) { return EPI == kLinearExpertUp ? g.slots.list[t] / g.slots.top : t; };
+  const int head = blockIdx.z;                          // (products by heads only)
+  activations += size_t(head) * g.head_in;
+  weight += size_t(head) * g.n * k_stride;
+  auto row_of = [&](int t) { return EPI == kLinearExpertUp || EPI == kLinearExpertStore ? g.slots.list[t] / g.slots.top : t; };
   float acc[4][4] = {};
   for (int k0 = 0; k0 < k_stride; k0 += kStep32) {
 #pragma unroll
     for (int i = threadIdx.x; i < kTile32 * kStep32; i += 256) {
       const int r = i / kStep32, k = i % kStep32;
-      as[k][r] = t0 + r < t_end && k0 + k < k_stride ? activations[size_t(row_of(t0 + r)) * k_stride + k0 + k] : 0.f;
+      as[k][r] = t0 + r < t_end && k0 + k < k_stride ? activations[size_t(row_of(t0 + r)) * in_stride + k0 + k] : 0.f;
       ws[k][r] = n0 + r < g.n && k0 + k < k_stride ? weight[size_t(n0 + r) * k_stride + k0 + k] : 0.f;
     }
     __syncthreads();
@@ -354,7 +374,7 @@ __global__ void __launch_bounds__(256) linear_f32(const float* activations, cons
       const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
       if (t >= t_end || n >= g.n) continue;
       const float v = acc[i][j] + (g.bias ? g.bias[n] : 0.f);
-      float* out = static_cast<float*>(g.out) + size_t(EPI == kLinearExpertDown ? g.slots.list[t] : t) * g.out_stride + n;
+      float* out = static_cast<float*>(g.out) + size_t(EPI == kLinearExpertDown ? g.slots.list[t] : t) * g.out_stride + size_t(head) * g.head_out + n;
       const float positive = fmaxf(EPI == kLinearExpertUp ? v * g.slots.score[t] : 0.f, 0.f);
       *out = EPI == kLinearAdd ? *out + v : EPI == kLinearExpertUp ? positive * positive : v;
     }
@@ -379,7 +399,8 @@ __global__ void __launch_bounds__(256) glu_rows(const T* in, T* out, int t, int 
 template <int BN> cudaError_t RaiseLimit() {
   const int smem = LinearShape<BN>::kSmem;
   for (auto kernel : {linear_tiles<BN, kLinearStore>, linear_tiles<BN, kLinearAdd>, linear_tiles<BN, kLinearGlu>, linear_tiles<BN, kLinearFloat>,
-                      linear_tiles<BN, kLinearExpertUp>, linear_tiles<BN, kLinearExpertDown>}) {
+                      linear_tiles<BN, kLinearExpertUp>, linear_tiles<BN, kLinearExpertDown>, linear_tiles<BN, kLinearHeads>,
+                      linear_tiles<BN, kLinearExpertGlu>}) {
     const cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (err != cudaSuccess) return err;
   }
@@ -393,9 +414,10 @@ template <int BN>
 cudaError_t LaunchTiles(const Queue& q, const LinearArgs& a, const LinearParams& p, int map, int splits) {
   auto kernel = a.epilogue == kLinearAdd ? linear_tiles<BN, kLinearAdd> : a.epilogue == kLinearGlu ? linear_tiles<BN, kLinearGlu>
                 : a.epilogue == kLinearFloat ? linear_tiles<BN, kLinearFloat> : a.epilogue == kLinearExpertUp ? linear_tiles<BN, kLinearExpertUp>
-                : a.epilogue == kLinearExpertDown ? linear_tiles<BN, kLinearExpertDown> : linear_tiles<BN, kLinearStore>;
+                : a.epilogue == kLinearExpertDown ? linear_tiles<BN, kLinearExpertDown> : a.epilogue == kLinearHeads ? linear_tiles<BN, kLinearHeads>
+                : a.epilogue == kLinearExpertGlu ? linear_tiles<BN, kLinearExpertGlu> : linear_tiles<BN, kLinearStore>;
   cudaLaunchConfig_t config{};
-  const unsigned weight_tiles = unsigned((a.n + kRowsM - 1) / kRowsM);
+  const unsigned weight_tiles = unsigned((a.n + kRowsM - 1) / kRowsM) * unsigned(std::max(a.heads, 1));
   config.gridDim = PerExpert(a.epilogue) ? dim3(weight_tiles, unsigned(MostTiles(a.slots)), unsigned(splits))
                                          : dim3(unsigned((a.t + BN - 1) / BN), weight_tiles, unsigned(splits));
   config.blockDim = dim3(kLinearThreads);
@@ -421,8 +443,8 @@ cudaError_t LaunchTiles(const Queue& q, const LinearArgs& a, const LinearParams&
 // Tile width (index into 16, 32, 64, 128, 256 tokens) and K splits: the widest tile that gives most SMs a CTA, else
 // the narrowest that covers the tokens (at most 128), with K split over a cluster until the SMs are covered; further, up
 // to two CTAs per SM, where a part keeps a long run of K.
-void ChooseLinear(int t, int n, int chunks, int sms, int* index, int* splits) {
-  const int tiles = (n + kRowsM - 1) / kRowsM;
+void ChooseLinear(int t, int n, int heads, int chunks, int sms, int* index, int* splits) {
+  const int tiles = (n + kRowsM - 1) / kRowsM * heads;
   *splits = 1;
   if (t > 128 && tiles * ((t + 255) / 256) * 10 >= sms * 8) {
     *index = 4;
@@ -464,9 +486,13 @@ int PrepareLinear() {
 }
 
 bool EncodeLinear(LinearMaps* maps, const void* weight, uint64_t n, const void* activations, uint64_t rows, uint64_t k_stride) {
+  return EncodeHeads(maps, weight, n, k_stride, activations, rows, k_stride);
+}
+
+bool EncodeHeads(LinearMaps* maps, const void* weight, uint64_t n, uint64_t k_stride, const void* activations, uint64_t rows, uint64_t in_stride) {
   if (!EncodeMatrix(&maps->weight, false, weight, n, k_stride, kRowsM)) return false;
   for (int i = 0; i < 5; ++i)
-    if (!EncodeMatrix(&maps->rows[i], false, activations, rows, k_stride, 16u << i)) return false;
+    if (!EncodeMatrix(&maps->rows[i], false, activations, rows, in_stride, 16u << i)) return false;
   return true;
 }
 
@@ -478,7 +504,11 @@ int Linear(const Queue& q, const LinearArgs& a) {
   if (a.t <= 0) return 0;
   const bool experts = PerExpert(a.epilogue);
   if (experts && (a.slots.slots <= 0 || a.slots.tile_rows < 16 || !a.slots.tiles)) return int(cudaErrorInvalidValue);
+  if (a.epilogue == kLinearHeads ? a.heads < 1 || a.head_in % 8 != 0 || a.bias : a.heads != 0) return int(cudaErrorInvalidValue);
+  if (a.epilogue == kLinearExpertStore && !q.f32) return int(cudaErrorInvalidValue);
   LinearParams p{};
+  p.head_in = a.head_in;
+  p.head_out = a.head_out;
   p.bias = a.bias;
   p.out = a.out;
   p.t = a.t;
@@ -489,18 +519,19 @@ int Linear(const Queue& q, const LinearArgs& a) {
   p.slots = a.slots;
   p.status = q.status;
   if (q.f32) {
-    if (a.epilogue == kLinearGlu) return int(cudaErrorInvalidValue);   // two operations in fp32: the product, then GluRows
+    if (IsGlu(a.epilogue)) return int(cudaErrorInvalidValue);   // two operations in fp32: the product, then GluRows
     auto kernel = a.epilogue == kLinearAdd ? linear_f32<kLinearAdd> : a.epilogue == kLinearExpertUp ? linear_f32<kLinearExpertUp>
-                  : a.epilogue == kLinearExpertDown ? linear_f32<kLinearExpertDown> : linear_f32<kLinearStore>;
+                  : a.epilogue == kLinearExpertDown ? linear_f32<kLinearExpertDown>
+                  : a.epilogue == kLinearExpertStore ? linear_f32<kLinearExpertStore> : linear_f32<kLinearStore>;
     if (experts && a.slots.tile_rows != kTile32) return int(cudaErrorInvalidValue);
-    const dim3 grid(unsigned((a.n + kTile32 - 1) / kTile32), unsigned(experts ? MostTiles(a.slots) : (a.t + kTile32 - 1) / kTile32));
+    const dim3 grid(unsigned((a.n + kTile32 - 1) / kTile32), unsigned(experts ? MostTiles(a.slots) : (a.t + kTile32 - 1) / kTile32), unsigned(std::max(a.heads, 1)));
     return int(Launch(kernel, grid, dim3(256), 0, q.stream, q.chained, static_cast<const float*>(a.activations),
-                      static_cast<const float*>(a.weight), p, a.k_stride));
+                      static_cast<const float*>(a.weight), p, a.k_stride, a.in_stride ? a.in_stride : a.k_stride));
   }
   p.chunks = (a.k_stride + kStepK - 1) / kStepK;
   int index = 0, splits = 1;
   if (experts) ChooseExpertLinear(a.slots, a.n, p.chunks, q.sm_count, &index, &splits);
-  else ChooseLinear(a.t, a.n, p.chunks, q.sm_count, &index, &splits);
+  else ChooseLinear(a.t, a.n, std::max(a.heads, 1), p.chunks, q.sm_count, &index, &splits);
   p.chunks_per_split = (p.chunks + splits - 1) / splits;
   switch (index) {
     case 0: return int(LaunchTiles<16>(q, a, p, 0, splits));

@@ -23,6 +23,7 @@ struct AppendParams {
   const float *q_norm, *k_norm;
   float eps;
   Rotary rot;
+  Blend blend;
 };
 
 template <typename T>
@@ -44,7 +45,7 @@ __global__ void __launch_bounds__(128) rotate_append(StepRows r, T* proj, T* k_p
   }
   const T* values = p.value_is_key ? keys : keys + size_t(p.kv_heads) * p.dim;
   for (int i = threadIdx.x; i < p.kv_heads * p.vdim; i += 128)
-    v_pool[pool_offset(kv, i / p.vdim, p.kv_heads, p.v_pool_dim) + i % p.vdim] = values[i];
+    v_pool[pool_offset(kv, i / p.vdim, p.kv_heads, p.v_pool_dim) + i % p.vdim] = blended(p.blend, values, row, i);
   for (int i = threadIdx.x; i < (p.heads + p.kv_heads) * units; i += 128) {
     const int head = i / units, u = i % units, group = head - p.heads;
     if (u >= half && group < 0 && !p.q_norm) continue;      // (an entry of q that stays as it is)
@@ -79,8 +80,16 @@ __global__ void __launch_bounds__(256) rotate_append_wide(StepRows r, __nv_bfloa
   const __nv_bfloat16* keys = line + size_t(p.heads) * p.dim;
   const __nv_bfloat16* values = p.value_is_key ? keys : keys + size_t(p.kv_heads) * p.dim;
   const int v_units = p.vdim / 8;
-  for (int i = threadIdx.x; i < p.kv_heads * v_units; i += 256)
-    *reinterpret_cast<uint4*>(v_pool + pool_offset(kv, i / v_units, p.kv_heads, p.v_pool_dim) + i % v_units * 8) = reinterpret_cast<const uint4*>(values)[i];
+  for (int i = threadIdx.x; i < p.kv_heads * v_units; i += 256) {
+    uint4 word = reinterpret_cast<const uint4*>(values)[i];
+    if (p.blend.by) {
+      alignas(16) __nv_bfloat16 mixed[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) mixed[j] = blended(p.blend, values, row, 8 * i + j);
+      word = *reinterpret_cast<const uint4*>(mixed);
+    }
+    *reinterpret_cast<uint4*>(v_pool + pool_offset(kv, i / v_units, p.kv_heads, p.v_pool_dim) + i % v_units * 8) = word;
+  }
   float2 inv = make_float2(1.f, 1.f);
   if (p.q_norm) {
     const int q_count = p.heads * p.dim, k_count = p.kv_heads * p.dim;
@@ -129,25 +138,33 @@ __global__ void __launch_bounds__(256) rotate_append_wide(StepRows r, __nv_bfloa
 }
 
 // ---- attention, one warp per (row, query head) -------------------------------------------------------------------------
+// Queries are rows of q_stride, heads q_head apart; outputs likewise. MAXD: most columns of a head's query or value.
 constexpr int kPlainWarps = 4;
 
-template <typename T>
-__global__ void __launch_bounds__(32 * kPlainWarps) attend_rows(StepRows r, const T* proj, int stride, const T* k_pool, const T* v_pool, T* out,
-                                                                int out_stride, int heads, int kv_heads, int dim, int vdim, int pool_dim,
-                                                                int v_pool_dim, int window, int keep, float scale, float sink, int gate_at) {
-  __shared__ float qs[kPlainWarps][kMaxHeadDim];
+struct PlainAttend {
+  int q_stride, q_head, out_stride, out_head, heads, kv_heads, dim, vdim, pool_dim, v_pool_dim, window, keep;
+  float scale, sink;
+  const float* sinks;
+  int gate_at;
+};
+
+template <typename T, int MAXD>
+__global__ void __launch_bounds__(32 * kPlainWarps) attend_rows(StepRows r, const T* q, const T* k_pool, const T* v_pool, T* out, PlainAttend p) {
+  __shared__ float qs[kPlainWarps][MAXD];
   dependency_wait();
   allow_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.x * kPlainWarps + warp, row = blockIdx.y;
-  if (head >= heads) return;
-  const int group = head / (heads / kv_heads);
+  if (head >= p.heads) return;
+  const int group = head / (p.heads / p.kv_heads);
   const int position = r.row_position[row];
   const int slot = r.entry[r.row_entry[row]].slot;
   const int* table = r.block_table + size_t(slot) * r.max_blocks;
-  for (int d = lane; d < dim; d += 32) qs[warp][d] = to_f(proj[size_t(row) * stride + size_t(head) * dim + d]);
+  const T* line = q + size_t(row) * p.q_stride;
+  for (int d = lane; d < p.dim; d += 32) qs[warp][d] = to_f(line[size_t(head) * p.q_head + d]);
   __syncwarp();
-  constexpr int N = kMaxHeadDim / 32;
+  constexpr int N = MAXD / 32;
+  const float sink = p.sinks ? p.sinks[head] : p.sink;
   float acc[N] = {}, top = sink, sum = sink == -INFINITY ? 0.f : 1.f;   // (the null key, if there is one)
   auto walk = [&](int from, int to) {
     for (int base = from; base < to; base += 32) {
@@ -156,38 +173,53 @@ __global__ void __launch_bounds__(32 * kPlainWarps) attend_rows(StepRows r, cons
       float score = -INFINITY;
       if (j < to) {
         const int key = key_row(table, j, r);
-        const size_t at = pool_offset(key, group, kv_heads, pool_dim);
-        v_at = (long long)(pool_offset(key, group, kv_heads, v_pool_dim));
+        const size_t at = pool_offset(key, group, p.kv_heads, p.pool_dim);
+        v_at = (long long)(pool_offset(key, group, p.kv_heads, p.v_pool_dim));
         float dot = 0.f;
-        for (int d = 0; d < dim; ++d) dot = fmaf(qs[warp][d], to_f(k_pool[at + d]), dot);
-        score = dot * scale;
+        for (int d = 0; d < p.dim; ++d) dot = fmaf(qs[warp][d], to_f(k_pool[at + d]), dot);
+        score = dot * p.scale;
       }
       const float high = fmaxf(top, warp_max(score));
-      const float fade = expf(top - high), p = j < to ? expf(score - high) : 0.f;
-      sum = sum * fade + warp_sum(p);
+      const float fade = expf(top - high), w = j < to ? expf(score - high) : 0.f;
+      sum = sum * fade + warp_sum(w);
       top = high;
 #pragma unroll
       for (int i = 0; i < N; ++i) acc[i] *= fade;
       const int count = min(32, to - base);
       for (int jj = 0; jj < count; ++jj) {
-        const float weight = __shfl_sync(0xffffffffu, p, jj);
+        const float weight = __shfl_sync(0xffffffffu, w, jj);
         const T* v = v_pool + __shfl_sync(0xffffffffu, v_at, jj);
 #pragma unroll
         for (int i = 0; i < N; ++i)
-          if (lane + 32 * i < vdim) acc[i] = fmaf(weight, to_f(v[lane + 32 * i]), acc[i]);
+          if (lane + 32 * i < p.vdim) acc[i] = fmaf(weight, to_f(v[lane + 32 * i]), acc[i]);
       }
     }
   };
-  const int low = max(0, position - window + 1);
-  walk(0, min(keep, low));
+  const int low = max(0, position - p.window + 1);
+  walk(0, min(p.keep, low));
   walk(low, position + 1);
 #pragma unroll
   for (int i = 0; i < N; ++i) {
     const int c = lane + 32 * i;
-    if (c >= vdim) continue;
-    const float gate = gate_at < 0 ? 1.f : sigmoid(to_f(proj[size_t(row) * stride + gate_at + size_t(head) * vdim + c]));
-    out[size_t(row) * out_stride + size_t(head) * vdim + c] = from_f<T>(acc[i] / sum * gate);
+    if (c >= p.vdim) continue;
+    const float gate = p.gate_at < 0 ? 1.f : sigmoid(to_f(line[p.gate_at + size_t(head) * p.vdim + c]));
+    out[size_t(row) * p.out_stride + size_t(head) * p.out_head + c] = from_f<T>(acc[i] / sum * gate);
   }
+}
+
+// ---- latent rows: normed into the pool ------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(128) append_latent(StepRows r, const T* raw, int stride, T* pool, int pool_dim, int rank, const float* norm, float eps,
+                                                     bool portions_only) {
+  __shared__ float2 part[4];
+  dependency_wait();
+  allow_dependents();
+  const int row = blockIdx.x;
+  if (portions_only && r.entry[r.row_entry[row]].rows == 1) return;
+  const T* line = raw + size_t(row) * stride;
+  T* to = pool + pool_offset(r.row_kv[row], 0, 1, pool_dim);
+  const float inv = inverse_rms<128>(make_float2(square_sum(line, rank, 128), 0.f), rank, 1, eps, part).x;
+  for (int d = threadIdx.x; d < rank; d += 128) to[d] = from_f<T>(to_f(line[d]) * inv * norm[d]);
 }
 
 // ---- retention by its recurrence ----------------------------------------------------------------------------------------
@@ -384,7 +416,8 @@ __global__ void __launch_bounds__(128) retention_gate(const float* raw, const T*
 }
 
 template <typename T> int RotateAppendAs(const Queue& q, const StepRows& r, const AttentionArgs& a) {
-  const AppendParams p{a.proj_stride, a.heads, a.kv_heads, a.dim, a.vdim, a.pool_dim, a.v_pool_dim, a.value_is_key, a.q_norm, a.k_norm, a.eps, a.rotary};
+  const AppendParams p{a.proj_stride, a.heads, a.kv_heads, a.dim, a.vdim, a.pool_dim, a.v_pool_dim, a.value_is_key, a.q_norm, a.k_norm, a.eps, a.rotary,
+                       {a.blend, a.blend_from, a.blend_stride}};
   if constexpr (sizeof(T) == 2) {
     if (a.dim % 8 == 0 && a.vdim % 8 == 0 && a.rotary.dims % 16 == 0 && a.proj_stride % 8 == 0)
       return int(Launch(rotate_append_wide, dim3(unsigned(r.rows)), dim3(256), 0, q.stream, q.chained, r, static_cast<T*>(a.proj),
@@ -394,11 +427,27 @@ template <typename T> int RotateAppendAs(const Queue& q, const StepRows& r, cons
                     static_cast<T*>(a.k_pool), static_cast<T*>(a.v_pool), p, !q.f32));
 }
 
+dim3 PlainGrid(int heads, int rows) { return dim3(unsigned((heads + kPlainWarps - 1) / kPlainWarps), unsigned(rows)); }
+
 template <typename T> int AttendAs(const Queue& q, const StepRows& r, const AttentionArgs& a) {
-  const dim3 grid(unsigned((a.heads + kPlainWarps - 1) / kPlainWarps), unsigned(r.rows));
-  return int(Launch(attend_rows<T>, grid, dim3(32 * kPlainWarps), 0, q.stream, q.chained, r, static_cast<const T*>(a.proj), a.proj_stride,
-                    static_cast<const T*>(a.k_pool), static_cast<const T*>(a.v_pool), static_cast<T*>(a.out), a.out_stride, a.heads,
-                    a.kv_heads, a.dim, a.vdim, a.pool_dim, a.v_pool_dim, a.window, a.keep, a.scale, a.sink, a.gate_at));
+  const PlainAttend p{a.proj_stride, a.dim, a.out_stride, a.vdim, a.heads, a.kv_heads, a.dim, a.vdim, a.pool_dim, a.v_pool_dim, a.window, a.keep,
+                      a.scale, a.sink, a.sinks, a.gate_at};
+  return int(Launch(attend_rows<T, kMaxHeadDim>, PlainGrid(a.heads, r.rows), dim3(32 * kPlainWarps), 0, q.stream, q.chained, r,
+                    static_cast<const T*>(a.proj), static_cast<const T*>(a.k_pool), static_cast<const T*>(a.v_pool), static_cast<T*>(a.out), p));
+}
+
+template <typename T> int AttendLatentAs(const Queue& q, const StepRows& r, const LatentArgs& a) {
+  const int stride = a.heads * a.rank_stride;
+  const PlainAttend p{stride, a.rank_stride, stride, a.rank_stride, a.heads, 1, a.rank, a.rank, a.pool_dim, a.pool_dim, a.window, 0,
+                      a.scale, a.sink, a.sinks, -1};
+  auto kernel = a.rank <= kMaxHeadDim ? attend_rows<T, kMaxHeadDim> : attend_rows<T, kMaxLatent>;
+  return int(Launch(kernel, PlainGrid(a.heads, r.rows), dim3(32 * kPlainWarps), 0, q.stream, q.chained, r, static_cast<const T*>(a.q),
+                    static_cast<const T*>(a.pool), static_cast<const T*>(a.pool), static_cast<T*>(a.out), p));
+}
+
+template <typename T> int AppendLatentAs(const Queue& q, const StepRows& r, const LatentArgs& a, bool portions_only) {
+  return int(Launch(append_latent<T>, dim3(unsigned(r.rows)), dim3(128), 0, q.stream, q.chained, r, static_cast<const T*>(a.raw), a.raw_stride,
+                    static_cast<T*>(a.pool), a.pool_dim, a.rank, a.norm, a.eps, portions_only));
 }
 
 template <typename T> int RetainAs(const Queue& q, const StepRows& r, const RetentionArgs& a, bool singles_only) {
@@ -438,6 +487,14 @@ int RotateAppend(const Queue& q, const StepRows& r, const AttentionArgs& a) {
 
 int Attend(const Queue& q, const StepRows& r, const AttentionArgs& a) {
   return q.f32 ? AttendAs<float>(q, r, a) : AttendTiles(q, r, a);
+}
+
+int AppendLatent(const Queue& q, const StepRows& r, const LatentArgs& a) {
+  return q.f32 ? AppendLatentAs<float>(q, r, a, false) : AppendLatentAs<__nv_bfloat16>(q, r, a, false);
+}
+
+int AttendLatent(const Queue& q, const StepRows& r, const LatentArgs& a) {
+  return q.f32 ? AttendLatentAs<float>(q, r, a) : AttendLatentAs<__nv_bfloat16>(q, r, a);
 }
 
 int Retain(const Queue& q, const StepRows& r, const RetentionArgs& a) {

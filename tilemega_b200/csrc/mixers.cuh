@@ -71,6 +71,19 @@ __device__ __forceinline__ float2 inverse_rms(float2 squares, int count_a, int c
   return make_float2(1.f / sqrtf(sum.x / float(count_a) + eps), 1.f / sqrtf(sum.y / float(count_b) + eps));
 }
 
+// A layer's values blended with those of another layer for the same rows, see AttentionArgs.
+struct Blend {
+  const float* by = nullptr;         // null: the layer's own as they are
+  const void* from = nullptr;
+  int stride = 0;
+};
+// Value i (of kv_heads x vdim) of a row; `own` points to the row's first.
+template <typename T> __device__ __forceinline__ T blended(const Blend& b, const T* own, int row, int i) {
+  if (!b.by) return own[i];
+  const float f = *b.by;
+  return from_f<T>((1.f - f) * to_f(own[i]) + f * to_f(static_cast<const T*>(b.from)[size_t(row) * b.stride + i]));
+}
+
 __device__ __forceinline__ float sigmoid(float v) { return 1.f / (1.f + expf(-v)); }
 
 }  // namespace tmb

@@ -69,6 +69,9 @@ struct AttendParams {
   float scale_log2, sink_log2, eps;
   bool value_is_key, even;
   Rotary rotary;
+  Blend blend;
+  const float* sinks;
+  __device__ float sink_of(int head) const { return sinks ? sinks[head] * 1.4426950408889634f : sink_log2; }
 };
 
 template <int DT, int WM> struct AttendShape {
@@ -231,7 +234,7 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
         if (first_head == 0) k_to[d] = kd;
       }
       for (int d = threadIdx.x; d < p.vdim; d += NT) {
-        const bf16 vd = v[d];
+        const bf16 vd = blended(p.blend, v - size_t(group) * p.vdim, e.first_row, group * p.vdim + d);
         vs[stage * Shape::kTile + key * P + d] = vd;
         if (first_head == 0) v_to[d] = vd;
       }
@@ -329,12 +332,13 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
   }
   if constexpr (WM > 1) {
     // (a null key that stands above every key takes the maximum's place: the values then count by the distance)
-    auto share = [&](float top, float sum) {
-      if (p.sink_log2 == -INFINITY) return 1.f / sum;
-      const float high = fmaxf(top, p.sink_log2), f = ex2(top - high);
-      return f / fmaf(sum, f, ex2(p.sink_log2 - high));
+    auto share = [&](int m, float top, float sum) {
+      const float sink = p.sink_of(head0 + m % gq);
+      if (sink == -INFINITY) return 1.f / sum;
+      const float high = fmaxf(top, sink), f = ex2(top - high);
+      return f / fmaf(sum, f, ex2(sink - high));
     };
-    const float inv_a = share(top_a, sum_a), inv_b = share(top_b, sum_b);
+    const float inv_a = share(ra, top_a, sum_a), inv_b = share(rb, top_b, sum_b);
     auto write = [&](int m, float inv, int i, int at) {
       const int t = m / gq, c = i * 8 + 2 * (lane & 3);
       if (t >= tokens || c >= p.vdim) return;
@@ -391,7 +395,8 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
     float* parts = p.part + (size_t(blockIdx.z) * p.heads + head0) * p.splits * record;   // [head of the unit][split][record]
     for (int i = threadIdx.x; i < gq * p.vdim; i += NT) {
       const int h = i / p.vdim, c = i % p.vdim;
-      float high = p.splits == 1 ? p.sink_log2 : -INFINITY, sum = 0.f, value = 0.f;
+      const float sink = p.sink_of(head0 + h);
+      float high = p.splits == 1 ? sink : -INFINITY, sum = 0.f, value = 0.f;
 #pragma unroll
       for (int w = 0; w < 4; ++w) high = fmaxf(high, ms[w * 16 + h]);
       const float ref = high == -INFINITY ? 0.f : high;
@@ -402,7 +407,7 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
         value = fmaf(os[(w * 16 + h) * D + c], f, value);
       }
       if (p.splits == 1) {
-        dst[i] = gated(value / (sum + ex2(p.sink_log2 - ref)), i);
+        dst[i] = gated(value / (sum + ex2(sink - ref)), i);
       } else {
         float* mine = parts + (size_t(h) * p.splits + split) * record;
         mine[2 + c] = value;
@@ -429,9 +434,10 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
       if (int(threadIdx.x) < gq) {
         float* f = factor + threadIdx.x * p.splits;
         const float* l = f + gq * p.splits;
-        float high = p.sink_log2;
+        const float sink = p.sink_of(head0 + int(threadIdx.x));
+        float high = sink;
         for (int s = 0; s < p.splits; ++s) high = fmaxf(high, f[s]);
-        float sum = ex2(p.sink_log2 - high);
+        float sum = ex2(sink - high);
         for (int s = 0; s < p.splits; ++s) {         // in split order
           f[s] = ex2(f[s] - high);
           sum = fmaf(l[s], f[s], sum);
@@ -831,6 +837,8 @@ int AttendTiles(const Queue& q, const StepRows& r, const AttentionArgs& a) {
   p.subs = (gq + p.sub_heads - 1) / p.sub_heads;
   p.scale_log2 = a.scale * 1.4426950408889634f;
   p.sink_log2 = a.sink * 1.4426950408889634f;
+  p.sinks = a.sinks;
+  p.blend = {a.blend, a.blend_from, a.blend_stride};
   const int tiles = (std::max(a.dim, a.vdim) + 15) / 16;
   return tiles <= 2 ? AttendWith<2>(q, r, a, p) : tiles <= 4 ? AttendWith<4>(q, r, a, p) : tiles <= 6 ? AttendWith<6>(q, r, a, p)
          : tiles <= 8 ? AttendWith<8>(q, r, a, p) : tiles <= 12 ? AttendWith<12>(q, r, a, p) : AttendWith<16>(q, r, a, p);

@@ -37,8 +37,9 @@ struct StepRows {
   int* row_kv = nullptr;                    // [rows] pool row: block * 16 + position mod 16
 };
 
-// x[row] = embed[token] (and as an element in `copy`, rows of copy_stride, unless null); the row tables.
-int StartStep(const Queue& q, const StepRows& r, const int* tokens, const void* embed, float* x, void* copy, int copy_stride, int width, int vocab);
+// Each of the `streams` copies of x[row] = embed[token] (and as an element in `copy`, rows of copy_stride, unless null); the row tables.
+int StartStep(const Queue& q, const StepRows& r, const int* tokens, const void* embed, float* x, int streams, void* copy, int copy_stride, int width,
+              int vocab);
 
 // out[i] = x[r] / sqrt(mean(x[r]^2) + eps) * weight, r = select ? select[i] : i. With `again`, x[r] += embed[token[r]]
 // first (and is written back). Rows of `out` are out_stride elements apart.
@@ -68,6 +69,31 @@ struct AddNormArgs {
 };
 int AddNorm(const Queue& q, const AddNormArgs& a);
 
+// One row operation between two sublayers of a model with residual streams x [row][streams][width]:
+//   update    x_t <- sum_s mix[s][t] x_s + out[t] y    (mix null: x_t itself, out null: 1), all t from the old streams
+//   collect   u = sum_t in[t] x_t (in null: 1), normed[i] = u / sqrt(mean(u^2) + eps) * weight, as elements
+// y = the weighted sum of `parts` elements rows, parts_of[i * parts + k] by part_scale[i * parts + k], plus branch[i] (fp32)
+// times sigmoid(branch_gate[i * gate_stride]) (null: 1); either may be absent. Without an update a row may be chosen:
+// r = select[i]. sum_of (or null): the streams' plain sum after the update.
+struct StreamArgs {
+  float* x;
+  int streams, rows, width, limit;
+  bool update;
+  const float *mix, *out;
+  const void* parts_of;
+  const float* part_scale;
+  int parts;
+  const float *branch, *branch_gate;
+  int gate_stride;
+  float* sum_of;
+  const float *in, *weight;  // weight null: no collect
+  void* normed;
+  int normed_stride;
+  const int* select;
+  float eps;
+};
+int StreamStep(const Queue& q, const StreamArgs& a);
+
 // Rotary table [capacity][dims / 2] of (cos, sin), or dims = 0: none.
 struct Rotary {
   const float2* table = nullptr;
@@ -81,7 +107,8 @@ struct Glu {
   bool gelu = false;
 };
 
-enum LinearEpilogue { kLinearStore = 0, kLinearAdd = 1, kLinearGlu = 2, kLinearFloat = 3, kLinearExpertUp = 4, kLinearExpertDown = 5 };
+enum LinearEpilogue { kLinearStore = 0, kLinearAdd = 1, kLinearGlu = 2, kLinearFloat = 3, kLinearExpertUp = 4, kLinearExpertDown = 5,
+                      kLinearHeads = 6, kLinearExpertGlu = 7, kLinearExpertStore = 8 };
 
 // The assignments of a step's rows to experts, sorted by expert (written by Route). Assignment a is the a % top-th choice
 // of row a / top; slot s, in sorted order, runs assignment list[s] on the expert of its tile.
@@ -101,7 +128,10 @@ struct ExpertSlots {
 // Activation and weight rows are k_stride elements long (a multiple of 8, zero weights behind k).
 // Per expert (weight rows expert * n ..., slots in place of t): ExpertUp reads activation row list[s] / top for slot s
 // (from `activations`; bf16 tiles of more than kGatherRows slots read row s of rows gathered before, see GatherRows) and
-// stores relu(score[s] D)^2 in row s; ExpertDown reads row s and stores D in row list[s]; both as elements.
+// stores relu(score[s] D)^2 in row s; ExpertGlu reads the same and stores the gated unit, ExpertStore (fp32) D itself;
+// ExpertDown reads row s and stores D in row list[s]; all as elements.
+// Heads: `heads` products side by side, head h of weight rows h * n ..., activation columns h * head_in ... and output
+// columns h * head_out ... (head_in a multiple of 8; n and k are one head's), stored as elements.
 constexpr int kGatherRows = 32;
 struct LinearMaps {
   CUtensorMap weight;        // bf16 only: 128-row boxes
@@ -115,6 +145,8 @@ struct LinearArgs {
   void* out;                 // element buffer, or the fp32 residual stream, or fp32
   const LinearMaps* maps;    // bf16 only
   int t, n, k_stride, out_stride;
+  int in_stride;             // elements of an activation row, if it is not k_stride (0)
+  int heads, head_in, head_out;   // kLinearHeads
   int outputs;               // kLinearGlu: columns stored (pairs beyond it are padding)
   int epilogue;
   Glu glu;
@@ -123,20 +155,28 @@ struct LinearArgs {
 int ExpertTileRows(const Queue& q, int slots, int experts);   // slots per tile that suits this many
 int PrepareLinear();         // raises the kernels' shared-memory limits (once per device)
 bool EncodeLinear(LinearMaps* maps, const void* weight, uint64_t n, const void* activations, uint64_t rows, uint64_t k_stride);
+bool EncodeHeads(LinearMaps* maps, const void* weight, uint64_t n, uint64_t k_stride, const void* activations, uint64_t rows, uint64_t in_stride);
 bool EncodeGathered(LinearMaps* maps, const void* activations, uint64_t rows, uint64_t k_stride);   // maps->row only
 int Linear(const Queue& q, const LinearArgs& a);
 
 // The gated unit by itself: in [t][2 * padded] interleaved pairs, out [t][outputs].
 int GluRows(const Queue& q, const void* in, void* out, int t, int in_stride, int out_stride, int outputs, const Glu& glu);
 
-// Mixture of experts: the `top` largest of z = router h per row (the smaller index on a tie), scores sigmoid(z), and the
+// Mixture of experts: per row z = router h, scores sigmoid(z) or softmax(z) over the experts, and the `top` largest of score
+// + correction (null: 0; the smaller index on a tie) among the keep_groups groups of neighbours whose largest is largest.
+// `weights`: the scores handed on are over their sum (+ 1e-20). `extra` more router rows are only multiplied. And the
 // assignments sorted by expert in tiles of slots->tile_rows. RouteFused: does Route compute z itself? (If not, the
 // caller has put it into `logits`.)
 struct RouteArgs {
   const void* h;             // elements, rows of k_stride
   const void* router;        // [experts][k_stride]
   int k_stride, rows, experts, top, tile_rows;
-  float* logits;             // [rows][experts]
+  int extra;
+  bool softmax, weights;
+  const float* correction;
+  int groups, keep_groups;
+  float* ranks;              // [rows][experts], scratch (softmax scores, corrections or groups)
+  float* logits;             // [rows][experts + extra]
   int* choice;               // [rows * top]
   float* score;              // [rows * top]
   int* list;                 // [rows * top], sorted
@@ -154,7 +194,8 @@ int GatherRows(const Queue& q, const void* h, int k_stride, const ExpertSlots& s
 // Attention with grouped heads, a sliding window of `window` positions and the first `keep` positions always seen.
 // proj rows hold q | k (| v) (| g): q heads x dim, k kv_heads x dim, v kv_heads x vdim, g heads x vdim; the values are v,
 // or k before rotation (value_is_key). q_norm / k_norm: RMS norm over all heads together before the rotation. A null key
-// of score `sink` (-infinity: none) without a value joins the softmax. gate_at >= 0: outputs times sigmoid(g).
+// of score `sink` (-infinity: none), or of sinks[head], without a value joins the softmax. Values are blended with
+// blend_from, those of another layer for the same rows: (1 - *blend) v + *blend * theirs. gate_at >= 0: outputs times sigmoid(g).
 struct AttentionArgs {
   void* proj;
   int proj_stride;
@@ -167,6 +208,10 @@ struct AttentionArgs {
   const float* q_norm;       // [heads * dim], or null
   const float* k_norm;       // [kv_heads * dim]
   float eps, sink;
+  const float* sinks;        // [heads], or null
+  const float* blend;        // or null
+  const void* blend_from;    // element rows of blend_stride, kv_heads x vdim
+  int blend_stride;
   int gate_at;               // first gate column of a projected row, or -1
   int window, keep;
   float scale;
@@ -182,6 +227,29 @@ int RotateAppend(const Queue& q, const StepRows& r, const AttentionArgs& a);
 int Attend(const Queue& q, const StepRows& r, const AttentionArgs& a);
 int AttendTiles(const Queue& q, const StepRows& r, const AttentionArgs& a);   // the bf16 form
 int PrepareMixers();
+
+// Attention whose keys and values are images, per head, of one cached latent row per token: scores and sums are taken
+// against the latent rows themselves, with queries `q` already multiplied by their heads' key matrices; `out` rows are the
+// heads' weighted sums of latent rows, for the heads' value matrices to follow. latent rows come from `raw` ([rows] of
+// raw_stride, normed by AppendLatent on their way into the pool).
+struct LatentArgs {
+  const void* q;             // [rows][heads][rank_stride]
+  void* out;                 // [rows][heads][rank_stride]
+  const void* raw;
+  int raw_stride;
+  const float* norm;         // [rank]
+  void* pool;                // [num_blocks][16][pool_dim]
+  int heads, rank, rank_stride, pool_dim;
+  float eps, scale, sink;
+  const float* sinks;        // [heads], or null
+  int window;
+  float* part;               // decode partials, part_floats floats
+  size_t part_floats;
+  unsigned* count;           // arrival counters, zero between launches
+  int count_words;
+};
+int AppendLatent(const Queue& q, const StepRows& r, const LatentArgs& a);
+int AttendLatent(const Queue& q, const StepRows& r, const LatentArgs& a);
 
 // Retention: per head S <- decay S + k v^T, o = S^T q, with rotary q and k, k scaled by key_scale. proj rows hold
 // q | k | v | g. state [slots][heads][dim][vdim] fp32; an entry that starts at position 0 starts from a zero state.

@@ -23,6 +23,9 @@ struct RaggedPlan {
   void* picked = nullptr;      // [max_wanted][padded width]: normed rows the head scores
   void* proj = nullptr;        // [max_rows][widest input projection]
   void* mixed = nullptr;       // [max_rows][widest mixer output]
+  void* source = nullptr;      // [max_rows][its input projection]: the projected rows of the layer whose values others blend in
+  int source_stride = 0, source_at = 0;   // ... and where its values start in a row
+  void *lookup = nullptr, *looked = nullptr;   // latent attention: queries against latent rows, weighted sums of latent rows
   void* mlp = nullptr;         // [max_rows][widest feed-forward]
   void* pairs = nullptr;       // fp32 plans: gate/up rows before the gated unit
   float* branch = nullptr;     // fp32 outputs of sublayers that are normed before they are added
@@ -33,6 +36,8 @@ struct RaggedPlan {
   ExpertTile* tiles = nullptr;
   unsigned* route_count = nullptr;
   void* gathered = nullptr;        // bf16 plans: [max_rows * most experts of a token][padded width]
+  float* ranks = nullptr;          // [max_rows][most experts]
+  void* expert_pairs = nullptr;    // fp32 plans: gate/up rows of experts before the gated unit
   void* expert_hidden = nullptr;   // [max_rows * most experts of a token][widest expert]
   void* expert_out = nullptr;      // [max_rows * most experts of a token][width]
   float* raw = nullptr;        // retention outputs before their norm
@@ -44,6 +49,7 @@ struct RaggedPlan {
   std::vector<float*> decay;   // per layer
   struct Maps {
     LinearMaps in, out, gate_up, down, router;   // (gate_up, down: of the gated unit or of the experts)
+    LinearMaps shared_up, shared_down, key_up, value_up;
   };
   std::vector<Maps> maps;      // per layer (bf16 plans)
   LinearMaps head;
@@ -83,7 +89,7 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     if (status_ != 0) return status_; \
   } while (0)
   const bool norm_output = s.layers[0].norm_output;   // sublayers then read the stream itself: `normed` holds it as elements
-  TMB_TRY(StartStep(q, r, tokens, buffer(s.embed), x, norm_output ? plan->normed : nullptr, W8, W, s.vocab));
+  TMB_TRY(StartStep(q, r, tokens, buffer(s.embed), x, s.streams, norm_output ? plan->normed : nullptr, W8, W, s.vocab));
   auto norm = [&](int weight, bool again) {
     NormArgs a{};
     a.x = x;
@@ -115,7 +121,7 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
   };
   // a sublayer's last product (rows of `in` times `weight`): added to the stream, or normed and added
   auto add_output = [&](const void* in, int weight, int bias, const LinearMaps* maps, int k) {
-    if (!norm_output) return Linear(q, linear(in, weight, bias, maps, W, k, x, W, kLinearAdd));
+    if (!norm_output && !s.combined) return Linear(q, linear(in, weight, bias, maps, W, k, x, W, kLinearAdd));
     return Linear(q, linear(in, weight, bias, maps, W, k, plan->branch, W, kLinearFloat));
   };
   auto add_norm = [&](int weight, int parts) {
@@ -132,14 +138,54 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     a.eps = float(s.eps);
     return AddNorm(q, a);
   };
+  // Several streams (combined): one row operation adds a sublayer's output and collects what the next one reads. `done`: the
+  // sublayer that ran (null: none yet), `next`: the one to come (null: the model's end).
+  StreamArgs step{};
+  step.x = x;
+  step.streams = s.streams;
+  step.rows = step.limit = r.rows;
+  step.width = W;
+  step.normed = plan->normed;
+  step.normed_stride = W8;
+  step.eps = float(s.eps);
+  auto restream = [&](const RaggedStreams* done, const RaggedMlp* mixture, const RaggedStreams* next, int norm_weight, float* sum_of) {
+    StreamArgs a = step;
+    if (done) {
+      a.update = true;
+      a.mix = floats(done->mix);
+      a.out = floats(done->out);
+      a.branch = plan->branch;
+      if (mixture) {
+        a.parts_of = plan->expert_out;
+        a.part_scale = plan->score;
+        a.parts = mixture->top;
+        a.branch = mixture->shared_ff ? plan->branch : nullptr;
+        a.branch_gate = mixture->shared_ff ? plan->logits + mixture->experts : nullptr;
+        a.gate_stride = mixture->logits();
+      }
+    }
+    if (next) {
+      a.in = floats(next->in);
+      a.weight = floats(norm_weight);
+    }
+    a.sum_of = sum_of;
+    return StreamStep(q, a);
+  };
+  if (s.combined) {
+    const RaggedLayer& first = s.layers[size_t(s.runs[0].layer)];
+    TMB_TRY(restream(nullptr, nullptr, &first.streams[0], first.norm1, nullptr));
+  }
   for (size_t i = 0; i < s.runs.size(); ++i) {
     const RaggedRun& run = s.runs[i];
+    const RaggedLayer* next = i + 1 < s.runs.size() ? &s.layers[size_t(s.runs[i + 1].layer)] : nullptr;
+    float* kept = s.write_residuals ? floats(s.residuals) + i * size_t(s.max_rows) * W : nullptr;
     const RaggedLayer& layer = s.layers[size_t(run.layer)];
     const RaggedMixer& m = layer.mixer;
     const RaggedPlan::Maps* maps = s.f32 ? nullptr : &plan->maps[size_t(run.layer)];
     const int stride = (m.proj_rows() + 7) / 8 * 8, mixed_stride = padded_columns(m.out_columns());
-    if (!norm_output) TMB_TRY(norm(layer.norm1, run.add_embedding));
-    TMB_TRY(Linear(q, linear(plan->normed, layer.in_weight, layer.in_bias, maps ? &maps->in : nullptr, m.proj_rows(), W, plan->proj, stride, kLinearStore)));
+    if (!norm_output && !s.combined) TMB_TRY(norm(layer.norm1, run.add_embedding));
+    void* proj = m.value_mix == RaggedMixer::kSource ? plan->source : plan->proj;
+    TMB_TRY(Linear(q, linear(plan->normed, layer.in_weight, layer.in_bias, maps ? &maps->in : nullptr, m.proj_rows(), W, proj, stride, kLinearStore)));
     Rotary rotary;
     if (m.rotary >= 0) {
       rotary.table = static_cast<const float2*>(buffer(s.rotaries[size_t(m.rotary)].buffer));
@@ -163,9 +209,45 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.eps = float(s.eps);
       a.rotary = rotary;
       TMB_TRY(Retain(q, r, a));
+    } else if (m.kind == RaggedMixer::kLatent) {
+      LatentArgs a{};
+      a.q = plan->lookup;
+      a.out = plan->looked;
+      a.raw = static_cast<const char*>(proj) + size_t(m.heads) * m.head_stride() * (s.f32 ? 4 : 2);
+      a.raw_stride = stride;
+      a.norm = floats(layer.latent_norm);
+      a.pool = buffer(run.k_pool);
+      a.heads = m.heads;
+      a.rank = m.rank;
+      a.rank_stride = m.rank_stride();
+      a.pool_dim = m.pool_dim();
+      a.eps = float(s.eps);
+      a.scale = float(m.scale);
+      a.sink = -INFINITY;
+      a.sinks = floats(layer.sinks);
+      a.window = m.window;
+      a.part = plan->part;
+      a.part_floats = plan->part_floats;
+      a.count = plan->count;
+      a.count_words = plan->count_words;
+      const int wide = m.heads * m.rank_stride();
+      TMB_TRY(AppendLatent(q, r, a));
+      LinearArgs up = linear(proj, layer.key_up, -1, maps ? &maps->key_up : nullptr, m.rank, m.head_stride(), plan->lookup, wide, kLinearHeads);
+      up.in_stride = stride;
+      up.heads = m.heads;
+      up.head_in = m.head_stride();
+      up.head_out = m.rank_stride();
+      TMB_TRY(Linear(q, up));
+      TMB_TRY(AttendLatent(q, r, a));
+      LinearArgs down = linear(plan->looked, layer.value_up, -1, maps ? &maps->value_up : nullptr, m.vdim, m.rank, plan->mixed, mixed_stride, kLinearHeads);
+      down.in_stride = wide;
+      down.heads = m.heads;
+      down.head_in = m.rank_stride();
+      down.head_out = m.vdim;
+      TMB_TRY(Linear(q, down));
     } else {
       AttentionArgs a{};
-      a.proj = plan->proj;
+      a.proj = proj;
       a.proj_stride = stride;
       a.k_pool = buffer(run.k_pool);
       a.v_pool = buffer(run.v_pool);
@@ -181,6 +263,10 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.k_norm = floats(layer.k_norm);
       a.eps = float(s.eps);
       a.sink = m.sink ? float(m.sink_score) : -INFINITY;
+      a.sinks = floats(layer.sinks);
+      a.blend = floats(layer.blend);
+      a.blend_from = static_cast<const char*>(plan->source) + size_t(plan->source_at) * (s.f32 ? 4 : 2);
+      a.blend_stride = plan->source_stride;
       a.gate_at = m.gate_at();
       a.value_is_key = m.value_is_key;
       a.window = m.window;
@@ -197,10 +283,16 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     TMB_TRY(add_output(plan->mixed, layer.out_weight, layer.out_bias, maps ? &maps->out : nullptr, m.out_columns()));
     if (norm_output) TMB_TRY(add_norm(layer.norm1, 0));
     const RaggedMlp& mlp = layer.mlp;
+    // what follows the mixer and what follows the layer, on several streams
+    const bool last = mlp.kind == RaggedMlp::kNone;
+    auto leave = [&](const RaggedStreams* done, const RaggedMlp* mixture) {
+      return restream(done, mixture, next ? &next->streams[0] : nullptr, next ? next->norm1 : -1, kept);
+    };
+    if (s.combined) TMB_TRY(last ? leave(&layer.streams[0], nullptr) : restream(&layer.streams[0], nullptr, &layer.streams[1], layer.norm2, nullptr));
     if (mlp.kind == RaggedMlp::kGlu) {
       const Glu glu{float(mlp.limit), float(mlp.alpha), float(mlp.shift), mlp.gelu};
       const int packed = mlp.packed_rows(), mlp_stride = padded_columns(mlp.ff);
-      if (!norm_output) TMB_TRY(norm(layer.norm2, false));
+      if (!norm_output && !s.combined) TMB_TRY(norm(layer.norm2, false));
       if (s.f32) {
         TMB_TRY(Linear(q, linear(plan->normed, layer.gate_up, -1, nullptr, packed, W, plan->pairs, packed, kLinearStore)));
         TMB_TRY(GluRows(q, plan->pairs, plan->mlp, r.rows, packed, mlp_stride, mlp.ff, glu));
@@ -212,6 +304,7 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       }
       TMB_TRY(add_output(plan->mlp, layer.down, -1, maps ? &maps->down : nullptr, mlp.ff));
       if (norm_output) TMB_TRY(add_norm(layer.norm2, 0));
+      if (s.combined) TMB_TRY(leave(&layer.streams[1], nullptr));
     } else if (mlp.kind == RaggedMlp::kExperts) {
       ExpertSlots slots;
       slots.tiles = plan->tiles;
@@ -230,6 +323,13 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.experts = mlp.experts;
       a.top = mlp.top;
       a.tile_rows = slots.tile_rows;
+      a.extra = mlp.logits() - mlp.experts;
+      a.softmax = mlp.softmax;
+      a.weights = mlp.output_weighted;
+      a.correction = floats(layer.correction);
+      a.groups = mlp.groups;
+      a.keep_groups = mlp.keep_groups;
+      a.ranks = mlp.output_weighted ? plan->ranks : nullptr;
       a.logits = plan->logits;
       a.choice = plan->choice;
       a.score = plan->score;
@@ -239,36 +339,70 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.tile_count = plan->tile_count;
       a.count = plan->route_count;
       if (!RouteFused(r.rows))
-        TMB_TRY(Linear(q, linear(plan->normed, layer.router, -1, maps ? &maps->router : nullptr, mlp.experts, W, plan->logits, mlp.experts, kLinearFloat)));
+        TMB_TRY(Linear(q, linear(plan->normed, layer.router, -1, maps ? &maps->router : nullptr, mlp.logits(), W, plan->logits, mlp.logits(), kLinearFloat)));
       TMB_TRY(Route(q, a));
       if (!s.f32 && slots.tile_rows > kGatherRows) TMB_TRY(GatherRows(q, plan->normed, W8, slots, plan->gathered));
       const int stride = padded_columns(mlp.ff);
+      const Glu glu{float(mlp.limit), float(mlp.alpha), float(mlp.shift), false};
       LinearArgs up = linear(plan->normed, layer.expert_up, -1, maps ? &maps->gate_up : nullptr, mlp.ff, W, plan->expert_hidden, stride, kLinearExpertUp);
       up.slots = slots;
+      if (mlp.output_weighted) {
+        up.n = mlp.packed_rows();
+        up.epilogue = s.f32 ? kLinearExpertStore : kLinearExpertGlu;
+        up.outputs = mlp.ff;
+        up.glu = glu;
+        if (s.f32) {
+          up.out = plan->expert_pairs;
+          up.out_stride = up.n;
+        }
+      }
       TMB_TRY(Linear(q, up));
+      if (mlp.output_weighted && s.f32) TMB_TRY(GluRows(q, plan->expert_pairs, plan->expert_hidden, slots.slots, up.n, stride, mlp.ff, glu));
       LinearArgs down = linear(plan->expert_hidden, layer.expert_down, -1, maps ? &maps->down : nullptr, W, mlp.ff, plan->expert_out, W, kLinearExpertDown);
       down.slots = slots;
       TMB_TRY(Linear(q, down));
-      TMB_TRY(add_norm(layer.norm2, mlp.top));
+      if (norm_output) TMB_TRY(add_norm(layer.norm2, mlp.top));
+      if (mlp.shared_ff) {
+        const Glu unit{float(mlp.shared_limit), float(mlp.alpha), float(mlp.shift), false};
+        const int packed = mlp.shared_rows(), unit_stride = padded_columns(mlp.shared_ff);
+        LinearArgs first = linear(plan->normed, layer.shared_up, -1, maps ? &maps->shared_up : nullptr, packed, W, s.f32 ? plan->pairs : plan->mlp,
+                                  s.f32 ? packed : unit_stride, s.f32 ? kLinearStore : kLinearGlu);
+        first.outputs = mlp.shared_ff;
+        first.glu = unit;
+        TMB_TRY(Linear(q, first));
+        if (s.f32) TMB_TRY(GluRows(q, plan->pairs, plan->mlp, r.rows, packed, unit_stride, mlp.shared_ff, unit));
+        TMB_TRY(add_output(plan->mlp, layer.shared_down, -1, maps ? &maps->shared_down : nullptr, mlp.shared_ff));
+      }
+      if (s.combined) TMB_TRY(leave(&layer.streams[1], &mlp));
     }
-    if (s.write_residuals) {
-      const cudaError_t err = cudaMemcpyAsync(floats(s.residuals) + i * size_t(s.max_rows) * W, x, size_t(rows) * W * sizeof(float),
+    if (kept && !s.combined) {
+      const cudaError_t err = cudaMemcpyAsync(kept, x, size_t(rows) * W * sizeof(float),
                                               cudaMemcpyDeviceToDevice, stream);
       if (err != cudaSuccess) return int(err);
     }
   }
   if (wanted) {
-    NormArgs a{};
-    a.x = x;
-    a.weight = floats(s.final_norm);
-    a.out = plan->picked;
-    a.select = static_cast<const int*>(buffer(s.wanted));
-    a.rows = int(wanted);
-    a.width = W;
-    a.out_stride = W8;
-    a.limit = r.rows;
-    a.eps = float(s.eps);
-    TMB_TRY(RmsNorm(q, a));
+    const int* select = static_cast<const int*>(buffer(s.wanted));
+    if (s.combined) {
+      StreamArgs a = step;
+      a.rows = int(wanted);
+      a.weight = floats(s.final_norm);
+      a.normed = plan->picked;
+      a.select = select;
+      TMB_TRY(StreamStep(q, a));
+    } else {
+      NormArgs a{};
+      a.x = x;
+      a.weight = floats(s.final_norm);
+      a.out = plan->picked;
+      a.select = select;
+      a.rows = int(wanted);
+      a.width = W;
+      a.out_stride = W8;
+      a.limit = r.rows;
+      a.eps = float(s.eps);
+      TMB_TRY(RmsNorm(q, a));
+    }
     LinearArgs h = linear(plan->picked, s.head, -1, s.f32 ? nullptr : &plan->head, s.vocab, W, buffer(s.logits), s.vocab, kLinearFloat);
     h.t = int(wanted);
     TMB_TRY(Linear(q, h));
@@ -294,25 +428,40 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
   };
   const size_t element = spec.f32 ? 4 : 2;
   size_t proj = 0, mixed = 0, mlp = 0, pairs = 0, raw = 0, split = 0, heads = 1, partial = 0;
-  size_t top = 0, experts = 0, expert_columns = 0;
+  size_t top = 0, experts = 0, expert_columns = 0, expert_pairs = 0, source = 0, latent = 0, ranks = 0;
   for (const RaggedLayer& layer : spec.layers) {
     const RaggedMixer& m = layer.mixer;
     proj = std::max(proj, size_t(m.proj_rows() + 7) / 8 * 8);
     mixed = std::max(mixed, size_t(padded_columns(m.out_columns())));
+    if (m.value_mix == RaggedMixer::kSource) {
+      source = size_t(m.proj_rows() + 7) / 8 * 8;
+      plan->source_stride = int(source);
+      plan->source_at = (m.heads + m.kv_heads) * m.dim;
+    }
     if (layer.mlp.kind == RaggedMlp::kGlu) {
       mlp = std::max(mlp, size_t(padded_columns(layer.mlp.ff)));
       pairs = std::max(pairs, size_t(layer.mlp.packed_rows()));
     } else if (layer.mlp.kind == RaggedMlp::kExperts) {
       top = std::max(top, size_t(layer.mlp.top));
-      experts = std::max(experts, size_t(layer.mlp.experts));
+      experts = std::max(experts, size_t(layer.mlp.logits()));
       expert_columns = std::max(expert_columns, size_t(padded_columns(layer.mlp.ff)));
+      if (layer.mlp.output_weighted) {
+        ranks = std::max(ranks, size_t(layer.mlp.experts));
+        expert_pairs = std::max(expert_pairs, size_t(layer.mlp.packed_rows()));
+      }
+      if (layer.mlp.shared_ff) {
+        mlp = std::max(mlp, size_t(padded_columns(layer.mlp.shared_ff)));
+        pairs = std::max(pairs, size_t(layer.mlp.shared_rows()));
+      }
     }
     if (m.kind == RaggedMixer::kRetention) {
       raw = std::max(raw, size_t(m.out_columns()));
       split = std::max(split, size_t(m.heads) * 4 * m.pool_dim());
     } else {
+      const size_t columns = m.kind == RaggedMixer::kLatent ? size_t(m.rank_stride()) : size_t(m.vdim);
       heads = std::max(heads, size_t(m.heads));
-      partial = std::max(partial, size_t(m.heads) * (m.vdim + 2));
+      partial = std::max(partial, size_t(m.heads) * (columns + 2));
+      if (m.kind == RaggedMixer::kLatent) latent = std::max(latent, size_t(m.heads) * m.rank_stride());
     }
   }
   const size_t rows = size_t(spec.max_rows), W8 = size_t(padded_columns(spec.width)), slots = rows * top;
@@ -322,7 +471,10 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
   if (!Own(plan, &plan->normed, rows * W8 * element) || !Own(plan, &plan->picked, size_t(spec.max_wanted) * W8 * element) ||
       !Own(plan, &plan->proj, rows * proj * element) || !Own(plan, &plan->mixed, rows * mixed * element) ||
       !Own(plan, &plan->mlp, rows * mlp * element) || !Own(plan, &plan->pairs, spec.f32 ? rows * pairs * element : 0) ||
-      !Own(plan, &plan->branch, spec.layers[0].norm_output ? rows * size_t(spec.width) * sizeof(float) : 0) ||
+      !Own(plan, &plan->branch, spec.layers[0].norm_output || spec.combined ? rows * size_t(spec.width) * sizeof(float) : 0) ||
+      !Own(plan, &plan->source, rows * source * element) || !Own(plan, &plan->lookup, rows * latent * element) ||
+      !Own(plan, &plan->looked, rows * latent * element) || !Own(plan, &plan->ranks, rows * ranks * sizeof(float)) ||
+      !Own(plan, &plan->expert_pairs, spec.f32 ? slots * expert_pairs * element : 0) ||
       !Own(plan, &plan->logits, rows * experts * sizeof(float)) || !Own(plan, &plan->choice, slots * sizeof(int)) ||
       !Own(plan, &plan->list, slots * sizeof(int)) || !Own(plan, &plan->tile_count, sizeof(int)) ||
       !Own(plan, &plan->score, slots * sizeof(float)) || !Own(plan, &plan->slot_score, slots * sizeof(float)) ||
@@ -366,12 +518,21 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
       bool ok = EncodeLinear(&maps.in, at(layer.in_weight), uint64_t(m.proj_rows()), plan->normed, rows, W8) &&
                 EncodeLinear(&maps.out, at(layer.out_weight), uint64_t(spec.width), plan->mixed, rows, uint64_t(padded_columns(m.out_columns())));
       const RaggedMlp& mlp = layer.mlp;
+      if (m.kind == RaggedMixer::kLatent)
+        ok = ok && EncodeHeads(&maps.key_up, at(layer.key_up), uint64_t(m.heads) * m.rank, uint64_t(m.head_stride()), plan->proj, rows,
+                               size_t(m.proj_rows() + 7) / 8 * 8) &&
+             EncodeHeads(&maps.value_up, at(layer.value_up), uint64_t(m.heads) * m.vdim, uint64_t(m.rank_stride()), plan->looked, rows,
+                         uint64_t(m.heads) * m.rank_stride());
       if (mlp.kind == RaggedMlp::kExperts)
-        ok = ok && EncodeLinear(&maps.router, at(layer.router), uint64_t(mlp.experts), plan->normed, rows, W8) &&
-             EncodeLinear(&maps.gate_up, at(layer.expert_up), uint64_t(mlp.experts) * mlp.ff, plan->gathered, slots, W8) &&
+        ok = ok && EncodeLinear(&maps.router, at(layer.router), uint64_t(mlp.logits()), plan->normed, rows, W8) &&
+             EncodeLinear(&maps.gate_up, at(layer.expert_up), uint64_t(mlp.experts) * (mlp.output_weighted ? mlp.packed_rows() : mlp.ff), plan->gathered,
+                          slots, W8) &&
              EncodeGathered(&maps.gate_up, plan->normed, rows, W8) &&
              EncodeLinear(&maps.down, at(layer.expert_down), uint64_t(mlp.experts) * spec.width, plan->expert_hidden, slots,
                           uint64_t(padded_columns(mlp.ff)));
+      if (mlp.shared_ff)
+        ok = ok && EncodeLinear(&maps.shared_up, at(layer.shared_up), uint64_t(mlp.shared_rows()), plan->normed, rows, W8) &&
+             EncodeLinear(&maps.shared_down, at(layer.shared_down), uint64_t(spec.width), plan->mlp, rows, uint64_t(padded_columns(mlp.shared_ff)));
       if (mlp.kind == RaggedMlp::kGlu)
         ok = ok && EncodeLinear(&maps.gate_up, at(layer.gate_up), uint64_t(mlp.packed_rows()), plan->normed, rows, W8) &&
              EncodeLinear(&maps.down, at(layer.down), uint64_t(spec.width), plan->mlp, rows, uint64_t(padded_columns(mlp.ff)));

@@ -33,6 +33,27 @@ std::string Name(const Json& object, const char* key) {
 
 std::string AliasRecipe(const std::string& name) { return "{\"kind\":\"alias\",\"source\":" + Json::Quote(name) + "}"; }
 
+std::string OffsetRecipe(const std::string& name, double offset) {
+  return offset == 0 ? AliasRecipe(name) : "{\"kind\":\"offset\",\"value\":" + std::to_string(offset) + ",\"source\":" + Json::Quote(name) + "}";
+}
+
+// Recipes one under the other, each a JSON object or a quoted tensor name.
+std::string Stack(const std::vector<std::string>& recipes) {
+  std::string out = "{\"kind\":\"stack\",\"sources\":[";
+  for (size_t i = 0; i < recipes.size(); ++i) out += (i ? "," : "") + recipes[i];
+  return out + "]}";
+}
+std::string PadColumns(const std::string& recipe, int columns) {
+  return "{\"kind\":\"pad_columns\",\"columns\":" + std::to_string(columns) + ",\"source\":" + recipe + "}";
+}
+std::string PerHead(const char* kind, const std::string& recipe, int heads, const char* key, int value) {
+  return "{\"kind\":\"" + std::string(kind) + "\",\"heads\":" + std::to_string(heads) + ",\"" + key + "\":" + std::to_string(value) +
+         ",\"source\":" + recipe + "}";
+}
+std::string GluRecipe(const std::string& gate, const std::string& up) {
+  return "{\"kind\":\"gate_up_interleave\",\"pad\":true,\"u\":" + std::to_string(kGluUnit) + ",\"sources\":[" + gate + "," + up + "]}";
+}
+
 std::string QuotedList(const Json& names, const char* key, int count) {
   Require(names.has(key) && names.at(key).kind == Json::kArray && int(names.at(key).items.size()) == count,
           std::string("a layer needs one tensor per expert for '") + key + "'");
@@ -57,6 +78,8 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
   s.width = int(model.integer("width", 0));
   s.vocab = int(model.integer("vocab", 0));
   s.eps = model.num("eps", -1);
+  s.streams = int(model.integer("streams", 1));
+  const double offset = model.num("norm_offset", 0);   // added to the stored weights of the residual norms
   s.slots = int(plan.integer("batch_hi", 0));
   s.capacity = int(plan.integer("capacity", 0));
   s.max_rows = int(plan.integer("max_rows", 0));
@@ -70,6 +93,12 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
   Require(s.max_rows >= 1 && s.max_rows <= 65535, "max_rows must lie in [1, 65535]");
   Require(s.max_wanted >= 1 && s.max_wanted <= 65535, "max_wanted must lie in [1, 65535]");
   Require(s.num_blocks >= 1, "kv.num_blocks must be positive");
+  Require(s.streams >= 1 && s.streams <= kMaxStreams, "a model has 1..16 residual streams");
+  s.combined = s.streams > 1;
+  for (const Json& in : model.at("layers").items) {
+    if (in.has("streams")) s.combined = true;
+    if (in.has("mlp") && in.at("mlp").str("weighted", "") == "output") s.combined = true;
+  }
 
   const uint32_t element = s.f32 ? 1u : 0u;
   const uint64_t element_bytes = s.f32 ? 4 : 2;
@@ -94,7 +123,7 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
   s.block_table = add("serving.block_table", 1, 2, 0, uint64_t(s.max_blocks), "");
   s.logits = add("step.logits", 1, 1, uint64_t(s.max_wanted) * s.vocab, 0, "");
   s.next = add("step.next", 1, 2, uint64_t(s.max_wanted), 0, "");
-  s.hidden = add("step.hidden", 0, 1, uint64_t(s.max_rows) * W, 0, "");
+  s.hidden = add("step.hidden", 0, 1, uint64_t(s.max_rows) * s.streams * W, 0, "");
   s.embed = add("embed", 1, element, uint64_t(s.vocab) * W, 0, AliasRecipe(Name(model, "embed")));
 
   Require(model.at("layers").kind == Json::kArray && !model.at("layers").items.empty(), "the model has no layers");
@@ -106,8 +135,8 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     const Json& mixer = in.at("mixer");
     const Json& names = mixer.at("tensors");
     const std::string kind = mixer.str("kind", "");
-    Require(kind == "attention" || kind == "retention", "unknown kind of mixer '" + kind + "'");
-    m.kind = kind == "retention" ? RaggedMixer::kRetention : RaggedMixer::kAttention;
+    Require(kind == "attention" || kind == "retention" || kind == "latent", "unknown kind of mixer '" + kind + "'");
+    m.kind = kind == "retention" ? RaggedMixer::kRetention : kind == "latent" ? RaggedMixer::kLatent : RaggedMixer::kAttention;
     m.heads = int(mixer.integer("heads", 0));
     m.kv_heads = int(mixer.integer("kv_heads", m.heads));
     m.dim = int(mixer.integer("dim", 0));
@@ -135,14 +164,37 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
         }
       }
     }
-    std::string sources;
+    std::string stacked;                 // recipe of the input projection
     const bool bias = mixer.flag("bias", false);
+    const bool pairs = m.rot_dims && mixer.at("rotary").str("layout", "halves") == "pairs";
+    // entries 2i and 2i + 1 of a head turn together: stored as i and i + dims/2, in queries and keys alike
+    auto arranged = [&](const std::string& name, int heads) {
+      return pairs ? PerHead("pairs_to_halves", name, heads, "dims", m.rot_dims) : name;
+    };
+    auto masked = [&]() {
+      const Json none;
+      const Json& mask = mixer.has("mask") && mixer.at("mask").kind == Json::kObject ? mixer.at("mask") : none;
+      m.window = int(std::min<long long>(mask.integer("size", s.capacity), s.capacity));   // no window: everything before
+      m.keep = int(std::min<long long>(mask.integer("keep_first", 0), s.capacity));
+      m.scale = mixer.num("scale", 0);
+      Require(m.window >= 1 && m.keep >= 0, "a window holds at least one position");
+    };
+    if (names.has("sink")) layer.sinks = add(p + "sinks", 1, 1, uint64_t(m.heads), 0, AliasRecipe(Name(names, "sink")));
     if (m.kind == RaggedMixer::kRetention) {
       Require(m.kv_heads == m.heads, "retention has one key and value head per query head");
       Require(m.vdim <= 4096 && !bias, "retention value heads are at most 4096 wide and its projections have no biases");
       Require(mixer.at("decay").kind == Json::kArray && int(mixer.at("decay").items.size()) == m.heads, "retention needs one decay per head");
       for (const Json& d : mixer.at("decay").items) m.decay.push_back(float(d.number));
-      sources = Quoted(names, {"q", "k", "v", "g"});
+      Require(!pairs, "retention turns the halves of a head");
+      stacked = "{\"kind\":\"stack_rows\",\"sources\":" + Quoted(names, {"q", "k", "v", "g"}) + "}";
+    } else if (m.kind == RaggedMixer::kLatent) {
+      m.rank = int(mixer.integer("rank", 0));
+      Require(m.kv_heads == m.heads && m.rotary < 0 && !bias, "latent attention has a key and a value per head, no rotation and no biases");
+      Require(m.vdim <= kMaxHeadDim, "head sizes must lie in [1, 256]");
+      Require(m.rank >= 1 && m.rank <= kMaxLatent, "a latent row has 1..1024 columns (rank)");
+      masked();
+      Require(m.keep == 0, "latent attention keeps no first positions");
+      stacked = Stack({PerHead("pad_heads", Json::Quote(Name(names, "q")), m.heads, "rows", m.head_stride()), Json::Quote(Name(names, "dkv"))});
     } else {
       m.value_is_key = mixer.str("values", "projected") == "keys";
       Require(m.vdim <= kMaxHeadDim, "head sizes must lie in [1, 256]");
@@ -151,31 +203,68 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
       m.gate = mixer.flag("gate", false);
       m.sink = mixer.has("sink") && mixer.at("sink").kind == Json::kNumber;
       m.sink_score = mixer.num("sink", 0);
-      const Json none;
-      const Json& mask = mixer.has("mask") && mixer.at("mask").kind == Json::kObject ? mixer.at("mask") : none;
-      m.window = int(std::min<long long>(mask.integer("size", s.capacity), s.capacity));   // no window: everything before
-      m.keep = int(std::min<long long>(mask.integer("keep_first", 0), s.capacity));
-      m.scale = mixer.num("scale", 0);
-      Require(m.window >= 1 && m.keep >= 0, "a window holds at least one position");
-      sources = m.value_is_key ? (m.gate ? Quoted(names, {"q", "k", "g"}) : Quoted(names, {"q", "k"}))
-                               : (m.gate ? Quoted(names, {"q", "k", "v", "g"}) : Quoted(names, {"q", "k", "v"}));
+      masked();
+      Require(!pairs || !m.value_is_key, "values that are keys take heads whose halves turn");
+      std::vector<std::string> parts = {arranged(Json::Quote(Name(names, "q")), m.heads), arranged(Json::Quote(Name(names, "k")), m.kv_heads)};
+      if (!m.value_is_key) parts.push_back(Json::Quote(Name(names, "v")));
+      if (m.gate) parts.push_back(Json::Quote(Name(names, "g")));
+      stacked = Stack(parts);
+      const std::string mixing = mixer.str("value_mix", "");
+      Require(mixing.empty() || mixing == "source" || mixing == "blend", "unknown way of mixing values");
+      m.value_mix = mixing.empty() ? RaggedMixer::kOwn : mixing == "source" ? RaggedMixer::kSource : RaggedMixer::kBlend;
+      if (m.value_mix != RaggedMixer::kOwn) {
+        Require(!m.value_is_key, "values that are keys are not mixed");
+        int sources = 0;
+        for (const RaggedLayer& before : s.layers)
+          if (before.mixer.value_mix == RaggedMixer::kSource) {
+            ++sources;
+            Require(before.mixer.kv_heads * before.mixer.vdim == m.kv_heads * m.vdim, "layers that mix values have as many of them");
+          }
+        Require(sources == (m.value_mix == RaggedMixer::kBlend ? 1 : 0), "values are mixed with those of one layer before");
+      }
+      if (m.value_mix == RaggedMixer::kBlend) layer.blend = add(p + "blend", 1, 1, 1, 0, AliasRecipe(Name(names, "vmix")));
       Require(!bias || !m.gate, "gated attention has no projection biases");
     }
     const std::string place = in.str("norm_at", "input");
     Require(place == "input" || place == "output", "a layer's norms act on its sublayers' input or output (norm_at)");
     layer.norm_output = place == "output";
     Require(i == 0 || layer.norm_output == s.layers[0].norm_output, "every layer of a model has its norms in the same place");
-    layer.norm1 = add(p + "norm1", 1, 1, W, 0, AliasRecipe(Name(in, "norm1")));
-    layer.in_weight = matrix(p + "in.weight", StackRecipe(sources, padded_columns(s.width)), m.proj_rows(), s.width);
+    Require(!s.combined || !layer.norm_output, "streams and experts whose outputs are weighted need the norms on the sublayers' inputs");
+    auto streams = [&](int which) {
+      if (!in.has("streams")) {
+        Require(s.streams == 1, "every layer of a model with several streams says how its sublayers use them");
+        return;
+      }
+      Require(int(in.at("streams").items.size()) > which, "a layer has stream weights for each of its sublayers");
+      const Json& parts = in.at("streams").items[size_t(which)];
+      const std::string at = p + "streams" + std::to_string(which + 1) + ".";
+      RaggedStreams& out = layer.streams[which];
+      out.in = add(at + "in", 1, 1, uint64_t(s.streams), 0, AliasRecipe(Name(parts, "in")));
+      out.out = add(at + "out", 1, 1, uint64_t(s.streams), 0, AliasRecipe(Name(parts, "out")));
+      out.mix = add(at + "mix", 1, 1, uint64_t(s.streams) * s.streams, 0, AliasRecipe(Name(parts, "mix")));
+    };
+    streams(0);
+    layer.norm1 = add(p + "norm1", 1, 1, W, 0, OffsetRecipe(Name(in, "norm1"), offset));
+    layer.in_weight = matrix(p + "in.weight", PadColumns(stacked, padded_columns(s.width)), m.proj_rows(), s.width);
+    if (m.kind == RaggedMixer::kLatent) {
+      const int rank = m.rank_stride();
+      layer.latent_norm = add(p + "latent.norm", 1, 1, uint64_t(m.rank), 0, AliasRecipe(Name(names, "dkv.norm")));
+      // a query against latent rows is its head's key matrix, transposed, times the query
+      layer.key_up = add(p + "key_up.weight", 1, element, uint64_t(m.heads) * m.rank * m.head_stride(), 0,
+                         PadColumns(PerHead("transpose_heads", Json::Quote(Name(names, "uk")), m.heads, "rows", m.dim), m.head_stride()));
+      layer.value_up = add(p + "value_up.weight", 1, element, uint64_t(m.heads) * m.vdim * rank, 0,
+                           PadColumns(Stack({Json::Quote(Name(names, "uv"))}), rank));
+    }
     layer.out_weight = matrix(p + "out.weight", StackRecipe(Quoted(names, {"o"}), padded_columns(m.out_columns())), s.width, m.out_columns());
     if (m.qk_norm) {
-      layer.q_norm = add(p + "q.norm", 1, 1, uint64_t(m.heads) * m.dim, 0, AliasRecipe(Name(names, "q.norm")));
-      layer.k_norm = add(p + "k.norm", 1, 1, uint64_t(m.kv_heads) * m.dim, 0, AliasRecipe(Name(names, "k.norm")));
+      layer.q_norm = add(p + "q.norm", 1, 1, uint64_t(m.heads) * m.dim, 0, Stack({arranged(Json::Quote(Name(names, "q.norm")), m.heads)}));
+      layer.k_norm = add(p + "k.norm", 1, 1, uint64_t(m.kv_heads) * m.dim, 0, Stack({arranged(Json::Quote(Name(names, "k.norm")), m.kv_heads)}));
     }
     if (bias) {
-      const std::string biases = m.value_is_key ? Quoted(names, {"q.b", "k.b"}) : Quoted(names, {"q.b", "k.b", "v.b"});
-      layer.in_bias = add(p + "in.bias", 1, 1, uint64_t(m.proj_rows()), 0, "{\"kind\":\"concat\",\"sources\":" + biases + "}");
-      layer.out_bias = add(p + "out.bias", 1, 1, W, 0, "{\"kind\":\"concat\",\"sources\":" + Quoted(names, {"o.b"}) + "}");
+      std::vector<std::string> biases = {arranged(Json::Quote(Name(names, "q.b")), m.heads), arranged(Json::Quote(Name(names, "k.b")), m.kv_heads)};
+      if (!m.value_is_key) biases.push_back(Json::Quote(Name(names, "v.b")));
+      layer.in_bias = add(p + "in.bias", 1, 1, uint64_t(m.proj_rows()), 0, Stack(biases));
+      if (names.has("o.b")) layer.out_bias = add(p + "out.bias", 1, 1, W, 0, AliasRecipe(Name(names, "o.b")));
     }
     if (in.has("mlp") && in.at("mlp").kind == Json::kObject) {
       const Json& mlp = in.at("mlp");
@@ -185,7 +274,8 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
       layer.mlp.kind = unit == "glu" ? RaggedMlp::kGlu : RaggedMlp::kExperts;
       layer.mlp.ff = int(mlp.integer("ff", 0));
       Require(layer.mlp.ff > 0, "the feed-forward width must be positive");
-      layer.norm2 = add(p + "norm2", 1, 1, W, 0, AliasRecipe(Name(in, "norm2")));
+      layer.norm2 = add(p + "norm2", 1, 1, W, 0, OffsetRecipe(Name(in, "norm2"), offset));
+      streams(1);
       const std::string activation = mlp.str("activation", "silu");
       if (layer.mlp.kind == RaggedMlp::kGlu) {
         Require(activation == "silu" || activation == "gelu_tanh", "unknown activation of a gated unit");
@@ -206,11 +296,46 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
         Require(e.experts >= 1 && e.experts <= kMaxExperts, "a layer has 1..1024 experts");
         Require(e.top >= 1 && e.top <= e.experts && e.top <= kMaxTop, "a token uses 1..32 of a layer's experts (top)");
         Require(uint64_t(s.max_rows) * e.top <= (1u << 20), "max_rows times the experts of a token is at most 2^20");
-        Require(activation == "relu2" && mlp.str("scores", "") == "sigmoid" && mlp.str("weighted", "") == "input",
-                "experts use the square of relu, sigmoid scores and weights on their inputs");
-        Require(layer.norm_output, "expert layers need their norms on the sublayers' outputs");
-        layer.router = matrix(p + "router.weight", StackRecipe(Quoted(parts, {"router"}), padded_columns(s.width)), e.experts, s.width);
-        layer.expert_up = matrix(p + "experts.up", StackRecipe(QuotedList(parts, "up", e.experts), padded_columns(s.width)), e.experts * e.ff, s.width);
+        const std::string scores = mlp.str("scores", "");
+        e.output_weighted = mlp.str("weighted", "") == "output";
+        e.softmax = scores == "softmax";
+        e.correction = parts.has("correction");
+        if (mlp.has("groups") && mlp.at("groups").kind == Json::kObject) {
+          e.groups = int(mlp.at("groups").integer("count", 1));
+          e.keep_groups = int(mlp.at("groups").integer("keep", e.groups));
+        }
+        Require(e.groups >= 1 && e.experts % e.groups == 0 && e.keep_groups >= 1 && e.keep_groups <= e.groups, "experts form equal groups, at least one of them kept");
+        Require(e.top <= e.keep_groups * (e.experts / e.groups), "the kept groups hold the experts of a token");
+        std::string router = Quoted(parts, {"router"});
+        if (e.output_weighted) {
+          Require(activation == "silu" && (e.softmax || scores == "sigmoid"), "experts with weighted outputs are gated units with softmax or sigmoid scores");
+          e.limit = mlp.num("limit", 3.0e38);
+          e.alpha = mlp.num("alpha", 1.0);
+          e.shift = mlp.num("shift", 0.0);
+          std::vector<std::string> units;
+          Require(parts.has("gate") && parts.has("up") && int(parts.at("gate").items.size()) == e.experts && int(parts.at("up").items.size()) == e.experts,
+                  "a layer needs one tensor per expert for 'gate' and 'up'");
+          for (int i = 0; i < e.experts; ++i)
+            units.push_back(GluRecipe(Json::Quote(parts.at("gate").items[size_t(i)].text), Json::Quote(parts.at("up").items[size_t(i)].text)));
+          layer.expert_up = matrix(p + "experts.gate_up", PadColumns(Stack(units), padded_columns(s.width)), e.experts * e.packed_rows(), s.width);
+          if (mlp.has("shared") && mlp.at("shared").kind == Json::kObject) {
+            e.shared_ff = int(mlp.at("shared").integer("ff", 0));
+            e.shared_limit = mlp.at("shared").num("limit", 3.0e38);
+            Require(e.shared_ff > 0, "the feed-forward width must be positive");
+            layer.shared_up = matrix(p + "shared.gate_up", PadColumns(GluRecipe(Json::Quote(Name(parts, "shared.gate")), Json::Quote(Name(parts, "shared.up"))),
+                                                                     padded_columns(s.width)), e.shared_rows(), s.width);
+            layer.shared_down = matrix(p + "shared.down", StackRecipe(Quoted(parts, {"shared.down"}), padded_columns(e.shared_ff)), s.width, e.shared_ff);
+            router = Quoted(parts, {"router", "shared.sg"});
+          }
+          if (e.correction) layer.correction = add(p + "correction", 1, 1, uint64_t(e.experts), 0, AliasRecipe(Name(parts, "correction")));
+        } else {
+          Require(activation == "relu2" && scores == "sigmoid" && mlp.str("weighted", "") == "input",
+                  "experts use the square of relu, sigmoid scores and weights on their inputs");
+          Require(layer.norm_output, "expert layers need their norms on the sublayers' outputs");
+          Require(e.groups == 1 && !e.correction && !mlp.has("shared"), "experts with weighted inputs are ranked by their scores alone, without a shared one");
+          layer.expert_up = matrix(p + "experts.up", StackRecipe(QuotedList(parts, "up", e.experts), padded_columns(s.width)), e.experts * e.ff, s.width);
+        }
+        layer.router = matrix(p + "router.weight", StackRecipe(router, padded_columns(s.width)), e.logits(), s.width);
         layer.expert_down = matrix(p + "experts.down", StackRecipe(QuotedList(parts, "down", e.experts), padded_columns(e.ff)), e.experts * s.width, e.ff);
       }
     }
@@ -225,6 +350,8 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     const std::string at = std::to_string(s.runs.size());
     if (m.kind == RaggedMixer::kRetention) {
       run.state = add("retention." + at, 1, 1, 0, uint64_t(m.heads) * m.dim * m.vdim, "");
+    } else if (m.kind == RaggedMixer::kLatent) {
+      run.k_pool = add("kv_pool.latent." + at, 1, element, uint64_t(s.num_blocks) * kRaggedBlock * m.pool_dim(), 0, "");
     } else {
       const uint64_t rows = uint64_t(s.num_blocks) * m.kv_heads * kRaggedBlock;
       run.k_pool = add("kv_pool.k." + at, 1, element, rows * m.pool_dim(), 0, "");
@@ -232,14 +359,17 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     }
     const RaggedMlp& mlp = s.layers[size_t(run.layer)].mlp;
     Require(!run.add_embedding || !s.layers[size_t(run.layer)].norm_output, "layers with norms on their outputs are not looped");
-    const int mlp_rows = mlp.kind == RaggedMlp::kGlu ? 3 * mlp.ff : mlp.kind == RaggedMlp::kExperts ? 2 * mlp.top * mlp.ff + mlp.experts : 0;
+    Require(!run.add_embedding || !s.combined, "layers of several streams are not looped");
+    const int unit = mlp.output_weighted ? 3 : 2;              // matrices of an expert
+    const int mlp_rows = mlp.kind == RaggedMlp::kGlu ? 3 * mlp.ff : mlp.kind == RaggedMlp::kExperts ? unit * mlp.top * mlp.ff + 3 * mlp.shared_ff + mlp.logits() : 0;
     s.weight_bytes += element_bytes * W * uint64_t(m.proj_rows() + m.out_columns() + mlp_rows);
+    if (m.kind == RaggedMixer::kLatent) s.weight_bytes += element_bytes * uint64_t(m.heads) * m.rank * (m.dim + m.vdim);
     s.runs.push_back(run);
   }
   Require(!s.runs.empty(), "the model runs no layer");
   s.weight_bytes += element_bytes * W * uint64_t(s.vocab);
   if (s.write_residuals) s.residuals = add("step.residuals", 0, 1, uint64_t(s.runs.size()) * s.max_rows * W, 0, "");
-  s.final_norm = add("final.norm", 1, 1, W, 0, AliasRecipe(Name(model, "final_norm")));
+  s.final_norm = add("final.norm", 1, 1, W, 0, OffsetRecipe(Name(model, "final_norm"), offset));
   s.head = matrix("head.weight", StackRecipe("[" + Json::Quote(Name(model, "head")) + "]", padded_columns(s.width)), s.vocab, s.width);
   return s;
 }

@@ -2,6 +2,8 @@
 // to it, greedy sampling, and the hand-over of sampled tokens to the next step.
 #include <cuda_bf16.h>
 
+#include <type_traits>
+
 #include "element.cuh"
 #include "ops.h"
 #include "ptx.cuh"
@@ -12,7 +14,7 @@ namespace {
 
 // One CTA per row. The row's entry is found by bisection over the entries' first rows (ascending, no gaps).
 template <typename T>
-__global__ void __launch_bounds__(256) start_step(StepRows r, const int* tokens, const T* embed, float* x, T* copy,
+__global__ void __launch_bounds__(256) start_step(StepRows r, const int* tokens, const T* embed, float* x, int streams, T* copy,
                                                   int copy_stride, int width, int vocab) {
   const int row = blockIdx.x;
   dependency_wait();
@@ -36,7 +38,7 @@ __global__ void __launch_bounds__(256) start_step(StepRows r, const int* tokens,
 #pragma unroll 8
   for (int i = threadIdx.x; i < width; i += 256) {
     const T value = embed[size_t(token) * width + i];
-    x[size_t(row) * width + i] = to_f(value);
+    for (int s = 0; s < streams; ++s) x[(size_t(row) * streams + s) * width + i] = to_f(value);
     if (copy) copy[size_t(row) * copy_stride + i] = value;
   }
 }
@@ -222,6 +224,157 @@ __global__ void __launch_bounds__(512) add_norm(AddNormArgs a) {
   }
 }
 
+// Streams updated by a sublayer's output and collected for the next one, see StreamArgs. S: streams held (at least those there
+// are). QUADS: widths that are multiples of 4 up to 8192 (what was collected stays in registers); otherwise a thread collects
+// its columns twice.
+template <typename T, int S, bool QUADS>
+__global__ void __launch_bounds__(512) stream_step(StreamArgs a) {
+  using V = std::conditional_t<QUADS, float4, float>;
+  constexpr int N = QUADS ? kQuads : 1, E = QUADS ? 4 : 1;   // E: columns of a V
+  __shared__ float part[16], mix[S * S], out[S], in[S];
+  const int i = blockIdx.x, units = a.width / E;
+  V weight[N], u[N];
+  if (threadIdx.x < S * S) {
+    const int from = threadIdx.x / S, to = threadIdx.x % S;
+    mix[threadIdx.x] = from >= a.streams || to >= a.streams ? 0.f : a.mix ? a.mix[from * a.streams + to] : from == to ? 1.f : 0.f;
+  }
+  if (threadIdx.x < S) {
+    const bool live = int(threadIdx.x) < a.streams;
+    out[threadIdx.x] = !live ? 0.f : a.out ? a.out[threadIdx.x] : 1.f;
+    in[threadIdx.x] = !live ? 0.f : a.in ? a.in[threadIdx.x] : 1.f;
+  }
+  if (QUADS && a.weight) {
+#pragma unroll
+    for (int n = 0; n < N; ++n)
+      if (int c = threadIdx.x + 512 * n; c < units) weight[n] = reinterpret_cast<const V*>(a.weight)[c];
+  }
+  dependency_wait();
+  allow_dependents();
+  __syncthreads();
+  const int row = a.select ? min(max(a.select[i], 0), a.limit - 1) : i;
+  float* x = a.x + size_t(row) * a.streams * a.width;
+  const float opened = a.branch_gate ? 1.f / (1.f + expf(-a.branch_gate[size_t(i) * a.gate_stride])) : 1.f;
+  const T* parts_of = static_cast<const T*>(a.parts_of) + size_t(i) * a.parts * a.width;
+  const float* scales = a.part_scale + size_t(i) * a.parts;
+  auto load = [&](const void* at, int c, float (&v)[E]) {         // fp32
+    if constexpr (QUADS) {
+      const float4 q = static_cast<const float4*>(at)[c];
+      v[0] = q.x, v[1] = q.y, v[2] = q.z, v[3] = q.w;
+    } else {
+      v[0] = static_cast<const float*>(at)[c];
+    }
+  };
+  auto store = [&](float* at, int c, const float (&v)[E]) {
+    if constexpr (QUADS) reinterpret_cast<float4*>(at)[c] = make_float4(v[0], v[1], v[2], v[3]);
+    else at[c] = v[0];
+  };
+  // column unit c of what the next sublayer reads; `write`: the update comes first
+  auto visit = [&](int c, bool write, float (&got)[E]) {
+    float old[S][E];
+#pragma unroll
+    for (int s = 0; s < S; ++s) {
+#pragma unroll
+      for (int e = 0; e < E; ++e) old[s][e] = 0.f;
+      if (s < a.streams) load(x + size_t(s) * a.width, c, old[s]);
+    }
+    if (write) {
+      float y[E] = {};
+      if (a.branch) {
+        load(a.branch + size_t(i) * a.width, c, y);
+#pragma unroll
+        for (int e = 0; e < E; ++e) y[e] *= opened;
+      }
+#pragma unroll 8
+      for (int k = 0; k < a.parts; ++k) {
+        const float f = scales[k];
+        if constexpr (QUADS) {
+          const float4 v = four<T>(parts_of + size_t(k) * a.width + 4 * c);
+          y[0] = fmaf(f, v.x, y[0]), y[1] = fmaf(f, v.y, y[1]), y[2] = fmaf(f, v.z, y[2]), y[3] = fmaf(f, v.w, y[3]);
+        } else {
+          y[0] = fmaf(f, to_f(parts_of[size_t(k) * a.width + c]), y[0]);
+        }
+      }
+      float sum[E] = {};
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        float now[S];
+#pragma unroll
+        for (int t = 0; t < S; ++t) {
+          now[t] = out[t] * y[e];
+#pragma unroll
+          for (int s = 0; s < S; ++s) now[t] = fmaf(mix[s * S + t], old[s][e], now[t]);
+          sum[e] += now[t];
+        }
+#pragma unroll
+        for (int t = 0; t < S; ++t) old[t][e] = now[t];
+      }
+#pragma unroll
+      for (int t = 0; t < S; ++t)
+        if (t < a.streams) store(x + size_t(t) * a.width, c, old[t]);
+      if (a.sum_of) store(a.sum_of + size_t(i) * a.width, c, sum);
+    }
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      got[e] = 0.f;
+#pragma unroll
+      for (int t = 0; t < S; ++t) got[e] = fmaf(in[t], old[t][e], got[e]);
+    }
+  };
+  float sq = 0.f;
+  if constexpr (QUADS) {
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      const int c = threadIdx.x + 512 * n;
+      float v[E] = {};
+      if (c < units) visit(c, a.update, v);
+      u[n] = make_float4(v[0], v[1], v[2], v[3]);
+      sq += v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
+    }
+  } else {
+    for (int c = threadIdx.x; c < units; c += 512) {
+      float v[E];
+      visit(c, a.update, v);
+      sq = fmaf(v[0], v[0], sq);
+    }
+  }
+  if (!a.weight) return;
+  sq = warp_sum(sq);
+  if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = sq;
+  __syncthreads();
+  sq = 0.f;
+#pragma unroll
+  for (int w = 0; w < 16; ++w) sq += part[w];
+  const float inv = 1.f / sqrtf(sq / float(a.width) + a.eps);
+  T* normed = static_cast<T*>(a.normed) + size_t(i) * a.normed_stride;
+  if constexpr (QUADS) {
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      const int c = threadIdx.x + 512 * n;
+      if (c >= units) continue;
+      alignas(16) T e[4] = {from_f<T>(u[n].x * inv * weight[n].x), from_f<T>(u[n].y * inv * weight[n].y), from_f<T>(u[n].z * inv * weight[n].z),
+                            from_f<T>(u[n].w * inv * weight[n].w)};
+      if (sizeof(T) == 2) reinterpret_cast<uint2*>(normed)[c] = *reinterpret_cast<const uint2*>(e);
+      else reinterpret_cast<uint4*>(normed)[c] = *reinterpret_cast<const uint4*>(e);
+    }
+  } else {
+    for (int c = threadIdx.x; c < units; c += 512) {   // (each thread re-reads its own columns)
+      float v[E];
+      visit(c, false, v);
+      normed[c] = from_f<T>(v[0] * inv * a.weight[c]);
+    }
+  }
+}
+
+template <typename T, int S> int StreamStepAs(const Queue& q, const StreamArgs& a) {
+  const bool quads = a.width % 4 == 0 && a.width <= 512 * 4 * kQuads;
+  auto kernel = quads ? stream_step<T, S, true> : stream_step<T, S, false>;
+  return int(Launch(kernel, dim3(unsigned(a.rows)), dim3(512), 0, q.stream, q.chained, a));
+}
+template <typename T> int StreamStepWith(const Queue& q, const StreamArgs& a) {
+  return a.streams == 1 ? StreamStepAs<T, 1>(q, a) : a.streams == 2 ? StreamStepAs<T, 2>(q, a) : a.streams <= 4 ? StreamStepAs<T, 4>(q, a)
+         : a.streams <= 8 ? StreamStepAs<T, 8>(q, a) : StreamStepAs<T, 16>(q, a);
+}
+
 __global__ void __launch_bounds__(1024) arg_max(const float* logits, int vocab, int* next) {
   __shared__ float best_v[32];
   __shared__ int best_i[32];
@@ -285,12 +438,13 @@ __global__ void feed(Entry* entries, int count, const int* next, int* tokens, in
 
 }  // namespace
 
-int StartStep(const Queue& q, const StepRows& r, const int* tokens, const void* embed, float* x, void* copy, int copy_stride, int width, int vocab) {
+int StartStep(const Queue& q, const StepRows& r, const int* tokens, const void* embed, float* x, int streams, void* copy, int copy_stride, int width,
+              int vocab) {
   const dim3 grid(unsigned(r.rows));
   if (q.f32)
-    return int(Launch(start_step<float>, grid, dim3(256), 0, q.stream, false, r, tokens, static_cast<const float*>(embed), x, static_cast<float*>(copy),
+    return int(Launch(start_step<float>, grid, dim3(256), 0, q.stream, false, r, tokens, static_cast<const float*>(embed), x, streams, static_cast<float*>(copy),
                       copy_stride, width, vocab));
-  return int(Launch(start_step<__nv_bfloat16>, grid, dim3(256), 0, q.stream, false, r, tokens, static_cast<const __nv_bfloat16*>(embed), x,
+  return int(Launch(start_step<__nv_bfloat16>, grid, dim3(256), 0, q.stream, false, r, tokens, static_cast<const __nv_bfloat16*>(embed), x, streams,
                     static_cast<__nv_bfloat16*>(copy), copy_stride, width, vocab));
 }
 
@@ -310,6 +464,12 @@ int AddNorm(const Queue& q, const AddNormArgs& a) {
   auto kernel = q.f32 ? (quads ? add_norm<float, true> : add_norm<float, false>)
                       : (quads ? add_norm<__nv_bfloat16, true> : add_norm<__nv_bfloat16, false>);
   return int(Launch(kernel, dim3(unsigned(a.rows)), dim3(512), 0, q.stream, q.chained, a));
+}
+
+int StreamStep(const Queue& q, const StreamArgs& a) {
+  if (a.rows <= 0) return 0;
+  if (a.streams < 1 || a.streams > kMaxStreams || (a.update && a.select)) return int(cudaErrorInvalidValue);
+  return q.f32 ? StreamStepWith<float>(q, a) : StreamStepWith<__nv_bfloat16>(q, a);
 }
 
 int ArgMax(const Queue& q, const float* logits, int rows, int vocab, int* next) {

@@ -104,12 +104,58 @@ def nadilorn_program(config: dict) -> dict:
             "head": "head", "layers": layers, "runs": looped_runs(len(layers), None)}
 
 
+def _mozidra_mixer(kind: str, mixer: dict, prefix: str, first_mixing: bool) -> dict:
+    shared = {"heads": mixer["heads"], "dim": mixer["dim"], "vdim": mixer["vdim"], "mask": mixer.get("mask"), "scale": mixer["scale"]}
+    if kind == "latent_attention":
+        return shared | {"kind": "latent", "rank": mixer["kv_rank"], "tensors": _names(prefix, "q", "dkv", "dkv.norm", "uk", "uv", "sink", "o")}
+    if kind != "attention":
+        raise ValueError(f"unknown layer type {kind!r}")
+    # biased projections, normed queries and keys, rotated pairs of neighbours, a learned sink per head; layers that mix
+    # values blend their own with those of the first such layer
+    rot, mixing = mixer.get("rot"), mixer.get("v_mix")
+    tensors = _names(prefix, "q", "k", "v", "o", "q.b", "k.b", "v.b", "q.norm", "k.norm", "sink")
+    if mixing and not first_mixing:
+        tensors |= _names(prefix, "vmix")
+    return shared | {"kind": kind, "kv_heads": mixer["kv_heads"], "rotary": rot and {"base": rot["base"], "dims": rot["dims"], "layout": "pairs"},
+                     "values": "projected", "qk_norm": True, "bias": True, "value_mix": ("source" if first_mixing else "blend") if mixing else "",
+                     "tensors": tensors}
+
+
+def _mozidra_mlp(mlp: dict | None, prefix: str) -> dict | None:
+    if mlp is None:
+        return None
+    if mlp["kind"] != "moe":
+        raise ValueError(f"unknown feed-forward {mlp['kind']!r}")
+    router, shared = mlp["router"], mlp.get("shared")
+    count = int(router["experts"])
+    tensors = _names(prefix, "router", "correction") | {part: [f"{prefix}e{expert}.{part}" for expert in range(count)] for part in ("gate", "up", "down")}
+    if shared:
+        tensors |= _names(prefix, "shared.gate", "shared.up", "shared.down", "shared.sg")
+    return {"kind": "experts", "ff": mlp["expert"]["ff"], "limit": mlp["expert"]["limit"], "alpha": 1.702, "shift": 1.0, "experts": count,
+            "top": router["top"], "groups": router.get("groups"), "activation": "silu", "scores": "softmax", "weighted": "output",
+            "shared": shared and {"ff": shared["ff"], "limit": shared["limit"]}, "tensors": tensors}
+
+
+def mozidra_program(config: dict) -> dict:
+    layers, mixing = [], [index for index, layer in enumerate(config["layers"]) if layer["mixer"].get("v_mix")]
+    for index, layer in enumerate(config["layers"]):
+        prefix = f"l{index}."
+        mlp = _mozidra_mlp(layer.get("mlp"), prefix + "mlp.")
+        layers.append({"norm1": prefix + "norm1", "norm2": prefix + "norm2" if mlp else None, "mlp": mlp,
+                       "mixer": _mozidra_mixer(layer["type"], layer["mixer"], prefix + "mix.", index in mixing[:1]),
+                       "streams": [_names(f"{prefix}hc{number}.", "in", "out", "mix") for number in ((1, 2) if mlp else (1,))]})
+    # stored norm weights are distances from one
+    return {"width": config["width"], "vocab": config["vocab"], "eps": config["norm"]["eps"], "norm_offset": 1.0, "streams": config["streams"],
+            "embed": "embed", "final_norm": "final.norm", "head": "head", "layers": layers, "runs": looped_runs(len(layers), None)}
+
+
 FAMILIES = {
     "LlamaForCausalLM": Family("llama", ("decode", "prefill")),
     "Qwen3MoeForCausalLM": Family("qwen3-moe", ("decode",)),
     "BertModel": Family("bert", ("forward",)),
     "Bamudra": Family("bamudra", ("ragged",), bamudra_program),
     "Nadilorn": Family("nadilorn", ("ragged",), nadilorn_program),
+    "Mozidra": Family("mozidra", ("ragged",), mozidra_program),
 }
 
 
@@ -142,23 +188,31 @@ def tensor_shapes(config: dict) -> dict[str, tuple[int, ...]]:
     shapes[program["embed"]] = (program["vocab"], width)
     for layer in program["layers"]:
         mixer, names = layer["mixer"], layer["mixer"]["tensors"]
-        q, out = mixer["heads"] * mixer["dim"], mixer["heads"] * mixer["vdim"]
-        k = mixer.get("kv_heads", mixer["heads"]) * mixer["dim"]
-        sizes = {"q": q, "k": k, "v": mixer.get("kv_heads", mixer["heads"]) * mixer["vdim"], "g": out}
+        heads, streams = mixer["heads"], program.get("streams", 1)
+        q, out = heads * mixer["dim"], heads * mixer["vdim"]
+        k, rank = mixer.get("kv_heads", heads) * mixer["dim"], mixer.get("rank", 0)
+        sizes = {"q": q, "k": k, "v": mixer.get("kv_heads", heads) * mixer["vdim"], "g": out, "dkv": rank, "o": width}
+        special = {"o": (width, out), "uk": (q, rank), "uv": (out, rank), "sink": (heads,), "vmix": ()}
         shapes[layer["norm1"]] = (width,)
         for part, name in names.items():
-            if part.endswith(".norm"):
-                shapes[name] = (sizes[part[:-5]],)
-            elif part.endswith(".b"):
-                shapes[name] = (width if part == "o.b" else sizes[part[:-2]],)
+            if part.endswith((".norm", ".b")):
+                shapes[name] = (sizes[part.rsplit(".", 1)[0]],)
             else:
-                shapes[name] = (width, out) if part == "o" else (sizes[part], width)
+                shapes[name] = special[part] if part in special else (sizes[part], width)
+        for parts in layer.get("streams", ()):
+            shapes |= {parts["in"]: (streams,), parts["out"]: (streams,), parts["mix"]: (streams, streams)}
         if layer["mlp"]:
             ff, parts = layer["mlp"]["ff"], layer["mlp"]["tensors"]
             shapes[layer["norm2"]] = (width,)
             if layer["mlp"]["kind"] == "experts":
                 shapes[parts["router"]] = (layer["mlp"]["experts"], width)
-                shapes |= {name: (ff, width) for name in parts["up"]} | {name: (width, ff) for name in parts["down"]}
+                shapes |= {name: (ff, width) for part in ("gate", "up") for name in parts.get(part, ())} | {name: (width, ff) for name in parts["down"]}
+                if "correction" in parts:
+                    shapes[parts["correction"]] = (layer["mlp"]["experts"],)
+                if layer["mlp"].get("shared"):
+                    wide = layer["mlp"]["shared"]["ff"]
+                    shapes |= {parts["shared.gate"]: (wide, width), parts["shared.up"]: (wide, width), parts["shared.down"]: (width, wide),
+                               parts["shared.sg"]: (1, width)}
             else:
                 shapes |= {parts["gate"]: (ff, width), parts["up"]: (ff, width), parts["down"]: (width, ff)}
     shapes[program["final_norm"]] = (width,)

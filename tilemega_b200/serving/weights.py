@@ -209,6 +209,28 @@ def dequantize_e4m3(codes: torch.Tensor, scale: torch.Tensor) -> torch.Tensor:
     return codes.view(torch.float8_e4m3fn).float() * scale[:, None].float()
 
 
+def per_head(recipe: Mapping[str, object], tensor: torch.Tensor) -> torch.Tensor:
+    """Recipes that treat each head's equal share of a tensor's rows by itself."""
+    kind, heads = recipe["kind"], int(recipe["heads"])
+    if heads < 1 or tensor.ndim < 1 or tensor.shape[0] % heads:
+        raise ValueError(f"{kind}: the rows do not split into {heads} heads")
+    rows = tensor.shape[0] // heads
+    split = tensor.reshape(heads, rows, *tensor.shape[1:])
+    if kind == "pad_heads":                      # zero rows behind every head's, up to `rows`
+        if tensor.ndim != 2 or int(recipe["rows"]) < rows:
+            raise ValueError("pad_heads takes a matrix of at most that many rows a head")
+        return torch.nn.functional.pad(split, (0, 0, 0, int(recipe["rows"]) - rows)).reshape(-1, tensor.shape[1])
+    if kind == "transpose_heads":                # every head's matrix of `rows` rows transposed
+        if tensor.ndim != 2 or rows != int(recipe["rows"]):
+            raise ValueError("transpose_heads takes a matrix of that many rows a head")
+        return split.transpose(1, 2).reshape(-1, rows)
+    # pairs_to_halves: of the first `dims` rows of a head the even ones, then the odd ones; the others stay
+    dims = int(recipe["dims"])
+    if dims % 2 or not 0 <= dims <= rows:
+        raise ValueError("pairs_to_halves takes an even number of a head's rows")
+    return torch.cat((split[:, 0:dims:2], split[:, 1:dims:2], split[:, dims:]), dim=1).reshape(tensor.shape)
+
+
 def pack(recipe: Mapping[str, object], source: Callable[[str], torch.Tensor], tp_rank: int = 0) -> torch.Tensor:
     kind = recipe["kind"]
     if kind in ("e4m3_pairs", "e4m3_scale"):
@@ -220,8 +242,19 @@ def pack(recipe: Mapping[str, object], source: Callable[[str], torch.Tensor], tp
             raise ValueError("e4m3 weight rows need an even number of columns")
         return codes.contiguous().view(torch.bfloat16)   # two codes per 2-byte unit: tile_pages applies unchanged
     source = sharded(recipe, source, tp_rank)
+    inner = lambda item: pack(item, source) if isinstance(item, Mapping) else source(str(item))   # a recipe or a tensor's name
     if kind == "alias":
         return source(str(recipe["source"]))
+    if kind == "offset":
+        return inner(recipe["source"]) + float(recipe["value"])
+    if kind == "stack":
+        # matrices of one width, or vectors, one behind the other
+        tensors = [inner(item) for item in recipe["sources"]]
+        if len({item.shape[1:] for item in tensors}) != 1 or tensors[0].ndim not in (1, 2):
+            raise ValueError("stack takes matrices of one width or vectors")
+        return torch.cat(tensors)
+    if kind in ("pad_heads", "transpose_heads", "pairs_to_halves"):
+        return per_head(recipe, inner(recipe["source"]))
     if kind == "tile_pages":
         inner = recipe["source"]
         if isinstance(inner, Mapping) and inner.get("kind") == "expert_stack":
