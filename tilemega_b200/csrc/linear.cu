@@ -29,6 +29,7 @@ struct LinearParams {
   void* out;
   int t, n, out_stride, outputs;
   int head_in, head_out;
+  const int* rows_there;
   int chunks, chunks_per_split;
   Glu glu;
   ExpertSlots slots;
@@ -118,6 +119,15 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
     weight_row = head * g.n + n0;
     k_at = head * g.head_in;
     out_at = head * g.head_out;
+  }
+  if constexpr (EPI == kLinearStore) {
+    if (g.rows_there) {
+      t_end = min(t_end, *g.rows_there);
+      if (t0 >= t_end) {
+        dependency_wait();
+        return;
+      }
+    }
   }
   // per expert only the tokens there are cost anything: wide tiles load them 32 rows at a time
   constexpr bool kGather = Gathers(EPI, BN);
@@ -505,10 +515,12 @@ int Linear(const Queue& q, const LinearArgs& a) {
   const bool experts = PerExpert(a.epilogue);
   if (experts && (a.slots.slots <= 0 || a.slots.tile_rows < 16 || !a.slots.tiles)) return int(cudaErrorInvalidValue);
   if (a.epilogue == kLinearHeads ? a.heads < 1 || a.head_in % 8 != 0 || a.bias : a.heads != 0) return int(cudaErrorInvalidValue);
+  if (a.rows_there && (q.f32 || a.epilogue != kLinearStore)) return int(cudaErrorInvalidValue);
   if (a.epilogue == kLinearExpertStore && !q.f32) return int(cudaErrorInvalidValue);
   LinearParams p{};
   p.head_in = a.head_in;
   p.head_out = a.head_out;
+  p.rows_there = a.rows_there;
   p.bias = a.bias;
   p.out = a.out;
   p.t = a.t;

@@ -490,11 +490,13 @@ int Attend(const Queue& q, const StepRows& r, const AttentionArgs& a) {
 }
 
 int AppendLatent(const Queue& q, const StepRows& r, const LatentArgs& a) {
-  return q.f32 ? AppendLatentAs<float>(q, r, a, false) : AppendLatentAs<__nv_bfloat16>(q, r, a, false);
+  if (q.f32 || !LatentTiled(a)) return q.f32 ? AppendLatentAs<float>(q, r, a, false) : AppendLatentAs<__nv_bfloat16>(q, r, a, false);
+  return r.singles == r.entries ? 0 : AppendLatentAs<__nv_bfloat16>(q, r, a, true);
 }
 
 int AttendLatent(const Queue& q, const StepRows& r, const LatentArgs& a) {
-  return q.f32 ? AttendLatentAs<float>(q, r, a) : AttendLatentAs<__nv_bfloat16>(q, r, a);
+  if (q.f32) return AttendLatentAs<float>(q, r, a);
+  return LatentTiled(a) ? AttendLatentTiles(q, r, a) : AttendLatentAs<__nv_bfloat16>(q, r, a);
 }
 
 int Retain(const Queue& q, const StepRows& r, const RetentionArgs& a) {

@@ -8,50 +8,13 @@
 
 #include "element.cuh"
 #include "mixers.cuh"
+#include "mma.cuh"
 #include "ops.h"
 #include "ptx.cuh"
 #include "tensor_map.h"
 
 namespace tmb {
 namespace {
-
-using bf16 = __nv_bfloat16;
-
-__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack(float lo, float hi) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
-  return *reinterpret_cast<const uint32_t*>(&h);
-}
-// What rounding to bf16 leaves behind.
-__device__ __forceinline__ float rest(float v) { return v - __bfloat162float(__float2bfloat16_rn(v)); }
-
-__device__ __forceinline__ void copy16(void* dst, const void* src, bool live) {   // 16 bytes, zero-filled unless live
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ void copy_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void copy_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
-// Operand tiles in shared memory are row-major with `pitch` elements per row, pitch = 16 n + 8: the eight rows of an
-// ldmatrix tile then start in eight different bank groups.
-__device__ __forceinline__ void load_a(uint32_t (&a)[4], const bf16* tile, int pitch, int row, int col, int lane) {
-  ldmatrix_x4(a, smem_u32(tile + (row + (lane & 15)) * pitch + col + (lane >> 4) * 8));
-}
-// A = tile^T: tile holds [k][m]
-__device__ __forceinline__ void load_a_transposed(uint32_t (&a)[4], const bf16* tile, int pitch, int k, int m, int lane) {
-  ldmatrix_x4_trans(a, smem_u32(tile + (k + (lane & 7) + (lane >> 4) * 8) * pitch + m + ((lane >> 3) & 1) * 8));
-}
-// two n8 tiles of B, tile holds [n][k]
-__device__ __forceinline__ void load_b(uint32_t (&b)[4], const bf16* tile, int pitch, int n, int k, int lane) {
-  ldmatrix_x4(b, smem_u32(tile + (n + (lane & 7) + (lane >> 4) * 8) * pitch + k + ((lane >> 3) & 1) * 8));
-}
-// two n8 tiles of B, tile holds [k][n]
-__device__ __forceinline__ void load_b_transposed(uint32_t (&b)[4], const bf16* tile, int pitch, int k, int n, int lane) {
-  ldmatrix_x4_trans(b, smem_u32(tile + (k + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + n + (lane >> 4) * 8));
-}
 
 // ---- attention ---------------------------------------------------------------------------------------------------------
 constexpr int kKeys = 64;   // keys per block
@@ -66,6 +29,9 @@ struct AttendParams {
   const float *q_norm, *k_norm;
   int proj_stride, out_stride, heads, kv_heads, dim, vdim, pool_dim, v_pool_dim, window, keep, splits, gate_at;
   int subs, sub_heads;      // query heads of one key head are served in `subs` units of up to `sub_heads`
+  int q_head;               // elements from one query head to the next
+  const int* context;       // portions whose keys and values are rows [.. + position] of k_pool and v_pool (see AttendContext), or null
+  int context_stride;
   float scale_log2, sink_log2, eps;
   bool value_is_key, even;
   Rotary rotary;
@@ -98,7 +64,7 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
   bf16* vs = ks + 2 * Shape::kTile;
   __shared__ unsigned last;
   __shared__ float2 square_part[NT / 32];
-  __shared__ int key_at[2][kKeys];   // pool rows of a block's keys (-1: none)
+  __shared__ long long key_at[2][kKeys], value_at[2][kKeys];   // element offsets of a block's keys (-1: none) and values
   // Every kernel of a step lets the next one start only behind its own dependency wait, so what kernels before the last
   // one wrote is there already: the step's tables, and the keys of earlier steps. A decoded token's first block of keys
   // is therefore requested before the wait (its own key, if the block holds it, is put over the copy later).
@@ -127,10 +93,24 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
   const int from = WM == 1 ? min(blocks, split * share) : 0, to = WM == 1 ? min(blocks, from + share) : blocks;
   auto block_base = [&](int b) { return b < kept_blocks ? b * kKeys : low + (b - kept_blocks) * kKeys; };
   auto block_limit = [&](int b) { return b < kept_blocks ? kept : p1 + 1; };
+  const int context = WM > 1 && p.context ? p.context[blockIdx.z] - max(0, e.first_position - p.window + 1) : 0;
   auto locate = [&](int b) {   // one block ahead of its fetch: the block-table loads are then off the copies' path
     if (threadIdx.x < kKeys && b < to) {
-      const int j = block_base(b) + int(threadIdx.x);
-      key_at[(b - from) & 1][threadIdx.x] = j < block_limit(b) ? key_row(table, j, r) : -1;
+      const int j = block_base(b) + int(threadIdx.x), stage = (b - from) & 1;
+      long long key = -1, value = -1;
+      if (j < block_limit(b)) {
+        if (WM > 1 && p.context) {
+          key = (long long)(context + j) * p.context_stride;
+          value = key + group * p.v_pool_dim;
+          key += group * p.pool_dim;
+        } else {
+          const int row = key_row(table, j, r);
+          key = (long long)(pool_offset(row, group, p.kv_heads, p.pool_dim));
+          value = (long long)(pool_offset(row, group, p.kv_heads, p.v_pool_dim));
+        }
+      }
+      key_at[stage][threadIdx.x] = key;
+      value_at[stage][threadIdx.x] = value;
     }
   };
   auto fetch = [&](int b) {
@@ -138,11 +118,11 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
     constexpr int C = DT * 2;   // 16-byte pieces of a row
 #pragma unroll 4
     for (int i = threadIdx.x; i < kKeys * C; i += NT) {
-      const int key = i / C, c = (i % C) * 8, row = key_at[stage][key];
-      const bool live = row >= 0;
-      const size_t line = live ? size_t(row / kRaggedBlock * p.kv_heads + group) * kRaggedBlock + row % kRaggedBlock : 0;
-      if (FULL || c < p.pool_dim) copy16(ks + stage * Shape::kTile + key * P + c, p.k_pool + line * p.pool_dim + c, live);
-      if (FULL || c < p.v_pool_dim) copy16(vs + stage * Shape::kTile + key * P + c, p.v_pool + line * p.v_pool_dim + c, live);
+      const int key = i / C, c = (i % C) * 8;
+      const long long at = key_at[stage][key];
+      const bool live = at >= 0;
+      if (FULL || c < p.pool_dim) copy16(ks + stage * Shape::kTile + key * P + c, p.k_pool + (live ? at + c : 0), live);
+      if (FULL || c < p.v_pool_dim) copy16(vs + stage * Shape::kTile + key * P + c, p.v_pool + (live ? value_at[stage][key] + c : 0), live);
     }
     copy_commit();
   };
@@ -183,10 +163,10 @@ __global__ void __launch_bounds__(AttendShape<DT, WM>::kThreads, DT > 8 ? 1 : WM
       qs[m * P + d] = __float2bfloat16_rn(a);
     }
   } else {
-    const bool wide = (p.dim & 7) == 0;
+    const bool wide = (p.dim & 7) == 0 && (p.q_head & 7) == 0;
     for (int i = threadIdx.x; i < Shape::kRows * (P / 8); i += NT) {
       const int m = i / (P / 8), c = (i % (P / 8)) * 8, t = m / gq;
-      const bf16* head = p.proj + size_t(e.first_row + t0 + t) * p.proj_stride + size_t(head0 + m % gq) * p.dim;
+      const bf16* head = p.proj + size_t(e.first_row + t0 + t) * p.proj_stride + size_t(head0 + m % gq) * p.q_head;
       uint4 word = make_uint4(0, 0, 0, 0);
       if (t < tokens && c < p.dim) {
         if (wide) {
@@ -806,7 +786,9 @@ template <int DT> cudaError_t Raise() {
 
 }  // namespace
 
-int AttendTiles(const Queue& q, const StepRows& r, const AttentionArgs& a) {
+namespace {
+
+AttendParams ParamsOf(const AttentionArgs& a) {
   AttendParams p{};
   p.proj = static_cast<const bf16*>(a.proj);
   p.k_pool = static_cast<bf16*>(a.k_pool);
@@ -839,9 +821,28 @@ int AttendTiles(const Queue& q, const StepRows& r, const AttentionArgs& a) {
   p.sink_log2 = a.sink * 1.4426950408889634f;
   p.sinks = a.sinks;
   p.blend = {a.blend, a.blend_from, a.blend_stride};
+  p.q_head = a.dim;
+  return p;
+}
+
+}  // namespace
+
+int AttendTiles(const Queue& q, const StepRows& r, const AttentionArgs& a) {
+  const AttendParams p = ParamsOf(a);
   const int tiles = (std::max(a.dim, a.vdim) + 15) / 16;
   return tiles <= 2 ? AttendWith<2>(q, r, a, p) : tiles <= 4 ? AttendWith<4>(q, r, a, p) : tiles <= 6 ? AttendWith<6>(q, r, a, p)
          : tiles <= 8 ? AttendWith<8>(q, r, a, p) : tiles <= 12 ? AttendWith<12>(q, r, a, p) : AttendWith<16>(q, r, a, p);
+}
+
+int AttendContext(const Queue& q, const StepRows& r, const AttentionArgs& a, int q_head, const int* context, int context_stride) {
+  AttendParams p = ParamsOf(a);
+  p.q_head = q_head;
+  p.context = context;
+  p.context_stride = context_stride;
+  p.splits = 1;
+  const int tiles = (std::max(a.dim, a.vdim) + 15) / 16, per_tile = 128 / p.sub_heads, x = (r.longest + per_tile - 1) / per_tile;
+  return tiles <= 2 ? LaunchAttend<2, 8>(q, r, p, x) : tiles <= 4 ? LaunchAttend<4, 8>(q, r, p, x) : tiles <= 6 ? LaunchAttend<6, 8>(q, r, p, x)
+         : tiles <= 8 ? LaunchAttend<8, 8>(q, r, p, x) : tiles <= 12 ? LaunchAttend<12, 8>(q, r, p, x) : LaunchAttend<16, 8>(q, r, p, x);
 }
 
 int RetainChunks(const Queue& q, const StepRows& r, const RetentionArgs& a) {

@@ -145,6 +145,7 @@ struct LinearArgs {
   void* out;                 // element buffer, or the fp32 residual stream, or fp32
   const LinearMaps* maps;    // bf16 only
   int t, n, k_stride, out_stride;
+  const int* rows_there;     // bf16: of the t rows only the first *rows_there are needed (null: all); written two kernels before, or earlier
   int in_stride;             // elements of an activation row, if it is not k_stride (0)
   int heads, head_in, head_out;   // kLinearHeads
   int outputs;               // kLinearGlu: columns stored (pairs beyond it are padding)
@@ -226,6 +227,10 @@ struct AttentionArgs {
 int RotateAppend(const Queue& q, const StepRows& r, const AttentionArgs& a);
 int Attend(const Queue& q, const StepRows& r, const AttentionArgs& a);
 int AttendTiles(const Queue& q, const StepRows& r, const AttentionArgs& a);   // the bf16 form
+// The portions of a step over keys and values that lie in rows of context_stride elements: position j of entry n in row
+// context[n] + j - max(0, first_position - window + 1), keys of head g at k_pool + g * pool_dim there, values at
+// v_pool + g * v_pool_dim. Query heads are q_head elements apart; nothing is rotated, normed or appended.
+int AttendContext(const Queue& q, const StepRows& r, const AttentionArgs& a, int q_head, const int* context, int context_stride);
 int PrepareMixers();
 
 // Attention whose keys and values are images, per head, of one cached latent row per token: scores and sums are taken
@@ -243,13 +248,23 @@ struct LatentArgs {
   float eps, scale, sink;
   const float* sinks;        // [heads], or null
   int window;
+  bool singles_only;         // portions are attended to elsewhere
   float* part;               // decode partials, part_floats floats
   size_t part_floats;
   unsigned* count;           // arrival counters, zero between launches
   int count_words;
 };
+// (bf16 rows that suit the tiled form: AppendLatent takes portions only, a decoded token's attention appends its own row.)
 int AppendLatent(const Queue& q, const StepRows& r, const LatentArgs& a);
 int AttendLatent(const Queue& q, const StepRows& r, const LatentArgs& a);
+constexpr int kTiledLatent = 512;   // widest latent row of the tiled form
+inline bool LatentTiled(const LatentArgs& a) { return a.rank <= kTiledLatent; }
+int AttendLatentTiles(const Queue& q, const StepRows& r, const LatentArgs& a);   // the tiled form
+int PrepareLatent();
+// Long portions expand the latent rows they see into keys and values first: where each entry's rows start in the expanded
+// ones (context [entries], and how many there are in all), and those rows gathered from the pool, `most` at most.
+int LatentContext(const Queue& q, const StepRows& r, int window, int* context, int* context_rows);
+int GatherLatent(const Queue& q, const StepRows& r, const LatentArgs& a, const int* context, const int* context_rows, int most, void* out);
 
 // Retention: per head S <- decay S + k v^T, o = S^T q, with rotary q and k, k scaled by key_scale. proj rows hold
 // q | k | v | g. state [slots][heads][dim][vdim] fp32; an entry that starts at position 0 starts from a zero state.

@@ -29,6 +29,10 @@ struct RaggedPlan {
   void* mlp = nullptr;         // [max_rows][widest feed-forward]
   void* pairs = nullptr;       // fp32 plans: gate/up rows before the gated unit
   float* branch = nullptr;     // fp32 outputs of sublayers that are normed before they are added
+  // bf16 plans with latent attention: the latent rows that portions see, gathered, and their keys and values
+  void *context = nullptr, *expanded = nullptr;
+  int *context_at = nullptr, *context_count = nullptr;
+  int context_rows = 0;
   // mixtures of experts: logits, choices and scores per row, the assignments sorted by expert, their hidden rows and outputs
   float* logits = nullptr;
   int *choice = nullptr, *list = nullptr, *tile_count = nullptr;
@@ -49,7 +53,7 @@ struct RaggedPlan {
   std::vector<float*> decay;   // per layer
   struct Maps {
     LinearMaps in, out, gate_up, down, router;   // (gate_up, down: of the gated unit or of the experts)
-    LinearMaps shared_up, shared_down, key_up, value_up;
+    LinearMaps shared_up, shared_down, key_up, value_up, expand;
   };
   std::vector<Maps> maps;      // per layer (bf16 plans)
   LinearMaps head;
@@ -67,6 +71,17 @@ template <typename T> bool Own(RaggedPlan* plan, T** out, size_t bytes) {
   plan->owned.push_back(p);
   *out = static_cast<T*>(p);
   return cudaMemset(p, 0, bytes) == cudaSuccess;
+}
+
+// Rows (at most) that a step's portions see of a latent layer, if these are to be expanded into keys and values: for long
+// portions that is less work than scores and sums over latent rows, by about three products' cost to one of attention.
+int ContextRows(const RaggedPlan* plan, const StepRows& r, const RaggedMixer& m) {
+  const int portions = r.entries - r.singles, rows = r.rows - r.singles;
+  if (!plan->context_rows || portions == 0) return 0;
+  const double reach = std::min(m.window, r.capacity), each = double(rows) / portions, head = m.dim + m.vdim;
+  const double most = rows + portions * (reach - 1);
+  if (most > plan->context_rows) return 0;
+  return each * reach * (2.0 * m.rank - head) > (each + reach) * m.rank * head / 3.0 ? int(most) : 0;
 }
 
 int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest, uint32_t singles, uint32_t wanted, bool feed, cudaStream_t stream) {
@@ -175,6 +190,7 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     const RaggedLayer& first = s.layers[size_t(s.runs[0].layer)];
     TMB_TRY(restream(nullptr, nullptr, &first.streams[0], first.norm1, nullptr));
   }
+  int context_window = -1;               // the window that the table of expanded rows is for
   for (size_t i = 0; i < s.runs.size(); ++i) {
     const RaggedRun& run = s.runs[i];
     const RaggedLayer* next = i + 1 < s.runs.size() ? &s.layers[size_t(s.runs[i + 1].layer)] : nullptr;
@@ -232,19 +248,51 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.count_words = plan->count_words;
       const int wide = m.heads * m.rank_stride();
       TMB_TRY(AppendLatent(q, r, a));
-      LinearArgs up = linear(proj, layer.key_up, -1, maps ? &maps->key_up : nullptr, m.rank, m.head_stride(), plan->lookup, wide, kLinearHeads);
-      up.in_stride = stride;
-      up.heads = m.heads;
-      up.head_in = m.head_stride();
-      up.head_out = m.rank_stride();
-      TMB_TRY(Linear(q, up));
-      TMB_TRY(AttendLatent(q, r, a));
-      LinearArgs down = linear(plan->looked, layer.value_up, -1, maps ? &maps->value_up : nullptr, m.vdim, m.rank, plan->mixed, mixed_stride, kLinearHeads);
-      down.in_stride = wide;
-      down.heads = m.heads;
-      down.head_in = m.rank_stride();
-      down.head_out = m.vdim;
-      TMB_TRY(Linear(q, down));
+      const int context = ContextRows(plan, r, m);
+      a.singles_only = context > 0;
+      if (!context || r.singles) {
+        LinearArgs up = linear(proj, layer.key_up, -1, maps ? &maps->key_up : nullptr, m.rank, m.head_stride(), plan->lookup, wide, kLinearHeads);
+        up.in_stride = stride;
+        up.heads = m.heads;
+        up.head_in = m.head_stride();
+        up.head_out = m.rank_stride();
+        TMB_TRY(Linear(q, up));
+        TMB_TRY(AttendLatent(q, r, a));
+        LinearArgs down = linear(plan->looked, layer.value_up, -1, maps ? &maps->value_up : nullptr, m.vdim, m.rank, plan->mixed, mixed_stride, kLinearHeads);
+        down.in_stride = wide;
+        down.heads = m.heads;
+        down.head_in = m.rank_stride();
+        down.head_out = m.vdim;
+        TMB_TRY(Linear(q, down));
+      }
+      if (context) {                     // (behind the products of all rows, whose result for the portions' rows it replaces)
+        if (context_window != m.window) TMB_TRY(LatentContext(q, r, m.window, plan->context_at, plan->context_count));
+        context_window = m.window;
+        TMB_TRY(GatherLatent(q, r, a, plan->context_at, plan->context_count, context, plan->context));
+        const int columns = m.expanded_columns();
+        LinearArgs expand = linear(plan->context, layer.expand, -1, &maps->expand, columns, m.rank, plan->expanded, columns, kLinearStore);
+        expand.t = context;
+        expand.rows_there = plan->context_count;
+        TMB_TRY(Linear(q, expand));
+        AttentionArgs seen{};
+        seen.proj = proj;
+        seen.proj_stride = stride;
+        seen.k_pool = plan->expanded;
+        seen.v_pool = static_cast<char*>(plan->expanded) + size_t(m.heads) * m.expanded_key() * 2;
+        seen.out = plan->mixed;
+        seen.out_stride = mixed_stride;
+        seen.heads = seen.kv_heads = m.heads;
+        seen.dim = m.dim;
+        seen.vdim = m.vdim;
+        seen.pool_dim = m.expanded_key();
+        seen.v_pool_dim = m.v_pool_dim();
+        seen.sink = a.sink;
+        seen.sinks = a.sinks;
+        seen.gate_at = -1;
+        seen.window = m.window;
+        seen.scale = a.scale;
+        TMB_TRY(AttendContext(q, r, seen, m.head_stride(), plan->context_at, columns));
+      }
     } else {
       AttentionArgs a{};
       a.proj = proj;
@@ -428,7 +476,8 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
   };
   const size_t element = spec.f32 ? 4 : 2;
   size_t proj = 0, mixed = 0, mlp = 0, pairs = 0, raw = 0, split = 0, heads = 1, partial = 0;
-  size_t top = 0, experts = 0, expert_columns = 0, expert_pairs = 0, source = 0, latent = 0, ranks = 0;
+  size_t top = 0, experts = 0, expert_columns = 0, expert_pairs = 0, source = 0, latent = 0, ranks = 0, context = 0, expanded = 0;
+  int reach = 0;
   for (const RaggedLayer& layer : spec.layers) {
     const RaggedMixer& m = layer.mixer;
     proj = std::max(proj, size_t(m.proj_rows() + 7) / 8 * 8);
@@ -460,11 +509,19 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
     } else {
       const size_t columns = m.kind == RaggedMixer::kLatent ? size_t(m.rank_stride()) : size_t(m.vdim);
       heads = std::max(heads, size_t(m.heads));
-      partial = std::max(partial, size_t(m.heads) * (columns + 2));
-      if (m.kind == RaggedMixer::kLatent) latent = std::max(latent, size_t(m.heads) * m.rank_stride());
+      // (latent attention fills an SM with one or two CTAs: a fourth of the parts)
+      partial = std::max(partial, size_t(m.heads) * (columns + 2) / (m.kind == RaggedMixer::kLatent ? 4 : 1));
+      if (m.kind == RaggedMixer::kLatent) {
+        latent = std::max(latent, size_t(m.heads) * m.rank_stride());
+        context = std::max(context, size_t(m.rank_stride()));
+        expanded = std::max(expanded, size_t(m.expanded_columns()));
+        reach = std::max(reach, std::min(m.window, spec.capacity));
+      }
     }
   }
   const size_t rows = size_t(spec.max_rows), W8 = size_t(padded_columns(spec.width)), slots = rows * top;
+  if (context && !spec.f32) plan->context_rows = int(std::min(size_t(spec.max_rows) + 2 * size_t(reach), size_t(spec.slots) * spec.capacity + spec.max_rows));
+  const size_t context_rows = size_t(plan->context_rows);
   plan->count_words = int(heads) * spec.slots;
   // a decode step cuts a long window into parts: at most eight CTAs per SM's worth of parts in all, one per head at least
   plan->part_floats = partial * (size_t(spec.slots) + 8 * size_t(sm_count));
@@ -472,6 +529,8 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
       !Own(plan, &plan->proj, rows * proj * element) || !Own(plan, &plan->mixed, rows * mixed * element) ||
       !Own(plan, &plan->mlp, rows * mlp * element) || !Own(plan, &plan->pairs, spec.f32 ? rows * pairs * element : 0) ||
       !Own(plan, &plan->branch, spec.layers[0].norm_output || spec.combined ? rows * size_t(spec.width) * sizeof(float) : 0) ||
+      !Own(plan, &plan->context, context_rows * context * element) || !Own(plan, &plan->expanded, context_rows * expanded * element) ||
+      !Own(plan, &plan->context_at, size_t(spec.slots) * sizeof(int)) || !Own(plan, &plan->context_count, sizeof(int)) ||
       !Own(plan, &plan->source, rows * source * element) || !Own(plan, &plan->lookup, rows * latent * element) ||
       !Own(plan, &plan->looked, rows * latent * element) || !Own(plan, &plan->ranks, rows * ranks * sizeof(float)) ||
       !Own(plan, &plan->expert_pairs, spec.f32 ? slots * expert_pairs * element : 0) ||
@@ -522,7 +581,8 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
         ok = ok && EncodeHeads(&maps.key_up, at(layer.key_up), uint64_t(m.heads) * m.rank, uint64_t(m.head_stride()), plan->proj, rows,
                                size_t(m.proj_rows() + 7) / 8 * 8) &&
              EncodeHeads(&maps.value_up, at(layer.value_up), uint64_t(m.heads) * m.vdim, uint64_t(m.rank_stride()), plan->looked, rows,
-                         uint64_t(m.heads) * m.rank_stride());
+                         uint64_t(m.heads) * m.rank_stride()) &&
+             EncodeLinear(&maps.expand, at(layer.expand), uint64_t(m.expanded_columns()), plan->context, context_rows, uint64_t(m.rank_stride()));
       if (mlp.kind == RaggedMlp::kExperts)
         ok = ok && EncodeLinear(&maps.router, at(layer.router), uint64_t(mlp.logits()), plan->normed, rows, W8) &&
              EncodeLinear(&maps.gate_up, at(layer.expert_up), uint64_t(mlp.experts) * (mlp.output_weighted ? mlp.packed_rows() : mlp.ff), plan->gathered,
@@ -541,7 +601,7 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
     if (!EncodeLinear(&plan->head, at(spec.head), uint64_t(spec.vocab), plan->picked, uint64_t(spec.max_wanted), W8))
       return fail("cuTensorMapEncodeTiled rejected the head");
   }
-  if (PrepareLinear() != 0 || PrepareMixers() != 0) return fail("cannot raise the kernels' shared-memory limit");
+  if (PrepareLinear() != 0 || PrepareMixers() != 0 || PrepareLatent() != 0) return fail("cannot raise the kernels' shared-memory limit");
   return plan;
 }
 

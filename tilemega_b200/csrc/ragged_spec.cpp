@@ -229,7 +229,7 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     Require(place == "input" || place == "output", "a layer's norms act on its sublayers' input or output (norm_at)");
     layer.norm_output = place == "output";
     Require(i == 0 || layer.norm_output == s.layers[0].norm_output, "every layer of a model has its norms in the same place");
-    Require(!s.combined || !layer.norm_output, "streams and experts whose outputs are weighted need the norms on the sublayers' inputs");
+    Require(!s.combined || !layer.norm_output, "layers with norms on their outputs have one stream, and experts with weights on their inputs");
     auto streams = [&](int which) {
       if (!in.has("streams")) {
         Require(s.streams == 1, "every layer of a model with several streams says how its sublayers use them");
@@ -252,6 +252,10 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
       // a query against latent rows is its head's key matrix, transposed, times the query
       layer.key_up = add(p + "key_up.weight", 1, element, uint64_t(m.heads) * m.rank * m.head_stride(), 0,
                          PadColumns(PerHead("transpose_heads", Json::Quote(Name(names, "uk")), m.heads, "rows", m.dim), m.head_stride()));
+      if (!s.f32)
+        layer.expand = add(p + "expand.weight", 1, element, uint64_t(m.expanded_columns()) * rank, 0,
+                           PadColumns(Stack({PerHead("pad_heads", Json::Quote(Name(names, "uk")), m.heads, "rows", m.expanded_key()),
+                                             PerHead("pad_heads", Json::Quote(Name(names, "uv")), m.heads, "rows", m.v_pool_dim())}), rank));
       layer.value_up = add(p + "value_up.weight", 1, element, uint64_t(m.heads) * m.vdim * rank, 0,
                            PadColumns(Stack({Json::Quote(Name(names, "uv"))}), rank));
     }

@@ -40,6 +40,8 @@ struct RaggedMixer {
   int out_columns() const { return heads * vdim; }
   int head_stride() const { return (dim + 7) / 8 * 8; }      // latent attention: columns of one head's query
   int rank_stride() const { return (rank + 7) / 8 * 8; }     // ... and of its query or output against latent rows
+  int expanded_key() const { return (dim + 15) / 16 * 16; }  // ... and of its key and value expanded from latent rows
+  int expanded_columns() const { return heads * (expanded_key() + v_pool_dim()); }
   int pool_dim() const { return ((kind == kLatent ? rank : dim) + 15) / 16 * 16; }
   int v_pool_dim() const { return (vdim + 15) / 16 * 16; }
 };
@@ -74,7 +76,7 @@ struct RaggedLayer {
   bool norm_output = false;               // the norms act on the sublayers' outputs; the sublayers read the stream itself
   // indices into the plan's buffer table
   int norm1 = -1, in_weight = -1, in_bias = -1, out_weight = -1, out_bias = -1, norm2 = -1, gate_up = -1, down = -1, decay = -1,
-      q_norm = -1, k_norm = -1, router = -1, expert_up = -1, expert_down = -1, sinks = -1, blend = -1, latent_norm = -1, key_up = -1, value_up = -1,
+      q_norm = -1, k_norm = -1, router = -1, expert_up = -1, expert_down = -1, sinks = -1, blend = -1, latent_norm = -1, key_up = -1, value_up = -1, expand = -1,
       correction = -1, shared_up = -1, shared_down = -1;
   RaggedStreams streams[2];               // of the mixer and of the feed-forward
 };
