@@ -70,8 +70,10 @@ MODELS = {"llama-3.1-8b": synthetic.LLAMA_3_1_8B, "llama-3.2-1b": synthetic.LLAM
           "llama-3.1-70b": synthetic.LLAMA_3_1_70B, "qwen3-30b-a3b": synthetic.QWEN3_30B_A3B,
           "bert-base": synthetic.BERT_BASE,   # the encoder forward workload (run_forward)
           "bamudra-8b": synthetic.BAMUDRA_8B, "bamudra-1b": synthetic.BAMUDRA_1B,   # ragged-step plans (run_ragged)
-          "nadilorn-8b": synthetic.NADILORN_8B, "nadilorn-1b": synthetic.NADILORN_1B, "nadilorn-30b-a3b": synthetic.NADILORN_30B_A3B}
-LAYERED = ("bamudra", "nadilorn")   # decoders given as a list of layers
+          "nadilorn-8b": synthetic.NADILORN_8B, "nadilorn-1b": synthetic.NADILORN_1B, "nadilorn-30b-a3b": synthetic.NADILORN_30B_A3B,
+          "nadilorn-7b-a1b": synthetic.NADILORN_7B_A1B, "nadilorn-47b-a13b": synthetic.NADILORN_47B_A13B,
+          "mozidra-30b-a3b": synthetic.MOZIDRA_30B_A3B, "mozidra-7b-a1b": synthetic.MOZIDRA_7B_A1B, "mozidra-47b-a13b": synthetic.MOZIDRA_47B_A13B}
+LAYERED = ("bamudra", "nadilorn", "mozidra")   # decoders given as a list of layers
 
 
 def workload(args) -> dict:
@@ -500,7 +502,7 @@ def run_forward(args) -> None:
 
 def run_ragged(args) -> None:
     """Secondary workload: a decoder given as a list of layers (`--model bamudra-8b | bamudra-1b | nadilorn-8b | nadilorn-1b |
-    nadilorn-30b-a3b`) through a ragged-step plan (phase 3 of the plan ABI). Decode: `--batch` sequences at `--context`
+    nadilorn-30b-a3b | nadilorn-7b-a1b | nadilorn-47b-a13b`, and `mozidra-` for the last three sizes) through a ragged-step plan (phase 3 of the plan ABI). Decode: `--batch` sequences at `--context`
     positions, one step = one decoded token of each, the sampled tokens fed back on the device. `--prefill T`: a prompt of T tokens in portions of `--portion` rows, one step =
     one portion. One JSON line in the shape of the decode line; same weights, widths and vocabulary as the Llama-shaped
     model of the same name, so the two lines stand side by side."""
@@ -543,8 +545,9 @@ def run_ragged(args) -> None:
         return min(position + 1, size) + min(keep, max(0, position + 1 - size))
 
     def cached(position: int) -> int:
-        """Bytes of keys and values one token at this position reads, all attention layers."""
-        return sum(seen(mixer, position) * 2 * mixer["kv_heads"] * (mixer["dim"] + mixer["vdim"]) for mixer in attention)
+        """Bytes of keys and values (or of latent rows) one token at this position reads, all attention layers."""
+        return sum(seen(mixer, position) * 2 * (mixer["kv_rank"] if "kv_rank" in mixer else mixer["kv_heads"] * (mixer["dim"] + mixer["vdim"]))
+                   for mixer in attention)
 
     def attention_flops(position: int) -> int:
         return sum(seen(mixer, position) * 2 * mixer["heads"] * (mixer["dim"] + mixer["vdim"]) for mixer in attention)
@@ -554,7 +557,7 @@ def run_ragged(args) -> None:
     mixtures = [layer["mlp"] for layer in config["layers"] if layer["mlp"] and layer["mlp"]["kind"] == "moe"]
     for mlp in mixtures:                                         # experts a batch reads, if its tokens spread evenly
         experts, top = mlp["router"]["experts"], mlp["router"]["top"]
-        weight_bytes += round(2 * 2 * width * mlp["expert"]["ff"] * (experts * (1.0 - (1.0 - top / experts) ** batch) - top))
+        weight_bytes += round(2 * (3 if "shared" in mlp else 2) * width * mlp["expert"]["ff"] * (experts * (1.0 - (1.0 - top / experts) ** batch) - top))
     peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
     if args.prefill:
         prompt = synthetic.seeded_tokens(1, context, vocab, seed=3)[0].tolist()
@@ -848,7 +851,7 @@ def main() -> None:
                         help="--model bert-base: element type of the forward plan (f16: the benchmark configuration; bf16: what the reference's export runs)")
     parser.add_argument("--prefill", type=int, default=0,
                         help="secondary workload: chunked prefill of one prompt of this many tokens (one GPU)")
-    parser.add_argument("--portion", type=int, default=2048, help="--model bamudra-* / nadilorn-*: rows per step of a prefilled prompt")
+    parser.add_argument("--portion", type=int, default=2048, help="--model bamudra-* / nadilorn-* / mozidra-*: rows per step of a prefilled prompt")
     parser.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     parser.add_argument("--trace", action="store_true",
                         help="after the timed runs, stamp one more step and print the per-stage table (rank 0)")

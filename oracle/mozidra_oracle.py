@@ -78,15 +78,15 @@ def window_of(spec: dict) -> int | None:
 
 
 def attention_mixer(h: torch.Tensor, positions: torch.Tensor, spec: dict, w, eps: float, first_values: torch.Tensor | None):
-    """(mixer output, the layer's own values before mixing [T, kv_heads, vdim])."""
+    """(mixer output, the layer's own values before mixing [T, kv_heads * vdim])."""
     heads, groups = spec["heads"], spec["kv_heads"]
     q = rms(h @ w("q").T + w("q.b"), eps) * w("q.norm")         # one mean over all heads together
     k = rms(h @ w("k").T + w("k.b"), eps) * w("k.norm")
-    own = (h @ w("v").T + w("v.b")).reshape(-1, groups, spec["vdim"])
+    own = h @ w("v").T + w("v.b")
     v = own
     if first_values is not None:
         v = (1.0 - w("vmix")) * own + w("vmix") * first_values
-    q, k = q.reshape(-1, heads, spec["dim"]), k.reshape(-1, groups, spec["dim"])
+    q, k, v = q.reshape(-1, heads, spec["dim"]), k.reshape(-1, groups, spec["dim"]), v.reshape(-1, groups, spec["vdim"])
     rot = spec.get("rot")
     if rot:
         q, k = rotate_pairs(q, positions, rot["base"], rot["dims"]), rotate_pairs(k, positions, rot["base"], rot["dims"])

@@ -234,10 +234,32 @@ NADILORN_8B = nadilorn_config(4096, 32, 8, 128, 14336, 32, 128256, 2048)
 NADILORN_1B = nadilorn_config(2048, 32, 8, 64, 8192, 16, 128256, 1024)
 NADILORN_30B_A3B = nadilorn_config(2048, 32, 4, 128, 6144, 48, 151936, 2048, 128, 8, 1152)
 
+NADILORN_7B_A1B = nadilorn_config(2048, 16, 4, 128, 6144, 16, 50304, 2048, 64, 8, 1536)
+NADILORN_47B_A13B = nadilorn_config(4096, 32, 8, 128, 14336, 32, 32000, 4096, 8, 2, 21504)
+
+
+# Mozidra-shaped decoders of the sizes of the mixtures above (an expert has three matrices, so its width is two thirds): of
+# three layers in a row two have latent attention, one grouped heads whose values are mixed across layers.
+def mozidra_config(width: int, heads: int, kv_heads: int, dim: int, rank: int, layers: int, vocab: int, window: int, streams: int,
+                   experts: int, top: int, groups: int, keep: int, expert_ff: int, shared_ff: int) -> dict:
+    sizes = {"heads": heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window}}
+    attention = sizes | {"kv_heads": kv_heads, "rot": {"base": 500000.0, "dims": dim // 2}, "v_mix": True}
+    mixture = {"kind": "moe", "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}},
+               "expert": {"ff": expert_ff, "limit": 7.0}, "shared": {"ff": shared_ff, "limit": 7.0}}
+    order = [{"type": "attention", "mixer": attention, "mlp": mixture} if index % 3 == 2 else
+             {"type": "latent_attention", "mixer": sizes | {"kv_rank": rank}, "mlp": mixture} for index in range(layers)]
+    return {"architecture": "Mozidra", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "streams": streams, "layers": order}
+
+
+MOZIDRA_30B_A3B = mozidra_config(2048, 32, 4, 128, 512, 48, 151936, 2048, 4, 128, 8, 8, 4, 768, 768)
+MOZIDRA_7B_A1B = mozidra_config(2048, 16, 4, 128, 256, 16, 50304, 2048, 2, 64, 8, 8, 4, 1024, 1024)
+MOZIDRA_47B_A13B = mozidra_config(4096, 32, 8, 128, 512, 32, 32000, 4096, 4, 8, 2, 4, 2, 14336, 2048)
+
 
 class LazyShapedCheckpoint:
     """Like LazySeededCheckpoint for any table of tensor shapes (registry.tensor_shapes): matrices N(0, std), norm
-    weights 1, biases N(0, std), each tensor from its own generator when it is asked for."""
+    weights 1, biases N(0, std), residual streams read in equal shares and kept as they are, each tensor from its own
+    generator when it is asked for."""
 
     def __init__(self, shapes: dict[str, tuple[int, ...]], seed: int = 0, dtype: torch.dtype = torch.bfloat16,
                  device: str | torch.device = "cuda", std: float = 0.02):
@@ -249,5 +271,10 @@ class LazyShapedCheckpoint:
             raise KeyError(f"checkpoint has no {name}")
         if name.split(".")[-1].startswith("norm"):
             return torch.ones(self.shapes[name], dtype=self.dtype, device=self.device)
+        if ".hc" in name:
+            shape = self.shapes[name]
+            if len(shape) == 2:
+                return torch.eye(shape[0], dtype=self.dtype, device=self.device)
+            return torch.full(shape, 1.0 / shape[0] if name.endswith(".in") else 1.0, dtype=self.dtype, device=self.device)
         generator = torch.Generator(device=self.device).manual_seed((self.seed << 32) ^ zlib.crc32(name.encode()))
         return torch.empty(self.shapes[name], dtype=self.dtype, device=self.device).normal_(0.0, self.std, generator=generator)
