@@ -86,61 +86,73 @@ template <bool HELD> __device__ __forceinline__ void choose(const RouteArgs& a, 
   }
 }
 // The same where scores are not the logits' order: ranked by score + correction, from the best groups only. `line` holds the
-// row's ranks (shared memory where HELD, else a.ranks).
-template <bool HELD> __device__ __forceinline__ void choose_ranked(const RouteArgs& a, int row, int lane, float* line) {
+// row's logits, then its ranks (shared memory where HELD, else a.ranks). One warp runs this once, so its loops stay short code.
+template <bool HELD> __device__ __forceinline__ void choose_ranked(const RouteArgs& a, int row, int lane, float* line, const float* correction) {
   const float* z = a.logits + size_t(row) * (a.experts + a.extra);
   float high = -INFINITY, sum = 0.f;
+#pragma unroll 4
+  for (int e = lane; e < a.experts; e += 32) {
+    const float v = __ldcg(z + e);
+    line[e] = v;
+    high = fmaxf(high, v);
+  }
   if (a.softmax) {
-    for (int e = lane; e < a.experts; e += 32) high = fmaxf(high, __ldcg(z + e));
     high = warp_max(high);
-    for (int e = lane; e < a.experts; e += 32) sum += expf(__ldcg(z + e) - high);
+#pragma unroll 1
+    for (int e = lane; e < a.experts; e += 32) sum += expf(line[e] - high);
     sum = warp_sum(sum);
   }
-  auto score = [&](int e) { return a.softmax ? expf(__ldcg(z + e) - high) / sum : 1.f / (1.f + expf(-__ldcg(z + e))); };
-  for (int e = lane; e < a.experts; e += 32) line[e] = score(e) + (a.correction ? a.correction[e] : 0.f);
+  auto score_of = [&](float logit) { return a.softmax ? expf(logit - high) / sum : 1.f / (1.f + expf(-logit)); };
+#pragma unroll 1
+  for (int e = lane; e < a.experts; e += 32) line[e] = score_of(line[e]) + (correction ? correction[e] : 0.f);
   __syncwarp();
   // the largest key behind (before, before_at) in falling order, the smaller index first where two are equal
-  auto next = [&](unsigned best, int at, unsigned& before, int& before_at) {
+  unsigned before = 0xffffffffu;
+  int before_at = -1;
+  auto next = [&](unsigned best, int at) {
     before = __reduce_max_sync(0xffffffffu, best);
     before_at = __reduce_min_sync(0xffffffffu, best == before ? at : 0x7fffffff);
   };
+  auto behind = [&](unsigned v, int at) { return v < before || (v == before && at > before_at); };
   if (a.keep_groups < a.groups) {
     const int size = a.experts / a.groups;
     auto largest = [&](int g) {
       unsigned v = 1u;
+#pragma unroll 4
       for (int e = g * size; e < (g + 1) * size; ++e) v = max(v, ordered(line[e]));
       return v;
     };
-    unsigned before = 0xffffffffu;
-    int before_at = -1;
+    const unsigned mine = lane < a.groups ? largest(lane) : 0u;
+    auto rank_of = [&](int g) { return g == lane ? mine : largest(g); };
+#pragma unroll 1
     for (int k = 0; k < a.keep_groups; ++k) {
       unsigned best = 0u;
       int at = 0x7fffffff;
+#pragma unroll 1
       for (int g = lane; g < a.groups; g += 32) {
-        const unsigned v = largest(g);
-        if (v > before || (v == before && g <= before_at)) continue;
-        if (v > best) {
+        const unsigned v = rank_of(g);
+        if (behind(v, g) && v > best) {
           best = v;
           at = g;
         }
       }
-      next(best, at, before, before_at);
+      next(best, at);
     }
     __syncwarp();
-    for (int g = lane; g < a.groups; g += 32) {
-      const unsigned v = largest(g);
-      if (v > before || (v == before && g <= before_at)) continue;
-      for (int e = g * size; e < (g + 1) * size; ++e) line[e] = -INFINITY;
-    }
+#pragma unroll 1
+    for (int g = lane; g < a.groups; g += 32)
+      if (behind(rank_of(g), g))
+        for (int e = g * size; e < (g + 1) * size; ++e) line[e] = -INFINITY;
     __syncwarp();
   }
   unsigned key[kMine];
   if (HELD)
 #pragma unroll
     for (int i = 0; i < kMine; ++i) key[i] = lane + 32 * i < a.experts ? max(ordered(line[lane + 32 * i]), 1u) : 0u;
-  unsigned before = 0xffffffffu;
-  int before_at = -1, mine_at = 0;
-  float total = 0.f, mine = 0.f;
+  before = 0xffffffffu;
+  before_at = -1;
+  int taken = 0;
+#pragma unroll 1
   for (int k = 0; k < a.top; ++k) {
     unsigned best = 0u;
     int at = 0x7fffffff;
@@ -154,37 +166,31 @@ template <bool HELD> __device__ __forceinline__ void choose_ranked(const RouteAr
     } else {
       for (int e = lane; e < a.experts; e += 32) {
         const unsigned v = max(ordered(line[e]), 1u);
-        if (v > before || (v == before && e <= before_at)) continue;
-        if (v > best) {
+        if (behind(v, e) && v > best) {
           best = v;
           at = e;
         }
       }
     }
-    next(best, at, before, before_at);
+    next(best, at);
     if (HELD) {
 #pragma unroll
       for (int i = 0; i < kMine; ++i)
         if (before_at == lane + 32 * i) key[i] = 0u;
     }
-    const int expert = min(before_at, a.experts - 1);
-    const float s = score(expert);
-    total += s;
-    if (lane == k) {
-      mine = s;
-      mine_at = expert;
-    }
+    if (lane == k) taken = min(before_at, a.experts - 1);
   }
+  const float score = lane < a.top ? score_of(__ldcg(z + taken)) : 0.f, total = warp_sum(score);
   if (lane < a.top) {
-    a.choice[row * a.top + lane] = mine_at;
-    a.score[row * a.top + lane] = a.weights ? mine / (total + 1e-20f) : mine;
+    a.choice[row * a.top + lane] = taken;
+    a.score[row * a.top + lane] = a.weights ? score / (total + 1e-20f) : score;
   }
 }
-__device__ __forceinline__ void choose(const RouteArgs& a, int row, int lane, float* line) {
+__device__ __forceinline__ void choose(const RouteArgs& a, int row, int lane, float* line, const float* correction) {
   const bool held = a.experts <= 32 * kMine;
   if (a.ranks) {
-    if (held) choose_ranked<true>(a, row, lane, line);
-    else choose_ranked<false>(a, row, lane, a.ranks + size_t(row) * a.experts);
+    if (held) choose_ranked<true>(a, row, lane, line, correction);
+    else choose_ranked<false>(a, row, lane, a.ranks + size_t(row) * a.experts, correction);
   } else {
     if (held) choose<true>(a, row, lane);
     else choose<false>(a, row, lane);
@@ -269,6 +275,10 @@ __global__ void __launch_bounds__(FUSED ? 256 : 1024) route(RouteArgs a) {
   __shared__ unsigned last;
   __shared__ float ranks[FUSED ? 8 : 32][32 * kMine];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5, logits = a.experts + a.extra;
+  // corrections wait in the table of slots, which is written behind their last use
+  float* correction = a.correction ? reinterpret_cast<float*>(first) : nullptr;
+  if (correction)
+    for (int e = threadIdx.x; e < a.experts; e += blockDim.x) correction[e] = a.correction[e];
   if constexpr (FUSED) {
     constexpr int N = 16 / sizeof(T);
     const int e = blockIdx.x * 8 + warp, pieces = a.k_stride / N, row0 = blockIdx.y * 8, rows = min(8, a.rows - row0);
@@ -292,14 +302,15 @@ __global__ void __launch_bounds__(FUSED ? 256 : 1024) route(RouteArgs a) {
         if (lane == 0) a.logits[size_t(row) * logits + e] = sum;
       }
     if (!arrives_last(a.count + 1 + blockIdx.y, gridDim.x, &last)) return;
-    if (warp < rows) choose(a, row0 + warp, lane, ranks[warp]);
+    if (warp < rows) choose(a, row0 + warp, lane, ranks[warp], correction);
     if (gridDim.y == 1) __syncthreads();
     else if (!arrives_last(a.count, gridDim.y, &last)) return;
   } else {
     dependency_wait();
     allow_dependents();
     const int row = blockIdx.x * warps + warp;
-    if (row < a.rows) choose(a, row, lane, ranks[warp]);
+    if (correction) __syncthreads();
+    if (row < a.rows) choose(a, row, lane, ranks[warp], correction);
     if (!arrives_last(a.count, gridDim.x, &last)) return;
   }
   sort_assignments(a, counts, first);

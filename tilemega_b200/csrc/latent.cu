@@ -16,7 +16,6 @@ namespace tmb {
 namespace {
 
 constexpr int kKeys = 64;          // latent rows per block
-constexpr int kWarps = 8, kThreads = 32 * kWarps;
 constexpr int kWeightPitch = kKeys + 8;
 
 struct LatentParams {
@@ -24,29 +23,32 @@ struct LatentParams {
   const bf16* raw;
   bf16* pool;
   bf16* out;
-  float* part;
-  unsigned* count;
+  float* part;                     // split sums: [entry][head][split][rank_stride] latent columns, then [entry][head][split] maxima and sums
   const float *norm, *sinks;
   int raw_stride, heads, rank, rank_stride, pool_dim, window, splits;
   int subs, sub_heads;             // the heads are served in `subs` units of up to `sub_heads`
   float scale_log2, sink_log2, eps;
+  __device__ float2* stats(int entries) const { return reinterpret_cast<float2*>(part + size_t(entries) * heads * splits * rank_stride); }
   __device__ float sink_of(int head) const { return sinks ? sinks[head] * 1.4426950408889634f : sink_log2; }
 };
 
 template <int RT, int WM> struct LatentShape {
+  static constexpr int kWarps = WM == 1 ? 8 : 16;
+  static constexpr int kThreads = 32 * kWarps;
   static constexpr int kPitch = RT * 16 + 8;
   static constexpr int kRows = 16 * WM;
   static constexpr int kTile = kKeys * kPitch;                                    // elements of one block
   static constexpr int kSmem = (kRows * kPitch + 2 * kTile + 2 * kRows * kWeightPitch) * 2;   // q, two blocks, weights as heads and remainders
 };
 
-// Rows of a tile are (token, head of the unit) pairs, token-major; the eight warps are WM row tiles times WN parts: of a
-// block's keys for the scores, of the latent columns for the sums. ONE: one decoded token, the keys cut over gridDim.x CTAs;
-// the CTA with the newest position norms and appends the token's own row. Otherwise a portion, whose rows are in the pool
+// Rows of a tile are (token, head of the unit) pairs, token-major; the warps are WM row tiles times WN parts: of a
+// block's keys for the scores, of the latent columns for the sums. ONE: one decoded token, the keys cut over gridDim.x CTAs
+// (merge_latent follows if there are several); the CTA with the newest position norms and appends the token's own row. Otherwise a portion, whose rows are in the pool
 // already. RT: 16-column tiles of a latent row; FULL: it fills them. blockIdx = (token tile | split, unit, entry).
 template <int RT, int WM, bool ONE, bool FULL>
-__global__ void __launch_bounds__(kThreads, 1) attend_latent(StepRows r, LatentParams p) {
+__global__ void __launch_bounds__(LatentShape<RT, WM>::kThreads, 1) attend_latent(StepRows r, LatentParams p) {
   using Shape = LatentShape<RT, WM>;
+  constexpr int kWarps = Shape::kWarps, kThreads = Shape::kThreads;
   constexpr int WN = kWarps / WM, KN = kKeys / WN, P = Shape::kPitch, CT = RT / WN;   // CT: column tiles of a warp
   static_assert(CT >= 1, "a warp sums at least one column tile");
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -57,7 +59,6 @@ __global__ void __launch_bounds__(kThreads, 1) attend_latent(StepRows r, LatentP
   __shared__ float high_part[WN][Shape::kRows], sum_part[WN][Shape::kRows];
   __shared__ float2 square_part[kWarps];
   __shared__ int key_at[2][kKeys];   // pool rows of a block's keys (-1: none)
-  __shared__ unsigned last;
   if (!ONE) dependency_wait();
   const Entry e = r.entry[blockIdx.z];
   if ((e.rows == 1) != ONE) {
@@ -280,8 +281,6 @@ __global__ void __launch_bounds__(kThreads, 1) attend_latent(StepRows r, LatentP
     sum_a += sum_part[w][ra];
     sum_b += sum_part[w][rb];
   }
-  const int record = p.rank + 2;
-  float* parts = p.part + (size_t(blockIdx.z) * p.heads + head0) * p.splits * record;   // [head of the unit][split][record]
   const bool whole = !ONE || p.splits == 1;
   auto finish = [&](int m, float top, float sum, int at) {
     const int t = m / gq, h = m % gq;
@@ -292,7 +291,8 @@ __global__ void __launch_bounds__(kThreads, 1) attend_latent(StepRows r, LatentP
       f = fade / fmaf(sum, fade, ex2(sink - high));
     }
     bf16* dst = p.out + (size_t(e.first_row + t0 + t) * p.heads + head0 + h) * p.rank_stride;
-    float* mine = parts + (size_t(h) * p.splits + split) * record;
+    const size_t record = (size_t(blockIdx.z) * p.heads + head0 + h) * p.splits + split;
+    float* mine = p.part + record * p.rank_stride;
 #pragma unroll
     for (int i = 0; i < 2 * CT; ++i) {
       const int c = wn * CT * 16 + i * 8 + 2 * (lane & 3);
@@ -301,66 +301,52 @@ __global__ void __launch_bounds__(kThreads, 1) attend_latent(StepRows r, LatentP
       if (whole) {                   // (a row has an even number of columns; the one behind an odd rank meets zero weights)
         *reinterpret_cast<uint32_t*>(dst + c) = pack(y0, c + 1 < p.rank ? y1 : 0.f);
       } else {
-        mine[2 + c] = y0;
-        if (c + 1 < p.rank) mine[3 + c] = y1;
+        *reinterpret_cast<float2*>(mine + c) = make_float2(y0, y1);
       }
     }
-    if (!whole && wn == 0 && (lane & 3) == 0) {
-      mine[0] = top;
-      mine[1] = sum;
-    }
+    if (!whole && wn == 0 && (lane & 3) == 0) p.stats(r.entries)[record] = make_float2(top, sum);
   };
   finish(ra, top_a, sum_a, 0);
   finish(rb, top_b, sum_b, 2);
-  if (whole) return;
-  unsigned* counter = p.count + size_t(blockIdx.z) * p.subs + blockIdx.y;
-  __syncthreads();
-  if (threadIdx.x == 0) last = atom_acq_rel_add(counter, 1u) == unsigned(p.splits) - 1 ? 1u : 0u;
-  __syncthreads();
-  if (!last) return;
-  if (threadIdx.x == 0) *counter = 0;   // for the next launch
-  // every split's share of the whole, once per head; then the sums, several splits' loads in flight at a time
-  float* factor = reinterpret_cast<float*>(smem_raw);   // [gq][splits], then the sums
-  for (int i = threadIdx.x; i < gq * p.splits; i += kThreads) {
-    factor[i] = __ldcg(parts + size_t(i) * record);
-    factor[gq * p.splits + i] = __ldcg(parts + size_t(i) * record + 1);
+}
+
+// A decoded token's splits put together, a CTA per head. blockIdx = (head, entry).
+constexpr int kMostSplits = 64;
+__global__ void __launch_bounds__(128) merge_latent(StepRows r, LatentParams p) {
+  __shared__ float factor[kMostSplits];
+  dependency_wait();
+  allow_dependents();
+  const Entry e = r.entry[blockIdx.y];
+  if (e.rows != 1) return;
+  const int head = blockIdx.x, lane = threadIdx.x & 31;
+  const size_t record = (size_t(blockIdx.y) * p.heads + head) * p.splits;
+  if (threadIdx.x < 32) {
+    const float2 none = make_float2(-INFINITY, 0.f);
+    const float2 a = lane < p.splits ? p.stats(r.entries)[record + lane] : none, b = lane + 32 < p.splits ? p.stats(r.entries)[record + lane + 32] : none;
+    const float sink = p.sink_of(head), high = fmaxf(warp_max(fmaxf(a.x, b.x)), sink), fa = ex2(a.x - high), fb = ex2(b.x - high);
+    const float sum = warp_sum(a.y * fa + b.y * fb) + ex2(sink - high);
+    factor[lane] = fa / sum;
+    factor[lane + 32] = fb / sum;
   }
   __syncthreads();
-  if (int(threadIdx.x) < gq) {
-    float* f = factor + threadIdx.x * p.splits;
-    const float* l = f + gq * p.splits;
-    const float sink = p.sink_of(head0 + int(threadIdx.x));
-    float high = sink;
-    for (int s = 0; s < p.splits; ++s) high = fmaxf(high, f[s]);
-    float sum = ex2(sink - high);
-    for (int s = 0; s < p.splits; ++s) {   // in split order
-      f[s] = ex2(f[s] - high);
-      sum = fmaf(l[s], f[s], sum);
-    }
-    for (int s = 0; s < p.splits; ++s) f[s] /= sum;
-  }
-  __syncthreads();
-  const int outputs = gq * p.rank;
-  bf16* dst = p.out + (size_t(e.first_row) * p.heads + head0) * p.rank_stride;
-  for (int i0 = threadIdx.x; i0 < outputs; i0 += 4 * kThreads) {
-    float value[4] = {};
-    const float* at[4];
-    const float* f[4];
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int i = min(i0 + j * kThreads, outputs - 1), h = i / p.rank;
-      at[j] = parts + size_t(h) * p.splits * record + 2 + i % p.rank;
-      f[j] = factor + h * p.splits;
-    }
+  const float4* parts = reinterpret_cast<const float4*>(p.part + record * p.rank_stride);
+  bf16* dst = p.out + (size_t(e.first_row) * p.heads + head) * p.rank_stride;
+  for (int c = threadIdx.x; c < p.rank_stride / 4; c += 128) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
-    for (int s = 0; s < p.splits; ++s)
-#pragma unroll
-      for (int j = 0; j < 4; ++j) value[j] = fmaf(__ldcg(at[j] + size_t(s) * record), f[j][s], value[j]);
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int i = i0 + j * kThreads;
-      if (i < outputs) dst[size_t(i / p.rank) * p.rank_stride + i % p.rank] = __float2bfloat16_rn(value[j]);
+    for (int s = 0; s < p.splits; ++s) {
+      const float4 w = parts[size_t(s) * (p.rank_stride / 4) + c];
+      v.x = fmaf(w.x, factor[s], v.x);
+      v.y = fmaf(w.y, factor[s], v.y);
+      v.z = fmaf(w.z, factor[s], v.z);
+      v.w = fmaf(w.w, factor[s], v.w);
     }
+    // (columns behind the rank were never written: they meet zero weights, as zeros)
+    const float y[4] = {v.x, v.y, v.z, v.w};
+    float z[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) z[j] = 4 * c + j < p.rank ? y[j] : 0.f;
+    *reinterpret_cast<uint2*>(dst + 4 * c) = make_uint2(pack(z[0], z[1]), pack(z[2], z[3]));
   }
 }
 
@@ -420,7 +406,7 @@ __global__ void __launch_bounds__(256) gather_latent(StepRows r, int window, con
 
 template <int RT, int WM, bool ONE> int LaunchLatent(const Queue& q, const StepRows& r, const LatentParams& p, int x) {
   auto kernel = p.pool_dim == 16 * RT ? attend_latent<RT, WM, ONE, true> : attend_latent<RT, WM, ONE, false>;
-  return int(Launch(kernel, dim3(unsigned(x), unsigned(p.subs), unsigned(r.entries)), dim3(kThreads), LatentShape<RT, WM>::kSmem, q.stream, q.chained, r, p));
+  return int(Launch(kernel, dim3(unsigned(x), unsigned(p.subs), unsigned(r.entries)), dim3(LatentShape<RT, WM>::kThreads), LatentShape<RT, WM>::kSmem, q.stream, q.chained, r, p));
 }
 
 template <int RT> int LatentWith(const Queue& q, const StepRows& r, const LatentArgs& a, LatentParams p) {
@@ -429,27 +415,30 @@ template <int RT> int LatentWith(const Queue& q, const StepRows& r, const Latent
     p.sub_heads = (a.heads + p.subs - 1) / p.subs;
     p.subs = (a.heads + p.sub_heads - 1) / p.sub_heads;
   };
-  divide(64);
   if (r.singles > 0) {
-    // the cut of a decoded token's keys that ends soonest: a CTA costs its blocks plus a few blocks' time to start and merge
-    const int blocks = std::min(a.window, r.capacity) / kKeys + 1, resident = (RT <= 16 ? 2 : 1) * q.sm_count;
+    // Units of 16 heads while these do not fill the GPU, else as few as there can be; then the cut of a decoded token's keys
+    // that ends soonest: a CTA costs its blocks plus a few blocks' time to start, a merge behind it two.
+    const int blocks = std::min(a.window, r.capacity) / kKeys + 1;
+    divide(size_t(r.singles) * ((a.heads + 15) / 16) * blocks <= size_t(q.sm_count) ? 16 : 64);
     LatentParams one = p;
     one.splits = 1;
     float least = 0.f;
-    for (int s = 1; s <= std::min(blocks, 64); ++s) {
-      if (s > 1 && size_t(r.singles) * p.subs * s > size_t(2 * q.sm_count)) break;
-      const int waves = (r.singles * p.subs * s + resident - 1) / resident;
-      const float cost = float(waves) * (float((blocks + s - 1) / s) + 3.f + float(s) / 8.f);
+    for (int s = 1; s <= std::min(blocks, kMostSplits); ++s) {
+      if (size_t(r.entries) * a.heads * s * (a.rank_stride + 2) > a.part_floats) break;
+      const int waves = (r.singles * p.subs * s + q.sm_count - 1) / q.sm_count;
+      const float cost = float(waves) * (float((blocks + s - 1) / s) + 2.f) + (s > 1 ? 2.f + float(s) / 16.f : 0.f);
       if (s == 1 || cost < least) {
         least = cost;
         one.splits = s;
       }
     }
-    if (size_t(r.entries) * a.heads * one.splits * (a.rank + 2) > a.part_floats || r.entries * p.subs > a.count_words) one.splits = 1;
-    const int status = p.sub_heads <= 16 ? LaunchLatent<RT, 1, true>(q, r, one, one.splits) : p.sub_heads <= 32 ? LaunchLatent<RT, 2, true>(q, r, one, one.splits)
-                       : LaunchLatent<RT, 4, true>(q, r, one, one.splits);
+    int status = p.sub_heads <= 16 ? LaunchLatent<RT, 1, true>(q, r, one, one.splits) : p.sub_heads <= 32 ? LaunchLatent<RT, 2, true>(q, r, one, one.splits)
+                 : LaunchLatent<RT, 4, true>(q, r, one, one.splits);
+    if (status == 0 && one.splits > 1)
+      status = int(Launch(merge_latent, dim3(unsigned(a.heads), unsigned(r.entries)), dim3(128), 0, q.stream, q.chained, r, one));
     if (status != 0) return status;
   }
+  divide(64);
   if (r.singles < r.entries && !a.singles_only) {
     const int per_tile = 64 / p.sub_heads;
     p.splits = 1;
@@ -482,7 +471,6 @@ int AttendLatentTiles(const Queue& q, const StepRows& r, const LatentArgs& a) {
   p.pool = static_cast<bf16*>(a.pool);
   p.out = static_cast<bf16*>(a.out);
   p.part = a.part;
-  p.count = a.count;
   p.norm = a.norm;
   p.sinks = a.sinks;
   p.raw_stride = a.raw_stride;

@@ -251,8 +251,6 @@ struct LatentArgs {
   bool singles_only;         // portions are attended to elsewhere
   float* part;               // decode partials, part_floats floats
   size_t part_floats;
-  unsigned* count;           // arrival counters, zero between launches
-  int count_words;
 };
 // (bf16 rows that suit the tiled form: AppendLatent takes portions only, a decoded token's attention appends its own row.)
 int AppendLatent(const Queue& q, const StepRows& r, const LatentArgs& a);

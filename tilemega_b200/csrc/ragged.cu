@@ -244,8 +244,6 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.window = m.window;
       a.part = plan->part;
       a.part_floats = plan->part_floats;
-      a.count = plan->count;
-      a.count_words = plan->count_words;
       const int wide = m.heads * m.rank_stride();
       TMB_TRY(AppendLatent(q, r, a));
       const int context = ContextRows(plan, r, m);
