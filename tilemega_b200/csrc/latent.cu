@@ -1,5 +1,6 @@
-// Latent attention of bf16 ragged steps on the tensor pipe (mma.sync): every head of a token reads the same cached rows, as
-// keys and as values, so a tile holds (token, head) rows against blocks of latent rows that are copied once for both.
+// Latent attention of bf16 ragged steps on the tensor pipe: every head of a token reads the same cached rows, as keys and as
+// values, so blocks of latent rows are copied once for both. Decoded tokens (decode_latent): tcgen05, latent rows by TMA.
+// Short portions (attend_latent): mma.sync tiles of (token, head) rows; long ones expand the rows they see first.
 #include <cuda_bf16.h>
 
 #include <algorithm>
@@ -16,14 +17,14 @@ namespace tmb {
 namespace {
 
 constexpr int kKeys = 64;          // latent rows per block
-constexpr int kWeightPitch = kKeys + 8;
 
 struct LatentParams {
   const bf16* q;
   const bf16* raw;
   bf16* pool;
   bf16* out;
-  float* part;                     // split sums: [entry][head][split][rank_stride] latent columns, then [entry][head][split] maxima and sums
+  float* part;                     // split sums: [entry][head][split][rank_stride] latent columns, then [entry][head][split] references and sums
+  unsigned* status;
   const float *norm, *sinks;
   int raw_stride, heads, rank, rank_stride, pool_dim, window, splits;
   int subs, sub_heads;             // the heads are served in `subs` units of up to `sub_heads`
@@ -32,23 +33,357 @@ struct LatentParams {
   __device__ float sink_of(int head) const { return sinks ? sinks[head] * 1.4426950408889634f : sink_log2; }
 };
 
-template <int RT, int WM> struct LatentShape {
-  static constexpr int kWarps = WM == 1 ? 8 : 16;
-  static constexpr int kThreads = 32 * kWarps;
+// ---- one decoded token ---------------------------------------------------------------------------------------------------
+// With C [64 keys][latent columns] a block of rows as TMA leaves it (128-byte swizzled chunks of 64 columns, two to a slot):
+//   S [head][key] = Q C^T       A = Q, B = C; of the 128 rows of the tile only a unit's (up to 32) mean anything
+//   O^T [column][head] += C^T P^T   A = C read transposed, 128 columns a slot; B = the weights P, each as a bf16 head (rows
+//                                   0 .. 31) and a bf16 remainder (rows 32 .. 63), summed at the end
+// so both products stream the rows through the tensor core from the one copy. Warp 0 requests rows, warp 1 issues products,
+// a thread of warp 4 owns one head's softmax, warps 4 to 7 own the columns of O (rescaled only when a maximum outgrows its
+// reference by 2^8) and put the token's own row, normed, and zeros for rows out of sight into the edge blocks.
+constexpr int kUnitHeads = 32, kLatentThreads = 256, kSlots = 10;
+constexpr int kChunkBytes = kKeys * 128, kSlotBytes = 2 * kChunkBytes, kQueryChunk = kUnitHeads * 128, kMostChunks = kTiledLatent / 64;
+constexpr int kQueryBytes = kMostChunks * kQueryChunk, kWeightBytes = 2 * kUnitHeads * 128;
+constexpr int kDecodeSmem = kQueryBytes + kSlots * kSlotBytes + 2 * kWeightBytes + 1024;
+constexpr int kScoreColumns = kKeys, kSumColumns = 2 * kUnitHeads;   // tensor memory: two blocks' scores, then a slot's sums each
+constexpr float kGrowth = 8.f;
+
+__device__ __forceinline__ void column_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+
+__global__ void __launch_bounds__(kLatentThreads, 1) decode_latent(const __grid_constant__ CUtensorMap pool_map, const __grid_constant__ CUtensorMap q_map,
+                                                                   StepRows r, LatentParams p) {
+  extern __shared__ unsigned char smem_raw[];
+  unsigned char* queries = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  unsigned char* slots = queries + kQueryBytes;        // (the score product reads rows behind a unit's out of whatever follows)
+  unsigned char* weights = slots + kSlots * kSlotBytes;
+  __shared__ uint64_t full[kSlots], empty[kSlots], query_full, score_full[2], weight_full[2], sum_done[2], patched;
+  __shared__ uint32_t tmem_slot;
+  __shared__ float fade[2][kUnitHeads], factor[kUnitHeads], square_part[4];
+  __shared__ int grown[2];
+  const Entry e = r.entry[blockIdx.z];   // (tables, the rows of earlier steps, this step's projection: there before the dependency wait)
+  if (e.rows != 1) {
+    dependency_wait();
+    allow_dependents();
+    return;
+  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int head0 = blockIdx.y * p.sub_heads, heads = min(p.sub_heads, p.heads - head0), split = blockIdx.x;
+  const int p1 = e.first_position, low = max(0, p1 - p.window + 1), start = low / kRaggedBlock * kRaggedBlock;
+  const int* table = r.block_table + size_t(e.slot) * r.max_blocks;
+  const int blocks = (p1 - start) / kKeys + 1, share = (blocks + p.splits - 1) / p.splits;
+  const int from = min(blocks, split * share), count = min(blocks, from + share) - from;
+  const int chunks = (p.pool_dim + 63) / 64, pairs = (chunks + 1) / 2;
+  auto edge = [&](int i) { return start + (from + i) * kKeys < low || from + i == blocks - 1; };   // a block with rows to put in
+
+  if (threadIdx.x == 0) {
+    prefetch_map(&pool_map);
+    prefetch_map(&q_map);
+    for (int s = 0; s < kSlots; ++s) {
+      mbar_init(&full[s], 1);
+      mbar_init(&empty[s], 1);
+    }
+    mbar_init(&query_full, 1);
+    for (int s = 0; s < 2; ++s) {
+      mbar_init(&score_full[s], 1);
+      mbar_init(&weight_full[s], 1);
+      mbar_init(&sum_done[s], 1);
+    }
+    mbar_init(&patched, 128);
+    mbar_fence_init();
+  }
+  if (warp == 1) tmem_alloc(&tmem_slot, 512);
+  tcgen05_fence_before();
+  __syncthreads();
+  tcgen05_fence_after();
+  const uint32_t tmem = tmem_slot;
+
+  if (warp == 0) {
+    // lane = (chunk of the slot, page of the block): one box of 16 rows x 64 columns each
+    const int total = count * pairs, page = lane & 3, chunk = (lane >> 2) & 1;
+    int issued = 0;
+    bool ok = true;
+    auto request = [&](int it) {
+      const int s = it % kSlots, block = it / pairs, pair = it % pairs, live = min(2, chunks - 2 * pair);
+      if (it >= kSlots) ok = __all_sync(0xffffffffu, wait_bounded(&empty[s], uint32_t(it / kSlots - 1) & 1u, p.status, 5));
+      if (!ok) return;
+      if (lane == 0) mbar_expect_tx(&full[s], uint32_t(live * kChunkBytes));
+      __syncwarp();
+      if (lane < 4 * live) {
+        const int position = min(start + (from + block) * kKeys + page * kRaggedBlock, r.capacity - 1);
+        tma_load_2d(slots + s * kSlotBytes + chunk * kChunkBytes + page * kRaggedBlock * 128, &pool_map, (2 * pair + chunk) * 64,
+                    key_row(table, position / kRaggedBlock * kRaggedBlock, r), &full[s]);
+      }
+      issued = it + 1;
+    };
+    const int early = min(total, kSlots);
+    for (int it = 0; it < early; ++it) request(it);
+    dependency_wait();
+    if (lane == 0 && count > 0) {
+      mbar_expect_tx(&query_full, uint32_t(chunks * kQueryChunk));
+      for (int c = 0; c < chunks; ++c) tma_load_2d(queries + c * kQueryChunk, &q_map, 64 * c, e.first_row * p.heads + head0, &query_full);
+    }
+    for (int it = early; it < total && ok; ++it) request(it);
+    if (!ok) {   // leaving early: let the copies already issued land first
+      for (int it = max(0, issued - kSlots); it < issued; ++it) wait_bounded(&full[it % kSlots], uint32_t(it / kSlots) & 1u, p.status, 6);
+      wait_bounded(&query_full, 0, p.status, 6);
+    }
+  } else {
+    dependency_wait();
+  }
+  allow_dependents();
+
+  if (warp == 1 && lane == 0) {
+    const uint32_t score_idesc = umma_idesc_bf16(128, kKeys), sum_idesc = umma_idesc_bf16(128, kSumColumns) | kUmmaATransposed;
+    bool ok = count > 0 && wait_bounded(&query_full, 0, p.status, 7);
+    unsigned patches = 0;
+    auto score = [&](int i) {
+      if (edge(i)) ok = ok && wait_bounded(&patched, patches++ & 1u, p.status, 8);
+      for (int j = 0; j < pairs && ok; ++j) {
+        const int it = i * pairs + j, s = it % kSlots;
+        ok = wait_bounded(&full[s], uint32_t(it / kSlots) & 1u, p.status, 9);
+        if (!ok) break;
+        tcgen05_fence_after();
+        for (int c = 2 * j; c < min(2 * j + 2, chunks); ++c) {
+          const uint32_t q = smem_u32(queries + c * kQueryChunk), k = smem_u32(slots + s * kSlotBytes + (c & 1) * kChunkBytes);
+#pragma unroll
+          for (int step = 0; step < 4; ++step)
+            umma_bf16(tmem + (i & 1) * kScoreColumns, umma_desc_k_sw128(q + 32 * step, 1024), umma_desc_k_sw128(k + 32 * step, 1024), score_idesc,
+                      uint32_t((c | step) != 0));
+        }
+      }
+      if (ok) umma_commit(&score_full[i & 1]);
+    };
+    if (ok) score(0);
+    for (int i = 0; i < count && ok; ++i) {
+      if (i + 1 < count) score(i + 1);
+      ok = ok && wait_bounded(&weight_full[i & 1], uint32_t(i >> 1) & 1u, p.status, 10);
+      if (!ok) break;
+      tcgen05_fence_after();
+      const uint32_t w = smem_u32(weights + (i & 1) * kWeightBytes);
+      for (int j = 0; j < pairs; ++j) {
+        const int s = (i * pairs + j) % kSlots;
+        const uint32_t c = smem_u32(slots + s * kSlotBytes);
+#pragma unroll
+        for (int step = 0; step < kKeys / 16; ++step)
+          umma_bf16(tmem + 2 * kScoreColumns + j * kSumColumns, umma_desc_mn_sw128(c + 2048 * step, kChunkBytes, 1024),
+                    umma_desc_k_sw128(w + 32 * step, 1024), sum_idesc, uint32_t((i | step) != 0));
+        umma_commit(&empty[s]);
+      }
+      umma_commit(&sum_done[i & 1]);
+    }
+  } else if (warp >= 4) {
+    // a wait that gave up does not leave the loop: its four warps meet at named barriers
+    const int quarter = warp - 4, t = threadIdx.x - 128, column = 32 * quarter + lane;
+    const uint32_t lanes = uint32_t(32 * quarter) << 16;
+    bool ok = true;
+    float inv = 1.f;
+    const bf16* raw = p.raw + size_t(e.first_row) * p.raw_stride;
+    const bool newest = count > 0 && from + count == blocks;
+    if (newest) {
+      float sq = 0.f;
+      for (int d = t; d < p.rank; d += 128) sq = fmaf(__bfloat162float(raw[d]), __bfloat162float(raw[d]), sq);
+      sq = warp_sum(sq);
+      if (lane == 0) square_part[quarter] = sq;
+      column_sync();
+      inv = 1.f / sqrtf((square_part[0] + square_part[1] + square_part[2] + square_part[3]) / float(p.rank) + p.eps);
+    }
+    float reference = -INFINITY, sum = 0.f;              // of the head `lane` (warp 4)
+    for (int i = 0; i < count; ++i) {
+      const int base = start + (from + i) * kKeys;
+      if (edge(i)) {
+        for (int j = 0; j < pairs; ++j) {
+          const int it = i * pairs + j;
+          ok = wait_bounded(&full[it % kSlots], uint32_t(it / kSlots) & 1u, p.status, 11) && ok;
+        }
+        auto place = [&](int key, int unit) {            // 16 bytes: columns 8 unit ... of the block's row `key`
+          const int it = i * pairs + unit / 16;
+          return reinterpret_cast<uint4*>(slots + (it % kSlots) * kSlotBytes + (unit / 8 % 2) * kChunkBytes + key * 128 + ((unit % 8) ^ (key & 7)) * 16);
+        };
+        const int units = chunks * 8, first = max(0, low - base), behind = min(kKeys, p1 + 1 - base);   // rows in sight: [first, behind)
+        for (int n = t; n < (first + kKeys - behind) * units; n += 128) {
+          const int row = n / units;
+          *place(row < first ? row : behind + row - first, n % units) = make_uint4(0, 0, 0, 0);
+        }
+        if (from + i == blocks - 1) {
+          bf16* to_pool = p.pool + size_t(key_row(table, p1, r)) * p.pool_dim;
+          for (int unit = t; unit < p.pool_dim / 8; unit += 128) {
+            float c[8];
+#pragma unroll
+            for (int x = 0; x < 8; ++x) {
+              const int d = 8 * unit + x;
+              c[x] = d < p.rank ? __bfloat162float(raw[d]) * inv * p.norm[d] : 0.f;
+            }
+            const uint4 word = make_uint4(pack(c[0], c[1]), pack(c[2], c[3]), pack(c[4], c[5]), pack(c[6], c[7]));
+            *place(p1 - base, unit) = word;
+            if (blockIdx.y == 0) *reinterpret_cast<uint4*>(to_pool + 8 * unit) = word;
+          }
+        }
+        fence_proxy_async();
+        mbar_arrive(&patched);
+      }
+      float s[kKeys];
+      if (quarter == 0) {
+        ok = wait_bounded(&score_full[i & 1], uint32_t(i >> 1) & 1u, p.status, 12) && ok;
+        ok = __all_sync(0xffffffffu, ok);
+        tcgen05_fence_after();
+        float high = -INFINITY;
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          float v[32];
+          tmem_load_32(tmem + lanes + uint32_t((i & 1) * kScoreColumns + 32 * half), v);
+#pragma unroll
+          for (int k = 0; k < 32; ++k) {
+            const int j = base + 32 * half + k;
+            s[32 * half + k] = j >= low && j <= p1 ? v[k] * p.scale_log2 : -INFINITY;
+            high = fmaxf(high, s[32 * half + k]);
+          }
+        }
+        const bool grows = lane < heads && high > reference + kGrowth;   // (the first block: from -infinity)
+        const float next = grows ? high : reference, f = grows && i > 0 ? ex2(reference - next) : 1.f;
+        reference = next;
+        sum *= f;
+        fade[i & 1][lane] = f;
+        const unsigned any = __ballot_sync(0xffffffffu, grows);
+        if (lane == 0) grown[i & 1] = i > 0 && any ? 1 : 0;
+      }
+      column_sync();
+      if (grown[i & 1]) {
+        ok = wait_bounded(&sum_done[(i - 1) & 1], uint32_t((i - 1) >> 1) & 1u, p.status, 13) && ok;
+        __syncwarp();
+        tcgen05_fence_after();
+        for (int c = 0; c < pairs * kSumColumns; c += 32) {
+          float v[32];
+          tmem_load_32(tmem + lanes + uint32_t(2 * kScoreColumns + c), v);
+#pragma unroll
+          for (int k = 0; k < 32; ++k) v[k] *= fade[i & 1][k];
+          tmem_store_32(tmem + lanes + uint32_t(2 * kScoreColumns + c), v);
+        }
+        tcgen05_fence_before();
+        column_sync();
+      }
+      if (quarter == 0) {
+        // the weights' place is free once the sums two blocks before are done
+        if (i >= 2) ok = wait_bounded(&sum_done[i & 1], uint32_t((i - 2) >> 1) & 1u, p.status, 14) && ok;
+        unsigned char* rows = weights + (i & 1) * kWeightBytes + lane * 128;
+        const bool live = lane < heads;
+#pragma unroll
+        for (int unit = 0; unit < kKeys / 8; ++unit) {
+          float w[8];
+#pragma unroll
+          for (int x = 0; x < 8; ++x) {
+            w[x] = live ? ex2(s[8 * unit + x] - reference) : 0.f;
+            sum += w[x];
+          }
+          const int at = (unit ^ (lane & 7)) * 16;
+          *reinterpret_cast<uint4*>(rows + at) = make_uint4(pack(w[0], w[1]), pack(w[2], w[3]), pack(w[4], w[5]), pack(w[6], w[7]));
+          *reinterpret_cast<uint4*>(rows + kUnitHeads * 128 + at) =
+              make_uint4(pack(rest(w[0]), rest(w[1])), pack(rest(w[2]), rest(w[3])), pack(rest(w[4]), rest(w[5])), pack(rest(w[6]), rest(w[7])));
+        }
+        fence_proxy_async();
+        tcgen05_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&weight_full[i & 1]);
+      }
+    }
+    const bool whole = p.splits == 1;
+    const size_t record = (size_t(blockIdx.z) * p.heads + head0) * p.splits + split;   // of the unit's head 0; heads are `splits` apart
+    if (quarter == 0 && lane < heads) {
+      if (whole) {
+        const float sink = p.sink_of(head0 + lane), high = fmaxf(reference, sink), f = ex2(reference - high);
+        factor[lane] = f / fmaf(sum, f, ex2(sink - high));
+      } else {
+        factor[lane] = 1.f;
+        p.stats(r.entries)[record + size_t(lane) * p.splits] = make_float2(reference, sum);
+      }
+    }
+    column_sync();
+    if (count > 0) {
+      ok = wait_bounded(&sum_done[(count - 1) & 1], uint32_t((count - 1) >> 1) & 1u, p.status, 15) && ok;
+      __syncwarp();
+      tcgen05_fence_after();
+    }
+    bf16* dst = p.out + (size_t(e.first_row) * p.heads + head0) * p.rank_stride;
+    for (int j = 0; j < pairs; ++j) {
+      float hi[32], lo[32];
+      const uint32_t at = tmem + lanes + uint32_t(2 * kScoreColumns + j * kSumColumns);
+      if (count > 0) {
+        tmem_load_32(at, hi);
+        tmem_load_32(at + kUnitHeads, lo);
+      }
+      const int c = 128 * j + column;
+      if (c < p.rank_stride) {
+#pragma unroll
+        for (int h = 0; h < kUnitHeads; ++h) {
+          if (h >= heads) break;
+          const float v = count > 0 && c < p.rank ? (hi[h] + lo[h]) * factor[h] : 0.f;
+          if (whole) dst[size_t(h) * p.rank_stride + c] = __float2bfloat16_rn(v);
+          else p.part[(record + size_t(h) * p.splits) * p.rank_stride + c] = v;
+        }
+      }
+      __syncwarp();
+    }
+  }
+  tcgen05_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tcgen05_fence_after();
+    tmem_dealloc(tmem, 512);
+  }
+}
+
+// A decoded token's splits put together, a CTA per head. blockIdx = (head, entry).
+constexpr int kMostSplits = 64;
+__global__ void __launch_bounds__(128) merge_latent(StepRows r, LatentParams p) {
+  __shared__ float factor[kMostSplits];
+  dependency_wait();
+  allow_dependents();
+  const Entry e = r.entry[blockIdx.y];
+  if (e.rows != 1) return;
+  const int head = blockIdx.x, lane = threadIdx.x & 31;
+  const size_t record = (size_t(blockIdx.y) * p.heads + head) * p.splits;
+  if (threadIdx.x < 32) {
+    const float2 none = make_float2(-INFINITY, 0.f);
+    const float2 a = lane < p.splits ? p.stats(r.entries)[record + lane] : none, b = lane + 32 < p.splits ? p.stats(r.entries)[record + lane + 32] : none;
+    const float sink = p.sink_of(head), high = fmaxf(warp_max(fmaxf(a.x, b.x)), sink), fa = ex2(a.x - high), fb = ex2(b.x - high);
+    const float sum = warp_sum(a.y * fa + b.y * fb) + ex2(sink - high);
+    factor[lane] = fa / sum;
+    factor[lane + 32] = fb / sum;
+  }
+  __syncthreads();
+  const float4* parts = reinterpret_cast<const float4*>(p.part + record * p.rank_stride);
+  bf16* dst = p.out + (size_t(e.first_row) * p.heads + head) * p.rank_stride;
+  for (int c = threadIdx.x; c < p.rank_stride / 4; c += 128) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int s = 0; s < p.splits; ++s) {
+      const float4 w = parts[size_t(s) * (p.rank_stride / 4) + c];
+      v.x = fmaf(w.x, factor[s], v.x);
+      v.y = fmaf(w.y, factor[s], v.y);
+      v.z = fmaf(w.z, factor[s], v.z);
+      v.w = fmaf(w.w, factor[s], v.w);
+    }
+    *reinterpret_cast<uint2*>(dst + 4 * c) = make_uint2(pack(v.x, v.y), pack(v.z, v.w));
+  }
+}
+
+// ---- a portion ------------------------------------------------------------------------------------------------------------
+constexpr int kWeightPitch = kKeys + 8;
+
+template <int RT> struct LatentShape {
+  static constexpr int WM = 4, kWarps = 16, kThreads = 32 * kWarps;
   static constexpr int kPitch = RT * 16 + 8;
   static constexpr int kRows = 16 * WM;
   static constexpr int kTile = kKeys * kPitch;                                    // elements of one block
   static constexpr int kSmem = (kRows * kPitch + 2 * kTile + 2 * kRows * kWeightPitch) * 2;   // q, two blocks, weights as heads and remainders
 };
 
-// Rows of a tile are (token, head of the unit) pairs, token-major; the warps are WM row tiles times WN parts: of a
-// block's keys for the scores, of the latent columns for the sums. ONE: one decoded token, the keys cut over gridDim.x CTAs
-// (merge_latent follows if there are several); the CTA with the newest position norms and appends the token's own row. Otherwise a portion, whose rows are in the pool
-// already. RT: 16-column tiles of a latent row; FULL: it fills them. blockIdx = (token tile | split, unit, entry).
-template <int RT, int WM, bool ONE, bool FULL>
-__global__ void __launch_bounds__(LatentShape<RT, WM>::kThreads, 1) attend_latent(StepRows r, LatentParams p) {
-  using Shape = LatentShape<RT, WM>;
-  constexpr int kWarps = Shape::kWarps, kThreads = Shape::kThreads;
+// Rows of a tile are (token, head of the unit) pairs, token-major; the warps are four row tiles times WN parts: of a block's
+// keys for the scores, of the latent columns for the sums. The portion's own rows are in the pool already. RT: 16-column
+// tiles of a latent row; FULL: it fills them. blockIdx = (token tile, unit, entry).
+template <int RT, bool FULL>
+__global__ void __launch_bounds__(LatentShape<RT>::kThreads, 1) attend_latent(StepRows r, LatentParams p) {
+  using Shape = LatentShape<RT>;
+  constexpr int WM = Shape::WM, kWarps = Shape::kWarps, kThreads = Shape::kThreads;
   constexpr int WN = kWarps / WM, KN = kKeys / WN, P = Shape::kPitch, CT = RT / WN;   // CT: column tiles of a warp
   static_assert(CT >= 1, "a warp sums at least one column tile");
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -57,35 +392,29 @@ __global__ void __launch_bounds__(LatentShape<RT, WM>::kThreads, 1) attend_laten
   bf16* wh = cs + 2 * Shape::kTile;
   bf16* wl = wh + Shape::kRows * kWeightPitch;
   __shared__ float high_part[WN][Shape::kRows], sum_part[WN][Shape::kRows];
-  __shared__ float2 square_part[kWarps];
   __shared__ int key_at[2][kKeys];   // pool rows of a block's keys (-1: none)
-  if (!ONE) dependency_wait();
+  dependency_wait();
+  allow_dependents();
   const Entry e = r.entry[blockIdx.z];
-  if ((e.rows == 1) != ONE) {
-    if (ONE) dependency_wait();
-    allow_dependents();
-    return;
-  }
+  if (e.rows == 1) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head0 = blockIdx.y * p.sub_heads, gq = min(p.sub_heads, p.heads - head0);
   const int per_tile = Shape::kRows / p.sub_heads;
-  const int t0 = ONE ? 0 : blockIdx.x * per_tile, split = ONE ? blockIdx.x : 0;
-  if (t0 >= e.rows) return;          // (portions only)
+  const int t0 = blockIdx.x * per_tile;
+  if (t0 >= e.rows) return;
   const int tokens = min(per_tile, e.rows - t0);
   const int p0 = e.first_position + t0, p1 = p0 + tokens - 1;
   const int* table = r.block_table + size_t(e.slot) * r.max_blocks;
 
   const int low = max(0, p0 - p.window + 1), blocks = (p1 + 1 - low + kKeys - 1) / kKeys;   // any row of the tile sees [low, p1]
-  const int share = (blocks + p.splits - 1) / p.splits;
-  const int from = ONE ? min(blocks, split * share) : 0, to = ONE ? min(blocks, from + share) : blocks;
   auto locate = [&](int b) {         // one block ahead of its fetch
-    if (threadIdx.x < kKeys && b < to) {
+    if (threadIdx.x < kKeys && b < blocks) {
       const int j = low + b * kKeys + int(threadIdx.x);
-      key_at[(b - from) & 1][threadIdx.x] = j <= p1 ? key_row(table, j, r) : -1;
+      key_at[b & 1][threadIdx.x] = j <= p1 ? key_row(table, j, r) : -1;
     }
   };
   auto fetch = [&](int b) {
-    const int stage = (b - from) & 1;
+    const int stage = b & 1;
     constexpr int C = RT * 2;        // 16-byte pieces of a row
 #pragma unroll 4
     for (int i = threadIdx.x; i < kKeys * C; i += kThreads) {
@@ -95,17 +424,10 @@ __global__ void __launch_bounds__(LatentShape<RT, WM>::kThreads, 1) attend_laten
     }
     copy_commit();
   };
-  locate(from);
-  locate(from + 1);
+  locate(0);
+  locate(1);
   __syncthreads();
-  if (from < to) fetch(from);        // (earlier steps' rows, and this portion's, are there; a token's own row comes later)
-  float inv = 1.f;
-  const bf16* raw = p.raw + size_t(e.first_row) * p.raw_stride;
-  const bool newest = ONE && to == blocks && from < to;
-  if (newest)                        // (the projection ran two kernels ago: there before the dependency wait)
-    inv = inverse_rms<kThreads>(make_float2(square_sum(raw, p.rank, kThreads), 0.f), p.rank, 1, p.eps, square_part).x;
-  if (ONE) dependency_wait();
-  allow_dependents();
+  fetch(0);
 
   for (int i = threadIdx.x; i < Shape::kRows * (P / 8); i += kThreads) {
     const int m = i / (P / 8), c = (i % (P / 8)) * 8, t = m / gq;
@@ -132,10 +454,10 @@ __global__ void __launch_bounds__(LatentShape<RT, WM>::kThreads, 1) attend_laten
   for (int i = 0; i < 2 * CT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float top_a = -INFINITY, top_b = -INFINITY, sum_a = 0.f, sum_b = 0.f;   // maxima of all keys, sums of this warp's
 
-  for (int b = from; b < to; ++b) {
-    const int stage = (b - from) & 1;
+  for (int b = 0; b < blocks; ++b) {
+    const int stage = b & 1;
     bf16* tile = cs + stage * Shape::kTile;
-    if (b + 1 < to) {
+    if (b + 1 < blocks) {
       fetch(b + 1);
       copy_wait<1>();
     } else {
@@ -143,48 +465,21 @@ __global__ void __launch_bounds__(LatentShape<RT, WM>::kThreads, 1) attend_laten
     }
     __syncthreads();
     locate(b + 2);
-    if (newest && b + 1 == blocks) {   // the token's own row: over whatever the copy found in its place
-      bf16* to_pool = p.pool + size_t(key_row(table, p1, r)) * p.pool_dim;
-      bf16* to_tile = tile + (p1 - low - b * kKeys) * P;
-      for (int d = threadIdx.x; d < p.rank; d += kThreads) {
-        const bf16 c = __float2bfloat16_rn(__bfloat162float(raw[d]) * inv * p.norm[d]);
-        to_tile[d] = c;
-        if (blockIdx.y == 0) to_pool[d] = c;
-      }
-      __syncthreads();
-    }
     float s[KN / 8][4];
 #pragma unroll
     for (int t = 0; t < KN / 8; ++t) s[t][0] = s[t][1] = s[t][2] = s[t][3] = 0.f;
-    if constexpr (KN >= 16) {
 #pragma unroll 8
-      for (int kk = 0; kk < RT; ++kk) {
-        if (!FULL && kk * 16 >= p.pool_dim) break;
-        uint32_t a[4];
-        load_a(a, qs, P, row0, kk * 16, lane);
+    for (int kk = 0; kk < RT; ++kk) {
+      if (!FULL && kk * 16 >= p.pool_dim) break;
+      uint32_t a[4];
+      load_a(a, qs, P, row0, kk * 16, lane);
 #pragma unroll
-        for (int t = 0; t < KN / 16; ++t) {
-          uint32_t bb[4];
-          load_b(bb, tile + key0 * P, P, t * 16, kk * 16, lane);
-          mma16816(s[2 * t], a, bb[0], bb[1]);
-          mma16816(s[2 * t + 1], a, bb[2], bb[3]);
-        }
+      for (int t = 0; t < KN / 16; ++t) {
+        uint32_t bb[4];
+        load_b(bb, tile + key0 * P, P, t * 16, kk * 16, lane);
+        mma16816(s[2 * t], a, bb[0], bb[1]);
+        mma16816(s[2 * t + 1], a, bb[2], bb[3]);
       }
-    } else {
-      float other[4] = {};             // two chains: the odd k steps apart
-#pragma unroll 8
-      for (int kk = 0; kk < RT; kk += 2) {
-        if (!FULL && kk * 16 >= p.pool_dim) break;
-        uint32_t a[4], bb[4];
-        load_b_narrow(bb, tile + key0 * P, P, 0, kk * 16, lane);
-        load_a(a, qs, P, row0, kk * 16, lane);
-        mma16816(s[0], a, bb[0], bb[1]);
-        if (!FULL && kk * 16 + 16 >= p.pool_dim) break;
-        load_a(a, qs, P, row0, kk * 16 + 16, lane);
-        mma16816(other, a, bb[2], bb[3]);
-      }
-#pragma unroll
-      for (int x = 0; x < 4; ++x) s[0][x] += other[x];
     }
     const int first = low + b * kKeys + key0 + 2 * (lane & 3);
     float high_a = -INFINITY, high_b = -INFINITY;
@@ -281,73 +576,21 @@ __global__ void __launch_bounds__(LatentShape<RT, WM>::kThreads, 1) attend_laten
     sum_a += sum_part[w][ra];
     sum_b += sum_part[w][rb];
   }
-  const bool whole = !ONE || p.splits == 1;
   auto finish = [&](int m, float top, float sum, int at) {
     const int t = m / gq, h = m % gq;
     if (t >= tokens) return;
-    float f = 1.f;
-    if (whole) {
-      const float sink = p.sink_of(head0 + h), high = fmaxf(top, sink), fade = ex2(top - high);
-      f = fade / fmaf(sum, fade, ex2(sink - high));
-    }
+    const float sink = p.sink_of(head0 + h), high = fmaxf(top, sink), fade = ex2(top - high);
+    const float f = fade / fmaf(sum, fade, ex2(sink - high));
     bf16* dst = p.out + (size_t(e.first_row + t0 + t) * p.heads + head0 + h) * p.rank_stride;
-    const size_t record = (size_t(blockIdx.z) * p.heads + head0 + h) * p.splits + split;
-    float* mine = p.part + record * p.rank_stride;
 #pragma unroll
     for (int i = 0; i < 2 * CT; ++i) {
       const int c = wn * CT * 16 + i * 8 + 2 * (lane & 3);
-      if (c >= p.rank) continue;
-      const float y0 = o[i][at] * f, y1 = o[i][at + 1] * f;
-      if (whole) {                   // (a row has an even number of columns; the one behind an odd rank meets zero weights)
-        *reinterpret_cast<uint32_t*>(dst + c) = pack(y0, c + 1 < p.rank ? y1 : 0.f);
-      } else {
-        *reinterpret_cast<float2*>(mine + c) = make_float2(y0, y1);
-      }
+      if (c >= p.rank) continue;     // (a row has an even number of columns; the one behind an odd rank meets zero weights)
+      *reinterpret_cast<uint32_t*>(dst + c) = pack(o[i][at] * f, c + 1 < p.rank ? o[i][at + 1] * f : 0.f);
     }
-    if (!whole && wn == 0 && (lane & 3) == 0) p.stats(r.entries)[record] = make_float2(top, sum);
   };
   finish(ra, top_a, sum_a, 0);
   finish(rb, top_b, sum_b, 2);
-}
-
-// A decoded token's splits put together, a CTA per head. blockIdx = (head, entry).
-constexpr int kMostSplits = 64;
-__global__ void __launch_bounds__(128) merge_latent(StepRows r, LatentParams p) {
-  __shared__ float factor[kMostSplits];
-  dependency_wait();
-  allow_dependents();
-  const Entry e = r.entry[blockIdx.y];
-  if (e.rows != 1) return;
-  const int head = blockIdx.x, lane = threadIdx.x & 31;
-  const size_t record = (size_t(blockIdx.y) * p.heads + head) * p.splits;
-  if (threadIdx.x < 32) {
-    const float2 none = make_float2(-INFINITY, 0.f);
-    const float2 a = lane < p.splits ? p.stats(r.entries)[record + lane] : none, b = lane + 32 < p.splits ? p.stats(r.entries)[record + lane + 32] : none;
-    const float sink = p.sink_of(head), high = fmaxf(warp_max(fmaxf(a.x, b.x)), sink), fa = ex2(a.x - high), fb = ex2(b.x - high);
-    const float sum = warp_sum(a.y * fa + b.y * fb) + ex2(sink - high);
-    factor[lane] = fa / sum;
-    factor[lane + 32] = fb / sum;
-  }
-  __syncthreads();
-  const float4* parts = reinterpret_cast<const float4*>(p.part + record * p.rank_stride);
-  bf16* dst = p.out + (size_t(e.first_row) * p.heads + head) * p.rank_stride;
-  for (int c = threadIdx.x; c < p.rank_stride / 4; c += 128) {
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
-    for (int s = 0; s < p.splits; ++s) {
-      const float4 w = parts[size_t(s) * (p.rank_stride / 4) + c];
-      v.x = fmaf(w.x, factor[s], v.x);
-      v.y = fmaf(w.y, factor[s], v.y);
-      v.z = fmaf(w.z, factor[s], v.z);
-      v.w = fmaf(w.w, factor[s], v.w);
-    }
-    // (columns behind the rank were never written: they meet zero weights, as zeros)
-    const float y[4] = {v.x, v.y, v.z, v.w};
-    float z[4];
-#pragma unroll
-    for (int j = 0; j < 4; ++j) z[j] = 4 * c + j < p.rank ? y[j] : 0.f;
-    *reinterpret_cast<uint2*>(dst + 4 * c) = make_uint2(pack(z[0], z[1]), pack(z[2], z[3]));
-  }
 }
 
 // First expanded row of every entry: the portions' reaches one after the other, decoded tokens' empty.
@@ -404,62 +647,48 @@ __global__ void __launch_bounds__(256) gather_latent(StepRows r, int window, con
   for (int c = lane; c < pieces; c += 32) out[size_t(i) * pieces + c] = pool[size_t(row) * pool_pieces + c];
 }
 
-template <int RT, int WM, bool ONE> int LaunchLatent(const Queue& q, const StepRows& r, const LatentParams& p, int x) {
-  auto kernel = p.pool_dim == 16 * RT ? attend_latent<RT, WM, ONE, true> : attend_latent<RT, WM, ONE, false>;
-  return int(Launch(kernel, dim3(unsigned(x), unsigned(p.subs), unsigned(r.entries)), dim3(LatentShape<RT, WM>::kThreads), LatentShape<RT, WM>::kSmem, q.stream, q.chained, r, p));
+// The heads in as few units of at most `most` as there can be.
+void Divide(LatentParams* p, int most) {
+  p->subs = (p->heads + most - 1) / most;
+  p->sub_heads = (p->heads + p->subs - 1) / p->subs;
+  p->subs = (p->heads + p->sub_heads - 1) / p->sub_heads;
 }
 
-template <int RT> int LatentWith(const Queue& q, const StepRows& r, const LatentArgs& a, LatentParams p) {
-  auto divide = [&](int most) {      // the heads in as few units of at most this many as there can be
-    p.subs = (a.heads + most - 1) / most;
-    p.sub_heads = (a.heads + p.subs - 1) / p.subs;
-    p.subs = (a.heads + p.sub_heads - 1) / p.sub_heads;
-  };
-  if (r.singles > 0) {
-    // Units of 16 heads while these do not fill the GPU, else as few as there can be; then the cut of a decoded token's keys
-    // that ends soonest: a CTA costs its blocks plus a few blocks' time to start, a merge behind it two.
-    const int blocks = std::min(a.window, r.capacity) / kKeys + 1;
-    divide(size_t(r.singles) * ((a.heads + 15) / 16) * blocks <= size_t(q.sm_count) ? 16 : 64);
-    LatentParams one = p;
-    one.splits = 1;
-    float least = 0.f;
-    for (int s = 1; s <= std::min(blocks, kMostSplits); ++s) {
-      if (size_t(r.entries) * a.heads * s * (a.rank_stride + 2) > a.part_floats) break;
-      const int waves = (r.singles * p.subs * s + q.sm_count - 1) / q.sm_count;
-      const float cost = float(waves) * (float((blocks + s - 1) / s) + 2.f) + (s > 1 ? 2.f + float(s) / 16.f : 0.f);
-      if (s == 1 || cost < least) {
-        least = cost;
-        one.splits = s;
-      }
+int DecodeLatent(const Queue& q, const StepRows& r, const LatentArgs& a, LatentParams p) {
+  // the cut of a token's keys that ends soonest: a CTA costs its blocks plus a few blocks' time to start, a merge behind it three
+  const int blocks = (std::min(a.window, r.capacity) + kRaggedBlock - 2) / kKeys + 1;
+  Divide(&p, kUnitHeads);
+  p.splits = 1;
+  float least = 0.f;
+  for (int s = 1; s <= std::min(blocks, kMostSplits); ++s) {
+    if (size_t(r.entries) * a.heads * s * (a.rank_stride + 2) > a.part_floats) break;
+    const int waves = (r.singles * p.subs * s + q.sm_count - 1) / q.sm_count;
+    const float cost = float(waves) * (float((blocks + s - 1) / s) + 3.f) + (s > 1 ? 3.f + float(s) / 16.f : 0.f);
+    if (s == 1 || cost < least) {
+      least = cost;
+      p.splits = s;
     }
-    int status = p.sub_heads <= 16 ? LaunchLatent<RT, 1, true>(q, r, one, one.splits) : p.sub_heads <= 32 ? LaunchLatent<RT, 2, true>(q, r, one, one.splits)
-                 : LaunchLatent<RT, 4, true>(q, r, one, one.splits);
-    if (status == 0 && one.splits > 1)
-      status = int(Launch(merge_latent, dim3(unsigned(a.heads), unsigned(r.entries)), dim3(128), 0, q.stream, q.chained, r, one));
-    if (status != 0) return status;
   }
-  divide(64);
-  if (r.singles < r.entries && !a.singles_only) {
-    const int per_tile = 64 / p.sub_heads;
-    p.splits = 1;
-    return LaunchLatent<RT, 4, false>(q, r, p, (r.longest + per_tile - 1) / per_tile);
-  }
-  return 0;
+  const int status = int(Launch(decode_latent, dim3(unsigned(p.splits), unsigned(p.subs), unsigned(r.entries)), dim3(kLatentThreads), kDecodeSmem, q.stream,
+                                q.chained, *a.pool_map, *a.q_map, r, p));
+  if (status != 0 || p.splits == 1) return status;
+  return int(Launch(merge_latent, dim3(unsigned(a.heads), unsigned(r.entries)), dim3(128), 0, q.stream, q.chained, r, p));
 }
 
-template <int RT, int WM, bool ONE> cudaError_t RaiseOne() {
-  for (auto kernel : {attend_latent<RT, WM, ONE, false>, attend_latent<RT, WM, ONE, true>}) {
-    const cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, LatentShape<RT, WM>::kSmem);
+template <int RT> int AttendWith(const Queue& q, const StepRows& r, LatentParams p) {
+  Divide(&p, 64);
+  auto kernel = p.pool_dim == 16 * RT ? attend_latent<RT, true> : attend_latent<RT, false>;
+  const int per_tile = 64 / p.sub_heads;
+  return int(Launch(kernel, dim3(unsigned((r.longest + per_tile - 1) / per_tile), unsigned(p.subs), unsigned(r.entries)), dim3(LatentShape<RT>::kThreads),
+                    LatentShape<RT>::kSmem, q.stream, q.chained, r, p));
+}
+
+template <int RT> cudaError_t Raise() {
+  for (auto kernel : {attend_latent<RT, false>, attend_latent<RT, true>}) {
+    const cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, LatentShape<RT>::kSmem);
     if (err != cudaSuccess) return err;
   }
   return cudaSuccess;
-}
-template <int RT> cudaError_t Raise() {
-  cudaError_t err = RaiseOne<RT, 1, true>();
-  if (err == cudaSuccess) err = RaiseOne<RT, 2, true>();
-  if (err == cudaSuccess) err = RaiseOne<RT, 4, true>();
-  if (err == cudaSuccess) err = RaiseOne<RT, 4, false>();
-  return err;
 }
 
 }  // namespace
@@ -482,7 +711,20 @@ int AttendLatentTiles(const Queue& q, const StepRows& r, const LatentArgs& a) {
   p.scale_log2 = a.scale * 1.4426950408889634f;
   p.sink_log2 = a.sink * 1.4426950408889634f;
   p.eps = a.eps;
-  return a.rank <= 128 ? LatentWith<8>(q, r, a, p) : a.rank <= 256 ? LatentWith<16>(q, r, a, p) : LatentWith<32>(q, r, a, p);
+  p.status = q.status;
+  if (r.singles > 0) {
+    const int status = DecodeLatent(q, r, a, p);
+    if (status != 0) return status;
+  }
+  if (r.singles == r.entries || a.singles_only) return 0;
+  return a.rank <= 128 ? AttendWith<8>(q, r, p) : a.rank <= 256 ? AttendWith<16>(q, r, p) : AttendWith<32>(q, r, p);
+}
+
+bool EncodeLatent(CUtensorMap* pool_map, const void* pool, uint64_t rows, uint64_t pool_dim) {
+  return EncodeMatrix(pool_map, false, pool, rows, pool_dim, kRaggedBlock);
+}
+bool EncodeLookup(CUtensorMap* q_map, const void* q, uint64_t rows, uint64_t rank_stride) {
+  return EncodeMatrix(q_map, false, q, rows, rank_stride, kUnitHeads);
 }
 
 int LatentContext(const Queue& q, const StepRows& r, int window, int* context, int* context_rows) {
@@ -496,7 +738,8 @@ int GatherLatent(const Queue& q, const StepRows& r, const LatentArgs& a, const i
 }
 
 int PrepareLatent() {
-  cudaError_t err = Raise<8>();
+  cudaError_t err = cudaFuncSetAttribute(decode_latent, cudaFuncAttributeMaxDynamicSharedMemorySize, kDecodeSmem);
+  if (err == cudaSuccess) err = Raise<8>();
   if (err == cudaSuccess) err = Raise<16>();
   if (err == cudaSuccess) err = Raise<32>();
   return int(err);

@@ -45,9 +45,5 @@ __device__ __forceinline__ void load_b(uint32_t (&b)[4], const bf16* tile, int p
 __device__ __forceinline__ void load_b_transposed(uint32_t (&b)[4], const bf16* tile, int pitch, int k, int n, int lane) {
   ldmatrix_x4_trans(b, smem_u32(tile + (k + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + n + (lane >> 4) * 8));
 }
-// one n8 tile of B for two k steps, tile holds [n][k]: b[0], b[1] for columns k .. k + 15, b[2], b[3] for the next 16
-__device__ __forceinline__ void load_b_narrow(uint32_t (&b)[4], const bf16* tile, int pitch, int n, int k, int lane) {
-  ldmatrix_x4(b, smem_u32(tile + (n + (lane & 7)) * pitch + k + (lane >> 3) * 8));
-}
 
 }  // namespace tmb

@@ -238,12 +238,13 @@ int PrepareMixers();
 // heads' weighted sums of latent rows, for the heads' value matrices to follow. latent rows come from `raw` ([rows] of
 // raw_stride, normed by AppendLatent on their way into the pool).
 struct LatentArgs {
-  const void* q;             // [rows][heads][rank_stride]
+  const void* q;             // [rows][heads][rank_stride], zeros behind the rank
   void* out;                 // [rows][heads][rank_stride]
   const void* raw;
   int raw_stride;
   const float* norm;         // [rank]
   void* pool;                // [num_blocks][16][pool_dim]
+  const CUtensorMap *pool_map, *q_map;   // bf16, tiled form: see EncodeLatent, EncodeLookup
   int heads, rank, rank_stride, pool_dim;
   float eps, scale, sink;
   const float* sinks;        // [heads], or null
@@ -259,6 +260,8 @@ constexpr int kTiledLatent = 512;   // widest latent row of the tiled form
 inline bool LatentTiled(const LatentArgs& a) { return a.rank <= kTiledLatent; }
 int AttendLatentTiles(const Queue& q, const StepRows& r, const LatentArgs& a);   // the tiled form
 int PrepareLatent();
+bool EncodeLatent(CUtensorMap* pool_map, const void* pool, uint64_t rows, uint64_t pool_dim);
+bool EncodeLookup(CUtensorMap* q_map, const void* q, uint64_t rows, uint64_t rank_stride);   // rows: one per token and head
 // Long portions expand the latent rows they see into keys and values first: where each entry's rows start in the expanded
 // ones (context [entries], and how many there are in all), and those rows gathered from the pool, `most` at most.
 int LatentContext(const Queue& q, const StepRows& r, int window, int* context, int* context_rows);

@@ -247,6 +247,15 @@ __device__ __forceinline__ uint64_t umma_desc_k_sw128(uint32_t address, uint32_t
   return lo | (hi << 32);
 }
 
+// The same for an operand that lies transposed (its M or N side contiguous, 64 elements to a 128-byte row, one row per k): 8-row
+// groups of k `k_group_bytes` apart, each further 64 elements of the M or N side `side_bytes` apart.
+__device__ __forceinline__ uint64_t umma_desc_mn_sw128(uint32_t address, uint32_t side_bytes, uint32_t k_group_bytes) {
+  const uint64_t lo = uint64_t((address >> 4) & 0x3FFFu) | (uint64_t((side_bytes >> 4) & 0x3FFFu) << 16);
+  const uint64_t hi = uint64_t((k_group_bytes >> 4) & 0x3FFFu) | (uint64_t(1) << 14) | (uint64_t(2) << 29);
+  return lo | (hi << 32);
+}
+constexpr uint32_t kUmmaATransposed = 1u << 15;   // instruction descriptor: A lies transposed
+
 // Instruction descriptor of kind::f16: bf16 x bf16 -> fp32, both operands K-major, M x N tile.
 __device__ __forceinline__ uint32_t umma_idesc_bf16(int m, int n) {
   return (1u << 4) | (1u << 7) | (1u << 10) | (uint32_t(n >> 3) << 17) | (uint32_t(m >> 4) << 24);
@@ -336,6 +345,21 @@ __device__ __forceinline__ void tmem_load_32(uint32_t address, float (&v)[32]) {
       : "memory");
 #pragma unroll
   for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
+}
+
+// The other way round; what is stored is there for later accesses of this thread once the function returns.
+__device__ __forceinline__ void tmem_store_32(uint32_t address, const float (&v)[32]) {
+  uint32_t r[32];
+#pragma unroll
+  for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(v[i]);
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, %17, %18, %19, "
+      "%20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};\n"
+      "tcgen05.wait::st.sync.aligned;" ::"r"(address),
+      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]),
+      "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]),
+      "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
+      : "memory");
 }
 
 // One 32-byte store (a whole sector) to a 32-byte aligned global address.

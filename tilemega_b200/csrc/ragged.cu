@@ -54,8 +54,10 @@ struct RaggedPlan {
   struct Maps {
     LinearMaps in, out, gate_up, down, router;   // (gate_up, down: of the gated unit or of the experts)
     LinearMaps shared_up, shared_down, key_up, value_up, expand;
+    CUtensorMap lookup;
   };
   std::vector<Maps> maps;      // per layer (bf16 plans)
+  std::vector<CUtensorMap> latent;   // per run (bf16 plans): pools of latent rows
   LinearMaps head;
   // recorded steps of single-row entries, by (entries, wanted, feed)
   std::map<std::tuple<uint32_t, uint32_t, bool>, cudaGraphExec_t> graphs;
@@ -233,6 +235,8 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.raw_stride = stride;
       a.norm = floats(layer.latent_norm);
       a.pool = buffer(run.k_pool);
+      a.pool_map = maps ? &plan->latent[i] : nullptr;
+      a.q_map = maps ? &maps->lookup : nullptr;
       a.heads = m.heads;
       a.rank = m.rank;
       a.rank_stride = m.rank_stride();
@@ -249,7 +253,7 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       const int context = ContextRows(plan, r, m);
       a.singles_only = context > 0;
       if (!context || r.singles) {
-        LinearArgs up = linear(proj, layer.key_up, -1, maps ? &maps->key_up : nullptr, m.rank, m.head_stride(), plan->lookup, wide, kLinearHeads);
+        LinearArgs up = linear(proj, layer.key_up, -1, maps ? &maps->key_up : nullptr, m.rank_stride(), m.head_stride(), plan->lookup, wide, kLinearHeads);
         up.in_stride = stride;
         up.heads = m.heads;
         up.head_in = m.head_stride();
@@ -576,7 +580,8 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
                 EncodeLinear(&maps.out, at(layer.out_weight), uint64_t(spec.width), plan->mixed, rows, uint64_t(padded_columns(m.out_columns())));
       const RaggedMlp& mlp = layer.mlp;
       if (m.kind == RaggedMixer::kLatent)
-        ok = ok && EncodeHeads(&maps.key_up, at(layer.key_up), uint64_t(m.heads) * m.rank, uint64_t(m.head_stride()), plan->proj, rows,
+        ok = ok && EncodeLookup(&maps.lookup, plan->lookup, rows * m.heads, uint64_t(m.rank_stride())) &&
+             EncodeHeads(&maps.key_up, at(layer.key_up), uint64_t(m.heads) * m.rank_stride(), uint64_t(m.head_stride()), plan->proj, rows,
                                size_t(m.proj_rows() + 7) / 8 * 8) &&
              EncodeHeads(&maps.value_up, at(layer.value_up), uint64_t(m.heads) * m.vdim, uint64_t(m.rank_stride()), plan->looked, rows,
                          uint64_t(m.heads) * m.rank_stride()) &&
@@ -595,6 +600,13 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
         ok = ok && EncodeLinear(&maps.gate_up, at(layer.gate_up), uint64_t(mlp.packed_rows()), plan->normed, rows, W8) &&
              EncodeLinear(&maps.down, at(layer.down), uint64_t(spec.width), plan->mlp, rows, uint64_t(padded_columns(mlp.ff)));
       if (!ok) return fail("cuTensorMapEncodeTiled rejected a layer's buffers");
+    }
+    plan->latent.resize(spec.runs.size());
+    for (size_t i = 0; i < spec.runs.size(); ++i) {
+      const RaggedMixer& m = spec.layers[size_t(spec.runs[i].layer)].mixer;
+      if (m.kind == RaggedMixer::kLatent &&
+          !EncodeLatent(&plan->latent[i], at(spec.runs[i].k_pool), uint64_t(spec.num_blocks) * kRaggedBlock, uint64_t(m.pool_dim())))
+        return fail("cuTensorMapEncodeTiled rejected a pool of latent rows");
     }
     if (!EncodeLinear(&plan->head, at(spec.head), uint64_t(spec.vocab), plan->picked, uint64_t(spec.max_wanted), W8))
       return fail("cuTensorMapEncodeTiled rejected the head");

@@ -250,8 +250,9 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
       const int rank = m.rank_stride();
       layer.latent_norm = add(p + "latent.norm", 1, 1, uint64_t(m.rank), 0, AliasRecipe(Name(names, "dkv.norm")));
       // a query against latent rows is its head's key matrix, transposed, times the query
-      layer.key_up = add(p + "key_up.weight", 1, element, uint64_t(m.heads) * m.rank * m.head_stride(), 0,
-                         PadColumns(PerHead("transpose_heads", Json::Quote(Name(names, "uk")), m.heads, "rows", m.dim), m.head_stride()));
+      layer.key_up = add(p + "key_up.weight", 1, element, uint64_t(m.heads) * rank * m.head_stride(), 0,
+                         PadColumns(PerHead("pad_heads", PerHead("transpose_heads", Json::Quote(Name(names, "uk")), m.heads, "rows", m.dim), m.heads, "rows", rank),
+                                    m.head_stride()));
       if (!s.f32)
         layer.expand = add(p + "expand.weight", 1, element, uint64_t(m.expanded_columns()) * rank, 0,
                            PadColumns(Stack({PerHead("pad_heads", Json::Quote(Name(names, "uk")), m.heads, "rows", m.expanded_key()),
