@@ -39,12 +39,13 @@ struct LatentParams {
 //   O^T [column][head] += C^T P^T   A = C read transposed, 128 columns a slot; B = the weights P, each as a bf16 head (rows
 //                                   0 .. 31) and a bf16 remainder (rows 32 .. 63), summed at the end
 // so both products stream the rows through the tensor core from the one copy. Warp 0 requests rows, warp 1 issues products,
-// a thread of warp 4 owns one head's softmax, warps 4 to 7 own the columns of O (rescaled only when a maximum outgrows its
-// reference by 2^8) and put the token's own row, normed, and zeros for rows out of sight into the edge blocks.
+// warps 4 to 7 share the softmax (a lane per head, 16 keys a warp), own the columns of O (rescaled only when a maximum outgrows
+// its reference by 2^8) and put the token's own row, normed, and zeros for rows out of sight into the edge blocks.
 constexpr int kUnitHeads = 32, kLatentThreads = 256, kSlots = 10;
 constexpr int kChunkBytes = kKeys * 128, kSlotBytes = 2 * kChunkBytes, kQueryChunk = kUnitHeads * 128, kMostChunks = kTiledLatent / 64;
 constexpr int kQueryBytes = kMostChunks * kQueryChunk, kWeightBytes = 2 * kUnitHeads * 128;
-constexpr int kDecodeSmem = kQueryBytes + kSlots * kSlotBytes + 2 * kWeightBytes + 1024;
+constexpr int kScorePitch = kKeys + 4;
+constexpr int kDecodeSmem = kQueryBytes + kSlots * kSlotBytes + 2 * kWeightBytes + kUnitHeads * kScorePitch * 4 + 1024;
 constexpr int kScoreColumns = kKeys, kSumColumns = 2 * kUnitHeads;   // tensor memory: two blocks' scores, then a slot's sums each
 constexpr float kGrowth = 8.f;
 
@@ -56,10 +57,10 @@ __global__ void __launch_bounds__(kLatentThreads, 1) decode_latent(const __grid_
   unsigned char* queries = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   unsigned char* slots = queries + kQueryBytes;        // (the score product reads rows behind a unit's out of whatever follows)
   unsigned char* weights = slots + kSlots * kSlotBytes;
+  float* scores = reinterpret_cast<float*>(weights + 2 * kWeightBytes);
   __shared__ uint64_t full[kSlots], empty[kSlots], query_full, score_full[2], weight_full[2], sum_done[2], patched;
   __shared__ uint32_t tmem_slot;
-  __shared__ float fade[2][kUnitHeads], factor[kUnitHeads], square_part[4];
-  __shared__ int grown[2];
+  __shared__ float exchange[4][kUnitHeads], factor[kUnitHeads], square_part[4];
   const Entry e = r.entry[blockIdx.z];   // (tables, the rows of earlier steps, this step's projection: there before the dependency wait)
   if (e.rows != 1) {
     dependency_wait();
@@ -85,7 +86,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) decode_latent(const __grid_
     mbar_init(&query_full, 1);
     for (int s = 0; s < 2; ++s) {
       mbar_init(&score_full[s], 1);
-      mbar_init(&weight_full[s], 1);
+      mbar_init(&weight_full[s], 4);
       mbar_init(&sum_done[s], 1);
     }
     mbar_init(&patched, 128);
@@ -187,7 +188,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) decode_latent(const __grid_
       column_sync();
       inv = 1.f / sqrtf((square_part[0] + square_part[1] + square_part[2] + square_part[3]) / float(p.rank) + p.eps);
     }
-    float reference = -INFINITY, sum = 0.f;              // of the head `lane` (warp 4)
+    float reference = -INFINITY, sum = 0.f;              // of the head `lane`: what its weights are relative to, this warp's sum
     for (int i = 0; i < count; ++i) {
       const int base = start + (from + i) * kKeys;
       if (edge(i)) {
@@ -221,33 +222,47 @@ __global__ void __launch_bounds__(kLatentThreads, 1) decode_latent(const __grid_
         fence_proxy_async();
         mbar_arrive(&patched);
       }
-      float s[kKeys];
+      // the scores lie in the first 32 lanes of tensor memory, which warp 4 alone reads: through shared memory every warp
+      // gets 16 keys of every head (a lane's)
       if (quarter == 0) {
         ok = wait_bounded(&score_full[i & 1], uint32_t(i >> 1) & 1u, p.status, 12) && ok;
-        ok = __all_sync(0xffffffffu, ok);
+        __syncwarp();
         tcgen05_fence_after();
-        float high = -INFINITY;
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           float v[32];
-          tmem_load_32(tmem + lanes + uint32_t((i & 1) * kScoreColumns + 32 * half), v);
+          tmem_load_32(tmem + uint32_t((i & 1) * kScoreColumns + 32 * half), v);
 #pragma unroll
-          for (int k = 0; k < 32; ++k) {
-            const int j = base + 32 * half + k;
-            s[32 * half + k] = j >= low && j <= p1 ? v[k] * p.scale_log2 : -INFINITY;
-            high = fmaxf(high, s[32 * half + k]);
-          }
+          for (int k = 0; k < 32; k += 4) *reinterpret_cast<float4*>(scores + lane * kScorePitch + 32 * half + k) = make_float4(v[k], v[k + 1], v[k + 2], v[k + 3]);
         }
-        const bool grows = lane < heads && high > reference + kGrowth;   // (the first block: from -infinity)
-        const float next = grows ? high : reference, f = grows && i > 0 ? ex2(reference - next) : 1.f;
-        reference = next;
-        sum *= f;
-        fade[i & 1][lane] = f;
-        const unsigned any = __ballot_sync(0xffffffffu, grows);
-        if (lane == 0) grown[i & 1] = i > 0 && any ? 1 : 0;
       }
       column_sync();
-      if (grown[i & 1]) {
+      float s[16], high = -INFINITY;
+#pragma unroll
+      for (int k = 0; k < 16; k += 4) {
+        const float4 v = *reinterpret_cast<const float4*>(scores + lane * kScorePitch + 16 * quarter + k);
+        s[k] = v.x * p.scale_log2;
+        s[k + 1] = v.y * p.scale_log2;
+        s[k + 2] = v.z * p.scale_log2;
+        s[k + 3] = v.w * p.scale_log2;
+      }
+      if (edge(i)) {
+#pragma unroll
+        for (int k = 0; k < 16; ++k) {
+          const int j = base + 16 * quarter + k;
+          if (j < low || j > p1) s[k] = -INFINITY;
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < 16; ++k) high = fmaxf(high, s[k]);
+      exchange[quarter][lane] = high;
+      column_sync();
+      high = fmaxf(fmaxf(exchange[0][lane], exchange[1][lane]), fmaxf(exchange[2][lane], exchange[3][lane]));
+      const bool live = lane < heads, grows = live && high > reference + kGrowth;   // (the first block: from -infinity)
+      const float next = grows ? high : reference, fade = grows && i > 0 ? ex2(reference - next) : 1.f;
+      reference = next;
+      sum *= fade;
+      if (__any_sync(0xffffffffu, grows) && i > 0) {
         ok = wait_bounded(&sum_done[(i - 1) & 1], uint32_t((i - 1) >> 1) & 1u, p.status, 13) && ok;
         __syncwarp();
         tcgen05_fence_after();
@@ -255,36 +270,42 @@ __global__ void __launch_bounds__(kLatentThreads, 1) decode_latent(const __grid_
           float v[32];
           tmem_load_32(tmem + lanes + uint32_t(2 * kScoreColumns + c), v);
 #pragma unroll
-          for (int k = 0; k < 32; ++k) v[k] *= fade[i & 1][k];
+          for (int k = 0; k < 32; ++k) v[k] *= __shfl_sync(0xffffffffu, fade, k);
           tmem_store_32(tmem + lanes + uint32_t(2 * kScoreColumns + c), v);
         }
-        tcgen05_fence_before();
-        column_sync();
       }
-      if (quarter == 0) {
-        // the weights' place is free once the sums two blocks before are done
-        if (i >= 2) ok = wait_bounded(&sum_done[i & 1], uint32_t((i - 2) >> 1) & 1u, p.status, 14) && ok;
-        unsigned char* rows = weights + (i & 1) * kWeightBytes + lane * 128;
-        const bool live = lane < heads;
+      // the weights' place is free once the sums two blocks before are done
+      if (i >= 2) ok = wait_bounded(&sum_done[i & 1], uint32_t((i - 2) >> 1) & 1u, p.status, 14) && ok;
+      unsigned char* rows = weights + (i & 1) * kWeightBytes + lane * 128;
 #pragma unroll
-        for (int unit = 0; unit < kKeys / 8; ++unit) {
-          float w[8];
+      for (int unit = 0; unit < 2; ++unit) {
+        float w[8], left[8];
+        uint32_t word[4];
 #pragma unroll
-          for (int x = 0; x < 8; ++x) {
-            w[x] = live ? ex2(s[8 * unit + x] - reference) : 0.f;
-            sum += w[x];
-          }
-          const int at = (unit ^ (lane & 7)) * 16;
-          *reinterpret_cast<uint4*>(rows + at) = make_uint4(pack(w[0], w[1]), pack(w[2], w[3]), pack(w[4], w[5]), pack(w[6], w[7]));
-          *reinterpret_cast<uint4*>(rows + kUnitHeads * 128 + at) =
-              make_uint4(pack(rest(w[0]), rest(w[1])), pack(rest(w[2]), rest(w[3])), pack(rest(w[4]), rest(w[5])), pack(rest(w[6]), rest(w[7])));
+        for (int x = 0; x < 8; ++x) {
+          w[x] = live ? ex2(s[8 * unit + x] - reference) : 0.f;
+          sum += w[x];
         }
-        fence_proxy_async();
-        tcgen05_fence_before();
-        __syncwarp();
-        if (lane == 0) mbar_arrive(&weight_full[i & 1]);
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          word[x] = pack(w[2 * x], w[2 * x + 1]);
+          left[2 * x] = w[2 * x] - bf_lo(word[x]);
+          left[2 * x + 1] = w[2 * x + 1] - bf_hi(word[x]);
+        }
+        const int at = ((2 * quarter + unit) ^ (lane & 7)) * 16;
+        *reinterpret_cast<uint4*>(rows + at) = make_uint4(word[0], word[1], word[2], word[3]);
+        *reinterpret_cast<uint4*>(rows + kUnitHeads * 128 + at) =
+            make_uint4(pack(left[0], left[1]), pack(left[2], left[3]), pack(left[4], left[5]), pack(left[6], left[7]));
       }
+      fence_proxy_async();
+      tcgen05_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&weight_full[i & 1]);
     }
+    column_sync();                                       // (the last maxima have been read)
+    exchange[quarter][lane] = sum;
+    column_sync();
+    sum = exchange[0][lane] + exchange[1][lane] + exchange[2][lane] + exchange[3][lane];
     const bool whole = p.splits == 1;
     const size_t record = (size_t(blockIdx.z) * p.heads + head0) * p.splits + split;   // of the unit's head 0; heads are `splits` apart
     if (quarter == 0 && lane < heads) {
