@@ -41,18 +41,26 @@ struct LatentParams {
 // so both products stream the rows through the tensor core from the one copy. Warp 0 requests rows, warp 1 issues products,
 // warps 4 to 7 share the softmax (a lane per head, 16 keys a warp), own the columns of O (rescaled only when a maximum outgrows
 // its reference by 2^8) and put the token's own row, normed, and zeros for rows out of sight into the edge blocks.
-constexpr int kUnitHeads = 32, kLatentThreads = 256, kSlots = 10;
+// A ring of slots holds blocks ahead: up to 256 columns four of them, two CTAs then share an SM and hide each other's waits.
+constexpr int kUnitHeads = 32, kLatentThreads = 256, kMostSlots = 10, kSharedSlots = 4, kSharedChunks = 4;
 constexpr int kChunkBytes = kKeys * 128, kSlotBytes = 2 * kChunkBytes, kQueryChunk = kUnitHeads * 128, kMostChunks = kTiledLatent / 64;
-constexpr int kQueryBytes = kMostChunks * kQueryChunk, kWeightBytes = 2 * kUnitHeads * 128;
+constexpr int kWeightBytes = 2 * kUnitHeads * 128;
 constexpr int kScorePitch = kKeys + 4;
-constexpr int kDecodeSmem = kQueryBytes + kSlots * kSlotBytes + 2 * kWeightBytes + kUnitHeads * kScorePitch * 4 + 1024;
+__host__ __device__ constexpr int DecodeSmem(int chunks, int ring) {
+  return chunks * kQueryChunk + ring * kSlotBytes + 2 * kWeightBytes + kUnitHeads * kScorePitch * 4 + 1024;
+}
+static_assert(kMostSlots * kSlotBytes >= 128 * 128, "a score product reads 128 query rows, past the last chunk's own");
+static_assert(kSharedSlots * kSlotBytes >= 128 * 128, "a score product reads 128 query rows, past the last chunk's own");
 constexpr int kScoreColumns = kKeys, kSumColumns = 2 * kUnitHeads;   // tensor memory: two blocks' scores, then a slot's sums each
 constexpr float kGrowth = 8.f;
 
 __device__ __forceinline__ void column_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
-__global__ void __launch_bounds__(kLatentThreads, 1) decode_latent(const __grid_constant__ CUtensorMap pool_map, const __grid_constant__ CUtensorMap q_map,
+template <bool SHARED>
+__global__ void __launch_bounds__(kLatentThreads, SHARED ? 2 : 1) decode_latent(const __grid_constant__ CUtensorMap pool_map, const __grid_constant__ CUtensorMap q_map,
                                                                    StepRows r, LatentParams p) {
+  constexpr int kSlots = SHARED ? kSharedSlots : kMostSlots, kQueryBytes = (SHARED ? kSharedChunks : kMostChunks) * kQueryChunk;
+  constexpr int kTensorColumns = SHARED ? 256 : 512;
   extern __shared__ unsigned char smem_raw[];
   unsigned char* queries = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   unsigned char* slots = queries + kQueryBytes;        // (the score product reads rows behind a unit's out of whatever follows)
@@ -92,7 +100,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) decode_latent(const __grid_
     mbar_init(&patched, 128);
     mbar_fence_init();
   }
-  if (warp == 1) tmem_alloc(&tmem_slot, 512);
+  if (warp == 1) tmem_alloc(&tmem_slot, kTensorColumns);
   tcgen05_fence_before();
   __syncthreads();
   tcgen05_fence_after();
@@ -348,7 +356,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1) decode_latent(const __grid_
   __syncthreads();
   if (warp == 1) {
     tcgen05_fence_after();
-    tmem_dealloc(tmem, 512);
+    tmem_dealloc(tmem, kTensorColumns);
   }
 }
 
@@ -678,19 +686,23 @@ void Divide(LatentParams* p, int most) {
 int DecodeLatent(const Queue& q, const StepRows& r, const LatentArgs& a, LatentParams p) {
   // the cut of a token's keys that ends soonest: a CTA costs its blocks plus a few blocks' time to start, a merge behind it three
   const int blocks = (std::min(a.window, r.capacity) + kRaggedBlock - 2) / kKeys + 1;
+  const bool shared = a.pool_dim <= 64 * kSharedChunks;
+  const int resident = (shared ? 2 : 1) * q.sm_count;
   Divide(&p, kUnitHeads);
   p.splits = 1;
   float least = 0.f;
   for (int s = 1; s <= std::min(blocks, kMostSplits); ++s) {
     if (size_t(r.entries) * a.heads * s * (a.rank_stride + 2) > a.part_floats) break;
-    const int waves = (r.singles * p.subs * s + q.sm_count - 1) / q.sm_count;
+    const int waves = (r.singles * p.subs * s + resident - 1) / resident;
     const float cost = float(waves) * (float((blocks + s - 1) / s) + 3.f) + (s > 1 ? 3.f + float(s) / 16.f : 0.f);
     if (s == 1 || cost < least) {
       least = cost;
       p.splits = s;
     }
   }
-  const int status = int(Launch(decode_latent, dim3(unsigned(p.splits), unsigned(p.subs), unsigned(r.entries)), dim3(kLatentThreads), kDecodeSmem, q.stream,
+  auto kernel = shared ? decode_latent<true> : decode_latent<false>;
+  const int smem = shared ? DecodeSmem(kSharedChunks, kSharedSlots) : DecodeSmem(kMostChunks, kMostSlots);
+  const int status = int(Launch(kernel, dim3(unsigned(p.splits), unsigned(p.subs), unsigned(r.entries)), dim3(kLatentThreads), smem, q.stream,
                                 q.chained, *a.pool_map, *a.q_map, r, p));
   if (status != 0 || p.splits == 1) return status;
   return int(Launch(merge_latent, dim3(unsigned(a.heads), unsigned(r.entries)), dim3(128), 0, q.stream, q.chained, r, p));
@@ -759,7 +771,9 @@ int GatherLatent(const Queue& q, const StepRows& r, const LatentArgs& a, const i
 }
 
 int PrepareLatent() {
-  cudaError_t err = cudaFuncSetAttribute(decode_latent, cudaFuncAttributeMaxDynamicSharedMemorySize, kDecodeSmem);
+  cudaError_t err = cudaFuncSetAttribute(decode_latent<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, DecodeSmem(kMostChunks, kMostSlots));
+  if (err == cudaSuccess)
+    err = cudaFuncSetAttribute(decode_latent<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DecodeSmem(kSharedChunks, kSharedSlots));
   if (err == cudaSuccess) err = Raise<8>();
   if (err == cudaSuccess) err = Raise<16>();
   if (err == cudaSuccess) err = Raise<32>();
