@@ -47,6 +47,8 @@ CASES = {
     # many heads on a latent row and per key head
     "crowd": model(96, 128, [latent(70, 16, 24, 140, 45, moe(9, 2, 48, 3, 2)), latent(20, 24, 8, 64, 300), grouped(34, 2, 16, 24, 8, 45, moe(8, 3, 20, 2, 2)),
                              grouped(20, 1, 48, 48, 24, 300), latent(33, 8, 16, 250, 37)], streams=2),
+    # latent rows wider than the tiles, windows over everything
+    "vast": model(64, 90, [latent(3, 16, 12, 600, None, moe(4, 2, 24, 2, 1)), grouped(4, 2, 16, 16, 16, None), latent(2, 24, 24, 1024, 40)], streams=2),
 }
 
 

@@ -129,7 +129,7 @@ def test_unsupported_programs_are_refused(break_it, message, plan_dir, capfd):
     so = emit_plan(case.CASES["odd"], plan_dir, phase="ragged", slots=2, capacity=32, num_blocks=5, max_rows=16)
     document = json.loads((so.parent / (so.name + ".plan.json")).read_text())
     break_it(document["model"]["layers"])
-    broken = so.parent / f"tilemega_b200_refused_{abs(hash(message)) % 10 ** 8}.so"
+    broken = so.parent / f"tilemega_b200_refused_mozidra_{abs(hash(message)) % 10 ** 8}.so"
     shutil.copyfile(so, broken)
     (so.parent / (broken.name + ".plan.json")).write_text(json.dumps(document))
     with pytest.raises(RuntimeError, match=message):

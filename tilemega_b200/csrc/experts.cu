@@ -337,7 +337,8 @@ bool RouteFused(int rows) { return rows <= kFusedRows; }
 
 int Route(const Queue& q, const RouteArgs& a) {
   if (a.rows <= 0) return 0;
-  if (a.experts > kMaxExperts || a.top > a.experts || a.tile_rows < 1 || a.k_stride % 8 || (!a.ranks && (a.softmax || a.correction || a.keep_groups < a.groups)) || a.top > kMaxTop)
+  if (a.experts > kMaxExperts || a.top > a.experts || a.top > kMaxTop || a.tile_rows < 1 || a.k_stride % 8 ||
+      (!a.ranks && (a.softmax || a.correction || a.keep_groups < a.groups)))
     return int(cudaErrorInvalidValue);
   return q.f32 ? RouteAs<float>(q, a) : RouteAs<__nv_bfloat16>(q, a);
 }

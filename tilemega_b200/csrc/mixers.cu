@@ -1,6 +1,7 @@
 // Token mixers of a ragged step, in the form that works for every size and both element types: rotary append into the
-// paged pools, attention with a sliding window and kept first positions, retention by its recurrence. Attention of
-// bf16 steps and retention inside bf16 prompt portions run in mixers_mma.cu.
+// paged pools, attention with a sliding window and kept first positions (over latent rows too), retention by its recurrence.
+// Attention of bf16 steps and retention inside bf16 prompt portions run in mixers_mma.cu, latent attention of bf16 steps in
+// latent.cu.
 #include <cuda_bf16.h>
 
 #include <algorithm>
