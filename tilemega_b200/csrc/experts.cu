@@ -48,7 +48,7 @@ template <bool HELD> __device__ __forceinline__ void choose(const RouteArgs& a, 
 #pragma unroll
     for (int i = 0; i < kMine; ++i) key[i] = lane + 32 * i < a.experts ? max(ordered(__ldcg(z + lane + 32 * i)), 1u) : 0u;   // 0: taken, or none
   unsigned before = 0xffffffffu;
-  int before_at = -1;
+  int before_at = -1, taken = 0;         // taken: the lane-th choice
   for (int k = 0; k < a.top; ++k) {
     unsigned best = 0u;
     int at = 0x7fffffff;
@@ -78,11 +78,17 @@ template <bool HELD> __device__ __forceinline__ void choose(const RouteArgs& a, 
     }
     before = high;
     before_at = at;
-    if (lane == 0) {
-      at = min(at, a.experts - 1);
-      a.choice[row * a.top + k] = at;
-      a.score[row * a.top + k] = 1.f / (1.f + expf(-__ldcg(z + at)));
-    }
+    if (lane == k) taken = min(at, a.experts - 1);
+  }
+  const float logit = lane < a.top ? __ldcg(z + taken) : -INFINITY;
+  float score = 1.f / (1.f + expf(-logit));
+  if (a.chosen) {
+    const float e = expf(logit - warp_max(logit));
+    score = e / warp_sum(e);
+  }
+  if (lane < a.top) {
+    a.choice[row * a.top + lane] = taken;
+    a.score[row * a.top + lane] = score;
   }
 }
 // The same where scores are not the logits' order: ranked by score + correction, from the best groups only. `line` holds the
@@ -338,7 +344,7 @@ bool RouteFused(int rows) { return rows <= kFusedRows; }
 int Route(const Queue& q, const RouteArgs& a) {
   if (a.rows <= 0) return 0;
   if (a.experts > kMaxExperts || a.top > a.experts || a.top > kMaxTop || a.tile_rows < 1 || a.k_stride % 8 ||
-      (!a.ranks && (a.softmax || a.correction || a.keep_groups < a.groups)))
+      (!a.ranks && (a.softmax || a.correction || a.keep_groups < a.groups)) || (a.chosen && a.ranks))
     return int(cudaErrorInvalidValue);
   return q.f32 ? RouteAs<float>(q, a) : RouteAs<__nv_bfloat16>(q, a);
 }

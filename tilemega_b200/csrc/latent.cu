@@ -20,7 +20,7 @@ constexpr int kKeys = 64;          // latent rows per block
 
 struct LatentParams {
   const bf16* q;
-  const bf16* raw;
+  const bf16* raw;                 // null: every row of the step lies in the pool already
   bf16* pool;
   bf16* out;
   float* part;                     // split sums: [entry][head][split][rank_stride] latent columns, then [entry][head][split] references and sums
@@ -187,7 +187,7 @@ __global__ void __launch_bounds__(kLatentThreads, SHARED ? 2 : 1) decode_latent(
     bool ok = true;
     float inv = 1.f;
     const bf16* raw = p.raw + size_t(e.first_row) * p.raw_stride;
-    const bool newest = count > 0 && from + count == blocks;
+    const bool newest = p.raw && count > 0 && from + count == blocks;
     if (newest) {
       float sq = 0.f;
       for (int d = t; d < p.rank; d += 128) sq = fmaf(__bfloat162float(raw[d]), __bfloat162float(raw[d]), sq);
@@ -213,7 +213,7 @@ __global__ void __launch_bounds__(kLatentThreads, SHARED ? 2 : 1) decode_latent(
           const int row = n / units;
           *place(row < first ? row : behind + row - first, n % units) = make_uint4(0, 0, 0, 0);
         }
-        if (from + i == blocks - 1) {
+        if (p.raw && from + i == blocks - 1) {
           bf16* to_pool = p.pool + size_t(key_row(table, p1, r)) * p.pool_dim;
           for (int unit = t; unit < p.pool_dim / 8; unit += 128) {
             float c[8];
@@ -403,7 +403,8 @@ template <int RT> struct LatentShape {
   static constexpr int kPitch = RT * 16 + 8;
   static constexpr int kRows = 16 * WM;
   static constexpr int kTile = kKeys * kPitch;                                    // elements of one block
-  static constexpr int kSmem = (kRows * kPitch + 2 * kTile + 2 * kRows * kWeightPitch) * 2;   // q, two blocks, weights as heads and remainders
+  static constexpr int kStages = RT <= 32 ? 2 : 1;
+  static constexpr int kSmem = (kRows * kPitch + kStages * kTile + 2 * kRows * kWeightPitch) * 2;   // q, blocks, weights as heads and remainders
 };
 
 // Rows of a tile are (token, head of the unit) pairs, token-major; the warps are four row tiles times WN parts: of a block's
@@ -413,12 +414,12 @@ template <int RT, bool FULL>
 __global__ void __launch_bounds__(LatentShape<RT>::kThreads, 1) attend_latent(StepRows r, LatentParams p) {
   using Shape = LatentShape<RT>;
   constexpr int WM = Shape::WM, kWarps = Shape::kWarps, kThreads = Shape::kThreads;
-  constexpr int WN = kWarps / WM, KN = kKeys / WN, P = Shape::kPitch, CT = RT / WN;   // CT: column tiles of a warp
+  constexpr int WN = kWarps / WM, KN = kKeys / WN, P = Shape::kPitch, CT = RT / WN, S = Shape::kStages;   // CT: column tiles of a warp
   static_assert(CT >= 1, "a warp sums at least one column tile");
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* qs = reinterpret_cast<bf16*>(smem_raw);
   bf16* cs = qs + Shape::kRows * P;
-  bf16* wh = cs + 2 * Shape::kTile;
+  bf16* wh = cs + S * Shape::kTile;
   bf16* wl = wh + Shape::kRows * kWeightPitch;
   __shared__ float high_part[WN][Shape::kRows], sum_part[WN][Shape::kRows];
   __shared__ int key_at[2][kKeys];   // pool rows of a block's keys (-1: none)
@@ -443,13 +444,12 @@ __global__ void __launch_bounds__(LatentShape<RT>::kThreads, 1) attend_latent(St
     }
   };
   auto fetch = [&](int b) {
-    const int stage = b & 1;
     constexpr int C = RT * 2;        // 16-byte pieces of a row
 #pragma unroll 4
     for (int i = threadIdx.x; i < kKeys * C; i += kThreads) {
-      const int key = i / C, c = (i % C) * 8, row = key_at[stage][key];
+      const int key = i / C, c = (i % C) * 8, row = key_at[b & 1][key];
       const bool live = row >= 0;
-      if (FULL || c < p.pool_dim) copy16(cs + stage * Shape::kTile + key * P + c, p.pool + size_t(live ? row : 0) * p.pool_dim + c, live);
+      if (FULL || c < p.pool_dim) copy16(cs + (b % S) * Shape::kTile + key * P + c, p.pool + size_t(live ? row : 0) * p.pool_dim + c, live);
     }
     copy_commit();
   };
@@ -484,9 +484,9 @@ __global__ void __launch_bounds__(LatentShape<RT>::kThreads, 1) attend_latent(St
   float top_a = -INFINITY, top_b = -INFINITY, sum_a = 0.f, sum_b = 0.f;   // maxima of all keys, sums of this warp's
 
   for (int b = 0; b < blocks; ++b) {
-    const int stage = b & 1;
-    bf16* tile = cs + stage * Shape::kTile;
-    if (b + 1 < blocks) {
+    bf16* tile = cs + (b % S) * Shape::kTile;
+    if (S == 1 && b > 0) fetch(b);
+    if (S > 1 && b + 1 < blocks) {
       fetch(b + 1);
       copy_wait<1>();
     } else {
@@ -729,7 +729,7 @@ template <int RT> cudaError_t Raise() {
 int AttendLatentTiles(const Queue& q, const StepRows& r, const LatentArgs& a) {
   LatentParams p{};
   p.q = static_cast<const bf16*>(a.q);
-  p.raw = static_cast<const bf16*>(a.raw);
+  p.raw = a.query_raw ? nullptr : static_cast<const bf16*>(a.raw);
   p.pool = static_cast<bf16*>(a.pool);
   p.out = static_cast<bf16*>(a.out);
   p.part = a.part;
@@ -750,7 +750,7 @@ int AttendLatentTiles(const Queue& q, const StepRows& r, const LatentArgs& a) {
     if (status != 0) return status;
   }
   if (r.singles == r.entries || a.singles_only) return 0;
-  return a.rank <= 128 ? AttendWith<8>(q, r, p) : a.rank <= 256 ? AttendWith<16>(q, r, p) : AttendWith<32>(q, r, p);
+  return a.rank <= 128 ? AttendWith<8>(q, r, p) : a.rank <= 256 ? AttendWith<16>(q, r, p) : a.rank <= 512 ? AttendWith<32>(q, r, p) : AttendWith<40>(q, r, p);
 }
 
 bool EncodeLatent(CUtensorMap* pool_map, const void* pool, uint64_t rows, uint64_t pool_dim) {
@@ -777,6 +777,7 @@ int PrepareLatent() {
   if (err == cudaSuccess) err = Raise<8>();
   if (err == cudaSuccess) err = Raise<16>();
   if (err == cudaSuccess) err = Raise<32>();
+  if (err == cudaSuccess) err = Raise<40>();
   return int(err);
 }
 

@@ -32,6 +32,10 @@ struct LinearParams {
   const int* rows_there;
   int chunks, chunks_per_split;
   Glu glu;
+  int tanh_below;
+  float gain;
+  RotateHeads rotate;
+  SideGate side;
   ExpertSlots slots;
   unsigned* status;
 };
@@ -64,6 +68,25 @@ __device__ __forceinline__ float glu_value(float g, float u, const Glu& p) {
   return g / (1.f + __expf(-p.alpha * g)) * (u + p.shift);
 }
 
+// Is column n of a product with rotated heads one that turns?
+__device__ __forceinline__ bool turns(const RotateHeads& p, int n) {
+  const int d = n % p.head - p.lead;
+  return d >= 0 && d < p.rotary.dims;
+}
+// ... and what becomes of it; `other` is its neighbour's value.
+__device__ __forceinline__ float turned(const RotateHeads& p, int t, int n, float v, float other) {
+  const int d = n % p.head - p.lead;
+  const float2 cs = p.rotary.table[size_t(min(p.positions[t], p.rotary.capacity - 1)) * (p.rotary.dims / 2) + d / 2];
+  return d & 1 ? v * cs.x + other * cs.y : v * cs.x - other * cs.y;
+}
+
+// gelu(z) times column n of the row's token's part
+template <typename T> __device__ __forceinline__ float side_value(const SideGate& p, int t, int n, float z) {
+  const T* part = static_cast<const T*>(p.part) + size_t(min(max(p.tokens[t], 0), p.vocab - 1)) * p.stride;
+  const float y = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  return (sizeof(T) == 4 ? 0.5f * z * (1.f + tanhf(y)) : z / (1.f + __expf(-2.f * y))) * to_f(part[n]);
+}
+
 __device__ __forceinline__ uint32_t cluster_rank() {
   uint32_t r;
   asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
@@ -81,9 +104,12 @@ __device__ __forceinline__ float ld_peer(uint32_t local, uint32_t rank) {
 }
 
 template <int EPI> __device__ __forceinline__ void emit(const LinearParams& g, int t, int n, float v) {
-  if (EPI == kLinearStore || EPI == kLinearHeads) static_cast<__nv_bfloat16*>(g.out)[size_t(t) * g.out_stride + n] = __float2bfloat16_rn(v);
+  if (EPI == kLinearStore && n < g.tanh_below) v = tanhf(v);
+  if (EPI == kLinearSide) v = side_value<__nv_bfloat16>(g.side, t, n, v);
+  if (EPI == kLinearStore || EPI == kLinearHeads || EPI == kLinearRotate || EPI == kLinearSide)
+    static_cast<__nv_bfloat16*>(g.out)[size_t(t) * g.out_stride + n] = __float2bfloat16_rn(v);
   if (EPI == kLinearAdd) static_cast<float*>(g.out)[size_t(t) * g.out_stride + n] += v;
-  if (EPI == kLinearFloat) static_cast<float*>(g.out)[size_t(t) * g.out_stride + n] = v;
+  if (EPI == kLinearFloat) static_cast<float*>(g.out)[size_t(t) * g.out_stride + n] = v * g.gain;
   if (EPI == kLinearExpertUp) {
     const float r = fmaxf(v * g.slots.score[t], 0.f);
     static_cast<__nv_bfloat16*>(g.out)[size_t(t) * g.out_stride + n] = __float2bfloat16_rn(r * r);
@@ -288,7 +314,12 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
         const int row = worker & (kRowsM - 1), n = n0 + row;
         if (n < g.n) {
           const float bias = g.bias ? g.bias[n] : 0.f;
-          for (int c = first + (worker >> 7); c < first + cols; c += 2) emit<EPI>(g, t0 + c, out_at + n, total(c, row) + bias);
+          const bool turning = EPI == kLinearRotate && turns(g.rotate, n);   // (neighbours lie in one tile)
+          for (int c = first + (worker >> 7); c < first + cols; c += 2) {
+            float v = total(c, row) + bias;
+            if (turning) v = turned(g.rotate, t0 + c, n, v, total(c, row ^ 1));
+            emit<EPI>(g, t0 + c, out_at + n, v);
+          }
         }
       }
     }
@@ -311,6 +342,13 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
           const int col = i + (upper ? 1 : 0);
           if (out < g.outputs && col < cols)
             static_cast<__nv_bfloat16*>(g.out)[size_t(t0 + c + col) * g.out_stride + out] = __float2bfloat16_rn(y);
+        }
+      } else if constexpr (EPI == kLinearRotate) {
+        const bool turning = turns(g.rotate, n);
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          const float other = __shfl_xor_sync(0xffffffffu, v[i], 1);
+          if (i < cols && n < g.n) emit<EPI>(g, t0 + c + i, n, turning ? turned(g.rotate, t0 + c + i, n, v[i], other) : v[i]);
         }
       } else if (n < g.n) {
         if constexpr (EPI == kLinearAdd) {
@@ -383,7 +421,11 @@ __global__ void __launch_bounds__(256) linear_f32(const float* activations, cons
     for (int j = 0; j < 4; ++j) {
       const int t = t0 + ty * 4 + i, n = n0 + tx * 4 + j;
       if (t >= t_end || n >= g.n) continue;
-      const float v = acc[i][j] + (g.bias ? g.bias[n] : 0.f);
+      float v = acc[i][j] + (g.bias ? g.bias[n] : 0.f);
+      if (EPI == kLinearStore && n < g.tanh_below) v = tanhf(v);
+      if (EPI == kLinearSide) v = side_value<float>(g.side, t, n, v);
+      if (EPI == kLinearFloat) v *= g.gain;
+      if (EPI == kLinearRotate && turns(g.rotate, n)) v = turned(g.rotate, t, n, v, acc[i][j ^ 1]);
       float* out = static_cast<float*>(g.out) + size_t(EPI == kLinearExpertDown ? g.slots.list[t] : t) * g.out_stride + size_t(head) * g.head_out + n;
       const float positive = fmaxf(EPI == kLinearExpertUp ? v * g.slots.score[t] : 0.f, 0.f);
       *out = EPI == kLinearAdd ? *out + v : EPI == kLinearExpertUp ? positive * positive : v;
@@ -410,7 +452,7 @@ template <int BN> cudaError_t RaiseLimit() {
   const int smem = LinearShape<BN>::kSmem;
   for (auto kernel : {linear_tiles<BN, kLinearStore>, linear_tiles<BN, kLinearAdd>, linear_tiles<BN, kLinearGlu>, linear_tiles<BN, kLinearFloat>,
                       linear_tiles<BN, kLinearExpertUp>, linear_tiles<BN, kLinearExpertDown>, linear_tiles<BN, kLinearHeads>,
-                      linear_tiles<BN, kLinearExpertGlu>}) {
+                      linear_tiles<BN, kLinearExpertGlu>, linear_tiles<BN, kLinearRotate>, linear_tiles<BN, kLinearSide>}) {
     const cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (err != cudaSuccess) return err;
   }
@@ -425,7 +467,8 @@ cudaError_t LaunchTiles(const Queue& q, const LinearArgs& a, const LinearParams&
   auto kernel = a.epilogue == kLinearAdd ? linear_tiles<BN, kLinearAdd> : a.epilogue == kLinearGlu ? linear_tiles<BN, kLinearGlu>
                 : a.epilogue == kLinearFloat ? linear_tiles<BN, kLinearFloat> : a.epilogue == kLinearExpertUp ? linear_tiles<BN, kLinearExpertUp>
                 : a.epilogue == kLinearExpertDown ? linear_tiles<BN, kLinearExpertDown> : a.epilogue == kLinearHeads ? linear_tiles<BN, kLinearHeads>
-                : a.epilogue == kLinearExpertGlu ? linear_tiles<BN, kLinearExpertGlu> : linear_tiles<BN, kLinearStore>;
+                : a.epilogue == kLinearExpertGlu ? linear_tiles<BN, kLinearExpertGlu> : a.epilogue == kLinearRotate ? linear_tiles<BN, kLinearRotate>
+                : a.epilogue == kLinearSide ? linear_tiles<BN, kLinearSide> : linear_tiles<BN, kLinearStore>;
   cudaLaunchConfig_t config{};
   const unsigned weight_tiles = unsigned((a.n + kRowsM - 1) / kRowsM) * unsigned(std::max(a.heads, 1));
   config.gridDim = PerExpert(a.epilogue) ? dim3(weight_tiles, unsigned(MostTiles(a.slots)), unsigned(splits))
@@ -517,7 +560,12 @@ int Linear(const Queue& q, const LinearArgs& a) {
   if (a.epilogue == kLinearHeads ? a.heads < 1 || a.head_in % 8 != 0 || a.bias : a.heads != 0) return int(cudaErrorInvalidValue);
   if (a.rows_there && (q.f32 || a.epilogue != kLinearStore)) return int(cudaErrorInvalidValue);
   if (a.epilogue == kLinearExpertStore && !q.f32) return int(cudaErrorInvalidValue);
+  if (a.epilogue == kLinearRotate && (a.rotate.head < 2 || a.rotate.head % 2 || a.rotate.lead % 2 || a.bias)) return int(cudaErrorInvalidValue);
   LinearParams p{};
+  p.tanh_below = a.tanh_below;
+  p.gain = a.gain;
+  p.rotate = a.rotate;
+  p.side = a.side;
   p.head_in = a.head_in;
   p.head_out = a.head_out;
   p.rows_there = a.rows_there;
@@ -534,7 +582,8 @@ int Linear(const Queue& q, const LinearArgs& a) {
     if (IsGlu(a.epilogue)) return int(cudaErrorInvalidValue);   // two operations in fp32: the product, then GluRows
     auto kernel = a.epilogue == kLinearAdd ? linear_f32<kLinearAdd> : a.epilogue == kLinearExpertUp ? linear_f32<kLinearExpertUp>
                   : a.epilogue == kLinearExpertDown ? linear_f32<kLinearExpertDown>
-                  : a.epilogue == kLinearExpertStore ? linear_f32<kLinearExpertStore> : linear_f32<kLinearStore>;
+                  : a.epilogue == kLinearExpertStore ? linear_f32<kLinearExpertStore> : a.epilogue == kLinearFloat ? linear_f32<kLinearFloat>
+                  : a.epilogue == kLinearRotate ? linear_f32<kLinearRotate> : a.epilogue == kLinearSide ? linear_f32<kLinearSide> : linear_f32<kLinearStore>;
     if (experts && a.slots.tile_rows != kTile32) return int(cudaErrorInvalidValue);
     const dim3 grid(unsigned((a.n + kTile32 - 1) / kTile32), unsigned(experts ? MostTiles(a.slots) : (a.t + kTile32 - 1) / kTile32), unsigned(std::max(a.heads, 1)));
     return int(Launch(kernel, grid, dim3(256), 0, q.stream, q.chained, static_cast<const float*>(a.activations),

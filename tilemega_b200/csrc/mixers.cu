@@ -208,19 +208,45 @@ __global__ void __launch_bounds__(32 * kPlainWarps) attend_rows(StepRows r, cons
   }
 }
 
-// ---- latent rows: normed into the pool ------------------------------------------------------------------------------------
+// ---- latent rows: normed (and their last columns rotated) into the pool; rows that queries are images of, normed -------------
+struct AppendLatentParams {
+  int raw_stride, pool_dim, rank;
+  const float* norm;
+  Rotary rotary;
+  const void* query_raw;
+  const float* query_norm;
+  void* query;
+  int query_rank, query_stride;
+  float eps;
+};
+
 template <typename T>
-__global__ void __launch_bounds__(128) append_latent(StepRows r, const T* raw, int stride, T* pool, int pool_dim, int rank, const float* norm, float eps,
-                                                     bool portions_only) {
+__global__ void __launch_bounds__(128) append_latent(StepRows r, const T* raw, T* pool, AppendLatentParams p, bool portions_only) {
   __shared__ float2 part[4];
   dependency_wait();
   allow_dependents();
   const int row = blockIdx.x;
   if (portions_only && r.entry[r.row_entry[row]].rows == 1) return;
-  const T* line = raw + size_t(row) * stride;
-  T* to = pool + pool_offset(r.row_kv[row], 0, 1, pool_dim);
-  const float inv = inverse_rms<128>(make_float2(square_sum(line, rank, 128), 0.f), rank, 1, eps, part).x;
-  for (int d = threadIdx.x; d < rank; d += 128) to[d] = from_f<T>(to_f(line[d]) * inv * norm[d]);
+  if (blockIdx.y == 1) {
+    const T* line = static_cast<const T*>(p.query_raw) + size_t(row) * p.raw_stride;
+    T* to = static_cast<T*>(p.query) + size_t(row) * p.query_stride;
+    const float inv = inverse_rms<128>(make_float2(square_sum(line, p.query_rank, 128), 0.f), p.query_rank, 1, p.eps, part).x;
+    for (int d = threadIdx.x; d < p.query_rank; d += 128) to[d] = from_f<T>(to_f(line[d]) * inv * p.query_norm[d]);
+    return;
+  }
+  const int half = p.rotary.dims / 2, normed = p.rank - p.rotary.dims;
+  const T* line = raw + size_t(row) * p.raw_stride;
+  T* to = pool + pool_offset(r.row_kv[row], 0, 1, p.pool_dim);
+  const float inv = inverse_rms<128>(make_float2(square_sum(line, normed, 128), 0.f), normed, 1, p.eps, part).x;
+  for (int d = threadIdx.x; d < normed; d += 128) to[d] = from_f<T>(to_f(line[d]) * inv * p.norm[d]);
+  const float2* angle = p.rotary.table + size_t(min(r.row_position[row], p.rotary.capacity - 1)) * half;
+  for (int i = threadIdx.x; i < half; i += 128) {
+    const int d = normed + 2 * i;
+    const float u = to_f(line[d]), v = to_f(line[d + 1]);
+    const float2 cs = angle[i];
+    to[d] = from_f<T>(u * cs.x - v * cs.y);
+    to[d + 1] = from_f<T>(v * cs.x + u * cs.y);
+  }
 }
 
 // ---- retention by its recurrence ----------------------------------------------------------------------------------------
@@ -370,18 +396,21 @@ __global__ void __launch_bounds__(kTokenThreads, NR <= 8 ? 2 : 1) retain_token(S
   }
 }
 
+// A warp per (row, head), see HeadGateArgs.
 template <typename T>
-__global__ void __launch_bounds__(128) retention_gate(const float* raw, const T* proj, int stride, int gate_offset, T* out, int out_stride, int rows,
-                                                      int heads, int vdim, float eps) {
+__global__ void __launch_bounds__(128) head_gate(HeadGateArgs p) {
   dependency_wait();
   allow_dependents();
-  const int unit = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (unit >= rows * heads) return;
-  const int row = unit / heads, head = unit % heads;
-  const float* o = raw + size_t(row) * heads * vdim + size_t(head) * vdim;
-  const T* gate = proj + size_t(row) * stride + gate_offset + size_t(head) * vdim;
+  const int unit = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, vdim = p.vdim;
+  if (unit >= p.rows * p.heads) return;
+  const int row = unit / p.heads, head = unit % p.heads;
+  const float* o = p.raw + size_t(row) * p.heads * vdim + size_t(head) * vdim;
+  const T* gate = static_cast<const T*>(p.proj) + size_t(row) * p.proj_stride + p.gate_at + size_t(head) * vdim;
+  const float* weight = p.weight ? p.weight + size_t(head) * vdim : nullptr;
+  T* out = static_cast<T*>(p.out) + size_t(row) * p.out_stride + size_t(head) * vdim;
+  auto opened = [&](float x) { return p.silu ? x / (1.f + expf(-x)) : sigmoid(x); };
   float sq = 0.f;
-  if (vdim % 4 == 0 && vdim <= 256 && stride % 4 == 0 && gate_offset % 4 == 0 && out_stride % 4 == 0) {
+  if (vdim % 4 == 0 && vdim <= 256 && p.proj_stride % 4 == 0 && p.gate_at % 4 == 0 && p.out_stride % 4 == 0) {
     float4 v[2];
     alignas(16) T g[2][4], y[4];
     using Word = std::conditional_t<sizeof(T) == 2, uint2, uint4>;
@@ -393,27 +422,22 @@ __global__ void __launch_bounds__(128) retention_gate(const float* raw, const T*
       *reinterpret_cast<Word*>(g[n]) = *reinterpret_cast<const Word*>(gate + d);
       sq += v[n].x * v[n].x + v[n].y * v[n].y + v[n].z * v[n].z + v[n].w * v[n].w;
     }
-    const float inv = 1.f / sqrtf(warp_sum(sq) / float(vdim) + eps);
+    const float inv = 1.f / sqrtf(warp_sum(sq) / float(vdim) + p.eps);
 #pragma unroll
     for (int n = 0; n < 2; ++n) {
       const int d = 4 * (lane + 32 * n);
       if (d >= vdim) continue;
-      const float value[4] = {v[n].x, v[n].y, v[n].z, v[n].w};
+      const float4 w = weight ? *reinterpret_cast<const float4*>(weight + d) : make_float4(1.f, 1.f, 1.f, 1.f);
+      const float value[4] = {v[n].x * w.x, v[n].y * w.y, v[n].z * w.z, v[n].w * w.w};
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float x = to_f(g[n][j]);
-        y[j] = from_f<T>(value[j] * inv * (x / (1.f + expf(-x))));
-      }
-      *reinterpret_cast<Word*>(out + size_t(row) * out_stride + size_t(head) * vdim + d) = *reinterpret_cast<const Word*>(y);
+      for (int j = 0; j < 4; ++j) y[j] = from_f<T>(value[j] * inv * opened(to_f(g[n][j])));
+      *reinterpret_cast<Word*>(out + d) = *reinterpret_cast<const Word*>(y);
     }
     return;
   }
   for (int d = lane; d < vdim; d += 32) sq = fmaf(o[d], o[d], sq);
-  const float inv = 1.f / sqrtf(warp_sum(sq) / float(vdim) + eps);
-  for (int d = lane; d < vdim; d += 32) {
-    const float g = to_f(gate[d]);
-    out[size_t(row) * out_stride + size_t(head) * vdim + d] = from_f<T>(o[d] * inv * (g / (1.f + expf(-g))));
-  }
+  const float inv = 1.f / sqrtf(warp_sum(sq) / float(vdim) + p.eps);
+  for (int d = lane; d < vdim; d += 32) out[d] = from_f<T>(o[d] * (weight ? weight[d] : 1.f) * inv * opened(to_f(gate[d])));
 }
 
 template <typename T> int RotateAppendAs(const Queue& q, const StepRows& r, const AttentionArgs& a) {
@@ -447,8 +471,9 @@ template <typename T> int AttendLatentAs(const Queue& q, const StepRows& r, cons
 }
 
 template <typename T> int AppendLatentAs(const Queue& q, const StepRows& r, const LatentArgs& a, bool portions_only) {
-  return int(Launch(append_latent<T>, dim3(unsigned(r.rows)), dim3(128), 0, q.stream, q.chained, r, static_cast<const T*>(a.raw), a.raw_stride,
-                    static_cast<T*>(a.pool), a.pool_dim, a.rank, a.norm, a.eps, portions_only));
+  const AppendLatentParams p{a.raw_stride, a.pool_dim, a.rank, a.norm, a.rotary, a.query_raw, a.query_norm, a.query, a.query_rank, a.query_stride, a.eps};
+  return int(Launch(append_latent<T>, dim3(unsigned(r.rows), a.query_raw ? 2u : 1u), dim3(128), 0, q.stream, q.chained, r, static_cast<const T*>(a.raw),
+                    static_cast<T*>(a.pool), p, portions_only));
 }
 
 template <typename T> int RetainAs(const Queue& q, const StepRows& r, const RetentionArgs& a, bool singles_only) {
@@ -472,11 +497,8 @@ template <typename T> int RetainTokenAs(const Queue& q, const StepRows& r, const
                     a.proj_stride, a.state, static_cast<T*>(a.out), a.out_stride, a.heads, a.dim, a.vdim, a.decay, a.key_scale, a.eps, a.rotary));
 }
 
-template <typename T> int GateAs(const Queue& q, const StepRows& r, const RetentionArgs& a) {
-  const unsigned blocks = unsigned((size_t(r.rows) * a.heads + 3) / 4);
-  return int(Launch(retention_gate<T>, dim3(blocks), dim3(128), 0, q.stream, q.chained, static_cast<const float*>(a.raw),
-                    static_cast<const T*>(a.proj), a.proj_stride, a.heads * (2 * a.dim + a.vdim), static_cast<T*>(a.out), a.out_stride,
-                    r.rows, a.heads, a.vdim, a.eps));
+int Gate(const Queue& q, const StepRows& r, const RetentionArgs& a) {
+  return HeadGate(q, {a.raw, a.proj, a.proj_stride, a.heads * (2 * a.dim + a.vdim), a.out, a.out_stride, r.rows, a.heads, a.vdim, nullptr, true, a.eps});
 }
 
 }  // namespace
@@ -491,7 +513,7 @@ int Attend(const Queue& q, const StepRows& r, const AttentionArgs& a) {
 }
 
 int AppendLatent(const Queue& q, const StepRows& r, const LatentArgs& a) {
-  if (q.f32 || !LatentTiled(a)) return q.f32 ? AppendLatentAs<float>(q, r, a, false) : AppendLatentAs<__nv_bfloat16>(q, r, a, false);
+  if (q.f32 || a.query_raw || !LatentTiled(a)) return q.f32 ? AppendLatentAs<float>(q, r, a, false) : AppendLatentAs<__nv_bfloat16>(q, r, a, false);
   return r.singles == r.entries ? 0 : AppendLatentAs<__nv_bfloat16>(q, r, a, true);
 }
 
@@ -500,19 +522,24 @@ int AttendLatent(const Queue& q, const StepRows& r, const LatentArgs& a) {
   return LatentTiled(a) ? AttendLatentTiles(q, r, a) : AttendLatentAs<__nv_bfloat16>(q, r, a);
 }
 
+int HeadGate(const Queue& q, const HeadGateArgs& a) {
+  const unsigned blocks = unsigned((size_t(a.rows) * a.heads + 3) / 4);
+  return int(Launch(q.f32 ? head_gate<float> : head_gate<__nv_bfloat16>, dim3(blocks), dim3(128), 0, q.stream, q.chained, a));
+}
+
 int Retain(const Queue& q, const StepRows& r, const RetentionArgs& a) {
   if (q.f32) {
     // a step of decoded tokens only takes the whole-token form; anything else the recurrence row by row
     if (r.singles == r.entries && TokenRows(a)) return RetainTokenAs<float>(q, r, a);
     const int status = RetainAs<float>(q, r, a, false);
-    return status != 0 ? status : GateAs<float>(q, r, a);
+    return status != 0 ? status : Gate(q, r, a);
   }
   // bf16: single tokens advance their states by the recurrence, portions by chunks
   const bool whole = TokenRows(a) != 0;
   int status = 0;
   if (r.singles < r.entries) status = RetainChunks(q, r, a);
   if (status == 0 && r.singles > 0 && !whole) status = RetainAs<__nv_bfloat16>(q, r, a, true);
-  if (status == 0 && (r.singles < r.entries || !whole)) status = GateAs<__nv_bfloat16>(q, r, a);
+  if (status == 0 && (r.singles < r.entries || !whole)) status = Gate(q, r, a);
   // (behind the gate of all rows, whose result for the single tokens it replaces)
   if (status == 0 && r.singles > 0 && whole) status = RetainTokenAs<__nv_bfloat16>(q, r, a);
   return status;

@@ -37,9 +37,10 @@ struct StepRows {
   int* row_kv = nullptr;                    // [rows] pool row: block * 16 + position mod 16
 };
 
-// Each of the `streams` copies of x[row] = embed[token] (and as an element in `copy`, rows of copy_stride, unless null); the row tables.
+// Each of the `streams` copies of x[row] = embed[token] * scale (and embed[token] as an element in `copy`, rows of copy_stride, unless null);
+// the row tables.
 int StartStep(const Queue& q, const StepRows& r, const int* tokens, const void* embed, float* x, int streams, void* copy, int copy_stride, int width,
-              int vocab);
+              int vocab, float scale);
 
 // out[i] = x[r] / sqrt(mean(x[r]^2) + eps) * weight, r = select ? select[i] : i. With `again`, x[r] += embed[token[r]]
 // first (and is written back). Rows of `out` are out_stride elements apart.
@@ -73,8 +74,8 @@ int AddNorm(const Queue& q, const AddNormArgs& a);
 //   update    x_t <- sum_s mix[s][t] x_s + out[t] y    (mix null: x_t itself, out null: 1), all t from the old streams
 //   collect   u = sum_t in[t] x_t (in null: 1), normed[i] = u / sqrt(mean(u^2) + eps) * weight, as elements
 // y = the weighted sum of `parts` elements rows, parts_of[i * parts + k] by part_scale[i * parts + k], plus branch[i] (fp32)
-// times sigmoid(branch_gate[i * gate_stride]) (null: 1); either may be absent. Without an update a row may be chosen:
-// r = select[i]. sum_of (or null): the streams' plain sum after the update.
+// times sigmoid(branch_gate[i * gate_stride]) (null: 1), the sum times `gain`; either may be absent. Without an update a row may be
+// chosen: r = select[i]. sum_of (or null): the streams' plain sum after the update. weight null: normed (or null) is u itself.
 struct StreamArgs {
   float* x;
   int streams, rows, width, limit;
@@ -85,14 +86,40 @@ struct StreamArgs {
   int parts;
   const float *branch, *branch_gate;
   int gate_stride;
+  float gain = 1.f;
   float* sum_of;
-  const float *in, *weight;  // weight null: no collect
+  const float *in, *weight;
   void* normed;
   int normed_stride;
   const int* select;
   float eps;
 };
 int StreamStep(const Queue& q, const StreamArgs& a);
+
+// The row operation in front of a layer whose mixer reads its norm through a short convolution over time:
+//   x'   = x + gain * side / sqrt(mean(side^2) + eps) * side_weight      (side null: x), written to x_out (or null; not x itself)
+//   h    = x' in `groups` runs of columns, each over its own root mean square, times weight; as elements in normed
+//   read = h + sum_j taps[j] h at position p - (count - 1) + j, as elements in convolved (count 0: none)
+// The h of the last count - 1 positions of a sequence lie in history [slots][count - 1][width], position p in row p mod
+// (count - 1); positions before the first count as zeros. With `select` (and no convolution) row i is row select[i] of x.
+struct ConvNormArgs {
+  const float* x;
+  const float* side;
+  const float* side_weight;
+  float* x_out;
+  float gain, eps;
+  const float* weight;
+  int groups, rows, width, limit;
+  void* normed;
+  int stride;                // of normed and convolved
+  const float* taps;         // [count][width]
+  int count;
+  float* history;
+  void* convolved;
+  const int* select;
+};
+int ConvNorm(const Queue& q, const StepRows& r, const ConvNormArgs& a);
+int PrepareConv();
 
 // Rotary table [capacity][dims / 2] of (cos, sin), or dims = 0: none.
 struct Rotary {
@@ -108,7 +135,21 @@ struct Glu {
 };
 
 enum LinearEpilogue { kLinearStore = 0, kLinearAdd = 1, kLinearGlu = 2, kLinearFloat = 3, kLinearExpertUp = 4, kLinearExpertDown = 5,
-                      kLinearHeads = 6, kLinearExpertGlu = 7, kLinearExpertStore = 8 };
+                      kLinearHeads = 6, kLinearExpertGlu = 7, kLinearExpertStore = 8, kLinearRotate = 9, kLinearSide = 10 };
+
+// kLinearRotate: output columns are heads of head_out, and in each the columns rotary.dims behind `lead` turn, neighbours 2i and
+// 2i + 1 by the row's position's angle i.
+struct RotateHeads {
+  Rotary rotary;
+  const int* positions = nullptr;   // [rows]
+  int lead = 0, head = 0;           // a head's columns: head
+};
+// kLinearSide: y = gelu(D) * part[token of the row], the tanh form; part rows of `stride` elements.
+struct SideGate {
+  const void* part = nullptr;
+  const int* tokens = nullptr;      // [rows]
+  int stride = 0, vocab = 0;
+};
 
 // The assignments of a step's rows to experts, sorted by expert (written by Route). Assignment a is the a % top-th choice
 // of row a / top; slot s, in sorted order, runs assignment list[s] on the expert of its tile.
@@ -130,6 +171,7 @@ struct ExpertSlots {
 // (from `activations`; bf16 tiles of more than kGatherRows slots read row s of rows gathered before, see GatherRows) and
 // stores relu(score[s] D)^2 in row s; ExpertGlu reads the same and stores the gated unit, ExpertStore (fp32) D itself;
 // ExpertDown reads row s and stores D in row list[s]; all as elements.
+// Rotate and Side store elements as their structs say. Store: columns below tanh_below as their hyperbolic tangent.
 // Heads: `heads` products side by side, head h of weight rows h * n ..., activation columns h * head_in ... and output
 // columns h * head_out ... (head_in a multiple of 8; n and k are one head's), stored as elements.
 constexpr int kGatherRows = 32;
@@ -149,7 +191,11 @@ struct LinearArgs {
   int in_stride;             // elements of an activation row, if it is not k_stride (0)
   int heads, head_in, head_out;   // kLinearHeads
   int outputs;               // kLinearGlu: columns stored (pairs beyond it are padding)
+  int tanh_below;            // kLinearStore
+  float gain = 1.f;          // kLinearFloat: factor of what is stored
   int epilogue;
+  RotateHeads rotate;
+  SideGate side;
   Glu glu;
   ExpertSlots slots;         // expert epilogues
 };
@@ -164,7 +210,8 @@ int Linear(const Queue& q, const LinearArgs& a);
 int GluRows(const Queue& q, const void* in, void* out, int t, int in_stride, int out_stride, int outputs, const Glu& glu);
 
 // Mixture of experts: per row z = router h, scores sigmoid(z) or softmax(z) over the experts, and the `top` largest of score
-// + correction (null: 0; the smaller index on a tie) among the keep_groups groups of neighbours whose largest is largest.
+// + correction (null: 0; the smaller index on a tie) among the keep_groups groups of neighbours whose largest is largest. `chosen`: ranked
+// by z, scores are a softmax over the chosen experts' z alone.
 // `weights`: the scores handed on are over their sum (+ 1e-20). `extra` more router rows are only multiplied. And the
 // assignments sorted by expert in tiles of slots->tile_rows. RouteFused: does Route compute z itself? (If not, the
 // caller has put it into `logits`.)
@@ -173,7 +220,7 @@ struct RouteArgs {
   const void* router;        // [experts][k_stride]
   int k_stride, rows, experts, top, tile_rows;
   int extra;
-  bool softmax, weights;
+  bool softmax, weights, chosen;
   const float* correction;
   int groups, keep_groups;
   float* ranks;              // [rows][experts], scratch (softmax scores, corrections or groups)
@@ -245,7 +292,12 @@ struct LatentArgs {
   const float* norm;         // [rank]
   void* pool;                // [num_blocks][16][pool_dim]
   const CUtensorMap *pool_map, *q_map;   // bf16, tiled form: see EncodeLatent, EncodeLookup
-  int heads, rank, rank_stride, pool_dim;
+  int heads, rank, rank_stride, pool_dim;   // rank: columns of a row, the rotated ones included
+  Rotary rotary;             // the last rotary.dims columns of a row turn, neighbours together, in place of being normed
+  const void* query_raw;     // rows of raw_stride beside `raw` that AppendLatent norms into query (null: none; then the heads' queries are images
+  const float* query_norm;   // of these, and AppendLatent takes every row)
+  void* query;               // [rows][query_stride]
+  int query_rank, query_stride;
   float eps, scale, sink;
   const float* sinks;        // [heads], or null
   int window;
@@ -256,7 +308,7 @@ struct LatentArgs {
 // (bf16 rows that suit the tiled form: AppendLatent takes portions only, a decoded token's attention appends its own row.)
 int AppendLatent(const Queue& q, const StepRows& r, const LatentArgs& a);
 int AttendLatent(const Queue& q, const StepRows& r, const LatentArgs& a);
-constexpr int kTiledLatent = 512;   // widest latent row of the tiled form
+constexpr int kTiledLatent = 640;   // widest latent row of the tiled form
 inline bool LatentTiled(const LatentArgs& a) { return a.rank <= kTiledLatent; }
 int AttendLatentTiles(const Queue& q, const StepRows& r, const LatentArgs& a);   // the tiled form
 int PrepareLatent();
@@ -285,6 +337,39 @@ struct RetentionArgs {
 // The mixer's output in a.out: o / rms(o) per head, times silu(g).
 int Retain(const Queue& q, const StepRows& r, const RetentionArgs& a);
 int RetainChunks(const Queue& q, const StepRows& r, const RetentionArgs& a);  // the bf16 form of entries of several rows
+
+// out = o / rms(o) of every head, times weight (null: 1), times the gate's sigmoid, or (silu) the gate times its sigmoid. o fp32
+// [rows][heads * vdim], gates at column gate_at of rows of `proj`.
+struct HeadGateArgs {
+  const float* raw;
+  const void* proj;
+  int proj_stride, gate_at;
+  void* out;
+  int out_stride, rows, heads, vdim;
+  const float* weight;       // [heads * vdim]
+  bool silu;
+  float eps;
+};
+int HeadGate(const Queue& q, const HeadGateArgs& a);
+
+// Generalised delta rule with a decay and a removal rate per head and key channel:
+//   u = k / sqrt(k^2 + unit_eps), w = exp(-decay_scale sigmoid(z)), S <- diag(w) S - (sigmoid(a) u) (u^T S) + k v^T, o = S^T r
+// proj rows hold r | k | v | a | g, heads x dim each; z fp32 [rows][heads * dim]. state [slots][heads][dim: value columns][padded dim: key
+// channels] fp32; an entry that starts at position 0 starts from a zero state. Out: o / rms(o) per head, times norm, times sigmoid(g).
+struct DeltaArgs {
+  const void* proj;
+  int proj_stride;
+  const float* z;
+  float* state;
+  float* raw;                // [rows][heads * dim]
+  void* out;
+  int out_stride;
+  int heads, dim, padded;
+  const float* norm;         // [heads * dim]
+  float decay_scale, unit_eps, eps;
+};
+int Delta(const Queue& q, const StepRows& r, const DeltaArgs& a);
+int PrepareDelta();
 
 // next[i] = index of the largest of logits[i][0..vocab), the smallest such index on a tie.
 int ArgMax(const Queue& q, const float* logits, int rows, int vocab, int* next);

@@ -28,7 +28,14 @@ struct RaggedPlan {
   void *lookup = nullptr, *looked = nullptr;   // latent attention: queries against latent rows, weighted sums of latent rows
   void* mlp = nullptr;         // [max_rows][widest feed-forward]
   void* pairs = nullptr;       // fp32 plans: gate/up rows before the gated unit
-  float* branch = nullptr;     // fp32 outputs of sublayers that are normed before they are added
+  float* branch = nullptr;     // fp32 outputs of sublayers that are normed, or summed, before they are added
+  // parallel layers: the stream's other place (rows are formed anew next to rows that still read the old ones), the stream and the
+  // convolved norm as elements, the side input's hidden rows and output
+  float* other = nullptr;
+  void *elements = nullptr, *convolved = nullptr, *side_hidden = nullptr;
+  float* side_out = nullptr;
+  void *query_latent = nullptr, *queries = nullptr;   // latent attention: normed rows that queries are images of, and these
+  float* decay_in = nullptr;   // delta rule: what decays are made of, [max_rows][heads * dim]
   // bf16 plans with latent attention: the latent rows that portions see, gathered, and their keys and values
   void *context = nullptr, *expanded = nullptr;
   int *context_at = nullptr, *context_count = nullptr;
@@ -53,7 +60,7 @@ struct RaggedPlan {
   std::vector<float*> decay;   // per layer
   struct Maps {
     LinearMaps in, out, gate_up, down, router;   // (gate_up, down: of the gated unit or of the experts)
-    LinearMaps shared_up, shared_down, key_up, value_up, expand;
+    LinearMaps shared_up, shared_down, key_up, value_up, expand, query_up, decay_up, side_gate, side_proj;
     CUtensorMap lookup;
   };
   std::vector<Maps> maps;      // per layer (bf16 plans)
@@ -80,10 +87,10 @@ template <typename T> bool Own(RaggedPlan* plan, T** out, size_t bytes) {
 int ContextRows(const RaggedPlan* plan, const StepRows& r, const RaggedMixer& m) {
   const int portions = r.entries - r.singles, rows = r.rows - r.singles;
   if (!plan->context_rows || portions == 0) return 0;
-  const double reach = std::min(m.window, r.capacity), each = double(rows) / portions, head = m.dim + m.vdim;
+  const double reach = std::min(m.window, r.capacity), each = double(rows) / portions, head = m.head_key() + m.vdim;
   const double most = rows + portions * (reach - 1);
   if (most > plan->context_rows) return 0;
-  return each * reach * (2.0 * m.rank - head) > (each + reach) * m.rank * head / 3.0 ? int(most) : 0;
+  return each * reach * (2.0 * m.columns() - head) > (each + reach) * m.columns() * head / 3.0 ? int(most) : 0;
 }
 
 int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest, uint32_t singles, uint32_t wanted, bool feed, cudaStream_t stream) {
@@ -106,7 +113,7 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     if (status_ != 0) return status_; \
   } while (0)
   const bool norm_output = s.layers[0].norm_output;   // sublayers then read the stream itself: `normed` holds it as elements
-  TMB_TRY(StartStep(q, r, tokens, buffer(s.embed), x, s.streams, norm_output ? plan->normed : nullptr, W8, W, s.vocab));
+  TMB_TRY(StartStep(q, r, tokens, buffer(s.embed), x, s.streams, norm_output ? plan->normed : nullptr, W8, W, s.vocab, float(s.embed_scale)));
   auto norm = [&](int weight, bool again) {
     NormArgs a{};
     a.x = x;
@@ -138,7 +145,7 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
   };
   // a sublayer's last product (rows of `in` times `weight`): added to the stream, or normed and added
   auto add_output = [&](const void* in, int weight, int bias, const LinearMaps* maps, int k) {
-    if (!norm_output && !s.combined) return Linear(q, linear(in, weight, bias, maps, W, k, x, W, kLinearAdd));
+    if (!norm_output && !s.combined && !s.parallel) return Linear(q, linear(in, weight, bias, maps, W, k, x, W, kLinearAdd));
     return Linear(q, linear(in, weight, bias, maps, W, k, plan->branch, W, kLinearFloat));
   };
   auto add_norm = [&](int weight, int parts) {
@@ -184,6 +191,8 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     if (next) {
       a.in = floats(next->in);
       a.weight = floats(norm_weight);
+    } else {
+      a.normed = nullptr;
     }
     a.sum_of = sum_of;
     return StreamStep(q, a);
@@ -192,6 +201,75 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     const RaggedLayer& first = s.layers[size_t(s.runs[0].layer)];
     TMB_TRY(restream(nullptr, nullptr, &first.streams[0], first.norm1, nullptr));
   }
+  // Parallel layers. In front of a layer: the side input of the layer before added, the grouped norm, the convolution. Behind it: both
+  // sublayers' outputs added at once, and the side input's products.
+  bool side_waits = false;
+  const RaggedSide* side = nullptr;
+  auto conv_norm = [&](int weight, const RaggedLayer* layer, const RaggedRun* run, const int* select, int count, void* normed) {
+    ConvNormArgs a{};
+    a.x = x;
+    if (side_waits) {
+      a.side = plan->side_out;
+      a.side_weight = floats(side->norm);
+      a.gain = float(s.residual_mult);
+    }
+    if (side_waits && !select) {
+      a.x_out = x == floats(s.hidden) ? plan->other : floats(s.hidden);
+      x = a.x_out;
+      side_waits = false;
+    }
+    a.eps = float(s.eps);
+    a.weight = floats(weight);
+    a.groups = s.norm_groups;
+    a.rows = count;
+    a.limit = r.rows;
+    a.width = W;
+    a.normed = normed;
+    a.stride = W8;
+    if (layer) {
+      a.taps = floats(layer->conv);
+      a.count = s.taps;
+      a.history = floats(run->history);
+      a.convolved = plan->convolved;
+    }
+    a.select = select;
+    return ConvNorm(q, r, a);
+  };
+  auto add_sublayers = [&](const RaggedLayer& layer, const RaggedPlan::Maps* maps) {
+    StreamArgs a{};
+    a.x = x;
+    a.streams = 1;
+    a.rows = a.limit = r.rows;
+    a.width = W;
+    a.update = true;
+    a.branch = plan->branch;
+    a.gain = float(s.residual_mult);
+    if (layer.mlp.kind == RaggedMlp::kExperts) {
+      a.parts_of = plan->expert_out;
+      a.part_scale = plan->score;
+      a.parts = layer.mlp.top;
+    }
+    if (s.side_dim) {
+      a.normed = plan->elements;
+      a.normed_stride = W8;
+    }
+    TMB_TRY(StreamStep(q, a));
+    if (!s.side_dim) return 0;
+    const int stride = padded_columns(s.side_dim);
+    LinearArgs gate = linear(plan->elements, layer.side.gate, -1, maps ? &maps->side_gate : nullptr, s.side_dim, W, plan->side_hidden, stride, kLinearSide);
+    gate.side.part = static_cast<const char*>(buffer(s.side_embed)) + size_t(layer.side.from) * (s.f32 ? 4 : 2);
+    gate.side.tokens = tokens;
+    gate.side.stride = s.side_columns;
+    gate.side.vocab = s.vocab;
+    TMB_TRY(Linear(q, gate));
+    TMB_TRY(Linear(q, linear(plan->side_hidden, layer.side.proj, -1, maps ? &maps->side_proj : nullptr, W, s.side_dim, plan->side_out, W, kLinearFloat)));
+    side = &layer.side;
+    side_waits = true;
+    return 0;
+  };
+  auto keep_stream = [&](size_t run) {       // (plans that write residuals)
+    return int(cudaMemcpyAsync(floats(s.residuals) + run * size_t(s.max_rows) * W, x, size_t(rows) * W * sizeof(float), cudaMemcpyDeviceToDevice, stream));
+  };
   int context_window = -1;               // the window that the table of expanded rows is for
   for (size_t i = 0; i < s.runs.size(); ++i) {
     const RaggedRun& run = s.runs[i];
@@ -201,9 +279,16 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     const RaggedMixer& m = layer.mixer;
     const RaggedPlan::Maps* maps = s.f32 ? nullptr : &plan->maps[size_t(run.layer)];
     const int stride = (m.proj_rows() + 7) / 8 * 8, mixed_stride = padded_columns(m.out_columns());
-    if (!norm_output && !s.combined) TMB_TRY(norm(layer.norm1, run.add_embedding));
+    if (s.parallel) {
+      TMB_TRY(conv_norm(layer.norm1, s.taps ? &layer : nullptr, &run, nullptr, r.rows, plan->normed));
+      if (s.write_residuals && i > 0) TMB_TRY(keep_stream(i - 1));
+    } else if (!norm_output && !s.combined) {
+      TMB_TRY(norm(layer.norm1, run.add_embedding));
+    }
     void* proj = m.value_mix == RaggedMixer::kSource ? plan->source : plan->proj;
-    TMB_TRY(Linear(q, linear(plan->normed, layer.in_weight, layer.in_bias, maps ? &maps->in : nullptr, m.proj_rows(), W, proj, stride, kLinearStore)));
+    LinearArgs in = linear(s.taps ? plan->convolved : plan->normed, layer.in_weight, layer.in_bias, maps ? &maps->in : nullptr, m.proj_rows(), W, proj, stride, kLinearStore);
+    if (m.kind == RaggedMixer::kDelta) in.tanh_below = m.decay_rank;
+    TMB_TRY(Linear(q, in));
     Rotary rotary;
     if (m.rotary >= 0) {
       rotary.table = static_cast<const float2*>(buffer(s.rotaries[size_t(m.rotary)].buffer));
@@ -227,18 +312,47 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.eps = float(s.eps);
       a.rotary = rotary;
       TMB_TRY(Retain(q, r, a));
+    } else if (m.kind == RaggedMixer::kDelta) {
+      const int all = m.heads * m.dim;
+      LinearArgs up = linear(proj, layer.decay_up, layer.decay_bias, maps ? &maps->decay_up : nullptr, all, m.decay_rank, plan->decay_in, all, kLinearFloat);
+      up.in_stride = stride;
+      TMB_TRY(Linear(q, up));
+      DeltaArgs a{};
+      a.proj = static_cast<const char*>(proj) + size_t(m.delta_at()) * (s.f32 ? 4 : 2);
+      a.proj_stride = stride;
+      a.z = plan->decay_in;
+      a.state = floats(run.state);
+      a.raw = plan->raw;
+      a.out = plan->mixed;
+      a.out_stride = mixed_stride;
+      a.heads = m.heads;
+      a.dim = m.dim;
+      a.padded = m.state_dim();
+      a.norm = floats(layer.out_norm);
+      a.decay_scale = float(m.decay_scale);
+      a.unit_eps = float(m.unit_eps);
+      a.eps = float(s.eps);
+      TMB_TRY(Delta(q, r, a));
     } else if (m.kind == RaggedMixer::kLatent) {
       LatentArgs a{};
       a.q = plan->lookup;
       a.out = plan->looked;
-      a.raw = static_cast<const char*>(proj) + size_t(m.heads) * m.head_stride() * (s.f32 ? 4 : 2);
+      a.raw = static_cast<const char*>(proj) + size_t(m.latent_at()) * (s.f32 ? 4 : 2);
       a.raw_stride = stride;
       a.norm = floats(layer.latent_norm);
       a.pool = buffer(run.k_pool);
       a.pool_map = maps ? &plan->latent[i] : nullptr;
       a.q_map = maps ? &maps->lookup : nullptr;
       a.heads = m.heads;
-      a.rank = m.rank;
+      a.rank = m.columns();
+      a.rotary = rotary;
+      if (m.q_rank) {
+        a.query_raw = proj;
+        a.query_norm = floats(layer.q_latent_norm);
+        a.query = plan->query_latent;
+        a.query_rank = m.q_rank;
+        a.query_stride = padded_columns(m.q_rank);
+      }
       a.rank_stride = m.rank_stride();
       a.pool_dim = m.pool_dim();
       a.eps = float(s.eps);
@@ -250,17 +364,30 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.part_floats = plan->part_floats;
       const int wide = m.heads * m.rank_stride();
       TMB_TRY(AppendLatent(q, r, a));
+      const void* heads = proj;            // the heads' queries
+      int heads_stride = stride;
+      if (m.q_rank) {
+        heads = plan->queries;
+        heads_stride = m.heads * m.head_stride();
+        LinearArgs up = linear(plan->query_latent, layer.query_up, -1, maps ? &maps->query_up : nullptr, heads_stride, m.q_rank, plan->queries, heads_stride,
+                               m.rot_dims ? kLinearRotate : kLinearStore);
+        up.rotate.rotary = rotary;
+        up.rotate.positions = r.row_position;
+        up.rotate.lead = m.head_lead();
+        up.rotate.head = m.head_stride();
+        TMB_TRY(Linear(q, up));
+      }
       const int context = ContextRows(plan, r, m);
       a.singles_only = context > 0;
       if (!context || r.singles) {
-        LinearArgs up = linear(proj, layer.key_up, -1, maps ? &maps->key_up : nullptr, m.rank_stride(), m.head_stride(), plan->lookup, wide, kLinearHeads);
-        up.in_stride = stride;
+        LinearArgs up = linear(heads, layer.key_up, -1, maps ? &maps->key_up : nullptr, m.rank_stride(), m.head_stride(), plan->lookup, wide, kLinearHeads);
+        up.in_stride = heads_stride;
         up.heads = m.heads;
         up.head_in = m.head_stride();
         up.head_out = m.rank_stride();
         TMB_TRY(Linear(q, up));
         TMB_TRY(AttendLatent(q, r, a));
-        LinearArgs down = linear(plan->looked, layer.value_up, -1, maps ? &maps->value_up : nullptr, m.vdim, m.rank, plan->mixed, mixed_stride, kLinearHeads);
+        LinearArgs down = linear(plan->looked, layer.value_up, -1, maps ? &maps->value_up : nullptr, m.vdim, m.rank_stride(), plan->mixed, mixed_stride, kLinearHeads);
         down.in_stride = wide;
         down.heads = m.heads;
         down.head_in = m.rank_stride();
@@ -272,19 +399,19 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
         context_window = m.window;
         TMB_TRY(GatherLatent(q, r, a, plan->context_at, plan->context_count, context, plan->context));
         const int columns = m.expanded_columns();
-        LinearArgs expand = linear(plan->context, layer.expand, -1, &maps->expand, columns, m.rank, plan->expanded, columns, kLinearStore);
+        LinearArgs expand = linear(plan->context, layer.expand, -1, &maps->expand, columns, m.rank_stride(), plan->expanded, columns, kLinearStore);
         expand.t = context;
         expand.rows_there = plan->context_count;
         TMB_TRY(Linear(q, expand));
         AttentionArgs seen{};
-        seen.proj = proj;
-        seen.proj_stride = stride;
+        seen.proj = const_cast<void*>(heads);
+        seen.proj_stride = heads_stride;
         seen.k_pool = plan->expanded;
         seen.v_pool = static_cast<char*>(plan->expanded) + size_t(m.heads) * m.expanded_key() * 2;
         seen.out = plan->mixed;
         seen.out_stride = mixed_stride;
         seen.heads = seen.kv_heads = m.heads;
-        seen.dim = m.dim;
+        seen.dim = m.head_key();
         seen.vdim = m.vdim;
         seen.pool_dim = m.expanded_key();
         seen.v_pool_dim = m.v_pool_dim();
@@ -342,7 +469,7 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     if (mlp.kind == RaggedMlp::kGlu) {
       const Glu glu{float(mlp.limit), float(mlp.alpha), float(mlp.shift), mlp.gelu};
       const int packed = mlp.packed_rows(), mlp_stride = padded_columns(mlp.ff);
-      if (!norm_output && !s.combined) TMB_TRY(norm(layer.norm2, false));
+      if (!norm_output && !s.combined && !s.parallel) TMB_TRY(norm(layer.norm2, false));
       if (s.f32) {
         TMB_TRY(Linear(q, linear(plan->normed, layer.gate_up, -1, nullptr, packed, W, plan->pairs, packed, kLinearStore)));
         TMB_TRY(GluRows(q, plan->pairs, plan->mlp, r.rows, packed, mlp_stride, mlp.ff, glu));
@@ -352,7 +479,8 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
         a.glu = glu;
         TMB_TRY(Linear(q, a));
       }
-      TMB_TRY(add_output(plan->mlp, layer.down, -1, maps ? &maps->down : nullptr, mlp.ff));
+      if (s.parallel) TMB_TRY(Linear(q, linear(plan->mlp, layer.down, -1, maps ? &maps->down : nullptr, W, mlp.ff, plan->branch, W, kLinearAdd)));
+      else TMB_TRY(add_output(plan->mlp, layer.down, -1, maps ? &maps->down : nullptr, mlp.ff));
       if (norm_output) TMB_TRY(add_norm(layer.norm2, 0));
       if (s.combined) TMB_TRY(leave(&layer.streams[1], nullptr));
     } else if (mlp.kind == RaggedMlp::kExperts) {
@@ -379,7 +507,8 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.correction = floats(layer.correction);
       a.groups = mlp.groups;
       a.keep_groups = mlp.keep_groups;
-      a.ranks = mlp.output_weighted ? plan->ranks : nullptr;
+      a.chosen = mlp.chosen;
+      a.ranks = mlp.output_weighted && !mlp.chosen ? plan->ranks : nullptr;
       a.logits = plan->logits;
       a.choice = plan->choice;
       a.score = plan->score;
@@ -425,15 +554,23 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       }
       if (s.combined) TMB_TRY(leave(&layer.streams[1], &mlp));
     }
-    if (kept && !s.combined) {
+    if (s.parallel) {
+      TMB_TRY(add_sublayers(layer, maps));
+    } else if (kept && !s.combined) {
       const cudaError_t err = cudaMemcpyAsync(kept, x, size_t(rows) * W * sizeof(float),
                                               cudaMemcpyDeviceToDevice, stream);
       if (err != cudaSuccess) return int(err);
     }
   }
+  if (s.parallel && s.write_residuals) {       // (the norm is not read)
+    TMB_TRY(conv_norm(s.final_norm, nullptr, nullptr, nullptr, r.rows, plan->normed));
+    TMB_TRY(keep_stream(s.runs.size() - 1));
+  }
   if (wanted) {
     const int* select = static_cast<const int*>(buffer(s.wanted));
-    if (s.combined) {
+    if (s.parallel) {
+      TMB_TRY(conv_norm(s.final_norm, nullptr, nullptr, select, int(wanted), plan->picked));
+    } else if (s.combined) {
       StreamArgs a = step;
       a.rows = int(wanted);
       a.weight = floats(s.final_norm);
@@ -455,6 +592,7 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
     }
     LinearArgs h = linear(plan->picked, s.head, -1, s.f32 ? nullptr : &plan->head, s.vocab, W, buffer(s.logits), s.vocab, kLinearFloat);
     h.t = int(wanted);
+    h.gain = float(s.logit_scale);
     TMB_TRY(Linear(q, h));
     TMB_TRY(ArgMax(q, floats(s.logits), int(wanted), s.vocab, static_cast<int*>(buffer(s.next))));
     if (feed)
@@ -477,7 +615,7 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
     return nullptr;
   };
   const size_t element = spec.f32 ? 4 : 2;
-  size_t proj = 0, mixed = 0, mlp = 0, pairs = 0, raw = 0, split = 0, heads = 1, partial = 0;
+  size_t proj = 0, mixed = 0, mlp = 0, pairs = 0, raw = 0, split = 0, heads = 1, partial = 0, query_latent = 0, queries = 0, decays = 0;
   size_t top = 0, experts = 0, expert_columns = 0, expert_pairs = 0, source = 0, latent = 0, ranks = 0, context = 0, expanded = 0;
   int reach = 0;
   for (const RaggedLayer& layer : spec.layers) {
@@ -508,6 +646,9 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
     if (m.kind == RaggedMixer::kRetention) {
       raw = std::max(raw, size_t(m.out_columns()));
       split = std::max(split, size_t(m.heads) * 4 * m.pool_dim());
+    } else if (m.kind == RaggedMixer::kDelta) {
+      raw = std::max(raw, size_t(m.out_columns()));
+      decays = std::max(decays, size_t(m.out_columns()));
     } else {
       const size_t columns = m.kind == RaggedMixer::kLatent ? size_t(m.rank_stride()) : size_t(m.vdim);
       heads = std::max(heads, size_t(m.heads));
@@ -515,6 +656,10 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
       partial = std::max(partial, size_t(m.heads) * (columns + 2) / (m.kind == RaggedMixer::kLatent ? 4 : 1));
       if (m.kind == RaggedMixer::kLatent) {
         latent = std::max(latent, size_t(m.heads) * m.rank_stride());
+        if (m.q_rank) {
+          query_latent = std::max(query_latent, size_t(padded_columns(m.q_rank)));
+          queries = std::max(queries, size_t(m.heads) * m.head_stride());
+        }
         context = std::max(context, size_t(m.rank_stride()));
         expanded = std::max(expanded, size_t(m.expanded_columns()));
         reach = std::max(reach, std::min(m.window, spec.capacity));
@@ -530,7 +675,13 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
   if (!Own(plan, &plan->normed, rows * W8 * element) || !Own(plan, &plan->picked, size_t(spec.max_wanted) * W8 * element) ||
       !Own(plan, &plan->proj, rows * proj * element) || !Own(plan, &plan->mixed, rows * mixed * element) ||
       !Own(plan, &plan->mlp, rows * mlp * element) || !Own(plan, &plan->pairs, spec.f32 ? rows * pairs * element : 0) ||
-      !Own(plan, &plan->branch, spec.layers[0].norm_output || spec.combined ? rows * size_t(spec.width) * sizeof(float) : 0) ||
+      !Own(plan, &plan->branch, spec.layers[0].norm_output || spec.combined || spec.parallel ? rows * size_t(spec.width) * sizeof(float) : 0) ||
+      !Own(plan, &plan->other, spec.side_dim ? rows * size_t(spec.width) * sizeof(float) : 0) || !Own(plan, &plan->elements, spec.side_dim ? rows * W8 * element : 0) ||
+      !Own(plan, &plan->convolved, spec.taps ? rows * W8 * element : 0) ||
+      !Own(plan, &plan->side_hidden, spec.side_dim ? rows * size_t(padded_columns(spec.side_dim)) * element : 0) ||
+      !Own(plan, &plan->side_out, spec.side_dim ? rows * size_t(spec.width) * sizeof(float) : 0) ||
+      !Own(plan, &plan->query_latent, rows * query_latent * element) || !Own(plan, &plan->queries, rows * queries * element) ||
+      !Own(plan, &plan->decay_in, rows * decays * sizeof(float)) ||
       !Own(plan, &plan->context, context_rows * context * element) || !Own(plan, &plan->expanded, context_rows * expanded * element) ||
       !Own(plan, &plan->context_at, size_t(spec.slots) * sizeof(int)) || !Own(plan, &plan->context_count, sizeof(int)) ||
       !Own(plan, &plan->source, rows * source * element) || !Own(plan, &plan->lookup, rows * latent * element) ||
@@ -576,16 +727,24 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
       const RaggedLayer& layer = spec.layers[i];
       const RaggedMixer& m = layer.mixer;
       RaggedPlan::Maps& maps = plan->maps[i];
-      bool ok = EncodeLinear(&maps.in, at(layer.in_weight), uint64_t(m.proj_rows()), plan->normed, rows, W8) &&
+      bool ok = EncodeLinear(&maps.in, at(layer.in_weight), uint64_t(m.proj_rows()), spec.taps ? plan->convolved : plan->normed, rows, W8) &&
                 EncodeLinear(&maps.out, at(layer.out_weight), uint64_t(spec.width), plan->mixed, rows, uint64_t(padded_columns(m.out_columns())));
       const RaggedMlp& mlp = layer.mlp;
       if (m.kind == RaggedMixer::kLatent)
         ok = ok && EncodeLookup(&maps.lookup, plan->lookup, rows * m.heads, uint64_t(m.rank_stride())) &&
-             EncodeHeads(&maps.key_up, at(layer.key_up), uint64_t(m.heads) * m.rank_stride(), uint64_t(m.head_stride()), plan->proj, rows,
-                               size_t(m.proj_rows() + 7) / 8 * 8) &&
+             EncodeHeads(&maps.key_up, at(layer.key_up), uint64_t(m.heads) * m.rank_stride(), uint64_t(m.head_stride()),
+                         m.q_rank ? plan->queries : plan->proj, rows, m.q_rank ? uint64_t(m.heads) * m.head_stride() : uint64_t(m.proj_rows() + 7) / 8 * 8) &&
              EncodeHeads(&maps.value_up, at(layer.value_up), uint64_t(m.heads) * m.vdim, uint64_t(m.rank_stride()), plan->looked, rows,
                          uint64_t(m.heads) * m.rank_stride()) &&
              EncodeLinear(&maps.expand, at(layer.expand), uint64_t(m.expanded_columns()), plan->context, context_rows, uint64_t(m.rank_stride()));
+      if (m.q_rank)
+        ok = ok && EncodeLinear(&maps.query_up, at(layer.query_up), uint64_t(m.heads) * m.head_stride(), plan->query_latent, rows, uint64_t(padded_columns(m.q_rank)));
+      if (m.kind == RaggedMixer::kDelta)
+        ok = ok && EncodeHeads(&maps.decay_up, at(layer.decay_up), uint64_t(m.out_columns()), uint64_t(padded_columns(m.decay_rank)), plan->proj, rows,
+                               uint64_t(m.proj_rows() + 7) / 8 * 8);
+      if (spec.side_dim)
+        ok = ok && EncodeLinear(&maps.side_gate, at(layer.side.gate), uint64_t(spec.side_dim), plan->elements, rows, W8) &&
+             EncodeLinear(&maps.side_proj, at(layer.side.proj), uint64_t(spec.width), plan->side_hidden, rows, uint64_t(padded_columns(spec.side_dim)));
       if (mlp.kind == RaggedMlp::kExperts)
         ok = ok && EncodeLinear(&maps.router, at(layer.router), uint64_t(mlp.logits()), plan->normed, rows, W8) &&
              EncodeLinear(&maps.gate_up, at(layer.expert_up), uint64_t(mlp.experts) * (mlp.output_weighted ? mlp.packed_rows() : mlp.ff), plan->gathered,
@@ -611,7 +770,7 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
     if (!EncodeLinear(&plan->head, at(spec.head), uint64_t(spec.vocab), plan->picked, uint64_t(spec.max_wanted), W8))
       return fail("cuTensorMapEncodeTiled rejected the head");
   }
-  if (PrepareLinear() != 0 || PrepareMixers() != 0 || PrepareLatent() != 0) return fail("cannot raise the kernels' shared-memory limit");
+  if (PrepareLinear() != 0 || PrepareMixers() != 0 || PrepareLatent() != 0 || PrepareConv() != 0 || PrepareDelta() != 0) return fail("cannot raise the kernels' shared-memory limit");
   return plan;
 }
 

@@ -7,6 +7,8 @@ constexpr int kGluUnit = 16;          // a packed gate/up matrix alternates this
 constexpr int kMaxHeadDim = 256;      // query/key (and attention value) columns of a head
 constexpr int kMaxLatent = 1024;      // columns of a cached latent row
 constexpr int kMaxStreams = 16;       // residual streams
+constexpr int kMaxTaps = 16;          // of a short convolution
+constexpr int kMaxConvWidth = 8192;   // residual columns of models with grouped norms, short convolutions or side inputs
 constexpr int kRaggedBlock = 16;      // positions per KV pool block
 constexpr int kMaxExperts = 1024;     // of a layer
 constexpr int kMaxTop = 32;           // experts a token uses

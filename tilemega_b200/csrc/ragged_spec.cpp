@@ -54,6 +54,18 @@ std::string GluRecipe(const std::string& gate, const std::string& up) {
   return "{\"kind\":\"gate_up_interleave\",\"pad\":true,\"u\":" + std::to_string(kGluUnit) + ",\"sources\":[" + gate + "," + up + "]}";
 }
 
+// Every head's matrix with an identity of `size` behind its rows and columns.
+std::string WithIdentity(const std::string& recipe, int heads, int size) { return size ? PerHead("append_identity", recipe, heads, "size", size) : recipe; }
+// Heads whose last `dims` rows are rotated: these as neighbours behind `lead` rows for the others, zero rows up to `rows`.
+std::string RotaryTail(const std::string& recipe, int heads, int dims, bool neighbours, int lead, int rows) {
+  return "{\"kind\":\"rotary_tail\",\"heads\":" + std::to_string(heads) + ",\"dims\":" + std::to_string(dims) + ",\"layout\":\"" +
+         (neighbours ? "pairs" : "halves") + "\",\"lead\":" + std::to_string(lead) + ",\"rows\":" + std::to_string(rows) + ",\"source\":" + recipe + "}";
+}
+// A vector between zeros.
+std::string Between(const std::string& name, int before, int behind) {
+  return "{\"kind\":\"pad_vector\",\"before\":" + std::to_string(before) + ",\"behind\":" + std::to_string(behind) + ",\"source\":" + Json::Quote(name) + "}";
+}
+
 std::string QuotedList(const Json& names, const char* key, int count) {
   Require(names.has(key) && names.at(key).kind == Json::kArray && int(names.at(key).items.size()) == count,
           std::string("a layer needs one tensor per expert for '") + key + "'");
@@ -95,7 +107,19 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
   Require(s.num_blocks >= 1, "kv.num_blocks must be positive");
   Require(s.streams >= 1 && s.streams <= kMaxStreams, "a model has 1..16 residual streams");
   s.combined = s.streams > 1;
-  for (const Json& in : model.at("layers").items) {
+  s.parallel = model.str("form", "sequential") == "parallel";
+  s.norm_groups = int(model.integer("norm_groups", 1));
+  s.taps = int(model.integer("taps", 0));
+  s.residual_mult = model.num("residual_mult", 1);
+  s.embed_scale = model.num("embed_scale", 1);
+  s.logit_scale = model.num("logit_scale", 1);
+  Require(s.norm_groups >= 1 && s.width % s.norm_groups == 0, "the norms' groups are equal runs of columns");
+  Require(s.taps >= 0 && s.taps <= kMaxTaps, "a short convolution has 1..16 taps");
+  Require(s.parallel || (s.norm_groups == 1 && s.taps == 0 && s.residual_mult == 1 && s.embed_scale == 1 && !model.has("side")),
+          "grouped norms, short convolutions, factors of the residual and side inputs are built for parallel layers");
+  Require(!s.parallel || (s.streams == 1 && s.width <= kMaxConvWidth && std::max(0, s.taps - 1) * s.width <= 40 * 1024 && offset == 0),
+          "parallel layers have one stream of at most 8192 columns, and at most 40960 values of a convolution's history");
+  if (!s.parallel) for (const Json& in : model.at("layers").items) {
     if (in.has("streams")) s.combined = true;
     if (in.has("mlp") && in.at("mlp").str("weighted", "") == "output") s.combined = true;
   }
@@ -125,6 +149,12 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
   s.next = add("step.next", 1, 2, uint64_t(s.max_wanted), 0, "");
   s.hidden = add("step.hidden", 0, 1, uint64_t(s.max_rows) * s.streams * W, 0, "");
   s.embed = add("embed", 1, element, uint64_t(s.vocab) * W, 0, AliasRecipe(Name(model, "embed")));
+  if (model.has("side") && model.at("side").kind == Json::kObject) {
+    s.side_dim = int(model.at("side").integer("dim", 0));
+    s.side_columns = s.side_dim * int(model.at("layers").items.size());
+    Require(s.side_dim >= 1, "a layer's part of the second embedding has at least one column");
+    s.side_embed = add("side.embed", 1, element, uint64_t(s.vocab) * s.side_columns, 0, AliasRecipe(Name(model.at("side"), "embed")));
+  }
 
   Require(model.at("layers").kind == Json::kArray && !model.at("layers").items.empty(), "the model has no layers");
   for (size_t i = 0; i < model.at("layers").items.size(); ++i) {
@@ -135,8 +165,8 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     const Json& mixer = in.at("mixer");
     const Json& names = mixer.at("tensors");
     const std::string kind = mixer.str("kind", "");
-    Require(kind == "attention" || kind == "retention" || kind == "latent", "unknown kind of mixer '" + kind + "'");
-    m.kind = kind == "retention" ? RaggedMixer::kRetention : kind == "latent" ? RaggedMixer::kLatent : RaggedMixer::kAttention;
+    Require(kind == "attention" || kind == "retention" || kind == "latent" || kind == "delta", "unknown kind of mixer '" + kind + "'");
+    m.kind = kind == "retention" ? RaggedMixer::kRetention : kind == "latent" ? RaggedMixer::kLatent : kind == "delta" ? RaggedMixer::kDelta : RaggedMixer::kAttention;
     m.heads = int(mixer.integer("heads", 0));
     m.kv_heads = int(mixer.integer("kv_heads", m.heads));
     m.dim = int(mixer.integer("dim", 0));
@@ -149,12 +179,22 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
       const double factor = rot.num("factor", 1);
       m.rot_dims = int(rot.integer("dims", 0));
       Require(factor > 0, "the rotary scaling factor must be positive");
-      Require(base > 0 && m.rot_dims >= 0 && m.rot_dims % 2 == 0 && m.rot_dims <= m.dim, "rotary dims must be even and at most the head size");
+      Require(base > 0 && m.rot_dims >= 0 && m.rot_dims % 2 == 0 && (m.rot_dims <= m.dim || m.kind == RaggedMixer::kLatent),
+              "rotary dims must be even and at most the head size");
       if (m.rot_dims) {
+        RotaryTable table;
+        if (rot.has("yarn") && rot.at("yarn").kind == Json::kObject) {
+          const char* keys[4] = {"factor", "original", "fast", "slow"};
+          for (int i = 0; i < 4; ++i) {
+            table.yarn[i] = rot.at("yarn").num(keys[i], 0);
+            Require(table.yarn[i] > 0, "a rotation's length scaling has a positive factor, original length and turns");
+          }
+        }
         for (size_t r = 0; r < s.rotaries.size(); ++r)
-          if (s.rotaries[r].base == base && s.rotaries[r].dims == m.rot_dims && s.rotaries[r].factor == factor) m.rotary = int(r);
+          if (s.rotaries[r].base == base && s.rotaries[r].dims == m.rot_dims && s.rotaries[r].factor == factor &&
+              std::equal(table.yarn, table.yarn + 4, s.rotaries[r].yarn))
+            m.rotary = int(r);
         if (m.rotary < 0) {
-          RotaryTable table;
           table.base = base;
           table.factor = factor;
           table.dims = m.rot_dims;
@@ -166,7 +206,8 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     }
     std::string stacked;                 // recipe of the input projection
     const bool bias = mixer.flag("bias", false);
-    const bool pairs = m.rot_dims && mixer.at("rotary").str("layout", "halves") == "pairs";
+    const bool neighbours = m.rot_dims && mixer.at("rotary").str("layout", "halves") == "pairs";
+    const bool pairs = m.kind != RaggedMixer::kLatent && neighbours;   // (latent attention turns neighbours where they are)
     // entries 2i and 2i + 1 of a head turn together: stored as i and i + dims/2, in queries and keys alike
     auto arranged = [&](const std::string& name, int heads) {
       return pairs ? PerHead("pairs_to_halves", name, heads, "dims", m.rot_dims) : name;
@@ -189,12 +230,27 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
       stacked = "{\"kind\":\"stack_rows\",\"sources\":" + Quoted(names, {"q", "k", "v", "g"}) + "}";
     } else if (m.kind == RaggedMixer::kLatent) {
       m.rank = int(mixer.integer("rank", 0));
-      Require(m.kv_heads == m.heads && m.rotary < 0 && !bias, "latent attention has a key and a value per head, no rotation and no biases");
-      Require(m.vdim <= kMaxHeadDim, "head sizes must lie in [1, 256]");
-      Require(m.rank >= 1 && m.rank <= kMaxLatent, "a latent row has 1..1024 columns (rank)");
+      m.q_rank = int(mixer.integer("q_rank", 0));
+      Require(m.kv_heads == m.heads && !bias, "latent attention has a key and a value per head and no biases");
+      Require(m.rotary < 0 || m.q_rank > 0, "latent attention turns queries that are images of a row of their own (q_rank)");
+      Require(m.vdim <= kMaxHeadDim && m.head_key() <= kMaxHeadDim, "head sizes must lie in [1, 256]");
+      Require(m.rank >= 1 && m.columns() <= kMaxLatent, "a latent row has 1..1024 columns (rank, rotated ones)");
       masked();
       Require(m.keep == 0, "latent attention keeps no first positions");
-      stacked = Stack({PerHead("pad_heads", Json::Quote(Name(names, "q")), m.heads, "rows", m.head_stride()), Json::Quote(Name(names, "dkv"))});
+      const std::string row = RotaryTail(Json::Quote(Name(names, "dkv")), 1, m.rot_dims, neighbours, m.rank, m.columns());
+      if (m.q_rank)
+        stacked = Stack({PerHead("pad_heads", Json::Quote(Name(names, "dq")), 1, "rows", m.latent_at()), row});
+      else
+        stacked = Stack({PerHead("pad_heads", Json::Quote(Name(names, "q")), m.heads, "rows", m.head_stride()), Json::Quote(Name(names, "dkv"))});
+    } else if (m.kind == RaggedMixer::kDelta) {
+      m.decay_rank = int(mixer.integer("decay_rank", 0));
+      m.decay_scale = mixer.num("decay_scale", 0);
+      m.unit_eps = mixer.num("unit_eps", 0);
+      Require(m.kv_heads == m.heads && m.vdim == m.dim && m.rotary < 0, "a delta rule has a key and a value of one size per head and no rotation");
+      Require(m.decay_rank >= 1 && m.decay_scale > 0 && m.unit_eps > 0, "a delta rule needs the size of its decays' row (decay_rank), decay_scale and unit_eps");
+      std::vector<std::string> parts = {PerHead("pad_heads", Json::Quote(Name(names, "w1")), 1, "rows", m.delta_at())};
+      for (const char* part : {"r", "k", "v", "a", "g"}) parts.push_back(Json::Quote(Name(names, part)));
+      stacked = Stack(parts);
     } else {
       m.value_is_key = mixer.str("values", "projected") == "keys";
       Require(m.vdim <= kMaxHeadDim, "head sizes must lie in [1, 256]");
@@ -229,6 +285,7 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     Require(place == "input" || place == "output", "a layer's norms act on its sublayers' input or output (norm_at)");
     layer.norm_output = place == "output";
     Require(i == 0 || layer.norm_output == s.layers[0].norm_output, "every layer of a model has its norms in the same place");
+    Require(!s.parallel || !layer.norm_output, "parallel layers read one norm");
     Require(!s.combined || !layer.norm_output, "layers with norms on their outputs have one stream, and experts with weights on their inputs");
     auto streams = [&](int which) {
       if (!in.has("streams")) {
@@ -248,24 +305,55 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     layer.in_weight = matrix(p + "in.weight", PadColumns(stacked, padded_columns(s.width)), m.proj_rows(), s.width);
     if (m.kind == RaggedMixer::kLatent) {
       const int rank = m.rank_stride();
+      const std::string uk = Json::Quote(Name(names, "uk"));
       layer.latent_norm = add(p + "latent.norm", 1, 1, uint64_t(m.rank), 0, AliasRecipe(Name(names, "dkv.norm")));
-      // a query against latent rows is its head's key matrix, transposed, times the query
+      if (m.q_rank) {
+        layer.q_latent_norm = add(p + "query.norm", 1, 1, uint64_t(m.q_rank), 0, AliasRecipe(Name(names, "dq.norm")));
+        layer.query_up = matrix(p + "query_up.weight",
+                                PadColumns(RotaryTail(Json::Quote(Name(names, "uq")), m.heads, m.rot_dims, neighbours, m.head_lead(), m.head_stride()),
+                                           padded_columns(m.q_rank)),
+                                m.heads * m.head_stride(), m.q_rank);
+      }
+      // a query against latent rows is its head's key matrix, transposed, times the query, and its rotated part as it is
+      std::string key_up = PerHead("transpose_heads", uk, m.heads, "rows", m.dim);
+      std::string key = uk;              // a key is the head's key matrix times the normed columns of a latent row, and the rotated ones as they are
+      if (m.rot_dims) {
+        key_up = WithIdentity(PadColumns(key_up, m.head_lead()), m.heads, m.rot_dims);
+        key = WithIdentity(PerHead("pad_heads", uk, m.heads, "rows", m.head_lead()), m.heads, m.rot_dims);
+      }
       layer.key_up = add(p + "key_up.weight", 1, element, uint64_t(m.heads) * rank * m.head_stride(), 0,
-                         PadColumns(PerHead("pad_heads", PerHead("transpose_heads", Json::Quote(Name(names, "uk")), m.heads, "rows", m.dim), m.heads, "rows", rank),
-                                    m.head_stride()));
+                         PadColumns(PerHead("pad_heads", key_up, m.heads, "rows", rank), m.head_stride()));
       if (!s.f32)
         layer.expand = add(p + "expand.weight", 1, element, uint64_t(m.expanded_columns()) * rank, 0,
-                           PadColumns(Stack({PerHead("pad_heads", Json::Quote(Name(names, "uk")), m.heads, "rows", m.expanded_key()),
-                                             PerHead("pad_heads", Json::Quote(Name(names, "uv")), m.heads, "rows", m.v_pool_dim())}), rank));
+                           PadColumns(Stack({PadColumns(PerHead("pad_heads", key, m.heads, "rows", m.expanded_key()), rank),
+                                             PadColumns(PerHead("pad_heads", Json::Quote(Name(names, "uv")), m.heads, "rows", m.v_pool_dim()), rank)}), rank));
       layer.value_up = add(p + "value_up.weight", 1, element, uint64_t(m.heads) * m.vdim * rank, 0,
                            PadColumns(Stack({Json::Quote(Name(names, "uv"))}), rank));
+    }
+    if (m.kind == RaggedMixer::kDelta) {
+      const int all = m.heads * m.dim;
+      layer.in_bias = add(p + "in.bias", 1, 1, uint64_t(m.proj_rows()), 0, Between(Name(names, "a.b"), m.delta_at() + 3 * all, all));
+      layer.decay_up = matrix(p + "decay_up.weight", PadColumns(Stack({Json::Quote(Name(names, "w2"))}), padded_columns(m.decay_rank)), all, m.decay_rank);
+      layer.decay_bias = add(p + "decay.bias", 1, 1, uint64_t(all), 0, AliasRecipe(Name(names, "w0")));
+      layer.out_norm = add(p + "out.norm", 1, 1, uint64_t(all), 0, AliasRecipe(Name(names, "norm")));
+    }
+    if (s.taps) {                        // one row per tap
+      layer.conv = add(p + "conv", 1, 1, uint64_t(s.taps) * W, 0, PerHead("transpose_heads", Json::Quote(Name(in, "conv")), 1, "rows", s.width));
+    }
+    if (s.side_dim) {
+      const Json& side = in.at("side");
+      layer.side.gate = matrix(p + "side.gate", StackRecipe(Quoted(side, {"gate"}), padded_columns(s.width)), s.side_dim, s.width);
+      layer.side.proj = matrix(p + "side.proj", StackRecipe(Quoted(side, {"proj"}), padded_columns(s.side_dim)), s.width, s.side_dim);
+      layer.side.norm = add(p + "side.norm", 1, 1, W, 0, AliasRecipe(Name(side, "norm")));
+      layer.side.from = int(side.integer("from", -1));
+      Require(layer.side.from >= 0 && layer.side.from + s.side_dim <= s.side_columns, "a layer's part lies inside the second embedding");
     }
     layer.out_weight = matrix(p + "out.weight", StackRecipe(Quoted(names, {"o"}), padded_columns(m.out_columns())), s.width, m.out_columns());
     if (m.qk_norm) {
       layer.q_norm = add(p + "q.norm", 1, 1, uint64_t(m.heads) * m.dim, 0, Stack({arranged(Json::Quote(Name(names, "q.norm")), m.heads)}));
       layer.k_norm = add(p + "k.norm", 1, 1, uint64_t(m.kv_heads) * m.dim, 0, Stack({arranged(Json::Quote(Name(names, "k.norm")), m.kv_heads)}));
     }
-    if (bias) {
+    if (bias && m.kind == RaggedMixer::kAttention) {
       std::vector<std::string> biases = {arranged(Json::Quote(Name(names, "q.b")), m.heads), arranged(Json::Quote(Name(names, "k.b")), m.kv_heads)};
       if (!m.value_is_key) biases.push_back(Json::Quote(Name(names, "v.b")));
       layer.in_bias = add(p + "in.bias", 1, 1, uint64_t(m.proj_rows()), 0, Stack(biases));
@@ -279,8 +367,10 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
       layer.mlp.kind = unit == "glu" ? RaggedMlp::kGlu : RaggedMlp::kExperts;
       layer.mlp.ff = int(mlp.integer("ff", 0));
       Require(layer.mlp.ff > 0, "the feed-forward width must be positive");
-      layer.norm2 = add(p + "norm2", 1, 1, W, 0, OffsetRecipe(Name(in, "norm2"), offset));
-      streams(1);
+      if (!s.parallel) {
+        layer.norm2 = add(p + "norm2", 1, 1, W, 0, OffsetRecipe(Name(in, "norm2"), offset));
+        streams(1);
+      }
       const std::string activation = mlp.str("activation", "silu");
       if (layer.mlp.kind == RaggedMlp::kGlu) {
         Require(activation == "silu" || activation == "gelu_tanh", "unknown activation of a gated unit");
@@ -304,6 +394,7 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
         const std::string scores = mlp.str("scores", "");
         e.output_weighted = mlp.str("weighted", "") == "output";
         e.softmax = scores == "softmax";
+        e.chosen = scores == "softmax_chosen";
         e.correction = parts.has("correction");
         if (mlp.has("groups") && mlp.at("groups").kind == Json::kObject) {
           e.groups = int(mlp.at("groups").integer("count", 1));
@@ -313,7 +404,10 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
         Require(e.top <= e.keep_groups * (e.experts / e.groups), "the kept groups hold the experts of a token");
         std::string router = Quoted(parts, {"router"});
         if (e.output_weighted) {
-          Require(activation == "silu" && (e.softmax || scores == "sigmoid"), "experts with weighted outputs are gated units with softmax or sigmoid scores");
+          Require(activation == "silu" && (e.softmax || e.chosen || scores == "sigmoid"),
+                  "experts with weighted outputs are gated units with softmax or sigmoid scores");
+          Require(!e.chosen || (e.groups == 1 && !e.correction), "experts weighted among the chosen ones are ranked by their logits alone");
+          Require(!s.parallel || !mlp.has("shared") || mlp.at("shared").kind != Json::kObject, "parallel layers have no shared expert");
           e.limit = mlp.num("limit", 3.0e38);
           e.alpha = mlp.num("alpha", 1.0);
           e.shift = mlp.num("shift", 0.0);
@@ -353,8 +447,11 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     Require(run.layer >= 0 && run.layer < int(s.layers.size()), "a run names a layer the model does not have");
     const RaggedMixer& m = s.layers[size_t(run.layer)].mixer;
     const std::string at = std::to_string(s.runs.size());
+    if (s.taps > 1) run.history = add("history." + at, 1, 1, 0, uint64_t(s.taps - 1) * W, "");
     if (m.kind == RaggedMixer::kRetention) {
       run.state = add("retention." + at, 1, 1, 0, uint64_t(m.heads) * m.dim * m.vdim, "");
+    } else if (m.kind == RaggedMixer::kDelta) {
+      run.state = add("delta." + at, 1, 1, 0, uint64_t(m.heads) * m.dim * m.state_dim(), "");
     } else if (m.kind == RaggedMixer::kLatent) {
       run.k_pool = add("kv_pool.latent." + at, 1, element, uint64_t(s.num_blocks) * kRaggedBlock * m.pool_dim(), 0, "");
     } else {
@@ -364,11 +461,14 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
     }
     const RaggedMlp& mlp = s.layers[size_t(run.layer)].mlp;
     Require(!run.add_embedding || !s.layers[size_t(run.layer)].norm_output, "layers with norms on their outputs are not looped");
-    Require(!run.add_embedding || !s.combined, "layers of several streams are not looped");
+    Require(!run.add_embedding || (!s.combined && !s.parallel), "layers of several streams, and parallel ones, are not looped with the embedding added");
     const int unit = mlp.output_weighted ? 3 : 2;              // matrices of an expert
     const int mlp_rows = mlp.kind == RaggedMlp::kGlu ? 3 * mlp.ff : mlp.kind == RaggedMlp::kExperts ? unit * mlp.top * mlp.ff + 3 * mlp.shared_ff + mlp.logits() : 0;
     s.weight_bytes += element_bytes * W * uint64_t(m.proj_rows() + m.out_columns() + mlp_rows);
-    if (m.kind == RaggedMixer::kLatent) s.weight_bytes += element_bytes * uint64_t(m.heads) * m.rank * (m.dim + m.vdim);
+    if (m.kind == RaggedMixer::kLatent)
+      s.weight_bytes += element_bytes * uint64_t(m.heads) * (uint64_t(m.rank) * (m.dim + m.vdim) + uint64_t(m.q_rank) * (m.dim + m.rot_dims));
+    if (m.kind == RaggedMixer::kDelta) s.weight_bytes += element_bytes * uint64_t(m.heads) * m.dim * m.decay_rank;
+    s.weight_bytes += element_bytes * 2 * W * uint64_t(s.side_dim);
     s.runs.push_back(run);
   }
   Require(!s.runs.empty(), "the model runs no layer");

@@ -15,7 +15,7 @@ namespace {
 // One CTA per row. The row's entry is found by bisection over the entries' first rows (ascending, no gaps).
 template <typename T>
 __global__ void __launch_bounds__(256) start_step(StepRows r, const int* tokens, const T* embed, float* x, int streams, T* copy,
-                                                  int copy_stride, int width, int vocab) {
+                                                  int copy_stride, int width, int vocab, float scale) {
   const int row = blockIdx.x;
   dependency_wait();
   allow_dependents();
@@ -38,7 +38,7 @@ __global__ void __launch_bounds__(256) start_step(StepRows r, const int* tokens,
 #pragma unroll 8
   for (int i = threadIdx.x; i < width; i += 256) {
     const T value = embed[size_t(token) * width + i];
-    for (int s = 0; s < streams; ++s) x[(size_t(row) * streams + s) * width + i] = to_f(value);
+    for (int s = 0; s < streams; ++s) x[(size_t(row) * streams + s) * width + i] = to_f(value) * scale;
     if (copy) copy[size_t(row) * copy_stride + i] = value;
   }
 }
@@ -296,6 +296,8 @@ __global__ void __launch_bounds__(512) stream_step(StreamArgs a) {
       }
       float sum[E] = {};
 #pragma unroll
+      for (int e = 0; e < E; ++e) y[e] *= a.gain;
+#pragma unroll
       for (int e = 0; e < E; ++e) {
         float now[S];
 #pragma unroll
@@ -337,7 +339,27 @@ __global__ void __launch_bounds__(512) stream_step(StreamArgs a) {
       sq = fmaf(v[0], v[0], sq);
     }
   }
-  if (!a.weight) return;
+  T* normed = static_cast<T*>(a.normed) + size_t(i) * a.normed_stride;
+  if (!a.weight) {
+    if (!a.normed) return;
+    if constexpr (QUADS) {
+#pragma unroll
+      for (int n = 0; n < N; ++n) {
+        const int c = threadIdx.x + 512 * n;
+        if (c >= units) continue;
+        alignas(16) T e[4] = {from_f<T>(u[n].x), from_f<T>(u[n].y), from_f<T>(u[n].z), from_f<T>(u[n].w)};
+        if (sizeof(T) == 2) reinterpret_cast<uint2*>(normed)[c] = *reinterpret_cast<const uint2*>(e);
+        else reinterpret_cast<uint4*>(normed)[c] = *reinterpret_cast<const uint4*>(e);
+      }
+    } else {
+      for (int c = threadIdx.x; c < units; c += 512) {
+        float v[E];
+        visit(c, false, v);
+        normed[c] = from_f<T>(v[0]);
+      }
+    }
+    return;
+  }
   sq = warp_sum(sq);
   if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = sq;
   __syncthreads();
@@ -345,7 +367,6 @@ __global__ void __launch_bounds__(512) stream_step(StreamArgs a) {
 #pragma unroll
   for (int w = 0; w < 16; ++w) sq += part[w];
   const float inv = 1.f / sqrtf(sq / float(a.width) + a.eps);
-  T* normed = static_cast<T*>(a.normed) + size_t(i) * a.normed_stride;
   if constexpr (QUADS) {
 #pragma unroll
     for (int n = 0; n < N; ++n) {
@@ -439,13 +460,13 @@ __global__ void feed(Entry* entries, int count, const int* next, int* tokens, in
 }  // namespace
 
 int StartStep(const Queue& q, const StepRows& r, const int* tokens, const void* embed, float* x, int streams, void* copy, int copy_stride, int width,
-              int vocab) {
+              int vocab, float scale) {
   const dim3 grid(unsigned(r.rows));
   if (q.f32)
     return int(Launch(start_step<float>, grid, dim3(256), 0, q.stream, false, r, tokens, static_cast<const float*>(embed), x, streams, static_cast<float*>(copy),
-                      copy_stride, width, vocab));
+                      copy_stride, width, vocab, scale));
   return int(Launch(start_step<__nv_bfloat16>, grid, dim3(256), 0, q.stream, false, r, tokens, static_cast<const __nv_bfloat16*>(embed), x, streams,
-                    static_cast<__nv_bfloat16*>(copy), copy_stride, width, vocab));
+                    static_cast<__nv_bfloat16*>(copy), copy_stride, width, vocab, scale));
 }
 
 int RmsNorm(const Queue& q, const NormArgs& a) {

@@ -8,6 +8,7 @@ csrc/ragged_spec.cpp reads. A new design of known mechanisms is one more functio
 from __future__ import annotations
 
 import json
+import math
 from dataclasses import dataclass
 from pathlib import Path
 from typing import Callable
@@ -18,17 +19,18 @@ class Family:
     name: str
     plans: tuple[str, ...]                          # phases emit_plan writes for it
     layer_program: Callable[[dict], dict] | None = None
+    complete: Callable[[dict, Callable], dict] | None = None   # fills in sizes only the checkpoint's tensor shapes tell
 
 
-def looped_runs(count: int, loop: dict | None) -> list[dict]:
-    """The order `count` layers run in when layers start .. stop-1 run `times` times in a row; every pass but the
-    first begins by adding the embedding output to the residual stream."""
+def looped_runs(count: int, loop: dict | None, add_embedding: bool = True) -> list[dict]:
+    """The order `count` layers run in when layers start .. stop-1 run `times` times in a row; with `add_embedding` every
+    pass but the first begins by adding the embedding output to the residual stream."""
     if not loop:
         return [{"layer": layer, "add_embedding": False} for layer in range(count)]
     start, stop, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
     if not 0 <= start <= stop <= count or times < 1:
         raise ValueError(f"loop {loop} does not fit {count} layers")
-    body = [(layer, turn > 0 and layer == start) for turn in range(times) for layer in range(start, stop)]
+    body = [(layer, add_embedding and turn > 0 and layer == start) for turn in range(times) for layer in range(start, stop)]
     order = [(layer, False) for layer in range(start)] + body + [(layer, False) for layer in range(stop, count)]
     return [{"layer": layer, "add_embedding": again} for layer, again in order]
 
@@ -149,6 +151,56 @@ def mozidra_program(config: dict) -> dict:
             "embed": "embed", "final_norm": "final.norm", "head": "head", "layers": layers, "runs": looped_runs(len(layers), None)}
 
 
+def _benarax_mixer(kind: str, mixer: dict, prefix: str) -> dict:
+    if kind == "general_delta":
+        # decay_rank: a completed config has it, see complete_benarax
+        return {"kind": "delta", "heads": mixer["heads"], "dim": mixer["dim"], "decay_rank": mixer["decay_rank"], "decay_scale": math.exp(-0.5),
+                "unit_eps": 1e-6, "tensors": _names(prefix, "r", "k", "v", "a", "a.b", "g", "w1", "w2", "w0", "norm", "o")}
+    if kind not in ("latent_attention", "latent_attention_2"):
+        raise ValueError(f"unknown layer type {kind!r}")
+    rot = mixer["rot"]
+    if rot["dims"] != mixer["rot_dim"]:
+        raise ValueError("the whole rotated part of a head turns")
+    # the two kinds differ in which entries of the rotated part turn together
+    return {"kind": "latent", "heads": mixer["heads"], "dim": mixer["dim"], "vdim": mixer["vdim"], "rank": mixer["kv_rank"], "q_rank": mixer["q_rank"],
+            "rotary": {"base": rot["base"], "dims": rot["dims"], "layout": "pairs" if kind == "latent_attention" else "halves", "yarn": rot.get("scaling")},
+            "scale": mixer["scale"], "tensors": _names(prefix, "dq", "dq.norm", "uq", "dkv", "dkv.norm", "uk", "uv", "o")}
+
+
+def _benarax_mlp(mlp: dict | None, prefix: str) -> dict | None:
+    if mlp is None:
+        return None
+    if mlp["kind"] != "moe":
+        raise ValueError(f"unknown feed-forward {mlp['kind']!r}")
+    count = int(mlp["router"]["experts"])
+    return {"kind": "experts", "ff": mlp["expert"]["ff"], "limit": mlp["expert"]["limit"], "alpha": 1.702, "shift": 1.0, "experts": count,
+            "top": mlp["router"]["top"], "activation": "silu", "scores": "softmax_chosen", "weighted": "output",
+            "tensors": {"router": prefix + "router"} | {part: [f"{prefix}e{expert}.{part}" for expert in range(count)] for part in ("gate", "up", "down")}}
+
+
+def benarax_program(config: dict) -> dict:
+    layers, side = [], config["token_side"]
+    for index, layer in enumerate(config["layers"]):
+        prefix = f"l{index}."
+        layers.append({"norm1": prefix + "norm1", "mixer": _benarax_mixer(layer["type"], layer["mixer"], prefix + "mix."),
+                       "mlp": _benarax_mlp(layer.get("mlp"), prefix + "mlp."), "conv": prefix + "canon1",
+                       "side": _names(prefix + "side.", "gate", "proj", "norm") | {"from": index * side["dim"]}})
+    return {"width": config["width"], "vocab": config["vocab"], "eps": config["norm"]["eps"], "form": "parallel", "norm_groups": config["norm"]["groups"],
+            "taps": config["canon"]["taps"], "residual_mult": config["residual_mult"], "embed_scale": config["embedding"]["scale"],
+            "logit_scale": config["logit_scale"], "side": {"embed": "side.embed", "dim": side["dim"]}, "embed": "embed", "final_norm": "final.norm",
+            "head": "head", "layers": layers, "runs": looped_runs(len(layers), config.get("loop"), add_embedding=False)}
+
+
+def complete_benarax(config: dict, shape_of: Callable) -> dict:
+    """The decays of a delta rule come through a row whose size no key of the config gives: that of the tensor."""
+    layers = []
+    for index, layer in enumerate(config["layers"]):
+        if layer["type"] == "general_delta" and "decay_rank" not in layer["mixer"]:
+            layer = layer | {"mixer": layer["mixer"] | {"decay_rank": int(shape_of(f"l{index}.mix.w1")[0])}}
+        layers.append(layer)
+    return config | {"layers": layers}
+
+
 FAMILIES = {
     "LlamaForCausalLM": Family("llama", ("decode", "prefill")),
     "Qwen3MoeForCausalLM": Family("qwen3-moe", ("decode",)),
@@ -156,6 +208,7 @@ FAMILIES = {
     "Bamudra": Family("bamudra", ("ragged",), bamudra_program),
     "Nadilorn": Family("nadilorn", ("ragged",), nadilorn_program),
     "Mozidra": Family("mozidra", ("ragged",), mozidra_program),
+    "Benarax": Family("benarax", ("ragged",), benarax_program, complete_benarax),
 }
 
 
@@ -174,7 +227,13 @@ def family_of(config: dict) -> Family:
 
 
 def load_config(model_dir: str | Path) -> dict:
-    return json.loads((Path(model_dir) / "config.json").read_text())
+    """config.json of a model folder, with the sizes its family takes from the checkpoint's tensor shapes."""
+    config = json.loads((Path(model_dir) / "config.json").read_text())
+    complete = FAMILIES[architecture_of(config)].complete if architecture_of(config) in FAMILIES else None
+    if complete is None:
+        return config
+    from .serving.weights import Checkpoint
+    return complete(config, Checkpoint(model_dir).shape)
 
 
 def vocab_of(config: dict) -> int:
@@ -189,21 +248,33 @@ def tensor_shapes(config: dict) -> dict[str, tuple[int, ...]]:
     for layer in program["layers"]:
         mixer, names = layer["mixer"], layer["mixer"]["tensors"]
         heads, streams = mixer["heads"], program.get("streams", 1)
-        q, out = heads * mixer["dim"], heads * mixer["vdim"]
-        k, rank = mixer.get("kv_heads", heads) * mixer["dim"], mixer.get("rank", 0)
-        sizes = {"q": q, "k": k, "v": mixer.get("kv_heads", heads) * mixer["vdim"], "g": out, "dkv": rank, "o": width}
-        special = {"o": (width, out), "uk": (q, rank), "uv": (out, rank), "sink": (heads,), "vmix": ()}
+        vdim = mixer.get("vdim", mixer["dim"])
+        q, out = heads * mixer["dim"], heads * vdim
+        k, rank, turned = mixer.get("kv_heads", heads) * mixer["dim"], mixer.get("rank", 0), (mixer.get("rotary") or {}).get("dims", 0)
+        q_rank, decay_rank = mixer.get("q_rank", 0), mixer.get("decay_rank", 0)
+        sizes = {"q": q, "k": k, "v": mixer.get("kv_heads", heads) * vdim, "g": out, "dkv": rank + (turned if q_rank else 0), "dq": q_rank, "r": q,
+                 "a": q, "w1": decay_rank, "o": width}
+        special = {"o": (width, out), "uk": (q, rank), "uv": (out, rank), "uq": (q + heads * turned, q_rank), "sink": (heads,), "vmix": (),
+                   "dkv.norm": (rank,), "w2": (q, decay_rank), "w0": (q,), "norm": (out,)}
         shapes[layer["norm1"]] = (width,)
         for part, name in names.items():
-            if part.endswith((".norm", ".b")):
+            if part in special:
+                shapes[name] = special[part]
+            elif part.endswith((".norm", ".b")):
                 shapes[name] = (sizes[part.rsplit(".", 1)[0]],)
             else:
-                shapes[name] = special[part] if part in special else (sizes[part], width)
+                shapes[name] = (sizes[part], width)
+        if program.get("taps"):
+            shapes[layer["conv"]] = (width, program["taps"])
+        if "side" in layer:
+            part = program["side"]["dim"]
+            shapes |= {layer["side"]["gate"]: (part, width), layer["side"]["proj"]: (width, part), layer["side"]["norm"]: (width,)}
         for parts in layer.get("streams", ()):
             shapes |= {parts["in"]: (streams,), parts["out"]: (streams,), parts["mix"]: (streams, streams)}
         if layer["mlp"]:
             ff, parts = layer["mlp"]["ff"], layer["mlp"]["tensors"]
-            shapes[layer["norm2"]] = (width,)
+            if "norm2" in layer:
+                shapes[layer["norm2"]] = (width,)
             if layer["mlp"]["kind"] == "experts":
                 shapes[parts["router"]] = (layer["mlp"]["experts"], width)
                 shapes |= {name: (ff, width) for part in ("gate", "up") for name in parts.get(part, ())} | {name: (width, ff) for name in parts["down"]}
@@ -215,6 +286,8 @@ def tensor_shapes(config: dict) -> dict[str, tuple[int, ...]]:
                                parts["shared.sg"]: (1, width)}
             else:
                 shapes |= {parts["gate"]: (ff, width), parts["up"]: (ff, width), parts["down"]: (width, ff)}
+    if "side" in program:
+        shapes[program["side"]["embed"]] = (program["vocab"], program["side"]["dim"] * len(program["layers"]))
     shapes[program["final_norm"]] = (width,)
     shapes[program["head"]] = (program["vocab"], width)
     return shapes

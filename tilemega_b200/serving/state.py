@@ -79,12 +79,24 @@ def rotary_tables(config: dict, capacity: int, device: torch.device | str) -> tu
             table.sin().to(torch.bfloat16).to(device).contiguous())
 
 
-def rotary_pairs(base: float, dims: int, capacity: int, factor: float = 1.0) -> torch.Tensor:
-    """fp32 [capacity][dims/2][2]: cosine and sine of position * base^(-2i/dims) / factor for the pairs of a rotate-half
-    rotation, the angles taken in float64."""
-    frequency = base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims) / factor
+def rotary_pairs(base: float, dims: int, capacity: int, factor: float = 1.0, yarn: dict | None = None) -> torch.Tensor:
+    """fp32 [capacity][dims/2][2]: cosine and sine of position * base^(-2i/dims) / factor for the pairs of a rotation, the
+    angles taken in float64.
+
+    `yarn` (factor, original, fast, slow; Peng et al., "YaRN: Efficient Context Window Extension of Large Language
+    Models"): pairs that turn less than `slow` times over the `original` length turn `factor` times slower, those that turn
+    more than `fast` times as before, a ramp over the pair's index between them; cosine and sine both grow by
+    0.1 ln(factor) + 1."""
+    index = torch.arange(dims // 2, dtype=torch.float64)
+    frequency, size = base ** (-2.0 * index / dims) / factor, 1.0
+    if yarn:
+        place = lambda turns: dims * math.log(yarn["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+        low, high = max(math.floor(place(yarn["fast"])), 0), min(math.ceil(place(yarn["slow"])), dims - 1)
+        ramp = ((index - low) / max(high - low, 0.001)).clamp(0.0, 1.0)
+        frequency = frequency / yarn["factor"] * ramp + frequency * (1.0 - ramp)
+        size = 0.1 * math.log(yarn["factor"]) + 1.0
     angles = torch.arange(capacity, dtype=torch.float64)[:, None] * frequency[None, :]
-    return torch.stack((angles.cos(), angles.sin()), dim=-1).float()
+    return torch.stack((size * angles.cos(), size * angles.sin()), dim=-1).float()
 
 
 def kv_row_swizzle(rows: torch.Tensor) -> torch.Tensor:
@@ -200,16 +212,16 @@ def allocate_ragged_state(ragged: PlanLibrary, device: str | torch.device = "cud
     tables = []
     for layer in model["layers"]:
         rot = layer["mixer"].get("rotary")
-        if rot and rot["dims"] and (rot["base"], rot["dims"], rot.get("factor", 1.0)) not in tables:
-            tables.append((rot["base"], rot["dims"], rot.get("factor", 1.0)))
+        if rot and rot["dims"] and (table := (rot["base"], rot["dims"], rot.get("factor", 1.0), rot.get("yarn"))) not in tables:
+            tables.append(table)
     result = {}
     for buffer in ragged.buffers:
         if buffer.role != 1 or buffer.pack_json:
             continue
         count = buffer.elements_constant + slots * buffer.elements_per_batch
         if buffer.name.startswith("rotary."):
-            base, dims, factor = tables[int(buffer.name.split(".")[1])]
-            tensor = rotary_pairs(base, dims, capacity, factor).to(device).reshape(-1).contiguous()
+            base, dims, factor, yarn = tables[int(buffer.name.split(".")[1])]
+            tensor = rotary_pairs(base, dims, capacity, factor, yarn).to(device).reshape(-1).contiguous()
         else:
             tensor = torch.zeros(count, dtype={0: torch.bfloat16, 1: torch.float32, 2: torch.int32}[buffer.dtype], device=device)
         if tensor.numel() != count:

@@ -49,6 +49,12 @@ class Checkpoint:
         if not self.files:
             raise FileNotFoundError(f"no safetensors in {self.model_dir}")
 
+    def shape(self, name: str) -> tuple[int, ...]:
+        if name not in self.files:
+            raise KeyError(f"checkpoint has no {name}")
+        with self._reader(self.files[name]) as handle:
+            return tuple(handle.get_slice(name).get_shape())
+
     def tensor(self, name: str) -> torch.Tensor:
         name = _tied_name(name, self.files, self.tie_word_embeddings)
         if name not in self.files:
@@ -224,6 +230,25 @@ def per_head(recipe: Mapping[str, object], tensor: torch.Tensor) -> torch.Tensor
         if tensor.ndim != 2 or rows != int(recipe["rows"]):
             raise ValueError("transpose_heads takes a matrix of that many rows a head")
         return split.transpose(1, 2).reshape(-1, rows)
+    if kind == "append_identity":                # behind every head's matrix: `size` columns of zeros, `size` rows of an identity on them
+        size = int(recipe["size"])
+        if tensor.ndim != 2 or size < 1:
+            raise ValueError("append_identity takes a matrix")
+        grown = torch.nn.functional.pad(split, (0, size, 0, size))
+        grown[:, rows:, tensor.shape[1]:] = torch.eye(size, dtype=tensor.dtype, device=tensor.device)
+        return grown.reshape(-1, grown.shape[2])
+    if kind == "rotary_tail":
+        # of every head the last `dims` rows as neighbours that turn together, behind `lead` rows for the others; zero rows up to `rows`
+        dims, lead, total = int(recipe["dims"]), int(recipe["lead"]), int(recipe["rows"])
+        others = rows - dims
+        if tensor.ndim != 2 or dims % 2 or not 0 <= others <= lead or lead + dims > total or recipe["layout"] not in ("pairs", "halves"):
+            raise ValueError("rotary_tail takes a matrix whose heads end in an even number of rotated rows")
+        tail = split[:, others:]
+        if recipe["layout"] == "halves":
+            tail = tail.reshape(heads, 2, dims // 2, -1).transpose(1, 2).reshape(heads, dims, -1)
+        placed = tensor.new_zeros((heads, total, tensor.shape[1]))
+        placed[:, :others], placed[:, lead:lead + dims] = split[:, :others], tail
+        return placed.reshape(-1, tensor.shape[1])
     # pairs_to_halves: of the first `dims` rows of a head the even ones, then the odd ones; the others stay
     dims = int(recipe["dims"])
     if dims % 2 or not 0 <= dims <= rows:
@@ -253,7 +278,12 @@ def pack(recipe: Mapping[str, object], source: Callable[[str], torch.Tensor], tp
         if len({item.shape[1:] for item in tensors}) != 1 or tensors[0].ndim not in (1, 2):
             raise ValueError("stack takes matrices of one width or vectors")
         return torch.cat(tensors)
-    if kind in ("pad_heads", "transpose_heads", "pairs_to_halves"):
+    if kind == "pad_vector":
+        vector = inner(recipe["source"])
+        if vector.ndim != 1:
+            raise ValueError("pad_vector takes a vector")
+        return torch.nn.functional.pad(vector, (int(recipe["before"]), int(recipe["behind"])))
+    if kind in ("pad_heads", "transpose_heads", "pairs_to_halves", "append_identity", "rotary_tail"):
         return per_head(recipe, inner(recipe["source"]))
     if kind == "tile_pages":
         inner = recipe["source"]
