@@ -72,8 +72,9 @@ MODELS = {"llama-3.1-8b": synthetic.LLAMA_3_1_8B, "llama-3.2-1b": synthetic.LLAM
           "bamudra-8b": synthetic.BAMUDRA_8B, "bamudra-1b": synthetic.BAMUDRA_1B,   # ragged-step plans (run_ragged)
           "nadilorn-8b": synthetic.NADILORN_8B, "nadilorn-1b": synthetic.NADILORN_1B, "nadilorn-30b-a3b": synthetic.NADILORN_30B_A3B,
           "nadilorn-7b-a1b": synthetic.NADILORN_7B_A1B, "nadilorn-47b-a13b": synthetic.NADILORN_47B_A13B,
-          "mozidra-30b-a3b": synthetic.MOZIDRA_30B_A3B, "mozidra-7b-a1b": synthetic.MOZIDRA_7B_A1B, "mozidra-47b-a13b": synthetic.MOZIDRA_47B_A13B}
-LAYERED = ("bamudra", "nadilorn", "mozidra")   # decoders given as a list of layers
+          "mozidra-30b-a3b": synthetic.MOZIDRA_30B_A3B, "mozidra-7b-a1b": synthetic.MOZIDRA_7B_A1B, "mozidra-47b-a13b": synthetic.MOZIDRA_47B_A13B,
+          "benarax-30b-a3b": synthetic.BENARAX_30B_A3B, "benarax-7b-a1b": synthetic.BENARAX_7B_A1B, "benarax-47b-a13b": synthetic.BENARAX_47B_A13B}
+LAYERED = ("bamudra", "nadilorn", "mozidra", "benarax")   # decoders given as a list of layers
 
 
 def workload(args) -> dict:
@@ -502,7 +503,7 @@ def run_forward(args) -> None:
 
 def run_ragged(args) -> None:
     """Secondary workload: a decoder given as a list of layers (`--model bamudra-8b | bamudra-1b | nadilorn-8b | nadilorn-1b |
-    nadilorn-30b-a3b | nadilorn-7b-a1b | nadilorn-47b-a13b`, and `mozidra-` for the last three sizes) through a ragged-step plan (phase 3 of the plan ABI). Decode: `--batch` sequences at `--context`
+    nadilorn-30b-a3b | nadilorn-7b-a1b | nadilorn-47b-a13b`, and `mozidra-` and `benarax-` for the last three sizes) through a ragged-step plan (phase 3 of the plan ABI). Decode: `--batch` sequences at `--context`
     positions, one step = one decoded token of each, the sampled tokens fed back on the device. `--prefill T`: a prompt of T tokens in portions of `--portion` rows, one step =
     one portion. One JSON line in the shape of the decode line; same weights, widths and vocabulary as the Llama-shaped
     model of the same name, so the two lines stand side by side."""
@@ -529,35 +530,38 @@ def run_ragged(args) -> None:
     executor = RaggedExecutor(synthetic.LazyShapedCheckpoint(tensor_shapes(config)), so)
     torch.cuda.empty_cache()
     for name, tensor in executor.state.items():
-        if name.startswith(("kv_pool", "retention")):
+        if name.startswith(("kv_pool", "retention", "delta", "history")):
             tensor.normal_(0.0, 0.5)
     stream = executor.stream
     vocab, width = config["vocab"], config["width"]
     begin, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
     clocks = ClockSampler(0)
     runs = executor.library.manifest["model"]["runs"]
-    state_bytes = sum(2 * 4 * m["heads"] * m["dim"] * m["vdim"] for m in (config["layers"][run["layer"]]["mixer"] for run in runs) if "decay" in m)
-
-    attention = [mixer for mixer in (config["layers"][run["layer"]]["mixer"] for run in runs) if "mask" in mixer]
+    ran = [config["layers"][run["layer"]] for run in runs]
+    recurrent = [layer["mixer"] for layer in ran if layer["type"] in ("retention", "general_delta")]
+    state_bytes = sum(2 * 4 * m["heads"] * m["dim"] * m.get("vdim", m["dim"]) for m in recurrent)
+    attention = [layer["mixer"] for layer in ran if layer["type"] not in ("retention", "general_delta")]
 
     def seen(mixer: dict, position: int) -> int:
-        size, keep = mixer["mask"]["size"], mixer["mask"].get("keep_first", 0)
+        mask = mixer.get("mask") or {}
+        size, keep = mask.get("size", position + 1), mask.get("keep_first", 0)
         return min(position + 1, size) + min(keep, max(0, position + 1 - size))
 
     def cached(position: int) -> int:
         """Bytes of keys and values (or of latent rows) one token at this position reads, all attention layers."""
-        return sum(seen(mixer, position) * 2 * (mixer["kv_rank"] if "kv_rank" in mixer else mixer["kv_heads"] * (mixer["dim"] + mixer["vdim"]))
+        return sum(seen(mixer, position) * 2 * (mixer["kv_rank"] + mixer.get("rot_dim", 0) if "kv_rank" in mixer else mixer["kv_heads"] * (mixer["dim"] + mixer["vdim"]))
                    for mixer in attention)
 
     def attention_flops(position: int) -> int:
-        return sum(seen(mixer, position) * 2 * mixer["heads"] * (mixer["dim"] + mixer["vdim"]) for mixer in attention)
+        return sum(seen(mixer, position) * 2 * mixer["heads"] * (mixer["dim"] + mixer.get("rot_dim", 0) + mixer["vdim"]) for mixer in attention)
 
     weight_bytes = executor.plan.step_bytes(0)
     weight_elements = weight_bytes // 2                          # of one token: its own experts
-    mixtures = [layer["mlp"] for layer in config["layers"] if layer["mlp"] and layer["mlp"]["kind"] == "moe"]
+    matrices = 2 if config["architecture"] == "Nadilorn" else 3   # of an expert
+    mixtures = [layer["mlp"] for layer in ran if layer["mlp"] and layer["mlp"]["kind"] == "moe"]
     for mlp in mixtures:                                         # experts a batch reads, if its tokens spread evenly
         experts, top = mlp["router"]["experts"], mlp["router"]["top"]
-        weight_bytes += round(2 * (3 if "shared" in mlp else 2) * width * mlp["expert"]["ff"] * (experts * (1.0 - (1.0 - top / experts) ** batch) - top))
+        weight_bytes += round(2 * matrices * width * mlp["expert"]["ff"] * (experts * (1.0 - (1.0 - top / experts) ** batch) - top))
     peaks = json.loads((ROOT / "MEASURED_PEAKS.json").read_text()) if (ROOT / "MEASURED_PEAKS.json").exists() else {}
     if args.prefill:
         prompt = synthetic.seeded_tokens(1, context, vocab, seed=3)[0].tolist()
@@ -590,7 +594,7 @@ def run_ragged(args) -> None:
         flops = 2.0 * (context * (weight_elements - head_elements) + head_elements)
         for position in range(context):
             flops += attention_flops(position)
-        flops += context * 4.0 * state_bytes / 8
+        flops += context * 4.0 * state_bytes / 8 * (2 if config["architecture"] == "Benarax" else 1)   # (products with the state per token: two, or four)
         peak = float(peaks.get("bf16_tflops", 1590.0))
         steps_run = -(-context // portion)
         line = {"metric": "prefill_tokens_per_s", "value": context / device_s, "unit": UNIT, "n_gpus": 1, "steps": steps_run, "warmup": 3,
@@ -851,7 +855,7 @@ def main() -> None:
                         help="--model bert-base: element type of the forward plan (f16: the benchmark configuration; bf16: what the reference's export runs)")
     parser.add_argument("--prefill", type=int, default=0,
                         help="secondary workload: chunked prefill of one prompt of this many tokens (one GPU)")
-    parser.add_argument("--portion", type=int, default=2048, help="--model bamudra-* / nadilorn-* / mozidra-*: rows per step of a prefilled prompt")
+    parser.add_argument("--portion", type=int, default=2048, help="--model bamudra-* / nadilorn-* / mozidra-* / benarax-*: rows per step of a prefilled prompt")
     parser.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     parser.add_argument("--trace", action="store_true",
                         help="after the timed runs, stamp one more step and print the per-stage table (rank 0)")

@@ -74,9 +74,8 @@ def rotate(x: torch.Tensor, positions: torch.Tensor, rot: dict, neighbours: bool
 
 def causal_softmax(score: torch.Tensor) -> torch.Tensor:
     """score [T, T]: row i over the keys j <= i."""
-    steps = score.shape[0]
-    hidden = torch.tensor([[j > i for j in range(steps)] for i in range(steps)]).reshape(steps, steps)
-    return torch.softmax(score.masked_fill(hidden, -math.inf), dim=-1)
+    places = torch.arange(score.shape[0])
+    return torch.softmax(score.masked_fill(places[None, :] > places[:, None], -math.inf), dim=-1)
 
 
 def latent_mixer(h: torch.Tensor, positions: torch.Tensor, spec: dict, w, eps: float, neighbours: bool) -> torch.Tensor:

@@ -110,7 +110,7 @@ def test_buffer_table_and_recipes(name, dtype, plan_dir):
 @pytest.mark.parametrize("break_it, message", [
     (lambda l: l[0]["mixer"].update(vdim=300), "head sizes"),
     (lambda l: l[0]["mixer"].update(rank=1025), "1..1024 columns"),
-    (lambda l: l[0]["mixer"].update(bias=True), "no rotation and no biases"),
+    (lambda l: l[0]["mixer"].update(bias=True), "per head and no biases"),
     (lambda l: l[0]["mixer"].update(mask={"size": 5, "keep_first": 2}), "keeps no first positions"),
     (lambda l: l[1]["mixer"].update(values="keys", vdim=20), "halves turn"),
     (lambda l: l[1]["mixer"].update(value_mix="other"), "way of mixing"),

@@ -256,6 +256,25 @@ MOZIDRA_7B_A1B = mozidra_config(2048, 16, 4, 128, 256, 16, 50304, 2048, 2, 64, 8
 MOZIDRA_47B_A13B = mozidra_config(4096, 32, 8, 128, 512, 32, 32000, 4096, 4, 8, 2, 4, 2, 14336, 2048)
 
 
+# Benarax-shaped decoders of the same sizes: of three layers in a row two have latent attention (one with a stretched rotation), one the
+# delta rule; every layer has a part of the second embedding in place of a shared expert.
+def benarax_config(width: int, heads: int, dim: int, rot: int, rank: int, q_rank: int, delta_heads: int, layers: int, vocab: int, side: int,
+                   experts: int, top: int, expert_ff: int) -> dict:
+    latent = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": dim, "kv_rank": rank, "q_rank": q_rank, "scale": (dim + rot) ** -0.5}
+    stretched = {"base": 10000.0, "dims": rot, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+    mixture = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": expert_ff, "limit": 7.0}}
+    kinds = [{"type": "latent_attention", "mixer": latent | {"rot": stretched}, "mlp": mixture},
+             {"type": "latent_attention_2", "mixer": latent | {"rot": {"base": 500000.0, "dims": rot}}, "mlp": mixture},
+             {"type": "general_delta", "mixer": {"heads": delta_heads, "dim": width // delta_heads, "decay_rank": 96}, "mlp": mixture}]
+    return {"architecture": "Benarax", "width": width, "vocab": vocab, "norm": {"eps": 1e-5, "groups": 8}, "canon": {"taps": 4}, "embedding": {"scale": 1.0},
+            "residual_mult": 1.0, "logit_scale": 1.0, "token_side": {"dim": side}, "layers": [kinds[index % 3] for index in range(layers)]}
+
+
+BENARAX_30B_A3B = benarax_config(2048, 32, 128, 64, 512, 768, 16, 48, 151936, 128, 128, 8, 768)
+BENARAX_7B_A1B = benarax_config(2048, 16, 128, 64, 256, 512, 16, 16, 50304, 128, 64, 8, 1024)
+BENARAX_47B_A13B = benarax_config(4096, 32, 128, 64, 512, 1024, 32, 32, 32000, 256, 8, 2, 14336)
+
+
 class LazyShapedCheckpoint:
     """Like LazySeededCheckpoint for any table of tensor shapes (registry.tensor_shapes): matrices N(0, std), norm
     weights 1, biases N(0, std), residual streams read in equal shares and kept as they are, each tensor from its own
