@@ -20,7 +20,7 @@ def test_layer_program_takes_every_size_and_constant_from_the_config():
     config = case.CASES["odd"]
     assert family_of(config).plans == ("ragged",)
     program = family_of(config).layer_program(config)
-    assert [program[key] for key in ("width", "vocab", "eps", "form", "norm_groups", "taps")] == [90, 203, 1e-3, "parallel", 3, 4]
+    assert [program[key] for key in ("width", "vocab", "eps", "form", "norm_groups", "taps")] == [90, 203, 2e-2, "parallel", 3, 4]
     assert [program[key] for key in ("residual_mult", "embed_scale", "logit_scale", "side")] == [0.8, 1.5, 0.5, {"embed": "side.embed", "dim": 7}]
     first, second, third, fourth, fifth = program["layers"]
     assert [first["mixer"][key] for key in ("kind", "heads", "dim", "vdim", "rank", "q_rank", "scale")] == ["latent", 5, 20, 28, 43, 21, 26 ** -0.5]

@@ -18,7 +18,9 @@ constexpr int kThreads = 512, kWarps = kThreads / 32;
 // units behind the other. It starts count - 1 rows before the tile, whose h it forms again (x is never written in place), so
 // tiles do not wait for one another; the first tile reads the history and writes the new one, and tiles are at least count - 1
 // rows long, so no other tile touches it. blockIdx = (tile, entry).
-template <typename T, int E, int N, bool SELECT>
+// HELD: up to four taps stay in registers.
+constexpr int kHeldTaps = 4;
+template <typename T, int E, int N, bool SELECT, bool HELD>
 __global__ void __launch_bounds__(kThreads) conv_norm(StepRows r, ConvNormArgs a, int tile) {
   extern __shared__ __align__(16) float memory[];
   __shared__ float side_part[kWarps];
@@ -29,7 +31,7 @@ __global__ void __launch_bounds__(kThreads) conv_norm(StepRows r, ConvNormArgs a
   float* partial = ring + size_t(lead) * a.width;
   float* inverse = partial + (whole ? units / 32 : units);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  float weight[N][E], side_weight[N][E];
+  float weight[N][E], side_weight[N][E], held[HELD ? kHeldTaps : 1][N][E];
   auto each = [&](auto&& visit) {
 #pragma unroll
     for (int n = 0; n < N; ++n)
@@ -61,7 +63,13 @@ __global__ void __launch_bounds__(kThreads) conv_norm(StepRows r, ConvNormArgs a
   each([&](int n, int c) {
     load(a.weight, c, weight[n]);
     if (a.side) load(a.side_weight, c, side_weight[n]);
-    for (int j = 0; j < a.count; ++j) asm volatile("prefetch.global.L2 [%0];" ::"l"(a.taps + size_t(j) * a.width + size_t(c) * E));
+    if constexpr (HELD) {                                 // held[j]: of j tokens before
+#pragma unroll
+      for (int j = 0; j < kHeldTaps; ++j)
+        if (j < a.count) load(a.taps + size_t(lead - j) * a.width, c, held[j][n]);
+    } else {
+      for (int j = 0; j < a.count; ++j) asm volatile("prefetch.global.L2 [%0];" ::"l"(a.taps + size_t(j) * a.width + size_t(c) * E));
+    }
   });
   Entry e{0, 0, 0, 0};
   int first = 0, end = 1;
@@ -87,13 +95,19 @@ __global__ void __launch_bounds__(kThreads) conv_norm(StepRows r, ConvNormArgs a
   dependency_wait();
   allow_dependents();
 
-  float x[N][E], h[N][E];
-  auto form = [&](int row) {               // x' and h of one row
-    float y[N][E], sq = 0.f;
+  float x[N][E], h[N][E], next_x[N][E], y[N][E];
+  auto request = [&](int row) {            // one row ahead of its use
     each([&](int n, int c) {
-      load(a.x + size_t(row) * a.width, c, x[n]);
+      load(a.x + size_t(row) * a.width, c, next_x[n]);
       if (a.side) load(a.side + size_t(row) * a.width, c, y[n]);
     });
+  };
+  auto form = [&](int following) {         // x' and h of the row requested last
+    float sq = 0.f;
+#pragma unroll
+    for (int n = 0; n < N; ++n)
+#pragma unroll
+      for (int i = 0; i < E; ++i) x[n][i] = next_x[n][i];
     if (a.side) {
       each([&](int n, int) {
 #pragma unroll
@@ -111,6 +125,7 @@ __global__ void __launch_bounds__(kThreads) conv_norm(StepRows r, ConvNormArgs a
         for (int i = 0; i < E; ++i) x[n][i] = fmaf(a.gain, y[n][i] * inv * side_weight[n][i], x[n][i]);
       });
     }
+    if (following >= 0) request(following);
 #pragma unroll
     for (int n = 0; n < N; ++n) {
       const int c = threadIdx.x + kThreads * n;
@@ -140,50 +155,69 @@ __global__ void __launch_bounds__(kThreads) conv_norm(StepRows r, ConvNormArgs a
     });
   };
   if constexpr (SELECT) {
-    form(a.select ? min(max(a.select[blockIdx.x], 0), a.limit - 1) : int(blockIdx.x));
+    request(a.select ? min(max(a.select[blockIdx.x], 0), a.limit - 1) : int(blockIdx.x));
+    form(-1);
     each([&](int n, int c) { store_elements(a.normed, blockIdx.x, c, h[n]); });
   } else {
-    auto keep = [&](int j) {
+    const int start = max(0, first - lead);
+    int at = lead ? slot_of(e.first_position + start) : 0;   // the row's place in the ring
+    auto keep = [&]() {
       if (lead == 0) return;
-      float* to = ring + size_t(slot_of(e.first_position + j)) * a.width;
+      float* to = ring + size_t(at) * a.width;
       each([&](int n, int c) { store(to, c, h[n]); });
+      at = at + 1 == lead ? 0 : at + 1;
     };
-    for (int j = max(0, first - lead); j < end; ++j) {
+    request(e.first_row + start);
+    for (int j = start; j < end; ++j) {
       const size_t row = size_t(e.first_row) + j;
-      form(int(row));
+      form(j + 1 < end ? int(row) + 1 : -1);
       if (j >= first) {
         each([&](int n, int c) {
           if (a.x_out) store(a.x_out + row * a.width, c, x[n]);
           store_elements(a.normed, row, c, h[n]);
           if (a.count == 0) return;
-          float sum[E], by[E];
-          load(a.taps + size_t(lead) * a.width, c, by);
+          float sum[E], by[E], old[E];
+          if constexpr (HELD) {
 #pragma unroll
-          for (int i = 0; i < E; ++i) sum[i] = fmaf(by[i], h[n][i], h[n][i]);
-          for (int back = 1; back <= lead; ++back) {
-            float old[E];
-            load(a.taps + size_t(lead - back) * a.width, c, by);
-            load(ring + size_t(slot_of(e.first_position + j - back)) * a.width, c, old);
+            for (int i = 0; i < E; ++i) sum[i] = fmaf(held[0][n][i], h[n][i], h[n][i]);
 #pragma unroll
-            for (int i = 0; i < E; ++i) sum[i] = fmaf(by[i], old[i], sum[i]);
+            for (int back = 1; back < kHeldTaps; ++back) {
+              if (back > lead) break;
+              load(ring + size_t(at >= back ? at - back : at - back + lead) * a.width, c, old);
+#pragma unroll
+              for (int i = 0; i < E; ++i) sum[i] = fmaf(held[back][n][i], old[i], sum[i]);
+            }
+          } else {
+            load(a.taps + size_t(lead) * a.width, c, by);
+#pragma unroll
+            for (int i = 0; i < E; ++i) sum[i] = fmaf(by[i], h[n][i], h[n][i]);
+            for (int back = 1; back <= lead; ++back) {
+              load(a.taps + size_t(lead - back) * a.width, c, by);
+              load(ring + size_t(at >= back ? at - back : at - back + lead) * a.width, c, old);
+#pragma unroll
+              for (int i = 0; i < E; ++i) sum[i] = fmaf(by[i], old[i], sum[i]);
+            }
           }
           store_elements(a.convolved, row, c, sum);
         });
       }
-      keep(j);
+      keep();
     }
     if (first == 0 && lead > 0) {
-      if (e.rows > tile)
+      if (e.rows > tile) {
+        at = slot_of(e.first_position + e.rows - lead);
+        request(e.first_row + e.rows - lead);
         for (int j = e.rows - lead; j < e.rows; ++j) {
-          form(e.first_row + j);
-          keep(j);
+          form(j + 1 < e.rows ? e.first_row + j + 1 : -1);
+          keep();
         }
+      }
       for (int j = max(0, e.rows - lead); j < e.rows; ++j) {
-        const int at = slot_of(e.first_position + j);
+        const int place = slot_of(e.first_position + j);
         each([&](int, int c) {
           float v[E];
-          load(ring + size_t(at) * a.width, c, v);
-          store(a.history + (size_t(e.slot) * lead + at) * a.width, c, v);
+          load(ring + size_t(place) * a.width, c, v);
+          store(a.history + (size_t(e.slot) * lead + place) * a.width, c, v);
         });
       }
     }
@@ -193,10 +227,12 @@ __global__ void __launch_bounds__(kThreads) conv_norm(StepRows r, ConvNormArgs a
 template <typename T, int E, int N> int ConvNormWith(const Queue& q, const StepRows& r, const ConvNormArgs& a) {
   const int lead = std::max(a.count - 1, 0), units = a.width / E;
   const size_t smem = (size_t(lead) * a.width + units + a.groups) * sizeof(float);
-  if (a.select) return int(Launch(conv_norm<T, E, N, true>, dim3(unsigned(a.rows)), dim3(kThreads), smem, q.stream, q.chained, r, a, 1));
+  if (a.select) return int(Launch(conv_norm<T, E, N, true, false>, dim3(unsigned(a.rows)), dim3(kThreads), smem, q.stream, q.chained, r, a, 1));
   const int tile = std::max({1, lead, std::min(8, (a.rows + 2 * q.sm_count - 1) / (2 * q.sm_count))});
-  return int(Launch(conv_norm<T, E, N, false>, dim3(unsigned((r.longest + tile - 1) / tile), unsigned(r.entries)), dim3(kThreads), smem, q.stream, q.chained,
-                    r, a, tile));
+  auto kernel = conv_norm<T, E, N, false, false>;
+  if constexpr (N * E <= 8)
+    if (a.count <= kHeldTaps) kernel = conv_norm<T, E, N, false, true>;
+  return int(Launch(kernel, dim3(unsigned((r.longest + tile - 1) / tile), unsigned(r.entries)), dim3(kThreads), smem, q.stream, q.chained, r, a, tile));
 }
 
 template <typename T> int ConvNormAs(const Queue& q, const StepRows& r, const ConvNormArgs& a) {
@@ -208,8 +244,11 @@ template <typename T> int ConvNormAs(const Queue& q, const StepRows& r, const Co
 constexpr int kMostMemory = 226 * 1024;
 
 template <typename T, int E, int N> cudaError_t Raise() {
-  cudaError_t err = cudaFuncSetAttribute(conv_norm<T, E, N, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMostMemory);
-  return err == cudaSuccess ? cudaFuncSetAttribute(conv_norm<T, E, N, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMostMemory) : err;
+  for (auto kernel : {conv_norm<T, E, N, false, false>, conv_norm<T, E, N, true, false>, conv_norm<T, E, N, false, (N * E <= 8)>}) {
+    const cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kMostMemory);
+    if (err != cudaSuccess) return err;
+  }
+  return cudaSuccess;
 }
 template <typename T> cudaError_t RaiseAll() {
   for (cudaError_t err : {Raise<T, 4, 1>(), Raise<T, 4, 2>(), Raise<T, 4, 4>(), Raise<T, 1, 4>(), Raise<T, 1, 16>()})

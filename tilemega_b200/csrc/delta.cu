@@ -1,8 +1,8 @@
 // The generalised delta rule of ragged steps, see DeltaArgs, by its recurrence in fp32 (both element types). With the old
 // state S, p = u^T S and q = (w r)^T S of a column come out of one pass over it, and with them
 //   S' = diag(w) S - (a u) p + k v,      o = S'^T r = q - (r . a u) p + (r . k) v,
-// so a token costs one reduction over the key channels. Columns of a state do not meet: a warp owns four, a lane every eighth
-// four of a column's key channels, and states lie with a column's key channels contiguous.
+// so a token costs one reduction over the key channels (and so do two, see below). Columns of a state do not meet: warps own some
+// each, lanes some of their key channels, and states lie with a column's key channels contiguous.
 #include <cuda_bf16.h>
 
 #include <algorithm>
@@ -92,7 +92,7 @@ template <typename T, int DP> __device__ __forceinline__ void stage_token(const 
   }
 }
 
-// One token on a lane's share of a column: returns o, the same in all lanes of the column.
+// One token on a lane's share of a column (every eighth four of its key channels): returns o, the same in all lanes of the column.
 template <int NQ> __device__ __forceinline__ float advance(float4 (&s)[NQ], const float* token, int group, float v) {
   constexpr int DP = NQ * 32;
   float p0 = 0.f, p1 = 0.f, q0 = 0.f, q1 = 0.f;
@@ -126,62 +126,236 @@ template <int NQ> __device__ __forceinline__ float advance(float4 (&s)[NQ], cons
   return fmaf(token[kVectors * DP + 1], v, fmaf(-token[kVectors * DP], p, q));
 }
 
-// An entry's rows one after the other, 32 columns of a head a CTA: warps 0 .. 7 own the columns, warps 8 .. 15 stage the next
-// batch of tokens meanwhile, one each. blockIdx = (slice, head, entry).
-constexpr int kBatch = 8, kSlice = 32, kStepThreads = 512;
-template <int NQ> constexpr int kTokenFloats = kVectors * NQ * 32 + kScalars;
-template <int NQ> constexpr int kStepMemory = 2 * kBatch * (kTokenFloats<NQ> + kSlice) * 4;
+// ---- portions: two tokens a turn ------------------------------------------------------------------------------------------
+// With the tokens 0 and 1 of a pair, both reductions are taken against the state S before them:
+//   p0 = u0^T S,  p1 = (w0 u1)^T S - (u1 . a0) p0 + (u1 . k0) v0,      a = removal rate times unit key
+//   o0 = (w0 r0)^T S - (r0 . a0) p0 + (r0 . k0) v0
+//   o1 = (w0 w1 r1)^T S - (w1 r1 . a0) p0 + (w1 r1 . k0) v0 - (r1 . a1) p1 + (r1 . k1) v1
+//   S' = diag(w0 w1) S - (w1 a0) p0 + (w1 k0) v0 - a1 p1 + k1 v1
+// A missing second token is one without a key, a query and a decay. A warp owns 32 / G groups of four columns, a lane every G-th
+// four of their key channels; sixteen sums (two kinds, two tokens, four columns) meet by halving the list at every step.
+enum { kU0, kR0, kU1, kR1, kW01, kA0, kK0, kA1, kK1, kPairVectors };
+enum { kU1A0, kU1K0, kR0A0, kR0K0, kR1A0, kR1K0, kR1A1, kR1K1, kPairScalars };
+constexpr int kPairs = 8, kOwners = 4, kPairThreads = 32 * (kOwners + kPairs);   // pairs a batch; warps that own columns
+template <int G, int NQ> struct PairShape {
+  static constexpr int DP = 4 * G * NQ;                    // key channels, padded
+  static constexpr int kColumns = 4 * 32 / G, kSlice = kOwners * kColumns;   // of a warp, of a CTA
+  static constexpr int kFloats = kPairVectors * DP + kPairScalars + 2 * kSlice;
+  static constexpr int kMemory = 2 * kPairs * kFloats * 4;
+};
 
-template <typename T, int NQ>
-__global__ void __launch_bounds__(kStepThreads, 1) delta_steps(StepRows r, DeltaParams p, bool portions_only) {
-  extern __shared__ __align__(16) float tokens[];         // [2][kBatch][vectors, scalars], then [2][kBatch][kSlice] values
-  float* values = tokens + 2 * kBatch * kTokenFloats<NQ>;
+// Sums over the warp of eight values each, the lane >> 2-th of them in every lane.
+__device__ __forceinline__ float sum_eight(float (&v)[8], int lane) {
+#pragma unroll
+  for (int half = 4; half; half >>= 1) {
+    const bool upper = lane & (4 * half);
+#pragma unroll
+    for (int j = 0; j < half; ++j) {
+      const float keep = upper ? v[j + half] : v[j], send = upper ? v[j] : v[j + half];
+      v[j] = keep + __shfl_xor_sync(0xffffffffu, send, 4 * half);
+    }
+  }
+  v[0] += __shfl_xor_sync(0xffffffffu, v[0], 2);
+  v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
+  return v[0];
+}
+
+// What a pair of tokens brings, by one warp: the vectors, the scalars, then the values of the CTA's columns.
+template <typename T, int G, int NQ>
+__device__ __forceinline__ void stage_pair(const DeltaParams& p, int row, bool second, int head, int column0, int lane, float* to) {
+  using Shape = PairShape<G, NQ>;
+  constexpr int DP = Shape::DP, M = (DP / 4 + 31) / 32;
+  const size_t all = size_t(p.heads) * p.dim;
+  const T* line = static_cast<const T*>(p.proj) + size_t(row) * p.proj_stride + size_t(head) * p.dim;
+  const float* z = p.z + size_t(row) * all + size_t(head) * p.dim;
+  float rv[2][M][4], kv[2][M][4], av[2][M][4], wv[2][M][4], square[2] = {};
+#pragma unroll
+  for (int t = 0; t < 2; ++t)
+#pragma unroll
+    for (int m = 0; m < M; ++m) {
+      const int d = 4 * (lane + 32 * m), count = t == 0 || second ? min(4, p.dim - d) : 0;
+      const T* r = line + size_t(t) * p.proj_stride + d;
+      load_four(r, count, p.wide, rv[t][m]);
+      load_four(r + all, count, p.wide, kv[t][m]);
+      load_four(r + 3 * all, count, p.wide, av[t][m]);
+      load_four(z + size_t(t) * all + d, count, p.wide, wv[t][m]);
+    }
+  float value[2 * Shape::kSlice / 32];
+#pragma unroll
+  for (int i = 0; i < 2 * Shape::kSlice / 32; ++i) {
+    const int at = lane + 32 * i, t = at / Shape::kSlice, c = column0 + at % Shape::kSlice;
+    value[i] = c < p.dim && (t == 0 || second) ? to_f(line[size_t(t) * p.proj_stride + 2 * all + c]) : 0.f;
+  }
+#pragma unroll
+  for (int t = 0; t < 2; ++t) {
+#pragma unroll
+    for (int m = 0; m < M; ++m)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) square[t] = fmaf(kv[t][m][i], kv[t][m][i], square[t]);
+    square[t] = 1.f / sqrtf(warp_sum(square[t]) + p.unit_eps);
+  }
+  float scalar[8] = {};
+#pragma unroll
+  for (int m = 0; m < M; ++m) {
+    const int d = 4 * (lane + 32 * m);
+    float vec[kPairVectors][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const bool live = d + i < p.dim;
+      float u[2], a[2], w[2];
+#pragma unroll
+      for (int t = 0; t < 2; ++t) {
+        u[t] = kv[t][m][i] * square[t];
+        a[t] = u[t] * sigmoid(av[t][m][i]);
+        w[t] = !live ? 0.f : t == 0 || second ? expf(-p.decay_scale * sigmoid(wv[t][m][i])) : 1.f;
+      }
+      const float r0 = rv[0][m][i], r1 = rv[1][m][i], k0 = kv[0][m][i], k1 = kv[1][m][i], r1w = r1 * w[1];
+      vec[kU0][i] = u[0];
+      vec[kR0][i] = r0 * w[0];
+      vec[kU1][i] = u[1] * w[0];
+      vec[kR1][i] = r1w * w[0];
+      vec[kW01][i] = w[0] * w[1];
+      vec[kA0][i] = a[0] * w[1];
+      vec[kK0][i] = k0 * w[1];
+      vec[kA1][i] = a[1];
+      vec[kK1][i] = k1;
+      scalar[kU1A0] = fmaf(u[1], a[0], scalar[kU1A0]);
+      scalar[kU1K0] = fmaf(u[1], k0, scalar[kU1K0]);
+      scalar[kR0A0] = fmaf(r0, a[0], scalar[kR0A0]);
+      scalar[kR0K0] = fmaf(r0, k0, scalar[kR0K0]);
+      scalar[kR1A0] = fmaf(r1w, a[0], scalar[kR1A0]);
+      scalar[kR1K0] = fmaf(r1w, k0, scalar[kR1K0]);
+      scalar[kR1A1] = fmaf(r1, a[1], scalar[kR1A1]);
+      scalar[kR1K1] = fmaf(r1, k1, scalar[kR1K1]);
+    }
+    if (d < DP)
+#pragma unroll
+      for (int n = 0; n < kPairVectors; ++n) *reinterpret_cast<float4*>(to + n * DP + d) = make_float4(vec[n][0], vec[n][1], vec[n][2], vec[n][3]);
+  }
+  const float sum = sum_eight(scalar, lane);
+  if ((lane & 3) == 0) to[kPairVectors * DP + lane / 4] = sum;
+#pragma unroll
+  for (int i = 0; i < 2 * Shape::kSlice / 32; ++i) to[kPairVectors * DP + kPairScalars + lane + 32 * i] = value[i];
+}
+
+// An entry's rows in pairs, a slice of a head's columns a CTA: the first warps own the columns, the others stage the next batch of
+// pairs meanwhile, one each. blockIdx = (slice, head, entry).
+template <typename T, int G, int NQ>
+__global__ void __launch_bounds__(kPairThreads, 1) delta_pairs(StepRows r, DeltaParams p, bool portions_only) {
+  using Shape = PairShape<G, NQ>;
+  constexpr int DP = Shape::DP;
+  extern __shared__ __align__(16) float pairs[];           // [2][kPairs]
   dependency_wait();
   allow_dependents();
   const Entry e = r.entry[blockIdx.z];
   if (portions_only && e.rows == 1) return;
-  const int head = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, group = lane >> 2;
-  const int mine = warp * 4 + (lane & 3), column = blockIdx.x * kSlice + mine;
+  const int head = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, part = lane & (G - 1);
+  const int column0 = blockIdx.x * Shape::kSlice, mine = warp * Shape::kColumns + lane / G * 4;   // the lane's four columns, in the slice
   const size_t all = size_t(p.heads) * p.dim;
-  const bool owner = warp < kBatch, live = owner && column < p.dim;
-  float* state = p.state + ((size_t(e.slot) * p.heads + head) * p.dim + min(column, p.dim - 1)) * p.padded;
-  float4 s[NQ];
+  const bool owner = warp < kOwners;
+  float* state = p.state + (size_t(e.slot) * p.heads + head) * p.dim * p.padded;
+  float4 s[NQ][4];
+  auto each_state = [&](auto&& visit) {
 #pragma unroll
-  for (int i = 0; i < NQ; ++i) {
-    const int d = 4 * (group + 8 * i);
-    s[i] = live && e.first_position > 0 && d < p.padded ? *reinterpret_cast<const float4*>(state + d) : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
-  const int batches = (e.rows + kBatch - 1) / kBatch;
+    for (int i = 0; i < NQ; ++i)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const int column = column0 + mine + c, d = 4 * (part + G * i);
+        if (owner && column < p.dim && d < p.padded) visit(*reinterpret_cast<float4*>(state + size_t(column) * p.padded + d), s[i][c]);
+      }
+  };
+#pragma unroll
+  for (int i = 0; i < NQ; ++i)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) s[i][c] = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (e.first_position > 0) each_state([](const float4& from, float4& to) { to = from; });
+  const int count = (e.rows + 1) / 2, batches = (count + kPairs - 1) / kPairs;
   auto stage = [&](int batch) {                            // (the staging warps)
-    const int t = batch * kBatch + warp - kBatch, at = (batch & 1) * kBatch + warp - kBatch;
-    if (t >= e.rows) return;
-    const int row = e.first_row + t, c = blockIdx.x * kSlice + lane;
-    values[at * kSlice + lane] = c < p.dim ? to_f(static_cast<const T*>(p.proj)[size_t(row) * p.proj_stride + 2 * all + size_t(head) * p.dim + c]) : 0.f;
-    stage_token<T, NQ * 32>(p, row, head, lane, tokens + at * kTokenFloats<NQ>);
+    const int n = batch * kPairs + warp - kOwners;
+    if (n < count)
+      stage_pair<T, G, NQ>(p, e.first_row + 2 * n, 2 * n + 1 < e.rows, head, column0, lane,
+                           pairs + size_t((batch & 1) * kPairs + warp - kOwners) * Shape::kFloats);
   };
   if (!owner) stage(0);
+  // (which sum a lane ends up with)
+  const int held = G == 32 ? lane >> 1 : lane & 15, held_column = held & 3, home = G == 32 ? 0 : lane & 16;
+  const bool query = held & 8, later = held & 4, writes = query && (G != 32 || (lane & 1) == 0) && column0 + mine + held_column < p.dim;
+  auto pick = [&](const float (&v)[4]) { return held_column & 2 ? (held_column & 1 ? v[3] : v[2]) : (held_column & 1 ? v[1] : v[0]); };
   for (int batch = 0; batch < batches; ++batch) {
     __syncthreads();
     if (!owner) {
       if (batch + 1 < batches) stage(batch + 1);
       continue;
     }
-    const int t0 = batch * kBatch, n = min(kBatch, e.rows - t0);
-    for (int t = 0; t < n; ++t) {
-      const int at = (batch & 1) * kBatch + t;
-      const float o = advance<NQ>(s, tokens + at * kTokenFloats<NQ>, group, values[at * kSlice + mine]);
-      if (group == 0 && live) p.raw[size_t(e.first_row + t0 + t) * all + size_t(head) * p.dim + column] = o;
+    const int n0 = batch * kPairs, here = min(kPairs, count - n0);
+    for (int n = 0; n < here; ++n) {
+      const float* pair = pairs + size_t((batch & 1) * kPairs + n) * Shape::kFloats;
+      const float4* vec = reinterpret_cast<const float4*>(pair) + part;
+      auto get = [&](int which, int i) { return vec[which * (DP / 4) + G * i]; };
+      float x[16] = {};                                    // [kind][token][column]
+#pragma unroll
+      for (int i = 0; i < NQ; ++i) {
+        const float4 by[4] = {get(kU0, i), get(kU1, i), get(kR0, i), get(kR1, i)};
+#pragma unroll
+        for (int b = 0; b < 4; ++b)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            float v = x[4 * b + c];
+            v = fmaf(by[b].x, s[i][c].x, v);
+            v = fmaf(by[b].y, s[i][c].y, v);
+            v = fmaf(by[b].z, s[i][c].z, v);
+            x[4 * b + c] = fmaf(by[b].w, s[i][c].w, v);
+          }
+      }
+#pragma unroll
+      for (int half = 8; half; half >>= 1) {
+        const int mask = G == 32 ? 2 * half : half;
+        const bool upper = lane & mask;
+#pragma unroll
+        for (int j = 0; j < half; ++j) {
+          const float keep = upper ? x[j + half] : x[j], send = upper ? x[j] : x[j + half];
+          x[j] = keep + __shfl_xor_sync(0xffffffffu, send, mask);
+        }
+      }
+      float sum = x[0];
+      if (G == 32) sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+      const float4 c01 = *reinterpret_cast<const float4*>(pair + kPairVectors * DP), c23 = *reinterpret_cast<const float4*>(pair + kPairVectors * DP + 4);
+      const float4 v0q = *reinterpret_cast<const float4*>(pair + kPairVectors * DP + kPairScalars + mine);
+      const float4 v1q = *reinterpret_cast<const float4*>(pair + kPairVectors * DP + kPairScalars + Shape::kSlice + mine);
+      const float v0[4] = {v0q.x, v0q.y, v0q.z, v0q.w}, v1[4] = {v1q.x, v1q.y, v1q.z, v1q.w};
+      float p0[4], p1[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        p0[c] = __shfl_sync(0xffffffffu, sum, G == 32 ? 2 * c : home + c);
+        p1[c] = __shfl_sync(0xffffffffu, sum, G == 32 ? 8 + 2 * c : home + 4 + c);
+        p1[c] = fmaf(c01.y, v0[c], fmaf(-c01.x, p0[c], p1[c]));
+      }
+#pragma unroll
+      for (int i = 0; i < NQ; ++i) {
+        const float4 w = get(kW01, i), a0 = get(kA0, i), k0 = get(kK0, i), a1 = get(kA1, i), k1 = get(kK1, i);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          s[i][c].x = fmaf(w.x, s[i][c].x, fmaf(-a0.x, p0[c], fmaf(k0.x, v0[c], fmaf(-a1.x, p1[c], k1.x * v1[c]))));
+          s[i][c].y = fmaf(w.y, s[i][c].y, fmaf(-a0.y, p0[c], fmaf(k0.y, v0[c], fmaf(-a1.y, p1[c], k1.y * v1[c]))));
+          s[i][c].z = fmaf(w.z, s[i][c].z, fmaf(-a0.z, p0[c], fmaf(k0.z, v0[c], fmaf(-a1.z, p1[c], k1.z * v1[c]))));
+          s[i][c].w = fmaf(w.w, s[i][c].w, fmaf(-a0.w, p0[c], fmaf(k0.w, v0[c], fmaf(-a1.w, p1[c], k1.w * v1[c]))));
+        }
+      }
+      const int t = 2 * (n0 + n) + (later ? 1 : 0);
+      if (writes && t < e.rows) {
+        float o = fmaf(later ? c23.y : c01.w, pick(v0), fmaf(later ? -c23.x : -c01.z, pick(p0), sum));
+        if (later) o = fmaf(c23.w, pick(v1), fmaf(-c23.z, pick(p1), o));
+        p.raw[size_t(e.first_row + t) * all + size_t(head) * p.dim + column0 + mine + held_column] = o;
+      }
     }
   }
-#pragma unroll
-  for (int i = 0; i < NQ; ++i) {
-    const int d = 4 * (group + 8 * i);
-    if (live && d < p.padded) *reinterpret_cast<float4*>(state + d) = s[i];
-  }
+  each_state([](float4& to, const float4& from) { to = from; });
 }
 
+// ---- one decoded token ------------------------------------------------------------------------------------------------------
 // One decoded token of an entry, whole: recurrence, per-head norm and gate. A CTA holds one head's state, a lane its share of
 // PASSES columns; every load of the state is in flight before the first is used. blockIdx = (head, entry).
+template <int NQ> constexpr int kTokenFloats = kVectors * NQ * 32 + kScalars;
 constexpr int kTokenThreads = 512, kTokenColumns = kTokenThreads / 8;
 
 template <typename T, int NQ, int PASSES>
@@ -249,9 +423,10 @@ __global__ void __launch_bounds__(kTokenThreads, NQ * PASSES <= 8 ? 2 : 1) delta
 
 constexpr int kWholeHead = 192;          // widest head whose state one CTA holds
 
-template <typename T, int NQ> int StepsWith(const Queue& q, const StepRows& r, const DeltaParams& p, bool portions_only) {
-  return int(Launch(delta_steps<T, NQ>, dim3(unsigned((p.dim + kSlice - 1) / kSlice), unsigned(p.heads), unsigned(r.entries)), dim3(kStepThreads),
-                    kStepMemory<NQ>, q.stream, q.chained, r, p, portions_only));
+template <typename T, int G, int NQ> int PairsWith(const Queue& q, const StepRows& r, const DeltaParams& p, bool portions_only) {
+  using Shape = PairShape<G, NQ>;
+  return int(Launch(delta_pairs<T, G, NQ>, dim3(unsigned((p.dim + Shape::kSlice - 1) / Shape::kSlice), unsigned(p.heads), unsigned(r.entries)),
+                    dim3(kPairThreads), Shape::kMemory, q.stream, q.chained, r, p, portions_only));
 }
 
 template <typename T> int DeltaAs(const Queue& q, const StepRows& r, const DeltaArgs& a) {
@@ -262,8 +437,7 @@ template <typename T> int DeltaAs(const Queue& q, const StepRows& r, const Delta
   const bool whole = a.dim <= kWholeHead;
   int status = 0;
   if (r.singles < r.entries || !whole) {
-    status = quads <= 1 ? StepsWith<T, 1>(q, r, p, whole) : quads <= 2 ? StepsWith<T, 2>(q, r, p, whole) : quads <= 3 ? StepsWith<T, 3>(q, r, p, whole)
-             : quads <= 4 ? StepsWith<T, 4>(q, r, p, whole) : quads <= 6 ? StepsWith<T, 6>(q, r, p, whole) : StepsWith<T, 8>(q, r, p, whole);
+    status = p.dim <= 64 ? PairsWith<T, 16, 1>(q, r, p, whole) : p.dim <= 128 ? PairsWith<T, 32, 1>(q, r, p, whole) : PairsWith<T, 32, 2>(q, r, p, whole);
     if (status == 0)
       status = HeadGate(q, {a.raw, a.proj, a.proj_stride, 4 * a.heads * a.dim, a.out, a.out_stride, r.rows, a.heads, a.dim, a.norm, false, a.eps});
   }
@@ -274,11 +448,11 @@ template <typename T> int DeltaAs(const Queue& q, const StepRows& r, const Delta
   return int(Launch(kernel, dim3(unsigned(a.heads), unsigned(r.entries)), dim3(kTokenThreads), 0, q.stream, q.chained, r, p));
 }
 
-template <typename T, int NQ> cudaError_t Raise() {
-  return cudaFuncSetAttribute(delta_steps<T, NQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, kStepMemory<NQ>);
+template <typename T, int G, int NQ> cudaError_t Raise() {
+  return cudaFuncSetAttribute(delta_pairs<T, G, NQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, PairShape<G, NQ>::kMemory);
 }
 template <typename T> cudaError_t RaiseAll() {
-  for (cudaError_t err : {Raise<T, 1>(), Raise<T, 2>(), Raise<T, 3>(), Raise<T, 4>(), Raise<T, 6>(), Raise<T, 8>()})
+  for (cudaError_t err : {Raise<T, 16, 1>(), Raise<T, 32, 1>(), Raise<T, 32, 2>()})
     if (err != cudaSuccess) return err;
   return cudaSuccess;
 }

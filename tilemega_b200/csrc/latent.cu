@@ -362,7 +362,8 @@ __global__ void __launch_bounds__(kLatentThreads, SHARED ? 2 : 1) decode_latent(
 
 // A decoded token's splits put together, a CTA per head. blockIdx = (head, entry).
 constexpr int kMostSplits = 64;
-__global__ void __launch_bounds__(128) merge_latent(StepRows r, LatentParams p) {
+constexpr int kMergeThreads = kTiledLatent / 4;   // a thread per four columns
+__global__ void __launch_bounds__(kMergeThreads) merge_latent(StepRows r, LatentParams p) {
   __shared__ float factor[kMostSplits];
   dependency_wait();
   allow_dependents();
@@ -381,7 +382,7 @@ __global__ void __launch_bounds__(128) merge_latent(StepRows r, LatentParams p) 
   __syncthreads();
   const float4* parts = reinterpret_cast<const float4*>(p.part + record * p.rank_stride);
   bf16* dst = p.out + (size_t(e.first_row) * p.heads + head) * p.rank_stride;
-  for (int c = threadIdx.x; c < p.rank_stride / 4; c += 128) {
+  for (int c = threadIdx.x; c < p.rank_stride / 4; c += kMergeThreads) {
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
     for (int s = 0; s < p.splits; ++s) {
@@ -705,7 +706,7 @@ int DecodeLatent(const Queue& q, const StepRows& r, const LatentArgs& a, LatentP
   const int status = int(Launch(kernel, dim3(unsigned(p.splits), unsigned(p.subs), unsigned(r.entries)), dim3(kLatentThreads), smem, q.stream,
                                 q.chained, *a.pool_map, *a.q_map, r, p));
   if (status != 0 || p.splits == 1) return status;
-  return int(Launch(merge_latent, dim3(unsigned(a.heads), unsigned(r.entries)), dim3(128), 0, q.stream, q.chained, r, p));
+  return int(Launch(merge_latent, dim3(unsigned(a.heads), unsigned(r.entries)), dim3(kMergeThreads), 0, q.stream, q.chained, r, p));
 }
 
 template <int RT> int AttendWith(const Queue& q, const StepRows& r, LatentParams p) {

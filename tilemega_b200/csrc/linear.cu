@@ -68,23 +68,34 @@ __device__ __forceinline__ float glu_value(float g, float u, const Glu& p) {
   return g / (1.f + __expf(-p.alpha * g)) * (u + p.shift);
 }
 
-// Is column n of a product with rotated heads one that turns?
-__device__ __forceinline__ bool turns(const RotateHeads& p, int n) {
+// Output column n of a product with rotated heads: whether it turns, by which angles, and with which sign its neighbour enters.
+struct Turn {
+  bool on;
+  const float2* angles;      // of position 0
+  int half;
+  float sign;
+};
+__device__ __forceinline__ Turn turn_of(const RotateHeads& p, int n) {
   const int d = n % p.head - p.lead;
-  return d >= 0 && d < p.rotary.dims;
+  return {d >= 0 && d < p.rotary.dims, p.rotary.table + d / 2, p.rotary.dims / 2, d & 1 ? 1.f : -1.f};
 }
-// ... and what becomes of it; `other` is its neighbour's value.
-__device__ __forceinline__ float turned(const RotateHeads& p, int t, int n, float v, float other) {
-  const int d = n % p.head - p.lead;
-  const float2 cs = p.rotary.table[size_t(min(p.positions[t], p.rotary.capacity - 1)) * (p.rotary.dims / 2) + d / 2];
-  return d & 1 ? v * cs.x + other * cs.y : v * cs.x - other * cs.y;
+__device__ __forceinline__ float2 angle_at(const RotateHeads& p, const Turn& turn, int t) {
+  return turn.on ? __ldg(turn.angles + size_t(min(__ldg(p.positions + t), p.rotary.capacity - 1)) * turn.half) : make_float2(1.f, 0.f);
 }
+__device__ __forceinline__ float turned(const Turn& turn, float2 angle, float v, float other) { return v * angle.x + turn.sign * other * angle.y; }
 
 // gelu(z) times column n of the row's token's part
 template <typename T> __device__ __forceinline__ float side_value(const SideGate& p, int t, int n, float z) {
   const T* part = static_cast<const T*>(p.part) + size_t(min(max(p.tokens[t], 0), p.vocab - 1)) * p.stride;
   const float y = 0.7978845608028654f * (z + 0.044715f * z * z * z);
   return (sizeof(T) == 4 ? 0.5f * z * (1.f + tanhf(y)) : z / (1.f + __expf(-2.f * y))) * to_f(part[n]);
+}
+
+// tanh to the precision of a 16-bit element
+__device__ __forceinline__ float tanh16(float v) {
+  float y;
+  asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(v));
+  return y;
 }
 
 __device__ __forceinline__ uint32_t cluster_rank() {
@@ -104,7 +115,6 @@ __device__ __forceinline__ float ld_peer(uint32_t local, uint32_t rank) {
 }
 
 template <int EPI> __device__ __forceinline__ void emit(const LinearParams& g, int t, int n, float v) {
-  if (EPI == kLinearStore && n < g.tanh_below) v = tanhf(v);
   if (EPI == kLinearSide) v = side_value<__nv_bfloat16>(g.side, t, n, v);
   if (EPI == kLinearStore || EPI == kLinearHeads || EPI == kLinearRotate || EPI == kLinearSide)
     static_cast<__nv_bfloat16*>(g.out)[size_t(t) * g.out_stride + n] = __float2bfloat16_rn(v);
@@ -314,11 +324,26 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
         const int row = worker & (kRowsM - 1), n = n0 + row;
         if (n < g.n) {
           const float bias = g.bias ? g.bias[n] : 0.f;
-          const bool turning = EPI == kLinearRotate && turns(g.rotate, n);   // (neighbours lie in one tile)
-          for (int c = first + (worker >> 7); c < first + cols; c += 2) {
-            float v = total(c, row) + bias;
-            if (turning) v = turned(g.rotate, t0 + c, n, v, total(c, row ^ 1));
-            emit<EPI>(g, t0 + c, out_at + n, v);
+          if constexpr (EPI == kLinearRotate) {           // (neighbours lie in one tile)
+            const Turn turn = turn_of(g.rotate, n);
+            constexpr int U = 8;
+            for (int c0 = first + (worker >> 7); c0 < first + cols; c0 += 2 * U) {
+              float2 angle[U];
+#pragma unroll
+              for (int i = 0; i < U; ++i) angle[i] = angle_at(g.rotate, turn, t0 + min(c0 + 2 * i, first + cols - 1));
+#pragma unroll
+              for (int i = 0; i < U; ++i)
+                if (const int c = c0 + 2 * i; c < first + cols) {
+                  const float v = total(c, row);
+                  emit<EPI>(g, t0 + c, n, turn.on ? turned(turn, angle[i], v, total(c, row ^ 1)) : v);
+                }
+            }
+          } else {
+            const bool bent = EPI == kLinearStore && n < g.tanh_below;
+            for (int c = first + (worker >> 7); c < first + cols; c += 2) {
+              const float v = total(c, row) + bias;
+              emit<EPI>(g, t0 + c, out_at + n, bent ? tanh16(v) : v);
+            }
           }
         }
       }
@@ -344,11 +369,21 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
             static_cast<__nv_bfloat16*>(g.out)[size_t(t0 + c + col) * g.out_stride + out] = __float2bfloat16_rn(y);
         }
       } else if constexpr (EPI == kLinearRotate) {
-        const bool turning = turns(g.rotate, n);
+        const Turn turn = turn_of(g.rotate, n);
+        if (__any_sync(0xffffffffu, turn.on)) {
 #pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          const float other = __shfl_xor_sync(0xffffffffu, v[i], 1);
-          if (i < cols && n < g.n) emit<EPI>(g, t0 + c + i, n, turning ? turned(g.rotate, t0 + c + i, n, v[i], other) : v[i]);
+          for (int i0 = 0; i0 < 32; i0 += 8) {
+            float2 angle[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) angle[i] = angle_at(g.rotate, turn, t0 + c + min(i0 + i, cols - 1));
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i0 + i] = turned(turn, angle[i], v[i0 + i], __shfl_xor_sync(0xffffffffu, v[i0 + i], 1));
+          }
+        }
+        if (n < g.n) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (i < cols) emit<EPI>(g, t0 + c + i, n, v[i]);
         }
       } else if (n < g.n) {
         if constexpr (EPI == kLinearAdd) {
@@ -361,6 +396,11 @@ __global__ void __launch_bounds__(kLinearThreads) linear_tiles(const __grid_cons
           for (int i = 0; i < 32; ++i)
             if (i < cols) x[size_t(i) * g.out_stride] = old[i] + (v[i] + bias);
         } else {
+          if (EPI == kLinearStore && n0 < g.tanh_below) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (n < g.tanh_below) v[i] = tanh16(v[i] + bias) - bias;
+          }
 #pragma unroll
           for (int i = 0; i < 32; ++i)
             if (i < cols) emit<EPI>(g, t0 + c + i, out_at + n, v[i] + bias);
@@ -425,7 +465,10 @@ __global__ void __launch_bounds__(256) linear_f32(const float* activations, cons
       if (EPI == kLinearStore && n < g.tanh_below) v = tanhf(v);
       if (EPI == kLinearSide) v = side_value<float>(g.side, t, n, v);
       if (EPI == kLinearFloat) v *= g.gain;
-      if (EPI == kLinearRotate && turns(g.rotate, n)) v = turned(g.rotate, t, n, v, acc[i][j ^ 1]);
+      if constexpr (EPI == kLinearRotate) {
+        const Turn turn = turn_of(g.rotate, n);
+        if (turn.on) v = turned(turn, angle_at(g.rotate, turn, t), v, acc[i][j ^ 1]);
+      }
       float* out = static_cast<float*>(g.out) + size_t(EPI == kLinearExpertDown ? g.slots.list[t] : t) * g.out_stride + size_t(head) * g.head_out + n;
       const float positive = fmaxf(EPI == kLinearExpertUp ? v * g.slots.score[t] : 0.f, 0.f);
       *out = EPI == kLinearAdd ? *out + v : EPI == kLinearExpertUp ? positive * positive : v;
