@@ -135,6 +135,7 @@ def test_rotary_tables_with_a_stretched_length():
     (lambda m: m["layers"][4]["mixer"]["rotary"]["yarn"].update(fast=0), "length scaling"),
     (lambda m: m["layers"][1]["mixer"].update(vdim=10), "one size per head"),
     (lambda m: m["layers"][1]["mixer"].update(decay_rank=0), "decays' row"),
+    (lambda m: m["layers"][1]["mixer"].update(decay_scale=4.5), "factor of e.4 per token"),
     (lambda m: m["layers"][0]["side"].update({"from": 30}), "second embedding"),
     (lambda m: m["layers"][0]["mlp"].update(shared={"ff": 8, "limit": 1.0}), "no shared expert"),
     (lambda m: m["layers"][0]["mlp"].update(groups={"count": 3, "keep": 1}), "logits alone"),

@@ -266,6 +266,13 @@ def test_states_that_remember(dim, heads, dtype, plan_dir):
             return out
         return recurrence
 
+    # decays as steep as they get, and removals of everything
+    steep = bf16(tensors | {"l0.mix.w0": torch.full_like(tensors["l0.mix.w0"], 9.0), "l0.mix.a.b": torch.full_like(tensors["l0.mix.a.b"], 9.0)})
+    expected = case.truth(config, steep, ids)[0]
+    with executor(config, steep, plan_dir, dtype) as ex:
+        for cuts in ([200], [1], [13, 21, 2]):
+            assert case.error(run_cut(ex, ids, cuts), expected) < case.TOLERANCE[dtype], cuts
+
     if dtype == "f32":
         unit = lambda k: k / torch.sqrt((k * k).sum(-1, keepdim=True) + 1e-6)
         for name, wrong in (("delta_recurrence", after_decay), ("delta_recurrence", lambda f: lambda r, k, v, w, a: f(r, unit(k), v, w, a)),

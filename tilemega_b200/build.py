@@ -27,7 +27,7 @@ UNITS = (("megakernel", "megakernel.cu", (), ALL), ("megakernel_extended", "mega
          ("pack", "pack.cu", (), ALL), ("calibrate", "calibrate.cu", (), ALL), ("encoder", "encoder.cu", (), ALL),
          ("ragged", "ragged.cu", (), BOTH), ("ragged_spec", "ragged_spec.cpp", (), BOTH), ("linear", "linear.cu", (), BOTH),
          ("experts", "experts.cu", (), BOTH), ("mixers", "mixers.cu", (), BOTH), ("mixers_mma", "mixers_mma.cu", (), BOTH),
-         ("latent", "latent.cu", (), BOTH), ("delta", "delta.cu", (), BOTH), ("conv", "conv.cu", (), BOTH),
+         ("latent", "latent.cu", (), BOTH), ("delta", "delta.cu", (), BOTH), ("delta_mma", "delta_mma.cu", (), BOTH), ("conv", "conv.cu", (), BOTH),
          ("rows", "rows.cu", (), BOTH), ("absent", "absent.cu", (), ("ragged",)))
 # headers a source includes (directly or through another header): a unit is rebuilt when one of ITS headers changed
 SPEC_HEADERS = ("plan_spec.h", "json.h", "params.h", "ragged_spec.h")
@@ -39,7 +39,7 @@ UNIT_HEADERS = {"megakernel.cu": KERNEL_HEADERS, "static_probe.cu": KERNEL_HEADE
                 "ragged_spec.cpp": SPEC_HEADERS + ("ragged_limits.h",), "ragged.cu": SPEC_HEADERS + OP_HEADERS + ("ragged.h",),
                 "linear.cu": OP_HEADERS, "rows.cu": OP_HEADERS, "experts.cu": OP_HEADERS, "mixers.cu": OP_HEADERS + ("mixers.cuh",),
                 "mixers_mma.cu": OP_HEADERS + ("mixers.cuh", "mma.cuh"), "latent.cu": OP_HEADERS + ("mixers.cuh", "mma.cuh"),
-                "delta.cu": OP_HEADERS + ("mixers.cuh",), "conv.cu": OP_HEADERS}
+                "delta.cu": OP_HEADERS + ("mixers.cuh",), "delta_mma.cu": OP_HEADERS + ("mixers.cuh", "mma.cuh"), "conv.cu": OP_HEADERS}
 SOURCES = tuple(sorted({unit[1] for unit in UNITS}))
 HEADERS = tuple(sorted({header for headers in UNIT_HEADERS.values() for header in headers}))
 ABI_HEADER = ROOT.parent / "include" / "tilemega_b200.h"

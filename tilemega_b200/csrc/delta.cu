@@ -1,4 +1,5 @@
-// The generalised delta rule of ragged steps, see DeltaArgs, by its recurrence in fp32 (both element types). With the old
+// The generalised delta rule of ragged steps, see DeltaArgs, by its recurrence in fp32: decoded tokens, and the portions of fp32 plans
+// (those of bf16 plans: delta_mma.cu). With the old
 // state S, p = u^T S and q = (w r)^T S of a column come out of one pass over it, and with them
 //   S' = diag(w) S - (a u) p + k v,      o = S'^T r = q - (r . a u) p + (r . k) v,
 // so a token costs one reduction over the key channels (and so do two, see below). Columns of a state do not meet: warps own some
@@ -29,21 +30,6 @@ struct DeltaParams {
 
 enum { kUnit, kTurnedDecay, kDecay, kRemoval, kKey, kVectors };   // u, r w, w, a u, k
 constexpr int kScalars = 4;              // r . a u, r . k
-
-template <typename T> __device__ __forceinline__ void load_four(const T* at, int count, bool wide, float (&v)[4]) {
-  if (wide && count >= 4) {
-    if constexpr (sizeof(T) == 4) {
-      const float4 q = *reinterpret_cast<const float4*>(at);
-      v[0] = q.x, v[1] = q.y, v[2] = q.z, v[3] = q.w;
-    } else {
-      const uint2 w = *reinterpret_cast<const uint2*>(at);
-      v[0] = bf_lo(w.x), v[1] = bf_hi(w.x), v[2] = bf_lo(w.y), v[3] = bf_hi(w.y);
-    }
-  } else {
-#pragma unroll
-    for (int i = 0; i < 4; ++i) v[i] = i < count ? to_f(at[i]) : 0.f;
-  }
-}
 
 // What one token brings, by one warp: the vectors of its head, DP floats each (zeros behind the head), then the scalars.
 template <typename T, int DP> __device__ __forceinline__ void stage_token(const DeltaParams& p, int row, int head, int lane, float* to) {
@@ -126,7 +112,7 @@ template <int NQ> __device__ __forceinline__ float advance(float4 (&s)[NQ], cons
   return fmaf(token[kVectors * DP + 1], v, fmaf(-token[kVectors * DP], p, q));
 }
 
-// ---- portions: two tokens a turn ------------------------------------------------------------------------------------------
+// ---- portions (fp32 plans): two tokens a turn ------------------------------------------------------------------------------------------
 // With the tokens 0 and 1 of a pair, both reductions are taken against the state S before them:
 //   p0 = u0^T S,  p1 = (w0 u1)^T S - (u1 . a0) p0 + (u1 . k0) v0,      a = removal rate times unit key
 //   o0 = (w0 r0)^T S - (r0 . a0) p0 + (r0 . k0) v0
@@ -161,12 +147,12 @@ __device__ __forceinline__ float sum_eight(float (&v)[8], int lane) {
 }
 
 // What a pair of tokens brings, by one warp: the vectors, the scalars, then the values of the CTA's columns.
-template <typename T, int G, int NQ>
+template <int G, int NQ>
 __device__ __forceinline__ void stage_pair(const DeltaParams& p, int row, bool second, int head, int column0, int lane, float* to) {
   using Shape = PairShape<G, NQ>;
   constexpr int DP = Shape::DP, M = (DP / 4 + 31) / 32;
   const size_t all = size_t(p.heads) * p.dim;
-  const T* line = static_cast<const T*>(p.proj) + size_t(row) * p.proj_stride + size_t(head) * p.dim;
+  const float* line = static_cast<const float*>(p.proj) + size_t(row) * p.proj_stride + size_t(head) * p.dim;
   const float* z = p.z + size_t(row) * all + size_t(head) * p.dim;
   float rv[2][M][4], kv[2][M][4], av[2][M][4], wv[2][M][4], square[2] = {};
 #pragma unroll
@@ -174,7 +160,7 @@ __device__ __forceinline__ void stage_pair(const DeltaParams& p, int row, bool s
 #pragma unroll
     for (int m = 0; m < M; ++m) {
       const int d = 4 * (lane + 32 * m), count = t == 0 || second ? min(4, p.dim - d) : 0;
-      const T* r = line + size_t(t) * p.proj_stride + d;
+      const float* r = line + size_t(t) * p.proj_stride + d;
       load_four(r, count, p.wide, rv[t][m]);
       load_four(r + all, count, p.wide, kv[t][m]);
       load_four(r + 3 * all, count, p.wide, av[t][m]);
@@ -184,7 +170,7 @@ __device__ __forceinline__ void stage_pair(const DeltaParams& p, int row, bool s
 #pragma unroll
   for (int i = 0; i < 2 * Shape::kSlice / 32; ++i) {
     const int at = lane + 32 * i, t = at / Shape::kSlice, c = column0 + at % Shape::kSlice;
-    value[i] = c < p.dim && (t == 0 || second) ? to_f(line[size_t(t) * p.proj_stride + 2 * all + c]) : 0.f;
+    value[i] = c < p.dim && (t == 0 || second) ? line[size_t(t) * p.proj_stride + 2 * all + c] : 0.f;
   }
 #pragma unroll
   for (int t = 0; t < 2; ++t) {
@@ -240,7 +226,7 @@ __device__ __forceinline__ void stage_pair(const DeltaParams& p, int row, bool s
 
 // An entry's rows in pairs, a slice of a head's columns a CTA: the first warps own the columns, the others stage the next batch of
 // pairs meanwhile, one each. blockIdx = (slice, head, entry).
-template <typename T, int G, int NQ>
+template <int G, int NQ>
 __global__ void __launch_bounds__(kPairThreads, 1) delta_pairs(StepRows r, DeltaParams p, bool portions_only) {
   using Shape = PairShape<G, NQ>;
   constexpr int DP = Shape::DP;
@@ -273,7 +259,7 @@ __global__ void __launch_bounds__(kPairThreads, 1) delta_pairs(StepRows r, Delta
   auto stage = [&](int batch) {                            // (the staging warps)
     const int n = batch * kPairs + warp - kOwners;
     if (n < count)
-      stage_pair<T, G, NQ>(p, e.first_row + 2 * n, 2 * n + 1 < e.rows, head, column0, lane,
+      stage_pair<G, NQ>(p, e.first_row + 2 * n, 2 * n + 1 < e.rows, head, column0, lane,
                            pairs + size_t((batch & 1) * kPairs + warp - kOwners) * Shape::kFloats);
   };
   if (!owner) stage(0);
@@ -423,9 +409,9 @@ __global__ void __launch_bounds__(kTokenThreads, NQ * PASSES <= 8 ? 2 : 1) delta
 
 constexpr int kWholeHead = 192;          // widest head whose state one CTA holds
 
-template <typename T, int G, int NQ> int PairsWith(const Queue& q, const StepRows& r, const DeltaParams& p, bool portions_only) {
+template <int G, int NQ> int PairsWith(const Queue& q, const StepRows& r, const DeltaParams& p, bool portions_only) {
   using Shape = PairShape<G, NQ>;
-  return int(Launch(delta_pairs<T, G, NQ>, dim3(unsigned((p.dim + Shape::kSlice - 1) / Shape::kSlice), unsigned(p.heads), unsigned(r.entries)),
+  return int(Launch(delta_pairs<G, NQ>, dim3(unsigned((p.dim + Shape::kSlice - 1) / Shape::kSlice), unsigned(p.heads), unsigned(r.entries)),
                     dim3(kPairThreads), Shape::kMemory, q.stream, q.chained, r, p, portions_only));
 }
 
@@ -437,7 +423,8 @@ template <typename T> int DeltaAs(const Queue& q, const StepRows& r, const Delta
   const bool whole = a.dim <= kWholeHead;
   int status = 0;
   if (r.singles < r.entries || !whole) {
-    status = p.dim <= 64 ? PairsWith<T, 16, 1>(q, r, p, whole) : p.dim <= 128 ? PairsWith<T, 32, 1>(q, r, p, whole) : PairsWith<T, 32, 2>(q, r, p, whole);
+    if (!q.f32) status = DeltaChunks(q, r, a, whole);
+    else status = p.dim <= 64 ? PairsWith<16, 1>(q, r, p, whole) : p.dim <= 128 ? PairsWith<32, 1>(q, r, p, whole) : PairsWith<32, 2>(q, r, p, whole);
     if (status == 0)
       status = HeadGate(q, {a.raw, a.proj, a.proj_stride, 4 * a.heads * a.dim, a.out, a.out_stride, r.rows, a.heads, a.dim, a.norm, false, a.eps});
   }
@@ -448,15 +435,9 @@ template <typename T> int DeltaAs(const Queue& q, const StepRows& r, const Delta
   return int(Launch(kernel, dim3(unsigned(a.heads), unsigned(r.entries)), dim3(kTokenThreads), 0, q.stream, q.chained, r, p));
 }
 
-template <typename T, int G, int NQ> cudaError_t Raise() {
-  return cudaFuncSetAttribute(delta_pairs<T, G, NQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, PairShape<G, NQ>::kMemory);
+template <int G, int NQ> cudaError_t Raise() {
+  return cudaFuncSetAttribute(delta_pairs<G, NQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, PairShape<G, NQ>::kMemory);
 }
-template <typename T> cudaError_t RaiseAll() {
-  for (cudaError_t err : {Raise<T, 16, 1>(), Raise<T, 32, 1>(), Raise<T, 32, 2>()})
-    if (err != cudaSuccess) return err;
-  return cudaSuccess;
-}
-
 }  // namespace
 
 int Delta(const Queue& q, const StepRows& r, const DeltaArgs& a) {
@@ -465,8 +446,9 @@ int Delta(const Queue& q, const StepRows& r, const DeltaArgs& a) {
 }
 
 int PrepareDelta() {
-  const cudaError_t err = RaiseAll<float>();
-  return int(err == cudaSuccess ? RaiseAll<__nv_bfloat16>() : err);
+  for (cudaError_t err : {Raise<16, 1>(), Raise<32, 1>(), Raise<32, 2>()})
+    if (err != cudaSuccess) return int(err);
+  return PrepareDeltaChunks();
 }
 
 }  // namespace tmb

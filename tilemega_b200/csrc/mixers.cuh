@@ -84,6 +84,22 @@ template <typename T> __device__ __forceinline__ T blended(const Blend& b, const
   return from_f<T>((1.f - f) * to_f(own[i]) + f * to_f(static_cast<const T*>(b.from)[size_t(row) * b.stride + i]));
 }
 
+// Four neighbours, of which the first `count` are there (zeros behind them); `wide`: their address suits one load.
+template <typename T> __device__ __forceinline__ void load_four(const T* at, int count, bool wide, float (&v)[4]) {
+  if (wide && count >= 4) {
+    if constexpr (sizeof(T) == 4) {
+      const float4 q = *reinterpret_cast<const float4*>(at);
+      v[0] = q.x, v[1] = q.y, v[2] = q.z, v[3] = q.w;
+    } else {
+      const uint2 w = *reinterpret_cast<const uint2*>(at);
+      v[0] = bf_lo(w.x), v[1] = bf_hi(w.x), v[2] = bf_lo(w.y), v[3] = bf_hi(w.y);
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) v[i] = i < count ? to_f(at[i]) : 0.f;
+  }
+}
+
 __device__ __forceinline__ float sigmoid(float v) { return 1.f / (1.f + expf(-v)); }
 
 }  // namespace tmb

@@ -367,9 +367,14 @@ struct DeltaArgs {
   int heads, dim, padded;
   const float* norm;         // [heads * dim]
   float decay_scale, unit_eps, eps;
+  void* chunks;              // bf16: DeltaChunkBytes bytes, the portions' chunks
 };
 int Delta(const Queue& q, const StepRows& r, const DeltaArgs& a);
 int PrepareDelta();
+size_t DeltaChunkBytes(int rows, int slots, int heads, int dim);
+// The bf16 form of portions (portions_only: of these alone), up to the heads' raw outputs.
+int DeltaChunks(const Queue& q, const StepRows& r, const DeltaArgs& a, bool portions_only);
+int PrepareDeltaChunks();
 
 // next[i] = index of the largest of logits[i][0..vocab), the smallest such index on a tie.
 int ArgMax(const Queue& q, const float* logits, int rows, int vocab, int* next);

@@ -36,6 +36,7 @@ struct RaggedPlan {
   float* side_out = nullptr;
   void *query_latent = nullptr, *queries = nullptr;   // latent attention: normed rows that queries are images of, and these
   float* decay_in = nullptr;   // delta rule: what decays are made of, [max_rows][heads * dim]
+  void* chunks = nullptr;      // ... bf16 plans: operands of the portions' chunks
   // bf16 plans with latent attention: the latent rows that portions see, gathered, and their keys and values
   void *context = nullptr, *expanded = nullptr;
   int *context_at = nullptr, *context_count = nullptr;
@@ -332,6 +333,7 @@ int Enqueue(RaggedPlan* plan, uint32_t entries, uint32_t rows, uint32_t longest,
       a.decay_scale = float(m.decay_scale);
       a.unit_eps = float(m.unit_eps);
       a.eps = float(s.eps);
+      a.chunks = plan->chunks;
       TMB_TRY(Delta(q, r, a));
     } else if (m.kind == RaggedMixer::kLatent) {
       LatentArgs a{};
@@ -615,7 +617,7 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
     return nullptr;
   };
   const size_t element = spec.f32 ? 4 : 2;
-  size_t proj = 0, mixed = 0, mlp = 0, pairs = 0, raw = 0, split = 0, heads = 1, partial = 0, query_latent = 0, queries = 0, decays = 0;
+  size_t proj = 0, mixed = 0, mlp = 0, pairs = 0, raw = 0, split = 0, heads = 1, partial = 0, query_latent = 0, queries = 0, decays = 0, chunks = 0;
   size_t top = 0, experts = 0, expert_columns = 0, expert_pairs = 0, source = 0, latent = 0, ranks = 0, context = 0, expanded = 0;
   int reach = 0;
   for (const RaggedLayer& layer : spec.layers) {
@@ -649,6 +651,7 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
     } else if (m.kind == RaggedMixer::kDelta) {
       raw = std::max(raw, size_t(m.out_columns()));
       decays = std::max(decays, size_t(m.out_columns()));
+      chunks = std::max(chunks, DeltaChunkBytes(spec.max_rows, spec.slots, m.heads, m.dim));
     } else {
       const size_t columns = m.kind == RaggedMixer::kLatent ? size_t(m.rank_stride()) : size_t(m.vdim);
       heads = std::max(heads, size_t(m.heads));
@@ -681,7 +684,7 @@ RaggedPlan* RaggedCreate(const RaggedSpec& spec, const std::vector<void*>& buffe
       !Own(plan, &plan->side_hidden, spec.side_dim ? rows * size_t(padded_columns(spec.side_dim)) * element : 0) ||
       !Own(plan, &plan->side_out, spec.side_dim ? rows * size_t(spec.width) * sizeof(float) : 0) ||
       !Own(plan, &plan->query_latent, rows * query_latent * element) || !Own(plan, &plan->queries, rows * queries * element) ||
-      !Own(plan, &plan->decay_in, rows * decays * sizeof(float)) ||
+      !Own(plan, &plan->decay_in, rows * decays * sizeof(float)) || !Own(plan, &plan->chunks, spec.f32 ? 0 : chunks) ||
       !Own(plan, &plan->context, context_rows * context * element) || !Own(plan, &plan->expanded, context_rows * expanded * element) ||
       !Own(plan, &plan->context_at, size_t(spec.slots) * sizeof(int)) || !Own(plan, &plan->context_count, sizeof(int)) ||
       !Own(plan, &plan->source, rows * source * element) || !Own(plan, &plan->lookup, rows * latent * element) ||

@@ -12,6 +12,7 @@ constexpr int kMaxConvWidth = 8192;   // residual columns of models with grouped
 constexpr int kRaggedBlock = 16;      // positions per KV pool block
 constexpr int kMaxExperts = 1024;     // of a layer
 constexpr int kMaxTop = 32;           // experts a token uses
+constexpr double kMostDecay = 4;       // of a delta rule in bf16 plans: largest scale of the log decays
 constexpr int kRetentionChunk = 64;   // positions a retention state advances by at once inside a prompt portion
 
 }  // namespace tmb

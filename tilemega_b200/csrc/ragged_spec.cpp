@@ -247,6 +247,7 @@ RaggedSpec RaggedSpec::FromJson(const Json& plan, std::vector<BufferSpec>* buffe
       m.decay_scale = mixer.num("decay_scale", 0);
       m.unit_eps = mixer.num("unit_eps", 0);
       Require(m.kv_heads == m.heads && m.vdim == m.dim && m.rotary < 0, "a delta rule has a key and a value of one size per head and no rotation");
+      Require(s.f32 || m.decay_scale <= kMostDecay, "a bf16 plan's delta rule forgets at most a factor of e^4 per token (decay_scale)");
       Require(m.decay_rank >= 1 && m.decay_scale > 0 && m.unit_eps > 0, "a delta rule needs the size of its decays' row (decay_rank), decay_scale and unit_eps");
       std::vector<std::string> parts = {PerHead("pad_heads", Json::Quote(Name(names, "w1")), 1, "rows", m.delta_at())};
       for (const char* part : {"r", "k", "v", "a", "g"}) parts.push_back(Json::Quote(Name(names, part)));
